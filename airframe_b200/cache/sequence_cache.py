@@ -133,14 +133,15 @@ class LayerCacheView:
     writes: bool                        # False: the run reads another run's keys and values
     keep_step_kv: bool                  # a later run reads this run's keys and values
     kv: Optional[KVView]
-    state: Optional[torch.Tensor]       # [slots, *shape]
+    state: Optional[torch.Tensor]       # [slots, *shape]: the mixer's
+    block_state: Optional[torch.Tensor] = None      # [slots, *shape]: what the layer's arrangement keeps
 
 
 class SequenceCache:
     """Slots, pages and fixed-size state for all runs of a model.
 
     ``needs`` lists, per schedule entry, ``(KVNeed | None, StateNeed | None,
-    cache_from | None)``.  ``max_tokens`` is the most tokens live sequences
+    cache_from | None)``, or four of them, the last a StateNeed | None of the run's block.  ``max_tokens`` is the most tokens live sequences
     hold together, each rounded up to whole pages; ``max_context`` the longest
     single sequence.  With ``device=None`` only the bookkeeping exists.
 
@@ -168,7 +169,8 @@ class SequenceCache:
         self.views: list = []
         by_need: dict = {}
         readers = {n[2] for n in needs if n[2] is not None}
-        for run, (kv_need, state_need, cache_from) in enumerate(needs):
+        needs = [(*n, None) if len(n) == 3 else tuple(n) for n in needs]
+        for run, (kv_need, state_need, cache_from, _) in enumerate(needs):
             if cache_from is None and kv_need is not None:
                 by_need.setdefault(kv_need, []).append(run)
         for need, runs in by_need.items():
@@ -177,7 +179,7 @@ class SequenceCache:
                 ring_pages = pages_for(min(pages_for(need.window) * PAGE, self.max_context))
                 n_pages = min(n_pages, self.n_slots * ring_pages)
             self.groups[need] = KVGroup(need, runs, self.n_slots, n_pages, self.max_context, dtype, device)
-        for run, (kv_need, state_need, cache_from) in enumerate(needs):
+        for run, (kv_need, state_need, cache_from, block_need) in enumerate(needs):
             src = run if cache_from is None else cache_from
             kv_view = None
             src_need = needs[src][0]
@@ -191,14 +193,16 @@ class SequenceCache:
                 i = g.index_of[src]
                 kv_view = KVView(g.k[i] if g.k is not None else None, g.v[i] if g.v is not None else None,
                                  g.table, g.ring_rows, src_need)
-            state = None
-            if state_need is not None:
-                if device is not None:
-                    state = torch.zeros((self.n_slots, *state_need.shape),
-                                        dtype=_STATE_DTYPES[state_need.dtype], device=device)
-                self.states[run] = state
+            held = []
+            for key, need in ((run, state_need), ((run, "block"), block_need)):
+                state = None
+                if need is not None:
+                    if device is not None:
+                        state = torch.zeros((self.n_slots, *need.shape), dtype=_STATE_DTYPES[need.dtype], device=device)
+                    self.states[key] = state
+                held.append(state)
             self.views.append(LayerCacheView(cache_id=src, writes=cache_from is None,
-                                             keep_step_kv=run in readers, kv=kv_view, state=state))
+                                             keep_step_kv=run in readers, kv=kv_view, state=held[0], block_state=held[1]))
 
     # ------------------------------------------------------------------ slots
 

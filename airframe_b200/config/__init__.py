@@ -5,6 +5,7 @@ from .banitar import BanitarConfig
 from .fiferax import FiferaxConfig
 from .gemma2 import Gemma2Config
 from .tarorax import TaroraxConfig
+from .teselix import TeselixConfig
 from .zatasun import ZatasunConfig
 from .registry import (architecture_name, config_from_dict, config_from_folder,
                        known_architectures, register_architecture)
@@ -14,9 +15,10 @@ register_architecture(FiferaxConfig.architecture, FiferaxConfig)
 register_architecture(BanitarConfig.architecture, BanitarConfig)
 register_architecture(ZatasunConfig.architecture, ZatasunConfig)
 register_architecture(TaroraxConfig.architecture, TaroraxConfig)
+register_architecture(TeselixConfig.architecture, TeselixConfig)
 
 __all__ = [
     "ConfigError", "KeyReader", "LayerSpec", "ModelConfig", "ModelSpec", "PartSpec", "ScheduleEntry",
-    "read_config_json", "BanitarConfig", "FiferaxConfig", "Gemma2Config", "TaroraxConfig", "ZatasunConfig", "architecture_name", "config_from_dict",
-    "config_from_folder", "known_architectures", "register_architecture",
+    "read_config_json", "BanitarConfig", "FiferaxConfig", "Gemma2Config", "TaroraxConfig", "TeselixConfig",
+    "ZatasunConfig", "architecture_name", "config_from_dict", "config_from_folder", "known_architectures", "register_architecture",
 ]

@@ -1,6 +1,6 @@
 """Named configurations for the random-weights mode: the two tiny test
-models, the layer sizes of the released Gemma-2 models, a small Fiferax, a small Banitar, a small Zatasun and a small Tarorax, as
-config.json dictionaries.  Nothing here is read by the model code: a configuration always
+models, the layer sizes of the released Gemma-2 models, a small Fiferax, a small Banitar, a small Zatasun, a small Tarorax
+and a small Teselix, as config.json dictionaries.  Nothing here is read by the model code: a configuration always
 reaches it through ``config_from_dict``."""
 from __future__ import annotations
 
@@ -99,6 +99,24 @@ def _tarorax_small() -> dict:
 
 
 PRESETS["tarorax-small"] = _tarorax_small()
+
+
+def _teselix_small() -> dict:
+    """Teselix with four layers, the last of which uses the second's weights (sizes of no released model)."""
+    ret = {"heads": 4, "dim": 64, "vdim": 128, "decay": [1.0 - 2.0 ** -(4 + h) for h in range(4)],
+           "rot": {"base": 10000.0, "dims": 64}}
+    lat = {"heads": 8, "dim": 64, "rot_dim": 32, "vdim": 64, "kv_rank": 160, "q_rank": 192, "scale": 0.1,
+           "rot": {"base": 10000.0, "dims": 32, "scaling": {"factor": 8.0, "original": 1024, "fast": 32.0, "slow": 1.0}}}
+    moe = {"kind": "moe", "expert": {"ff": 256, "limit": 7.0}, "router": {"experts": 8, "top": 2},
+           "shared": {"ff": 512, "limit": 7.0}}
+    layers = [{"type": "retention", "mixer": ret, "mlp": None}, {"type": "latent_attention", "mixer": lat, "mlp": moe},
+              {"type": "retention", "mixer": ret, "mlp": moe},
+              {"type": "latent_attention", "mixer": lat, "mlp": moe, "weights_of": 1}]
+    return {"architecture": "Teselix", "vocab": 8192, "width": 512, "norm": {"eps": 1e-5}, "postln_alpha": 1.5,
+            "layers": layers}
+
+
+PRESETS["teselix-small"] = _teselix_small()
 
 
 def preset(name: str) -> dict:

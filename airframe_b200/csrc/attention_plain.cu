@@ -970,94 +970,166 @@ AF_EXPORT int af_qk_norm_rope_store(void* qkv, int dtype, long long out_stride, 
 
 // ---------------------------------------------------------------- keys and values from a latent vector
 
-// From float projection rows [q heads of (dim + rot) | latent of `rank` | shared key part of `rot`]:
-//   q heads: the last `rot` elements of every head rotated (pairs i, i + rot / 2), the first `dim` kept,
-//            into the rows `q` of the compute dtype, head u at u * pitch (pitch >= dim + rot; the elements
-//            between a head's end and the next head's start are set to zero);
-//   the latent divided by its root mean square (eps inside the root) times `norm_w`, and the shared key
-//   part rotated, into the row `kv` [rank + rot] of the compute dtype and into the token's row of its cache
-//   page (one kv head of rank + rot elements; the values are the latent part of the same row).
+// Three jobs of latent attention, each done when its source is given, from float projection rows:
+//   q       heads of (dim + rot) elements (from `q_parts` partial sums, added in order): the last `rot` elements of every
+//           head rotated, the first `dim` kept, into the rows `q` of the compute dtype, head u at u * pitch
+//           (pitch >= dim + rot; the elements between a head's end and the next head's start are set to zero);
+//   kv      [latent of `rank` | shared key part of `rot`]: the latent divided by its root mean square (eps inside the
+//           root) times `norm_w`, and the shared key part rotated, into the row `kv` [rank + rot] of the compute
+//           dtype and into the token's row of its cache page (one kv head of rank + rot elements; the values are
+//           the latent part of the same row);
+//   side    another latent of `side_n` elements (the queries'), normed with `side_w` into rows of the compute dtype.
+// Rotation: pairs (i, i + rot / 2), or (2 i, 2 i + 1) with `adjacent`; cosines and sines from `table` (of the step's
+// tokens) or worked out from `inv_freq`, times `magnitude`.
 // One block per token.
 template <typename T>
+struct LatentPrepArgs {
+  T* q;
+  long long q_stride;
+  const float* q_src;
+  long long q_ld, q_part_stride;
+  int q_parts, heads, dim, rot, pitch;
+  T* kv;
+  long long kv_stride;
+  const float* kv_src;
+  long long kv_ld;
+  const float* norm_w;
+  int rank;
+  T* side;
+  long long side_stride;
+  const float* side_src;
+  long long side_ld;
+  const float* side_w;
+  int side_n;
+  float eps, magnitude;
+  int adjacent;
+  const float* inv_freq;
+  const float2* table;
+  const int *positions, *seq_of_token, *slots, *len_after;
+  T* kcache;
+  const int* page_table;
+  int max_pages, ring_rows;
+};
+
+template <typename T>
 __global__ void __launch_bounds__(256)
-latent_prep_kernel(T* __restrict__ q, long long q_stride, T* __restrict__ kv, long long kv_stride,
-                   const float* __restrict__ proj, long long ld, const float* __restrict__ norm_w, float eps,
-                   const int* __restrict__ positions, const int* __restrict__ seq_of_token,
-                   const int* __restrict__ slots, const int* __restrict__ len_after,
-                   const float* __restrict__ inv_freq, int heads, int dim, int rot, int rank, int pitch,
-                   T* __restrict__ kcache, const int* __restrict__ page_table, int max_pages, int ring_rows) {
+latent_prep_kernel(LatentPrepArgs<T> p) {
   pdl_launch_dependents();
   __shared__ float scratch[33];
-  const int t = blockIdx.x;
-  const int pos = positions[t];
-  const int width = rank + rot;
+  const int t = blockIdx.x, rot = p.rot, rank = p.rank, dim = p.dim;
+  const int pos = p.positions[t];
   T* kdst = nullptr;
-  if (kcache != nullptr) {
-    const int seq = seq_of_token[t];
-    const int slot = slots[seq];
-    if (slot >= 0 && !(ring_rows > 0 && pos + ring_rows < len_after[seq])) {
-      const int r = ring_rows > 0 ? pos % ring_rows : pos;
-      if (AF_INDEX_OK(pos >= 0 && r / AF_PAGE < max_pages, r)) {
-        const int page = page_table[(size_t)slot * max_pages + r / AF_PAGE];
-        if (AF_INDEX_OK(page >= 0, page)) kdst = kcache + ((size_t)page * AF_PAGE + r % AF_PAGE) * width;
+  if (p.kcache != nullptr && p.kv_src != nullptr) {
+    const int seq = p.seq_of_token[t];
+    const int slot = p.slots[seq];
+    if (slot >= 0 && !(p.ring_rows > 0 && pos + p.ring_rows < p.len_after[seq])) {
+      const int r = p.ring_rows > 0 ? pos % p.ring_rows : pos;
+      if (AF_INDEX_OK(pos >= 0 && r / AF_PAGE < p.max_pages, r)) {
+        const int page = p.page_table[(size_t)slot * p.max_pages + r / AF_PAGE];
+        if (AF_INDEX_OK(page >= 0, page)) kdst = p.kcache + ((size_t)page * AF_PAGE + r % AF_PAGE) * (rank + rot);
       }
     }
   }
   pdl_wait();
-  const float* x = proj + (size_t)t * ld;
-  const float* lat = x + (size_t)heads * (dim + rot);
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < rank; i += blockDim.x) ss += lat[i] * lat[i];
-  ss = block_sum(ss, scratch);
-  const float inv = rsqrtf(ss / (float)rank + eps);
-  T* kvr = kv + (size_t)t * kv_stride;
-  for (int i = threadIdx.x; i < rank; i += blockDim.x) {
-    const T v = from_f32<T>(lat[i] * inv * norm_w[i]);
-    kvr[i] = v;
-    if (kdst != nullptr) kdst[i] = v;
-  }
   const int half = rot / 2;
-  T* qr = q + (size_t)t * q_stride;
-  // rotated pairs: unit heads + 1 is the shared key part
-  for (int i = threadIdx.x; i < (heads + 1) * half; i += blockDim.x) {
-    const int u = i / half, p = i - u * half;
-    float s, c;
-    sincosf((float)pos * inv_freq[p], &s, &c);
-    const float* src = u < heads ? x + (size_t)u * (dim + rot) + dim : lat + rank;
-    const float a = src[p], b = src[p + half];
-    const T ra = from_f32<T>(a * c - b * s), rb = from_f32<T>(b * c + a * s);
-    if (u < heads) {
-      T* d = qr + (size_t)u * pitch + dim;
-      d[p] = ra, d[p + half] = rb;
-    } else {
-      kvr[rank + p] = ra, kvr[rank + p + half] = rb;
-      if (kdst != nullptr) kdst[rank + p] = ra, kdst[rank + p + half] = rb;
+  const float2* tab = p.table != nullptr ? pdl_fresh(p.table) + (size_t)t * half : nullptr;
+  auto turn = [&](int i) {
+    float2 cs;
+    if (tab != nullptr) cs = tab[i];
+    else sincosf((float)pos * p.inv_freq[i], &cs.y, &cs.x);
+    cs.x *= p.magnitude, cs.y *= p.magnitude;
+    return cs;
+  };
+  auto first_of = [&](int i) { return p.adjacent ? 2 * i : i; };
+  auto second_of = [&](int i) { return p.adjacent ? 2 * i + 1 : i + half; };
+  if (p.kv_src != nullptr) {
+    const float* lat = p.kv_src + (size_t)t * p.kv_ld;
+    T* kvr = p.kv + (size_t)t * p.kv_stride;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < rank; i += blockDim.x) ss += lat[i] * lat[i];
+    ss = block_sum(ss, scratch);
+    const float inv = rsqrtf(ss / (float)rank + p.eps);
+    for (int i = threadIdx.x; i < rank; i += blockDim.x) {
+      const T v = from_f32<T>(lat[i] * inv * p.norm_w[i]);
+      kvr[i] = v;
+      if (kdst != nullptr) kdst[i] = v;
+    }
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+      const float2 cs = turn(i);
+      const int e0 = first_of(i), e1 = second_of(i);
+      const float a = lat[rank + e0], b = lat[rank + e1];
+      const T ra = from_f32<T>(a * cs.x - b * cs.y), rb = from_f32<T>(b * cs.x + a * cs.y);
+      kvr[rank + e0] = ra, kvr[rank + e1] = rb;
+      if (kdst != nullptr) kdst[rank + e0] = ra, kdst[rank + e1] = rb;
     }
   }
-  for (int i = threadIdx.x; i < heads * dim; i += blockDim.x) {
-    const int u = i / dim, e = i - u * dim;
-    qr[(size_t)u * pitch + e] = from_f32<T>(x[(size_t)u * (dim + rot) + e]);
+  if (p.side_src != nullptr) {
+    const float* src = p.side_src + (size_t)t * p.side_ld;
+    T* dst = p.side + (size_t)t * p.side_stride;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < p.side_n; i += blockDim.x) ss += src[i] * src[i];
+    ss = block_sum(ss, scratch);
+    const float inv = rsqrtf(ss / (float)p.side_n + p.eps);
+    for (int i = threadIdx.x; i < p.side_n; i += blockDim.x) dst[i] = from_f32<T>(src[i] * inv * p.side_w[i]);
   }
-  const int pad = pitch - dim - rot;
-  for (int i = threadIdx.x; i < heads * pad; i += blockDim.x) {
+  if (p.q_src == nullptr) return;
+  const float* x = p.q_src + (size_t)t * p.q_ld;
+  auto q_at = [&](int i) {
+    float s = x[i];
+    for (int u = 1; u < p.q_parts; ++u) s += x[(size_t)u * p.q_part_stride + i];
+    return s;
+  };
+  T* qr = p.q + (size_t)t * p.q_stride;
+  for (int i = threadIdx.x; i < p.heads * half; i += blockDim.x) {
+    const int u = i / half, e = i - u * half;
+    const float2 cs = turn(e);
+    const int e0 = first_of(e), e1 = second_of(e);
+    const float a = q_at(u * (dim + rot) + dim + e0), b = q_at(u * (dim + rot) + dim + e1);
+    T* d = qr + (size_t)u * p.pitch + dim;
+    d[e0] = from_f32<T>(a * cs.x - b * cs.y), d[e1] = from_f32<T>(b * cs.x + a * cs.y);
+  }
+  for (int i = threadIdx.x; i < p.heads * dim; i += blockDim.x) {
+    const int u = i / dim, e = i - u * dim;
+    qr[(size_t)u * p.pitch + e] = from_f32<T>(q_at(u * (dim + rot) + e));
+  }
+  const int pad = p.pitch - dim - rot;
+  for (int i = threadIdx.x; i < p.heads * pad; i += blockDim.x) {
     const int u = i / pad, e = i - u * pad;
-    qr[(size_t)u * pitch + dim + rot + e] = from_f32<T>(0.f);
+    qr[(size_t)u * p.pitch + dim + rot + e] = from_f32<T>(0.f);
   }
 }
 
-AF_EXPORT int af_latent_prep(void* q, long long q_stride, void* kv, long long kv_stride, int dtype, const float* proj,
-                             long long ld, const float* norm_w, float eps, const int* positions,
-                             const int* seq_of_token, const int* slots, const int* len_after, const float* inv_freq,
-                             int n_tokens, int heads, int dim, int rot, int rank, int pitch, void* kcache,
-                             const int* page_table, int max_pages, int ring_rows, cudaStream_t stream) {
+AF_EXPORT int af_latent_prep(void* q, long long q_stride, const float* q_src, long long q_ld, int q_parts,
+                             long long q_part_stride, void* kv, long long kv_stride, const float* kv_src, long long kv_ld,
+                             const float* norm_w, void* side, long long side_stride, const float* side_src,
+                             long long side_ld, const float* side_w, int side_n, int dtype, float eps,
+                             const int* positions, const int* seq_of_token, const int* slots, const int* len_after,
+                             const float* inv_freq, const float* table, int adjacent, float magnitude, int n_tokens,
+                             int heads, int dim, int rot, int rank, int pitch, void* kcache, const int* page_table,
+                             int max_pages, int ring_rows, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
-  AF_REQUIRE(n_tokens > 0 && heads > 0 && dim >= 0 && rot >= 0 && rot % 2 == 0 && rank > 0 && dim + rot > 0 &&
-             pitch >= dim + rot, "af_latent_prep: bad sizes");
+  AF_REQUIRE(n_tokens > 0 && dim >= 0 && rot >= 0 && rot % 2 == 0, "af_latent_prep: bad sizes");
+  AF_REQUIRE(q_src == nullptr || (q != nullptr && heads > 0 && dim + rot > 0 && pitch >= dim + rot && q_parts >= 1),
+             "af_latent_prep: bad sizes of the query heads");
+  AF_REQUIRE(kv_src == nullptr || (kv != nullptr && rank > 0 && norm_w != nullptr), "af_latent_prep: bad sizes of the latent");
+  AF_REQUIRE(side_src == nullptr || (side != nullptr && side_n > 0 && side_w != nullptr),
+             "af_latent_prep: bad sizes of the second latent");
   AF_REQUIRE(ring_rows % AF_PAGE == 0, "af_latent_prep: ring rows %d not whole pages", ring_rows);
-  AF_DISPATCH_DTYPE(dtype, T,
-                    af_launch(latent_prep_kernel<T>, dim3(n_tokens), dim3(256), 0, stream, (T*)q, q_stride, (T*)kv,
-                              kv_stride, proj, ld, norm_w, eps, positions, seq_of_token, slots, len_after, inv_freq,
-                              heads, dim, rot, rank, pitch, (T*)kcache, page_table, max_pages, ring_rows));
+#define LATENT_PREP(T)                                                                                                  \
+  do {                                                                                                                  \
+    LatentPrepArgs<T> p;                                                                                                \
+    p.q = (T*)q, p.q_stride = q_stride, p.q_src = q_src, p.q_ld = q_ld, p.q_parts = q_parts;                            \
+    p.q_part_stride = q_part_stride, p.heads = heads, p.dim = dim, p.rot = rot, p.pitch = pitch;                        \
+    p.kv = (T*)kv, p.kv_stride = kv_stride, p.kv_src = kv_src, p.kv_ld = kv_ld, p.norm_w = norm_w, p.rank = rank;       \
+    p.side = (T*)side, p.side_stride = side_stride, p.side_src = side_src, p.side_ld = side_ld, p.side_w = side_w;      \
+    p.side_n = side_n, p.eps = eps, p.magnitude = magnitude, p.adjacent = adjacent, p.inv_freq = inv_freq;              \
+    p.table = (const float2*)table, p.positions = positions, p.seq_of_token = seq_of_token, p.slots = slots;            \
+    p.len_after = len_after, p.kcache = (T*)kcache, p.page_table = page_table, p.max_pages = max_pages;                 \
+    p.ring_rows = ring_rows;                                                                                            \
+    af_launch(latent_prep_kernel<T>, dim3(n_tokens), dim3(256), 0, stream, p);                                          \
+  } while (0)
+  AF_DISPATCH_DTYPE(dtype, T, LATENT_PREP(T));
+#undef LATENT_PREP
   AF_CHECK_LAUNCH("af_latent_prep");
 }
 

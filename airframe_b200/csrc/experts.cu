@@ -213,10 +213,13 @@ AF_EXPORT int af_expert_route(int* ids, float* wts, float* shared_gate, float* s
 
 // ---------------------------------------------------------------- pairs by expert
 
-// One block.  plan: [0] tiles in use; then per tile (expert, first sorted row, rows).  perm[sorted row] = pair.
+// One block a plan.  plan: [0] tiles in use; then per tile (expert, first sorted row, rows).  perm[sorted row] = pair.
+// The experts of pair p come from `ids`, or with `table` (rows of `top` expert numbers, one row a token id) from the
+// token that the pair belongs to: expert = table[tokens[p / top]][p % top].  Block b takes the b-th table of
+// [blocks][vocab][top] and writes the b-th perm [n_pairs] and plan.
 __global__ void __launch_bounds__(1024)
-expert_plan_kernel(int* __restrict__ perm, int* __restrict__ plan, const int* __restrict__ ids, int n_pairs,
-                   int n_experts, int max_tiles, int tile) {
+expert_plan_kernel(int* __restrict__ perm, int* __restrict__ plan, const int* __restrict__ ids,
+                   const int* __restrict__ table, int vocab, int top, int n_pairs, int n_experts, int max_tiles, int tile) {
   pdl_launch_dependents();
   extern __shared__ int sh[];                       // count[E], first[E], cursor[E]
   int* count = sh;
@@ -226,9 +229,21 @@ expert_plan_kernel(int* __restrict__ perm, int* __restrict__ plan, const int* __
   __syncthreads();
   pdl_wait();
   ids = pdl_fresh(ids);
+  perm += (size_t)blockIdx.x * n_pairs;
+  plan += (size_t)blockIdx.x * (1 + 3 * max_tiles);
+  if (table != nullptr) table += (size_t)blockIdx.x * vocab * top;
+  auto expert_of = [&](int p) {
+    if (table == nullptr) return ids[p];
+    const int token = ids[p / top];                 // (with a table `ids` holds the tokens)
+    const bool known = token >= 0 && token < vocab;   // (ids are validated on the host; a bad one has no expert)
+    (void)AF_INDEX_OK(known, token);
+    return known ? table[(size_t)token * top + p % top] : -1;
+  };
   for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
-    const int e = ids[p];
-    if (AF_INDEX_OK(e >= 0 && e < n_experts, e)) atomicAdd(&count[e], 1);
+    const int e = expert_of(p);
+    const bool ok = e >= 0 && e < n_experts;
+    (void)AF_INDEX_OK(ok, e);
+    if (ok) atomicAdd(&count[e], 1);
   }
   __syncthreads();
   if (threadIdx.x == 0) {
@@ -250,7 +265,7 @@ expert_plan_kernel(int* __restrict__ perm, int* __restrict__ plan, const int* __
   }
   __syncthreads();
   for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
-    const int e = ids[p];
+    const int e = expert_of(p);
     if (e >= 0 && e < n_experts) perm[first[e] + atomicAdd(&cursor[e], 1)] = p;
   }
 }
@@ -263,8 +278,24 @@ AF_EXPORT int af_expert_plan(int* perm, int* plan, const int* ids, int n_pairs, 
   AF_REQUIRE(max_tiles >= n_pairs / tile + n_experts || max_tiles >= n_pairs,
              "af_expert_plan: room for %d tiles is too little", max_tiles);
   af_launch(expert_plan_kernel, dim3(1), dim3(1024), (size_t)3 * n_experts * sizeof(int), stream, perm, plan, ids,
-            n_pairs, n_experts, max_tiles, tile);
+            (const int*)nullptr, 0, 1, n_pairs, n_experts, max_tiles, tile);
   AF_CHECK_LAUNCH("af_expert_plan");
+}
+
+// n_tables plans at once, the experts looked up by token: tables [n_tables][vocab][top], perm [n_tables][n_tokens top],
+// plan [n_tables][1 + 3 max_tiles].
+AF_EXPORT int af_expert_table_plan(int* perm, int* plan, const int* tokens, const int* tables, int n_tables, int vocab,
+                                   int top, int n_tokens, int n_experts, int max_tiles, int tile, cudaStream_t stream) {
+  if (n_tokens == 0 || n_tables == 0) return 0;
+  AF_REQUIRE(n_tokens > 0 && n_tables > 0 && vocab > 0 && top > 0 && n_experts > 0 && n_experts <= 4096 && tile > 0,
+             "af_expert_table_plan: bad sizes");
+  AF_REQUIRE((long long)n_tokens * top < (1ll << 31), "af_expert_table_plan: too many pairs");
+  const int n_pairs = n_tokens * top;
+  AF_REQUIRE(max_tiles >= n_pairs / tile + n_experts || max_tiles >= n_pairs,
+             "af_expert_table_plan: room for %d tiles is too little", max_tiles);
+  af_launch(expert_plan_kernel, dim3(n_tables), dim3(n_pairs <= 256 ? 256 : 1024), (size_t)3 * n_experts * sizeof(int), stream, perm, plan,
+            tokens, tables, vocab, top, n_pairs, n_experts, max_tiles, tile);
+  AF_CHECK_LAUNCH("af_expert_table_plan");
 }
 
 // ---------------------------------------------------------------- the tokens' rows in sorted order

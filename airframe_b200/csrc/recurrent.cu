@@ -572,10 +572,45 @@ AF_EXPORT int af_state_scan(int mode, const float* r, long long r_ts, const floa
   }
 }
 
+// ---------------------------------------------------------------- rotated queries and keys of a recurrence
+
+// In place on float rows: in every head of two sections of a row (queries and keys, heads of `dk` elements) the pairs
+// (i, i + n), or (2 i, 2 i + 1) with `adjacent`, i < n, turned by the token's cosines and sines (table [tokens][n],
+// times `magnitude`); the elements from 2 n on stay.  One thread a pair of one head of both sections.
+__global__ void __launch_bounds__(256)
+rotate_rows_kernel(float* __restrict__ q, long long q_ts, float* __restrict__ k, long long k_ts,
+                   const float2* __restrict__ table, float magnitude, int adjacent, int heads, int dk, int n) {
+  pdl_launch_dependents();
+  pdl_wait();
+  table = pdl_fresh(table);
+  const int t = blockIdx.x;
+  float* qr = q + (size_t)t * q_ts;
+  float* kr = k + (size_t)t * k_ts;
+  for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < heads * n; i += gridDim.y * blockDim.x) {
+    const int h = i / n, e = i - h * n;
+    const int e0 = h * dk + (adjacent ? 2 * e : e), e1 = h * dk + (adjacent ? 2 * e + 1 : e + n);
+    const float2 cs = table[(size_t)t * n + e];
+    const float c = cs.x * magnitude, s = cs.y * magnitude;
+    const float qa = qr[e0], qb = qr[e1], ka = kr[e0], kb = kr[e1];
+    qr[e0] = qa * c - qb * s, qr[e1] = qb * c + qa * s;
+    kr[e0] = ka * c - kb * s, kr[e1] = kb * c + ka * s;
+  }
+}
+
+AF_EXPORT int af_rotate_rows(float* q, long long q_ts, float* k, long long k_ts, const float* table, float magnitude,
+                             int adjacent, int n_tokens, int heads, int dk, int n, cudaStream_t stream) {
+  if (n_tokens == 0 || n == 0) return 0;
+  AF_REQUIRE(n_tokens > 0 && heads > 0 && n > 0 && 2 * n <= dk, "af_rotate_rows: %d pairs in heads of %d", n, dk);
+  const int pairs = heads * n;
+  af_launch(rotate_rows_kernel, dim3(n_tokens, (pairs + 1023) / 1024), dim3(pairs >= 256 ? 256 : (pairs + 31) / 32 * 32), 0,
+            stream, q, q_ts, k, k_ts, (const float2*)table, magnitude, adjacent, heads, dk, n);
+  AF_CHECK_LAUNCH("af_rotate_rows");
+}
+
 // ---------------------------------------------------------------- the output of a state mixer
 
 // y[t][i] = o'[t][i] * rsqrt(mean over i's group of o'^2 + eps) * w[i] * sigmoid(gate[t][i]), o' = in_scale * o: a norm
-// over groups of `group` values (a head, or the whole row) with a weight vector (no offset), times a gate (its sigmoid,
+// over groups of `group` values (a head, or the whole row) with a weight vector (no offset; null: none), times a gate (its sigmoid,
 // or with gate_act 1 the gate times its sigmoid).  One block per token.
 template <typename TY>
 __global__ void __launch_bounds__(256)
@@ -587,6 +622,7 @@ gated_group_norm_kernel(TY* __restrict__ y, const float* __restrict__ o, const f
   __shared__ float scratch[33];
   // the gate: its sigmoid, or (gate_act 1) the gate itself times its sigmoid
   auto gated = [&](float g) { const float sg = 1.f / (1.f + expf(-g)); return gate_act ? g * sg : sg; };
+  auto weight = [&](int i) { return w != nullptr ? w[i] : 1.f; };
   const int t = blockIdx.x;
   const float* orow = o + (size_t)t * n;
   const float* grow = gate + (size_t)t * gate_ts;
@@ -597,7 +633,7 @@ gated_group_norm_kernel(TY* __restrict__ y, const float* __restrict__ o, const f
     ss = block_sum(ss, scratch);
     const float inv = rsqrtf(ss / (float)n + eps);
     for (int i = threadIdx.x; i < n; i += blockDim.x)
-      yrow[i] = from_f32<TY>(orow[i] * in_scale * inv * w[i] * gated(grow[i]));
+      yrow[i] = from_f32<TY>(orow[i] * in_scale * inv * weight(i) * gated(grow[i]));
     return;
   }
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
@@ -608,7 +644,7 @@ gated_group_norm_kernel(TY* __restrict__ y, const float* __restrict__ o, const f
     const float inv = rsqrtf(ss / (float)group + eps);
     for (int c = lane; c < group; c += 32) {
       const int i = g * group + c;
-      yrow[i] = from_f32<TY>(orow[i] * in_scale * inv * w[i] * gated(grow[i]));
+      yrow[i] = from_f32<TY>(orow[i] * in_scale * inv * weight(i) * gated(grow[i]));
     }
   }
 }

@@ -12,7 +12,7 @@ from __future__ import annotations
 import torch
 
 from ..config.base import ConfigError, ModelSpec
-from ..parts import BuildContext, build_part
+from ..parts import Block, BuildContext, build_part
 
 
 def _build_layers(spec: ModelSpec, ctx: BuildContext):
@@ -64,6 +64,12 @@ class Model:
     def load(self, weights: dict) -> None:
         for p in self.parts():
             p.load(weights)
+        by_class: dict = {}
+        for p in self.parts():
+            for part in (p, *(p.children() if isinstance(p, Block) else ())):
+                by_class.setdefault(type(part), []).append(part)
+        for cls, parts in by_class.items():
+            cls.link(parts)
         self.loaded = True
 
     @property
@@ -74,11 +80,12 @@ class Model:
     # ------------------------------------------------------------------ cache
 
     def cache_needs(self) -> list:
-        """Per schedule entry: (KVNeed | None, StateNeed | None, cache_from | None)."""
+        """Per schedule entry: (the mixer's KVNeed | None, the mixer's StateNeed | None, cache_from | None, the
+        block's own StateNeed | None)."""
         out = []
         for e in self.spec.schedule:
-            m = self.blocks[e.layer].mixer
-            out.append((m.kv_need(), m.state_need(), e.cache_from))
+            b = self.blocks[e.layer]
+            out.append((b.mixer.kv_need(), b.mixer.state_need(), e.cache_from, b.state_need()))
         return out
 
     # ------------------------------------------------------------------ what a step costs
@@ -128,12 +135,12 @@ class Model:
         for i, e in enumerate(sched):
             blk = self.blocks[e.layer]
             if e.enter is not None:
-                normed = self.junctions[e.enter].forward(x, x0, e.enter_index, batch, then=blk.first_norm(),
-                                                         out_dtype=self.ctx.compute_dtype)
+                normed = self.junctions[e.enter].forward(x, x0, e.enter_index, batch,
+                                                         then=blk.reader(cache.views[i], batch), out_dtype=self.ctx.compute_dtype)
             # the last kernel of a run also makes the next run's first norm, unless a junction rewrites the stream first
             nxt = None
             if i + 1 < len(sched) and sched[i + 1].enter is None:
-                nxt = self.blocks[sched[i + 1].layer].first_norm()
+                nxt = self.blocks[sched[i + 1].layer].reader(cache.views[i + 1], batch)
             normed = blk.forward(x, batch, cache.views[i], normed=normed, next_pre=nxt)
             if probe is not None:
                 probe.after(i, e.layer, self._sum_streams(x) if self.streams > 1 else x, batch)

@@ -920,20 +920,35 @@ def state_scan(mode: str, out, r, k, v, state, batch, heads: int, dk: int, dv: i
                                 _stream()))
 
 
+def rotate_rows(q, k, table, heads: int, dk: int, pairing: str = "half", magnitude: float = 1.0) -> None:
+    """In place on float32 rows q and k [T, heads * dk] (column sections allowed): in every head the pairs (i, i + n), or
+    neighbours, turned by the step's ``table`` (float32 [T, n, 2] of cosines and sines, both times ``magnitude``)."""
+    T = q.shape[0]
+    if tuple(q.shape) != (T, heads * dk) or tuple(k.shape) != (T, heads * dk) or pairing not in PAIRINGS:
+        raise KernelError(f"rotate_rows: q and k [{T}, {heads * dk}]")
+    n = table.shape[1]
+    if tuple(table.shape) != (T, n, 2) or not table.is_contiguous():
+        raise KernelError(f"rotate_rows: a table of cosines and sines [{T}, n, 2]")
+    qp, kp = _f32_rows(q, "q"), _f32_rows(k, "k")
+    _check(_lib().af_rotate_rows(*qp, *kp, _ptr(table, "table", torch.float32), c_float(magnitude), c_int(PAIRINGS[pairing]),
+                                 c_int(T), c_int(heads), c_int(dk), c_int(n), _stream()))
+
+
 GATE_ACTS = {"sigmoid": 0, "silu": 1}
 
 
 def gated_group_norm(y, o, w, gate, group: int, eps: float, gate_act: str = "sigmoid", in_scale: float = 1.0) -> None:
     """y = o' * rsqrt(mean over each group of ``group`` values of o'^2 + eps) * w * act(gate), o' = in_scale * o,
     act the sigmoid or ("silu") the gate times its sigmoid;
-    o float32 [T, n] contiguous, gate float32 rows [T, n] (a column section is fine), w float32 [n]."""
+    o float32 [T, n] contiguous, gate float32 rows [T, n] (a column section is fine), w float32 [n] (None: no weight)."""
     T, n = o.shape
     if o.dtype != torch.float32 or not o.is_contiguous() or tuple(y.shape) != (T, n) or not y.is_contiguous():
         raise KernelError("gated_group_norm: o float32 and y, both contiguous [T, n]")
-    if w.numel() != n or tuple(gate.shape) != (T, n):
+    if (w is not None and w.numel() != n) or tuple(gate.shape) != (T, n):
         raise KernelError("gated_group_norm: weight [n] and gate [T, n]")
     gp, gts = _f32_rows(gate, "gate")
-    _check(_lib().af_gated_group_norm(_ptr(y), c_int(dtype_code(y.dtype)), _ptr(o), _ptr(w, "w", torch.float32), gp, gts,
+    _check(_lib().af_gated_group_norm(_ptr(y), c_int(dtype_code(y.dtype)), _ptr(o),
+                                      _ptr(w, "w", torch.float32, allow_none=True), gp, gts,
                                       c_int(T), c_int(n), c_int(group), c_float(eps), c_int(GATE_ACTS[gate_act]),
                                       c_float(in_scale), _stream()))
 
@@ -1025,34 +1040,64 @@ def attn_prefill_fast_head(size: int) -> int:
     return 0
 
 
-def latent_prep(q, kvrow, proj, batch, heads: int, dim: int, rot: int, rank: int, norm_w, eps: float, inv_freq,
-                kv=None, pitch: int = 0) -> None:
-    """From float32 projection rows [q heads of (dim + rot) | latent of ``rank`` | shared key part of ``rot``]:
-    the q heads with their last ``rot`` elements rotated (pairs i, i + rot / 2) into ``q`` [T, heads pitch]
-    (``pitch`` >= dim + rot, by default that: a head's elements beyond dim + rot are set to zero);
-    the latent over its root mean square (eps inside the root) times ``norm_w`` and the rotated shared key part
-    into ``kvrow`` [T, rank + rot], and, with ``kv`` (the layer's view of its cache: one kv head of rank + rot
-    elements, no value pages), into each token's row of its page."""
-    T = proj.shape[0]
+def latent_prep(batch, heads: int, dim: int, rot: int, rank: int, eps: float, inv_freq, q=None, q_src=None, kvrow=None,
+                kv_src=None, norm_w=None, side=None, side_src=None, side_w=None, kv=None, pitch: int = 0,
+                pairing: str = "half", magnitude: float = 1.0, table=None) -> None:
+    """What latent attention makes of float32 projection rows; each part is done when its source is given:
+
+    ``q_src`` [T, heads (dim + rot)] (or partial sums of it [n, T, ...], added in order): the heads with their last
+    ``rot`` elements rotated into ``q`` [T, heads pitch] (``pitch`` >= dim + rot, by default that: a head's elements
+    beyond dim + rot are set to zero);
+    ``kv_src`` [T, rank + rot]: the latent over its root mean square (eps inside the root) times ``norm_w`` and the
+    rotated shared key part into ``kvrow`` [T, rank + rot], and, with ``kv`` (the layer's view of its cache: one kv
+    head of rank + rot elements, no value pages), into each token's row of its page;
+    ``side_src`` [T, n]: a second latent, normed with ``side_w``, into ``side`` [T, n].
+
+    The rotation: ``pairing``, frequencies ``inv_freq`` or the step's ``table`` (float32 [T, rot / 2, 2]) of cosines and
+    sines, both times ``magnitude``."""
+    T = batch.positions.shape[0]
     pitch = pitch or dim + rot
-    if proj.shape[1] < heads * (dim + rot) + rank + rot or tuple(q.shape) != (T, heads * pitch) \
-            or tuple(kvrow.shape) != (T, rank + rot) or q.dtype != kvrow.dtype:
-        raise KernelError("latent_prep: shapes of the projection, q and kv rows do not fit")
-    if inv_freq.numel() != rot // 2 or norm_w.numel() != rank:
-        raise KernelError("latent_prep: inv_freq holds rot / 2 values, the norm weight rank values")
+    dts = {t.dtype for t in (q, kvrow, side) if t is not None}
+    if len(dts) != 1 or pairing not in PAIRINGS:
+        raise KernelError("latent_prep: outputs of one dtype, a known pairing")
+    dtype = dts.pop()
+    null = (c_void_p(0), c_longlong(0))
+    q_args, kv_args, side_args = (*null, *null, c_int(1), c_longlong(0)), (*null, *null, c_void_p(0)), (*null, *null, c_void_p(0), c_int(0))
+    if q_src is not None:
+        parts, part_stride, rows = 1, 0, q_src
+        if q_src.dim() == 3:
+            parts, part_stride, rows = q_src.shape[0], q_src.stride(0), q_src[0]
+        if tuple(rows.shape) != (T, heads * (dim + rot)) or tuple(q.shape) != (T, heads * pitch):
+            raise KernelError("latent_prep: shapes of the query heads do not fit")
+        sp, sld = _f32_rows(rows, "q_src")
+        q_args = (_ptr(q), c_longlong(_rows(q, "q")), sp, sld, c_int(parts), c_longlong(part_stride))
+    if kv_src is not None:
+        if tuple(kv_src.shape) != (T, rank + rot) or tuple(kvrow.shape) != (T, rank + rot) or norm_w.numel() != rank:
+            raise KernelError("latent_prep: shapes of the latent rows do not fit")
+        sp, sld = _f32_rows(kv_src, "kv_src")
+        kv_args = (_ptr(kvrow), c_longlong(_rows(kvrow, "kvrow")), sp, sld, _ptr(norm_w, "norm_w", torch.float32))
+    if side_src is not None:
+        if side_src.shape != side.shape or side.shape[0] != T or side_w.numel() != side.shape[1]:
+            raise KernelError("latent_prep: shapes of the second latent do not fit")
+        sp, sld = _f32_rows(side_src, "side_src")
+        side_args = (_ptr(side), c_longlong(_rows(side, "side")), sp, sld, _ptr(side_w, "side_w", torch.float32),
+                     c_int(side.shape[1]))
+    if inv_freq.numel() != rot // 2:
+        raise KernelError("latent_prep: inv_freq holds rot / 2 values")
+    if table is not None and (tuple(table.shape) != (T, rot // 2, 2) or table.dtype != torch.float32 or not table.is_contiguous()):
+        raise KernelError(f"latent_prep: a table of cosines and sines [{T}, {rot // 2}, 2]")
     kc = pt = None
     max_pages = ring = 0
     if kv is not None:
         kc, pt, ring = kv.k, kv.page_table, kv.ring_rows
-        if kc.dtype != q.dtype or tuple(kc.shape[1:]) != (1, PAGE, rank + rot) or not kc.is_contiguous():
+        if kc.dtype != dtype or tuple(kc.shape[1:]) != (1, PAGE, rank + rot) or not kc.is_contiguous():
             raise KernelError(f"latent_prep: cache pages must be [pages, 1, {PAGE}, {rank + rot}] of the rows' dtype")
         max_pages = pt.shape[1]
-    pp, ld = _f32_rows(proj, "proj")
     _check(_lib().af_latent_prep(
-        _ptr(q), c_longlong(_rows(q, "q")), _ptr(kvrow), c_longlong(_rows(kvrow, "kvrow")), c_int(dtype_code(q.dtype)),
-        pp, ld, _ptr(norm_w, "norm_w", torch.float32), c_float(eps), _ptr(batch.positions, "positions", torch.int32),
+        *q_args, *kv_args, *side_args, c_int(dtype_code(dtype)), c_float(eps), _ptr(batch.positions, "positions", torch.int32),
         _ptr(batch.seq_of_token, "seq_of_token", torch.int32), _ptr(batch.slots, "slots", torch.int32),
-        _ptr(batch.len_after, "len_after", torch.int32), _ptr(inv_freq, "inv_freq", torch.float32), c_int(T),
+        _ptr(batch.len_after, "len_after", torch.int32), _ptr(inv_freq, "inv_freq", torch.float32),
+        _ptr(table, "table", torch.float32, allow_none=True), c_int(PAIRINGS[pairing]), c_float(magnitude), c_int(T),
         c_int(heads), c_int(dim), c_int(rot), c_int(rank), c_int(pitch), _ptr(kc, allow_none=True),
         _ptr(pt, "page_table", torch.int32, allow_none=True), c_int(max_pages), c_int(ring), _stream()))
 
@@ -1365,6 +1410,22 @@ def expert_plan(perm, plan, ids, n_experts: int, tile: int = EXPERT_TILE) -> Non
                                  c_int(tile), _stream()))
 
 
+def expert_table_plan(perm, plan, tokens, tables, n_experts: int, tile: int = EXPERT_TILE) -> None:
+    """:func:`expert_plan` for layers whose experts are looked up by token id: ``tables`` int32 [n, vocab, top] (every
+    entry a valid expert), perm int32 [n, T * top], plan int32 [n, 1 + 3 * expert_max_tiles], tokens int32 [T]; the plans
+    of all n tables in one kernel."""
+    n, vocab, top = tables.shape
+    T = tokens.shape[0]
+    max_tiles = (plan.shape[1] - 1) // 3
+    if tuple(perm.shape) != (n, T * top) or plan.shape[0] != n or not (perm.is_contiguous() and plan.is_contiguous()
+                                                                     and tables.is_contiguous()):
+        raise KernelError("expert_table_plan: one row of perm and plan a table")
+    i32 = torch.int32
+    _check(_lib().af_expert_table_plan(_ptr(perm, "perm", i32), _ptr(plan, "plan", i32), _ptr(tokens, "tokens", i32),
+                                       _ptr(tables, "tables", i32), c_int(n), c_int(vocab), c_int(top), c_int(T),
+                                       c_int(n_experts), c_int(max_tiles), c_int(tile), _stream()))
+
+
 EXPERT_ACTS = {None: 0, "gelu_erf": 1}
 
 
@@ -1653,3 +1714,75 @@ def diff_join(y, ctx, gate, H: int, G: int, dv: int, pv: int, lam: float, eps: f
 
 
 __all__ = [n for n in dir() if not n.startswith("_")]
+
+
+# ---------------------------------------------------------------- a norm behind the residual sum, the token shift
+
+LAYER_NORM_MAX = 12288     # values a row of these kernels
+
+
+def layer_norm(y, x, w, b, eps: float, rows=None) -> None:
+    """y[r] = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b of row rows[r] (or r) of x (float32 [T, H])."""
+    n, H = y.shape
+    if not (x.is_contiguous() and y.is_contiguous()) or x.shape[1] != H or w.numel() != H or b.numel() != H:
+        raise KernelError("layer_norm: contiguous rows of one size, weight and bias of that size")
+    _check(_lib().af_layer_norm(_ptr(y, "y"), c_int(dtype_code(y.dtype)), _ptr(x, "x", torch.float32),
+                                _ptr(w, "w", torch.float32), _ptr(b, "b", torch.float32),
+                                _ptr(rows, "rows", torch.int32, allow_none=True), c_int(n), c_int(H), c_float(eps), _stream()))
+
+
+def norm_of_sum(x, terms, alpha: float, w, bias, eps: float, gate=None, gate_bias=None, y=None, shifted=None, shift=None,
+                prev=None, slots=None) -> None:
+    """x <- layer_norm(alpha x + g * (sum of scale * term)) in place (float32 [rows, H]; all sums 32-bit): ``terms`` as in
+    :func:`add_scaled_rmsnorm` (at most two, or they are added up first), g = sigmoid(gate + gate_bias) with ``gate``
+    a tensor [rows, H] or float32 partial sums of it, or 1.  ``y``: the new row in y's dtype.  ``shifted`` (rows that are
+    single tokens, one a sequence): the new row plus (prev[slot] - new row) * ``shift`` in its dtype, prev (float32
+    [slots, H]) then holding the new row; rows with slot -1 touch no state."""
+    n, H = x.shape
+    outs = [t for t in (y, shifted) if t is not None]
+    if not x.is_contiguous() or any(tuple(t.shape) != (n, H) or not t.is_contiguous() for t in outs) \
+            or len({t.dtype for t in outs}) > 1:
+        raise KernelError("norm_of_sum: contiguous rows of one size, outputs of one dtype")
+    if w.numel() != H or bias.numel() != H or (gate is not None and (gate_bias is None or gate_bias.numel() != H)):
+        raise KernelError("norm_of_sum: weight, bias and the gate's bias of the row's size")
+    if shifted is not None and (shift is None or shift.numel() != H or prev is None or prev.dtype != torch.float32
+                                or prev.shape[1:] != (H,) or not prev.is_contiguous() or slots.shape[0] != n):
+        raise KernelError("norm_of_sum: a shifted row needs factors [H], float32 state [slots, H] and one slot a row")
+    if not terms:
+        raise KernelError("norm_of_sum: at least one term")
+    if len(terms) > 2:
+        total = torch.zeros(n, H, dtype=torch.float32, device=x.device)
+        add_scaled_rmsnorm(total, terms)
+        terms = [(total, 1.0)]
+    none = (c_void_p(0), c_int(F32), c_int(1))
+    a, sa = terms[0]
+    b, sb = terms[1] if len(terms) > 1 else (None, 0.0)
+    barg = _term_arg(b, n, H, "norm_of_sum") if b is not None else none
+    zarg = _term_arg(gate, n, H, "norm_of_sum") if gate is not None else none
+    f32 = torch.float32
+    _check(_lib().af_norm_of_sum(
+        _ptr(x, "x", f32), *_term_arg(a, n, H, "norm_of_sum"), c_float(sa), *barg, c_float(sb), *zarg,
+        _ptr(gate_bias if gate is not None else None, "gate_bias", f32, allow_none=True), c_float(alpha), _ptr(w, "w", f32),
+        _ptr(bias, "bias", f32), c_float(eps), _ptr(y, "y", allow_none=True), _ptr(shifted, "shifted", allow_none=True),
+        c_int(dtype_code(outs[0].dtype) if outs else F32), _ptr(shift, "shift", f32, allow_none=True),
+        _ptr(prev, "prev", f32, allow_none=True), _ptr(slots, "slots", torch.int32, allow_none=True), c_int(n), c_int(H),
+        _stream()))
+
+
+def token_shift(shifted, x, shift, prev, batch, y=None) -> None:
+    """shifted[t] = x[t] + (before - x[t]) * shift, ``before`` the row in front in the same sequence: of the step, or for
+    a sequence's first row of the step ``prev`` of its slot (float32 [slots, H]; zeros at position 0), which is left
+    holding the sequence's last row.  x float32 [T, H]; ``y``: x in y's dtype."""
+    T, H = x.shape
+    outs = [t for t in (y, shifted) if t is not None]
+    if not x.is_contiguous() or any(tuple(t.shape) != (T, H) or not t.is_contiguous() for t in outs) \
+            or len({t.dtype for t in outs}) > 1 or shift.numel() != H:
+        raise KernelError("token_shift: contiguous rows of one size, outputs of one dtype, factors of the row's size")
+    if prev.dtype != torch.float32 or prev.shape[1:] != (H,) or not prev.is_contiguous():
+        raise KernelError(f"token_shift: state must be contiguous float32 [slots, {H}]")
+    i32 = torch.int32
+    _check(_lib().af_token_shift(_ptr(shifted), _ptr(y, allow_none=True), c_int(dtype_code(shifted.dtype)),
+                                 _ptr(x, "x", torch.float32), _ptr(shift, "shift", torch.float32), _ptr(prev, "prev"),
+                                 _ptr(batch.positions, "positions", i32), _ptr(batch.seq_of_token, "seq_of_token", i32),
+                                 _ptr(batch.seq_starts, "seq_starts", i32), _ptr(batch.slots, "slots", i32), c_int(T), c_int(H),
+                                 _stream()))

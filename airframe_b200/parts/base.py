@@ -117,6 +117,11 @@ class Part:
     def load(self, weights: dict) -> None:
         pass
 
+    @classmethod
+    def link(cls, parts) -> None:
+        """Called once a model is loaded with all its parts of this class: what they can share they may put together
+        (one kernel that serves all layers at once, say)."""
+
     # ---- what a step costs, for measurement (rooflines): every part answers for itself
 
     def decode_bytes(self, lens) -> int:
@@ -272,6 +277,16 @@ class Block(Part):
         """The norm this block applies to x first, or None.  The layer before
         may compute it in its last kernel and pass the result as ``normed``."""
         return None
+
+    def state_need(self) -> Optional[StateNeed]:
+        """What the arrangement itself keeps per sequence and run, beside what its mixer asks for (its view has it as
+        ``block_state``)."""
+        return None
+
+    def reader(self, view, batch):
+        """What a run of this block with the cache view ``view`` reads first in the step ``batch``: something with a
+        ``forward(x, out_dtype)`` that the run before may compute in its last kernel (the first norm, for most blocks)."""
+        return self.first_norm()
 
     def decode_bytes(self, lens) -> int:
         return sum(c.decode_bytes(lens) for c in self.children())

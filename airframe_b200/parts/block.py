@@ -14,13 +14,22 @@ stream itself and the only norms stand behind them (each on the sublayer's outpu
 not on the sum); a layer whose feed-forward is of the kind ``none`` has the first
 half only.  On the 16-bit path the kernel of a residual sum also writes the new
 stream in 16 bits for the sublayer that reads it next.
+``normed_sum``: x <- norm1(alpha x + mixer(x)); x <- norm2(alpha x + ff(x)): the norm is
+taken of the residual sum, so the stream itself is a norm's output; the sublayers read it as it stands.
+Each sublayer's result may be multiplied element by element by sigmoid(W x + b) first, and what the
+mixer reads may be shifted towards the token before, x_t + (x_(t-1) - x_t) * mu, whose row
+is then part of a sequence's state, one for every run of the layer.
 """
 from __future__ import annotations
 
+import torch
+
 from .. import kernels
-from ..config.base import PartSpec
-from .base import Block, build_part, register_part
-from .linear import as_terms
+from ..config.base import ConfigError, PartSpec
+from ..weights.loader import WeightDecl
+from .base import Block, StateNeed, build_part, register_part
+from .linear import PartialSums, as_terms, linear_split
+from .norm import LayerNorm
 
 
 @register_part("block", "sandwich")
@@ -104,3 +113,128 @@ class PostNormBlock(Block):
 
     def first_norm(self):
         return self.reader
+
+
+class ShiftedReader:
+    """What a run of a :class:`NormedSumBlock` reads first: the stream in the compute dtype and, for the mixer, its rows
+    shifted towards the row before (the same tensor where the block shifts nothing)."""
+    graph_safe = True
+
+    def __init__(self, block, view, batch):
+        self.block, self.view, self.batch = block, view, batch
+
+    def forward(self, x, out_dtype, rows=None):
+        blk = self.block
+        y = x if out_dtype == torch.float32 else torch.empty_like(x, dtype=out_dtype)
+        if blk.shift is None:
+            if y is not x:
+                kernels.cast_rows(y, x)
+            return y, y
+        h = torch.empty_like(x, dtype=out_dtype)
+        kernels.token_shift(h, x, blk.shift, self.view.block_state, self.batch, y=y if y is not x else None)
+        return y, h
+
+    def outputs(self, x, out_dtype):
+        """(the arguments that make :func:`kernels.norm_of_sum` write what this reader reads, the tensors it writes),
+        for a step of single tokens (or a block that shifts nothing)."""
+        blk = self.block
+        y = x if out_dtype == torch.float32 else torch.empty_like(x, dtype=out_dtype)
+        args = {} if y is x else {"y": y}
+        if blk.shift is None:
+            return args, (y, y)
+        h = torch.empty_like(x, dtype=out_dtype)
+        args.update(shifted=h, shift=blk.shift, prev=self.view.block_state, slots=self.batch.slots)
+        return args, (y, h)
+
+
+@register_part("block", "normed_sum")
+class NormedSumBlock(Block):
+    """Parameters: ``hidden_size``, ``alpha``; optional ``shift_weight`` (tensor name, [hidden]) and ``gates``: for the
+    mixer and for the feed-forward {``weight`` ([hidden, hidden]), ``bias`` ([hidden])} of tensor names, or None.
+    Norm roles ``mixer_sum`` and ``feed_forward_sum`` (``layer_norm``).  A layer whose feed-forward is of the kind
+    ``none`` has the first half only."""
+    roles = ("mixer_sum", "feed_forward_sum")
+
+    def __init__(self, params, ctx, mixer, feed_forward, norms):
+        if not feed_forward.present:
+            self.roles = ("mixer_sum",)
+        super().__init__(params, ctx, mixer, feed_forward, norms)
+        self.hidden = int(self.param("hidden_size"))
+        self.alpha = float(self.param("alpha"))
+        self.shift_name = self.params.get("shift_weight")
+        halves = 2 if feed_forward.present else 1
+        self.gate_names = [g for g in (self.params.get("gates") or [None, None])][:halves]
+        for n in norms.values():
+            if not isinstance(n, LayerNorm):
+                raise ConfigError("normed_sum: the norms of the sums are of the kind layer_norm")
+        self.shift = None
+        self.gates = [None] * halves
+
+    def state_need(self):
+        return StateNeed((self.hidden,)) if self.shift_name else None
+
+    def weight_decls(self):
+        h, decls = self.hidden, super().weight_decls()
+        if self.shift_name:
+            decls.append(WeightDecl(self.shift_name, (h,), "blend"))
+        for g in self.gate_names:
+            if g is not None:
+                decls += [WeightDecl(g["weight"], (h, h)), WeightDecl(g["bias"], (h,), "norm")]
+        return decls
+
+    def load(self, weights):
+        super().load(weights)
+        if self.shift_name:
+            self.shift = weights[self.shift_name].to(torch.float32).contiguous()
+        for q, g in enumerate(self.gate_names):
+            if g is not None:
+                self.gates[q] = (weights[g["weight"]].to(self.ctx.compute_dtype).contiguous(),
+                                 weights[g["bias"]].to(torch.float32).contiguous())
+
+    def _gate_numel(self) -> int:
+        return sum(self.hidden * self.hidden for g in self.gate_names if g is not None)
+
+    def decode_bytes(self, lens) -> int:
+        state = len(lens) * 2 * 4 * self.hidden if self.shift_name else 0
+        el = 4 if self.ctx.compute_dtype == torch.float32 else 2
+        return super().decode_bytes(lens) + self._gate_numel() * el + state
+
+    def prefill_flops(self, lens) -> int:
+        return super().prefill_flops(lens) + 2 * sum(lens) * self._gate_numel()
+
+    def first_norm(self):
+        raise ConfigError("normed_sum: what a run reads first depends on its state (see Block.reader)")
+
+    def reader(self, view, batch):
+        return ShiftedReader(self, view, batch)
+
+    def _gate(self, which: int, y):
+        """The arguments that put this sublayer's gate into the kernel of its residual sum."""
+        if self.gates[which] is None:
+            return {}
+        w, b = self.gates[which]
+        z = linear_split(y, w, wide=True)
+        return {"gate": z.parts if isinstance(z, PartialSums) else z, "gate_bias": b}
+
+    def forward(self, x, batch, view, normed=None, next_pre=None):
+        dt = self.ctx.compute_dtype
+        y, h = normed if normed is not None else ShiftedReader(self, view, batch).forward(x, dt)
+        gate = self._gate(0, y)
+        a = self.mixer.forward(h, batch, view)
+        if not self.feed_forward.present:
+            return self._close(self.norms["mixer_sum"], x, a, gate, batch, next_pre)
+        y = x if dt == torch.float32 else torch.empty_like(x, dtype=dt)
+        self.norms["mixer_sum"].of_sum(x, a, self.alpha, y=None if y is x else y, **gate)
+        gate = self._gate(1, y)
+        return self._close(self.norms["feed_forward_sum"], x, self.feed_forward.forward(y, batch), gate, batch, next_pre)
+
+    def _close(self, norm, x, a, gate, batch, next_pre):
+        """The layer's last residual sum; returns what ``next_pre`` reads of the new stream."""
+        dt = self.ctx.compute_dtype
+        if isinstance(next_pre, ShiftedReader) and (not batch.is_prefill or next_pre.block.shift is None):
+            args, out = next_pre.outputs(x, dt)
+            norm.of_sum(x, a, self.alpha, **gate, **args)
+            return out
+        # a prompt: a row's shift wants its neighbour's new row, which another block of the kernel makes
+        norm.of_sum(x, a, self.alpha, **gate)
+        return None if next_pre is None else next_pre.forward(x, dt)

@@ -22,6 +22,10 @@ divide the chosen scores by their sum and multiply them by a constant.  An exper
 may be of one matrix and an activation, E(h) = W_down gelu(W_up h) with the exact
 (erf) GELU (``expert`` = "gelu_erf"); its weight then multiplies the expert's
 *output* (it is applied behind the activation, in front of the linear down product).
+
+There may be no router at all: a table of integers then names the ``top`` experts of every token id, each with the
+weight 1 / top on its output, which the residual sum applies.  Which experts a step's tokens use is then known before its
+first layer runs: the pairs of all such layers are sorted by one kernel, at the first of them.
 """
 from __future__ import annotations
 
@@ -99,7 +103,9 @@ class RoutedExperts(FeedForward):
     """Parameters: ``hidden_size``, ``intermediate_size``, ``num_experts``, ``top``, ``limit``,
     ``router_weight`` ([experts, hidden]) and ``expert_weights``: a pattern with ``{e}`` for the expert's number
     and ``{role}`` for gate / up / down; optional ``shared``: {``intermediate_size``, ``limit``,
-    ``gate_weight``, ``up_weight``, ``down_weight``, ``mix_weight`` ([1, hidden])}.  Optional ``expert``:
+    ``gate_weight``, ``up_weight``, ``down_weight``, optional ``mix_weight`` ([1, hidden]; without it the shared expert is
+    added as it is)}.  Instead of ``router_weight``: ``table_weight`` (tensor name, int32 [``vocab_size``, top]) and
+    ``vocab_size``.  Optional ``expert``:
     "clamped_glu" (the default, with ``limit``) or "gelu_erf" (up and down only; the weight on the output; no
     ``limit``).  Optional ``router``: {``correction_weight`` (tensor name, [experts]), ``groups``: {``count``,
     ``keep``}, ``normalise`` (bool), ``scale``}.  The result is a sum of 32-bit terms that the residual kernel takes."""
@@ -128,21 +134,33 @@ class RoutedExperts(FeedForward):
             raise ConfigError(f"routed_experts: the kept groups hold fewer than the {self.top} experts a token uses")
         if not 1 <= self.top <= self.n_experts:
             raise ConfigError(f"routed_experts: {self.top} of {self.n_experts} experts")
-        self.router_name = self.param("router_weight")
+        self.table_name = self.params.get("table_weight")
+        self.router_name = None if self.table_name else self.param("router_weight")
+        self.vocab = int(self.param("vocab_size")) if self.table_name else 0
+        if self.table_name and (ro or not self.gated):
+            raise ConfigError("routed_experts: experts chosen by a table have no router and are of the kind clamped_glu")
+        self.table = self.tables = None      # this layer's table; those of all layers that share a plan
+        self.table_index = 0
         self.pattern = self.param("expert_weights")
         self.shared = self.params.get("shared")
         if self.shared is not None:
-            missing = [k for k in ("intermediate_size", "limit", "gate_weight", "up_weight", "down_weight", "mix_weight")
+            missing = [k for k in ("intermediate_size", "limit", "gate_weight", "up_weight", "down_weight")
                        if k not in self.shared]
             if missing:
                 raise ConfigError(f"routed_experts: 'shared' needs {missing}")
+        self.mixed = self.shared is not None and bool(self.shared.get("mix_weight"))
+        if self.mixed and self.table_name:
+            raise ConfigError("routed_experts: a shared expert's 'mix_weight' rides with the router, which a table replaces")
 
     def _name(self, e: int, role: str) -> str:
         return self.pattern.format(e=e, role=role)
 
     def weight_decls(self):
         h, f = self.hidden, self.inter
-        decls = [WeightDecl(self.router_name, (self.n_experts, h))]
+        if self.table_name:
+            decls = [WeightDecl(self.table_name, (self.vocab, self.top), "choice_table", below=self.n_experts)]
+        else:
+            decls = [WeightDecl(self.router_name, (self.n_experts, h))]
         if self.correction_name:
             decls.append(WeightDecl(self.correction_name, (self.n_experts,), "norm"))
         for e in range(self.n_experts):
@@ -152,7 +170,9 @@ class RoutedExperts(FeedForward):
         if self.shared is not None:
             sf, sh = int(self.shared["intermediate_size"]), self.shared
             decls += [WeightDecl(sh["gate_weight"], (sf, h)), WeightDecl(sh["up_weight"], (sf, h)),
-                      WeightDecl(sh["down_weight"], (h, sf)), WeightDecl(sh["mix_weight"], (1, h))]
+                      WeightDecl(sh["down_weight"], (h, sf))]
+            if self.mixed:
+                decls.append(WeightDecl(sh["mix_weight"], (1, h)))
         return decls
 
     def load(self, weights):
@@ -164,48 +184,86 @@ class RoutedExperts(FeedForward):
                            if self.correction_name else None)
         self.w_up = torch.stack([weights[self._name(e, "up")] for e in E]).to(dt).contiguous()
         self.w_down = torch.stack([weights[self._name(e, "down")] for e in E]).to(dt).contiguous()
-        rows = [weights[self.router_name]]
+        rows = [] if self.table_name else [weights[self.router_name]]
+        if self.mixed:
+            rows.append(weights[self.shared["mix_weight"]].reshape(1, self.hidden))       # the shared expert's gate rides with the router
         if self.shared is not None:
             sh = self.shared
-            rows.append(weights[sh["mix_weight"]].reshape(1, self.hidden))       # the shared expert's gate rides with the router
             self.s_gate = weights[sh["gate_weight"]].to(dt).unsqueeze(0).contiguous()
             self.s_up = weights[sh["up_weight"]].to(dt).unsqueeze(0).contiguous()
             self.s_down = weights[sh["down_weight"]].to(dt).unsqueeze(0).contiguous()
-        self.router = torch.cat(rows, dim=0).to(torch.float32).contiguous()      # (router logits are 32-bit)
+        self.router = torch.cat(rows, dim=0).to(torch.float32).contiguous() if rows else None     # (router logits are 32-bit)
+        if self.table_name:
+            self.table = weights[self.table_name].to(torch.int32).contiguous()
+            if not 0 <= int(self.table.min()) <= int(self.table.max()) < self.n_experts:
+                raise ConfigError(f"routed_experts: {self.table_name} names an expert outside 0 .. {self.n_experts - 1}")
+            self.tables = self.table.unsqueeze(0)
+
+    @classmethod
+    def link(cls, parts) -> None:
+        groups: dict = {}
+        for p in parts:
+            if p.table is not None:
+                groups.setdefault((p.n_experts, p.top, p.vocab), []).append(p)
+        for same in groups.values():
+            tables = torch.stack([p.table for p in same]).contiguous()
+            for i, p in enumerate(same):
+                p.tables, p.table_index, p.table = tables, i, tables[i]
 
     def _el(self) -> int:
         return 4 if self.ctx.compute_dtype == torch.float32 else 2
+
+    def _router_numel(self) -> int:
+        return self.router.numel() if self.router is not None else 0
 
     def decode_bytes(self, lens) -> int:
         # the experts whose matrices are read: the expected number under a router that chooses evenly
         used = self.n_experts * (1.0 - (1.0 - self.top / self.n_experts) ** len(lens))
         mats = 3 if self.gated else 2
-        total = int(mats * used * self.hidden * self.inter * self._el()) + 4 * self.router.numel()
+        total = int(mats * used * self.hidden * self.inter * self._el()) + 4 * self._router_numel()
         if self.shared is not None:
             total += 3 * self.hidden * int(self.shared["intermediate_size"]) * self._el()
         return total
 
     def prefill_flops(self, lens) -> int:
-        per_token = (3 if self.gated else 2) * self.hidden * self.inter * self.top + self.router.numel()
+        per_token = (3 if self.gated else 2) * self.hidden * self.inter * self.top + self._router_numel()
         if self.shared is not None:
             per_token += 3 * self.hidden * int(self.shared["intermediate_size"])
         return 2 * sum(lens) * per_token
 
-    def forward(self, x, batch):
-        T, top, dev = x.shape[0], self.top, x.device
-        ids = torch.empty(T, top, dtype=torch.int32, device=dev)
+    def _plan(self, x, batch, tile: int):
+        """(perm, plan, weights of the pairs or None, the shared expert's factor or None): the step's (token, choice)
+        pairs sorted by expert."""
+        T, top, dev, i32 = x.shape[0], self.top, x.device, torch.int32
+        cells = 1 + 3 * kernels.expert_max_tiles(T * top, self.n_experts, tile)
+        if self.table is not None:       # known from the tokens: the plans of all layers that choose alike, made once a step
+            key = ("expert_plans", self.tables.data_ptr(), tile)
+            if key not in batch.aux:
+                n = self.tables.shape[0]
+                perms = torch.empty(n, T * top, dtype=i32, device=dev)
+                plans = torch.empty(n, cells, dtype=i32, device=dev)
+                kernels.expert_table_plan(perms, plans, batch.tokens, self.tables, self.n_experts, tile)
+                batch.aux[key] = (perms, plans)
+            perms, plans = batch.aux[key]
+            return perms[self.table_index], plans[self.table_index], None, None
+        ids = torch.empty(T, top, dtype=i32, device=dev)
         wts = torch.empty(T, top, dtype=torch.float32, device=dev)
-        mix = torch.empty(T, dtype=torch.float32, device=dev) if self.shared is not None else None
+        mix = torch.empty(T, dtype=torch.float32, device=dev) if self.mixed else None
         kernels.expert_route(ids, wts, mix, x, self.router, self.n_experts, correction=self.correction,
                              groups=self.groups, keep=self.keep, normalise=self.normalise, out_scale=self.route_scale)
+        perm = torch.empty(T * top, dtype=i32, device=dev)
+        plan = torch.empty(cells, dtype=i32, device=dev)
+        kernels.expert_plan(perm, plan, ids, self.n_experts, tile)
+        return perm, plan, wts, mix
+
+    def forward(self, x, batch):
+        T, top, dev = x.shape[0], self.top, x.device
         # bfloat16 with sizes the tensor-core products take: the rows in sorted order, then grouped products;
         # else the products on the CUDA cores (32-bit, or odd sizes), which fetch their rows themselves
         fast = (kernels.expert_rows_tc_supported(x, self.w_up) and self.inter % 8 == 0)
         act = None if self.gated else "gelu_erf"
         tile = kernels.expert_tc_tile(T * top, self.n_experts) if fast else kernels.EXPERT_TILE
-        perm = torch.empty(T * top, dtype=torch.int32, device=dev)
-        plan = torch.empty(1 + 3 * kernels.expert_max_tiles(T * top, self.n_experts, tile), dtype=torch.int32, device=dev)
-        kernels.expert_plan(perm, plan, ids, self.n_experts, tile)
+        perm, plan, wts, mix = self._plan(x, batch, tile)
         mid = torch.empty(T * top, self.inter, dtype=x.dtype, device=dev)
         out = torch.empty(top, T, self.hidden, dtype=torch.float32, device=dev)
         if fast:
@@ -225,7 +283,7 @@ class RoutedExperts(FeedForward):
             else:
                 kernels.expert_rows(mid, x, self.w_up, perm=perm, plan=plan, pair_weight=wts, n_tokens=T, top=top, act=act)
             kernels.expert_rows(out, mid, self.w_down, perm=perm, plan=plan, n_tokens=T, top=top)
-        terms = [(PartialSums(out), 1.0)]
+        terms = [(PartialSums(out), 1.0 / top if self.table is not None else 1.0)]
         if self.shared is not None:
             sf = int(self.shared["intermediate_size"])
             smid = torch.empty(T, sf, dtype=x.dtype, device=dev)

@@ -3,6 +3,8 @@
 ``rms_norm``: y = x * rsqrt(mean(x^2) + eps) * (offset + w).
 ``tanh_norm``: y = tanh(alpha x) w + b with a scalar alpha: no mean and no
 variance, so it is elementwise and a row needs no reduction.
+``layer_norm``: y = (x - mean) / sqrt(variance + eps) * w + b, the variance the mean of
+the squared deviations.
 ``as_is``: y = x in the compute dtype: what a sublayer is given that reads the
 stream itself (a norm only behind it); a residual kernel writes it beside the sum.
 
@@ -16,6 +18,7 @@ from __future__ import annotations
 import torch
 
 from .. import kernels
+from ..config.base import ConfigError
 from ..weights.loader import WeightDecl
 from .base import Norm, register_part
 from .linear import PartialSums, as_terms
@@ -139,6 +142,49 @@ class TanhNorm(Norm):
                               b_next=then.b if then is not None else None,
                               alpha_next=then.alpha if then is not None else 0.0)
         return y
+
+
+@register_part("norm", "layer_norm")
+class LayerNorm(Norm):
+    """Centred, divided by the standard deviation, times a weight, plus a bias.  Parameters: ``weight``, ``bias`` (tensor
+    names), ``size``, ``eps``.  A block whose norm stands behind the residual sum asks :meth:`of_sum`."""
+    graph_safe = True
+
+    def __init__(self, params, ctx):
+        super().__init__(params, ctx)
+        self.names = (self.param("weight"), self.param("bias"))
+        self.size = int(self.param("size"))
+        self.eps = float(self.param("eps"))
+        if self.size > kernels.LAYER_NORM_MAX:
+            raise ConfigError(f"layer_norm: rows of up to {kernels.LAYER_NORM_MAX} values, got {self.size}")
+        self.w = self.b = None
+
+    def weight_decls(self):
+        w, b = self.names
+        return [WeightDecl(w, (self.size,), "gain"), WeightDecl(b, (self.size,), "norm")]
+
+    def load(self, weights):
+        self.w, self.b = (weights[n].to(torch.float32).contiguous() for n in self.names)
+
+    def decode_bytes(self, lens) -> int:
+        return 8 * self.size
+
+    def forward(self, x, out_dtype, rows=None):
+        n = x.shape[0] if rows is None else rows.shape[0]
+        y = torch.empty(n, self.size, dtype=out_dtype, device=x.device)
+        kernels.layer_norm(y, x, self.w, self.b, self.eps, rows)
+        return y
+
+    def add_normed(self, x, a, then=None, out_dtype=None):
+        y = torch.zeros_like(x)
+        kernels.add_scaled_rmsnorm(y, as_terms(a))
+        kernels.add_scaled_rmsnorm(x, [(self.forward(y, torch.float32), 1.0)])
+        return None if then is None else then.forward(x, out_dtype)
+
+    def of_sum(self, x, a, alpha: float, **outputs) -> None:
+        """x <- this norm of alpha x + ``a`` (a tensor, partial sums or a weighted sum of them), in place; ``outputs``: a
+        gate on ``a`` and what else the kernel writes (:func:`kernels.norm_of_sum`)."""
+        kernels.norm_of_sum(x, as_terms(a), alpha, self.w, self.b, self.eps, **outputs)
 
 
 @register_part("norm", "as_is")

@@ -17,6 +17,10 @@ weight vector (no offset), times sigmoid(Wg h), then the output projection.
 q, k, v = silu of their projections, S <- decay_h S + k v^T, o = S^T q; the heads
 together are RMS-normed with a weight vector (no offset), times sigmoid(Wg h), then projected.
 
+``retention``: linear attention with a fixed decay per head and rotated queries and
+keys: q, k turned by their positions, S <- decay_h S + k v^T, o = key_scale S^T q; each
+head's o is divided by its root mean square, times silu(Wg h), then projected.
+
 ``mingru``: a gated recurrence over a vector: z = sigmoid(Wz h + bz),
 c = Wx h + bx, candidate = c + 1/2 where c >= 0 and sigmoid(c) below,
 S <- (1 - z) S + z * candidate, output Wo (S * silu(Wg h)).
@@ -40,8 +44,9 @@ import torch
 from .. import kernels
 from ..config.base import ConfigError
 from ..weights.loader import WeightDecl
-from .base import Mixer, StateNeed, register_part
+from .base import Mixer, StateNeed, build_part, register_part
 from .linear import linear, linear_split
+from .rope import Rope
 
 
 def _el(ctx) -> int:
@@ -202,6 +207,71 @@ class LightningAttention(_StateMixer):
                            decay=self.decay, silu=True)
         y = torch.empty(T, nv, dtype=x.dtype, device=x.device)
         kernels.gated_group_norm(y, o, self.norm_w, proj[:, off["g"]: off["g"] + nv], nv, self.eps)
+        return linear_split(y, self.w_o, wide=self.wide)
+
+
+@register_part("mixer", "retention")
+class Retention(_StateMixer):
+    """Parameters: ``hidden_size``, ``num_heads``, ``head_dim`` (queries and keys), ``value_dim``, ``decay`` (one factor per
+    head), ``eps`` (of the heads' norm, which has no weight), ``position`` (a ``rope`` PartSpec), ``weights``: tensor
+    names for ``q, k, v, g, o``; optional ``key_scale`` (default head_dim^-1/2; every output is linear in the keys, so it
+    is applied to them) and ``gate`` ("silu", the default, or "sigmoid")."""
+    ROLES = ("q", "k", "v", "g", "o")
+
+    def __init__(self, params, ctx):
+        super().__init__(params, ctx)
+        self.hidden = int(self.param("hidden_size"))
+        self.heads = int(self.param("num_heads"))
+        self.dk = int(self.param("head_dim"))
+        self.dv = int(self.param("value_dim"))
+        self.eps = float(self.param("eps"))
+        decay = self.param("decay")
+        if not isinstance(decay, (list, tuple)) or len(decay) != self.heads:
+            raise ConfigError(f"retention: 'decay' must list one factor for each of the {self.heads} heads")
+        self.decay_host = torch.tensor([float(d) for d in decay], dtype=torch.float64).to(torch.float32)
+        self.key_scale = float(self.params.get("key_scale", self.dk ** -0.5))
+        self.gate = self.params.get("gate", "silu")
+        if self.gate not in kernels.GATE_ACTS:
+            raise ConfigError(f"retention: unknown gate '{self.gate}' (known: {sorted(kernels.GATE_ACTS)})")
+        self.position = build_part("position", self.param("position"), ctx)
+        if not isinstance(self.position, Rope) or self.position.rotary_dim > self.dk:
+            raise ConfigError("retention: the position encoding is a rotation over at most head_dim elements")
+        self.names = self._names(self.ROLES)
+
+    def state_need(self):
+        return StateNeed((self.heads, self.dv, self.dk), "float32")      # [head][value column][key channel]
+
+    def weight_decls(self):
+        nk, nv, h, nm = self.heads * self.dk, self.heads * self.dv, self.hidden, self.names
+        return [WeightDecl(nm["q"], (nk, h)), WeightDecl(nm["k"], (nk, h)), WeightDecl(nm["v"], (nv, h)),
+                WeightDecl(nm["g"], (nv, h)), WeightDecl(nm["o"], (h, nv))]
+
+    def load(self, weights):
+        self.w_in, self.off = self._pack(weights, ("q", "k", "v", "g"))
+        self.w_o = weights[self.names["o"]].to(self.ctx.compute_dtype).contiguous()
+        self.decay = self.decay_host.to(self.ctx.device)
+        self.position.load(weights)
+
+    def decode_bytes(self, lens) -> int:
+        return ((self.w_in.numel() + self.w_o.numel()) * _el(self.ctx)
+                + len(lens) * 2 * 4 * self.heads * self.dk * self.dv)      # the state, read and written
+
+    def prefill_flops(self, lens) -> int:
+        T = sum(lens)
+        return 2 * T * (self.w_in.numel() + self.w_o.numel()) + T * self.heads * 4 * self.dk * self.dv
+
+    def forward(self, x, batch, view):
+        T, off, pos = x.shape[0], self.off, self.position
+        nk, nv = self.heads * self.dk, self.heads * self.dv
+        proj = linear(x, self.w_in, out_dtype=torch.float32)
+        q, k, v = (proj[:, off[n]: off[n] + w] for n, w in (("q", nk), ("k", nk), ("v", nv)))
+        if pos.rotary_dim:
+            kernels.rotate_rows(q, k, pos.step_table(batch), self.heads, self.dk, pairing=pos.pairing, magnitude=pos.magnitude)
+        o = torch.empty(T, nv, dtype=torch.float32, device=x.device)
+        kernels.state_scan("decay", o, q, k, v, view.state, batch, self.heads, self.dk, self.dv, decay=self.decay)
+        y = torch.empty(T, nv, dtype=x.dtype, device=x.device)
+        kernels.gated_group_norm(y, o, None, proj[:, off["g"]: off["g"] + nv], self.dv, self.eps, gate_act=self.gate,
+                                 in_scale=self.key_scale)
         return linear_split(y, self.w_o, wide=self.wide)
 
 

@@ -102,6 +102,11 @@ class Rope(PositionEncoding):
             batch.aux[key] = kernels.rope_table_precise(batch.positions, self.inv_freq64)
         return batch.aux[key]
 
+    def step_table(self, batch):
+        """float32 [T, rotary_dim / 2, 2] of (cos, sin) for the step's tokens, made once per pass for all layers that rotate
+        alike (from 64-bit angles with ``precise_angles``)."""
+        return self.precise_table(batch) if self.precise else self.rotary_table(batch, self.rotary_dim)
+
     def rotates_half_pairs(self, hd):
         return self.pairing == "half" and self.rotary_dim == hd and self.magnitude == 1.0
 

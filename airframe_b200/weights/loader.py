@@ -25,13 +25,14 @@ from .safetensors_io import SafetensorsError, SafetensorsFile
 @dataclass
 class WeightDecl:
     """A tensor that a part needs.  ``kind`` tells the random-weights mode how
-    to fill it: ``matrix`` and ``table`` N(0, 0.02), ``norm`` N(0, 0.1), ``gain`` N(1, 0.1), ``mixing`` identity + N(0, 0.1), ``share`` N(1, 0.1) / n,
-    ``int_table`` integers.  A ``None`` in ``shape`` stands for a size that only
+    to fill it: ``matrix`` and ``table`` N(0, 0.02), ``norm`` N(0, 0.1), ``gain`` N(1, 0.1), ``mixing`` identity + N(0, 0.1), ``share`` N(1, 0.1) / n, ``blend`` N(0.5, 0.1),
+    ``int_table`` integers, ``choice_table`` rows of distinct integers below ``below``.  A ``None`` in ``shape`` stands for a size that only
     the stored tensor gives (the part reads it when it loads)."""
     name: str
     shape: tuple
     kind: str = "matrix"
     optional: bool = False
+    below: int = 0
 
 
 def shape_fits(declared, got) -> bool:

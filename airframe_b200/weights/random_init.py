@@ -2,7 +2,8 @@
 (seed, tensor name), and a writer of whole model folders (config.json and
 model.safetensors).  Matrices and tables are N(0, 0.02), norm weights
 N(0, 0.1) (they act as ``offset + w``), gains (factors used as they stand) N(1, 0.1),
-mixing matrices the identity + N(0, 0.1), shares (the n factors of a weighted mean) N(1, 0.1) / n.
+mixing matrices the identity + N(0, 0.1), shares (the n factors of a weighted mean) N(1, 0.1) / n,
+blends (factors between two things) N(0.5, 0.1); the rows of a choice table are distinct integers below a bound.
 
 The reference has no such mode (its tests use zeros and ones,
 ``src/family/llama.rs:625-682``).
@@ -18,8 +19,9 @@ import torch
 from .loader import WeightDecl
 from .safetensors_io import write_safetensors
 
-_STD = {"matrix": 0.02, "table": 0.02, "norm": 0.1, "gain": 0.1, "mixing": 0.1, "share": 0.1}
-_MEAN = {"gain": 1.0}      # a factor that is used as it stands (a norm weight that acts as ``offset + w`` is "norm")
+_STD = {"matrix": 0.02, "table": 0.02, "norm": 0.1, "gain": 0.1, "mixing": 0.1, "share": 0.1, "blend": 0.1}
+_MEAN = {"gain": 1.0, "blend": 0.5}      # a factor that is used as it stands (a norm weight that acts as ``offset + w`` is "norm")
+INT_KINDS = ("int_table", "choice_table")      # tensors of integers
 _STORE = {"bfloat16": torch.bfloat16, "float32": torch.float32, "float16": torch.float16}
 
 
@@ -38,6 +40,9 @@ def random_tensor(decl: WeightDecl, seed: int, dtype: torch.dtype, device="cpu")
     gen.manual_seed(tensor_seed(seed, decl.name))
     if decl.kind == "int_table":
         return torch.randint(0, 1 << 15, tuple(decl.shape), generator=gen, device=device, dtype=torch.int32)
+    if decl.kind == "choice_table":      # every row: distinct integers in 0 .. below - 1, in random order
+        rows, n = decl.shape
+        return torch.rand(rows, decl.below, generator=gen, device=device).argsort(dim=1)[:, :n].to(torch.int32)
     if decl.kind not in _STD:
         raise ValueError(f"tensor '{decl.name}': unknown kind '{decl.kind}'")
     t = torch.empty(tuple(decl.shape), dtype=torch.float32, device=device)
@@ -68,7 +73,7 @@ class RandomSource:
 
     def info(self, name):
         d = self.decls[name]
-        return (torch.int32 if d.kind == "int_table" else self.store_dtype), tuple(d.shape)
+        return (torch.int32 if d.kind in INT_KINDS else self.store_dtype), tuple(d.shape)
 
     def read(self, name, device=None) -> torch.Tensor:
         return random_tensor(self.decls[name], self.seed, self.store_dtype, self.device)
@@ -91,7 +96,7 @@ def write_random_model(folder, config, seed: int, store_dtype: str = "bfloat16",
 
     def entries():
         for d in decls:
-            dt = torch.int32 if d.kind == "int_table" else dtype
+            dt = torch.int32 if d.kind in INT_KINDS else dtype
             yield d.name, tuple(d.shape), dt, (lambda d=d: random_tensor(d, seed, dtype, device))
 
     write_safetensors(folder / "model.safetensors", entries(), metadata={"format": "pt", "seed": seed})

@@ -159,7 +159,9 @@ def test_latent_rows_and_the_product_per_head(K, heads, dim, rot, rank, pitch, d
     P = pitch or dim + rot
     q = torch.full((T, heads * P), float("nan"), dtype=dtype, device=DEV)
     kvrow = torch.empty(T, rank + rot, dtype=dtype, device=DEV)
-    K.latent_prep(q, kvrow, proj, batch, heads, dim, rot, rank, norm_w, 1e-5, inv, kv=kv_view(kc, None, table, 0), pitch=pitch)
+    nq = heads * (dim + rot)
+    K.latent_prep(batch, heads, dim, rot, rank, 1e-5, inv, q=q, q_src=proj[:, :nq], pitch=pitch, kvrow=kvrow,
+                  kv_src=proj[:, nq:], norm_w=norm_w, kv=kv_view(kc, None, table, 0))
     x = proj.double().cpu()
     pos = batch.positions.cpu()
     qh = x[:, : heads * (dim + rot)].view(T, heads, dim + rot)
