@@ -344,7 +344,8 @@ __device__ __forceinline__ float clamped_glu(float g, float u, float limit) {
 
 // DUAL: out[sorted row][n] = act(s (x . w0[e][n]), s (x . w1[e][n])) * post, x the row of `a` that the pair's
 //       token names, s the pair's weight (a weight on an expert's input goes through its products, which have no
-//       bias), post the token's `scale_out` (1 without); out of the compute dtype, rows of N values.
+//       bias), post the token's `scale_out` (1 without); out of the compute dtype, rows of N values.  With split > 0
+//       the experts from there on have the limit limit_b.
 // MODE 2: out[sorted row][n] = gelu(x . w0[e][n]) * s * post with the exact (erf) GELU: an expert of one matrix, whose
 //       weight stands behind the activation.
 // else: out[(choice, token)][n] = a[sorted row] . w0[e][n] as floats: [top][tokens][N], partial sums that the
@@ -354,7 +355,8 @@ template <typename T, int MODE>
 __global__ void __launch_bounds__(256)
 expert_rows_kernel(void* __restrict__ out_, const T* __restrict__ a, const T* __restrict__ w0, const T* __restrict__ w1,
                    const int* __restrict__ perm, const int* __restrict__ plan, const float* __restrict__ pair_weight,
-                   const float* __restrict__ scale_out, int n_rows, int n_tokens, int top, int N, int K, float limit) {
+                   const float* __restrict__ scale_out, int n_rows, int n_tokens, int top, int N, int K, float limit, int split,
+                   float limit_b) {
   pdl_launch_dependents();
   constexpr bool DUAL = MODE == 1;                  // gate and up with the clamped activation
   constexpr bool MID = MODE != 0;                   // rows out in sorted order, of the compute dtype (MODE 2: one matrix, exact GELU)
@@ -383,6 +385,7 @@ expert_rows_kernel(void* __restrict__ out_, const T* __restrict__ a, const T* __
     src_row[m] = pair < 0 ? -1 : (MID ? pair / top : row0 + m);
   }
   __syncthreads();
+  if (split > 0 && expert >= split) limit = limit_b;
   const T* w0e = w0 + (size_t)expert * N * K;
   const T* w1e = DUAL ? w1 + (size_t)expert * N * K : nullptr;
   float acc0[AF_EX_TM / 4], acc1[AF_EX_TM / 4];
@@ -436,7 +439,7 @@ expert_rows_kernel(void* __restrict__ out_, const T* __restrict__ a, const T* __
 
 AF_EXPORT int af_expert_rows(void* out, const void* a, const void* w0, const void* w1, int dtype, const int* perm,
                              const int* plan, const float* pair_weight, const float* scale_out, int n_rows,
-                             int n_tokens, int top, int max_tiles, int N, int K, float limit, int act,
+                             int n_tokens, int top, int max_tiles, int N, int K, float limit, int split, float limit_b, int act,
                              cudaStream_t stream) {
   if (n_rows == 0) return 0;
   AF_REQUIRE(n_rows > 0 && n_tokens > 0 && top >= 1 && N > 0 && K > 0, "af_expert_rows: bad sizes");
@@ -449,15 +452,18 @@ AF_EXPORT int af_expert_rows(void* out, const void* a, const void* w0, const voi
   if (w1 != nullptr) {
     AF_DISPATCH_DTYPE(dtype, T,
                       af_launch(expert_rows_kernel<T, 1>, grid, dim3(256), 0, stream, out, (const T*)a, (const T*)w0,
-                                (const T*)w1, perm, plan, pair_weight, scale_out, n_rows, n_tokens, top, N, K, limit));
+                                (const T*)w1, perm, plan, pair_weight, scale_out, n_rows, n_tokens, top, N, K, limit, split,
+                                limit_b));
   } else if (act == 1) {
     AF_DISPATCH_DTYPE(dtype, T,
                       af_launch(expert_rows_kernel<T, 2>, grid, dim3(256), 0, stream, out, (const T*)a, (const T*)w0,
-                                (const T*)nullptr, perm, plan, pair_weight, scale_out, n_rows, n_tokens, top, N, K, limit));
+                                (const T*)nullptr, perm, plan, pair_weight, scale_out, n_rows, n_tokens, top, N, K, limit, split,
+                                limit_b));
   } else {
     AF_DISPATCH_DTYPE(dtype, T,
                       af_launch(expert_rows_kernel<T, 0>, grid, dim3(256), 0, stream, out, (const T*)a, (const T*)w0,
-                                (const T*)nullptr, perm, plan, pair_weight, scale_out, n_rows, n_tokens, top, N, K, limit));
+                                (const T*)nullptr, perm, plan, pair_weight, scale_out, n_rows, n_tokens, top, N, K, limit, split,
+                                limit_b));
   }
   AF_CHECK_LAUNCH("af_expert_rows");
 }

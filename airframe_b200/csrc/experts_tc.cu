@@ -62,6 +62,9 @@ struct ExArgs {
   const float* ba;
   const float* bi;
   const float* rate;
+  // EX_ACT: experts from `split` on are limited to limit_b (split 0: all to limit)
+  int split;
+  float limit_b;
 };
 
 enum { EX_DOWN = 0, EX_ACT = 1, EX_GATES = 2, EX_GELU = 3 };
@@ -287,6 +290,7 @@ expert_rows_tc_kernel(const __grid_constant__ CUtensorMap map_w0, const __grid_c
         }
         const int n = min(CW, rows - c0);                 // (sorted rows: the chunk's first n are the tile's)
         if constexpr (DUAL || SINGLE) {
+          const float limit = a.split > 0 && expert >= a.split ? a.limit_b : a.limit;
           const bool scaled = a.pair_weight != nullptr, posted = a.scale_out != nullptr;
           __nv_bfloat16* o = static_cast<__nv_bfloat16*>(a.out) + (size_t)(row0 + c0) * a.N + f;
 #pragma unroll
@@ -297,7 +301,7 @@ expert_rows_tc_kernel(const __grid_constant__ CUtensorMap map_w0, const __grid_c
             if constexpr (SINGLE)       // (the weight stands behind the activation: it is the expert's output that is weighed)
               o[(size_t)j * a.N] = __float2bfloat16_rn(0.5f * g[j] * (1.f + erff(g[j] * 0.70710678118654752f)) * s * post);
             else
-              o[(size_t)j * a.N] = __float2bfloat16_rn(ex_act(s * g[j], s * u[j], a.limit) * post);
+              o[(size_t)j * a.N] = __float2bfloat16_rn(ex_act(s * g[j], s * u[j], limit) * post);
           }
         } else {
 #pragma unroll
@@ -362,11 +366,12 @@ int ex_launch_bn(int bn, const CUtensorMap& m0, const CUtensorMap& m1, const CUt
 // the pairs' tokens name, gathered; else the first product's output); w0, w1 [experts, N, K] bfloat16; tile: the
 // plan's row tile (16, 32, 64, 128 or 256; at most so many rows a plan entry).  K a multiple of 8, bases 16-byte
 // aligned.  act 1 (no w1): out[sorted row] = gelu(a w0[e]^T) * s * post with the exact (erf) GELU, rows of the
-// compute dtype like the two-matrix form's.  Otherwise as af_expert_rows.
+// compute dtype like the two-matrix form's.  Otherwise as af_expert_rows (split > 0: experts from there on have the
+// limit limit_b).
 AF_EXPORT int af_expert_rows_tc(void* out, const void* a, const void* w0, const void* w1, int n_experts, const int* perm,
                                 const int* plan, const float* pair_weight, const float* scale_out, int n_rows,
-                                int n_tokens, int top, int max_tiles, int tile, int N, int K, float limit, int act,
-                                int* err, cudaStream_t stream) {
+                                int n_tokens, int top, int max_tiles, int tile, int N, int K, float limit, int split,
+                                float limit_b, int act, int* err, cudaStream_t stream) {
   if (n_rows == 0) return 0;
   AF_REQUIRE(n_rows > 0 && n_tokens > 0 && top >= 1 && N > 0 && K > 0 && n_experts > 0, "af_expert_rows_tc: bad sizes");
   AF_REQUIRE((plan == nullptr) == (perm == nullptr), "af_expert_rows_tc: a plan and its permutation, or neither");
@@ -385,6 +390,7 @@ AF_EXPORT int af_expert_rows_tc(void* out, const void* a, const void* w0, const 
   if (rc) return rc;
   ExArgs args{out, N, K, n_rows, n_tokens, top, (N + EX_BM - 1) / EX_BM,
               plan != nullptr ? max_tiles : (n_rows + tile - 1) / tile, perm, plan, pair_weight, scale_out, limit, err};
+  args.split = split, args.limit_b = limit_b;
   AF_REQUIRE(args.max_row_tiles > 0, "af_expert_rows_tc: no tiles");
   AF_REQUIRE(act == 0 || (act == 1 && w1 == nullptr), "af_expert_rows_tc: the exact GELU stands behind one matrix");
   if (w1 != nullptr) return ex_launch_bn<EX_ACT>(tile, m0, m1, mx, args, stream);

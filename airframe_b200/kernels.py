@@ -1426,15 +1426,24 @@ def expert_table_plan(perm, plan, tokens, tables, n_experts: int, tile: int = EX
                                        c_int(n_experts), c_int(max_tiles), c_int(tile), _stream()))
 
 
+def _second_limit(second):
+    if second is None:
+        return c_int(0), c_float(0.0)
+    if second[0] < 1:
+        raise KernelError("expert_rows: a second limit begins behind the first expert")
+    return c_int(second[0]), c_float(second[1])
+
+
 EXPERT_ACTS = {None: 0, "gelu_erf": 1}
 
 
 def expert_rows(out, a, w0, w1=None, perm=None, plan=None, pair_weight=None, scale_out=None, n_tokens: int = 0,
-                top: int = 1, limit: float = 0.0, act=None) -> None:
+                top: int = 1, limit: float = 0.0, act=None, second=None) -> None:
     """Rows times the matrices of the expert they belong to (the CUDA-core path; 32-bit sums in index order).
     With ``w1``: out[sorted row] = act(s x w0[e]^T, s x w1[e]^T) * post in the compute dtype, x = row
     pair // top of ``a``, s = pair_weight[pair], post = scale_out[token], act(g, u) = min(g, limit)
-    sigmoid(1.702 min(g, limit)) (clamp(u, +-limit) + 1).  Without: out float32 [top, tokens, N] with
+    sigmoid(1.702 min(g, limit)) (clamp(u, +-limit) + 1); ``second`` = (expert, limit): the experts from that one on have
+    that limit.  Without: out float32 [top, tokens, N] with
     out[choice, token] = a[sorted row] w0[e]^T.  Without ``w1`` but with ``act`` = "gelu_erf": an expert of one
     matrix, out[sorted row] = gelu(x w0[e]^T) * s * post with the exact GELU (the weight stands behind the
     activation).  w0, w1: [experts, N, K].  Without a plan: one expert, the rows in order."""
@@ -1460,7 +1469,7 @@ def expert_rows(out, a, w0, w1=None, perm=None, plan=None, pair_weight=None, sca
                                  _ptr(pair_weight, "pair_weight", torch.float32, allow_none=True),
                                  _ptr(scale_out, "scale_out", torch.float32, allow_none=True), c_int(n_rows),
                                  c_int(n_tokens), c_int(top), c_int(max_tiles), c_int(N), c_int(K), c_float(limit),
-                                 c_int(EXPERT_ACTS[act]), _stream()))
+                                 *_second_limit(second), c_int(EXPERT_ACTS[act]), _stream()))
 
 
 def expert_gather(out, x, perm, top: int) -> None:
@@ -1481,7 +1490,7 @@ def expert_rows_tc_supported(a, w0) -> bool:
 
 
 def expert_rows_tc(out, a, w0, w1=None, perm=None, plan=None, pair_weight=None, scale_out=None, n_tokens: int = 0,
-                   top: int = 1, limit: float = 0.0, tile: int = 0, act=None) -> None:
+                   top: int = 1, limit: float = 0.0, tile: int = 0, act=None, second=None) -> None:
     """:func:`expert_rows` on the tcgen05 tensor cores (bfloat16 operands, 32-bit sums in TMEM), with one
     difference: ``a`` holds the sorted rows themselves also for the first product (:func:`expert_gather`).
     ``tile``: the row tile the plan was made for (without a plan: chosen here)."""
@@ -1511,7 +1520,7 @@ def expert_rows_tc(out, a, w0, w1=None, perm=None, plan=None, pair_weight=None, 
                                     _ptr(pair_weight, "pair_weight", torch.float32, allow_none=True),
                                     _ptr(scale_out, "scale_out", torch.float32, allow_none=True), c_int(n_rows),
                                     c_int(n_tokens), c_int(top), c_int(max_tiles), c_int(tile), c_int(N), c_int(K),
-                                    c_float(limit), c_int(EXPERT_ACTS[act]),
+                                    c_float(limit), *_second_limit(second), c_int(EXPERT_ACTS[act]),
                                     _ptr(error_word(a.device), "err", torch.int32), _stream()))
 
 
@@ -1654,6 +1663,100 @@ def state_scan_chunked(out, r, k, v, w, state, batch, heads: int, dk: int, dv: i
                                 _ptr(chunk_starts, "chunk_starts", i32), _ptr(seq_first, "seq_first", i32),
                                 _ptr(tiles, "tiles", i32), _ptr(batch.slots, "slots", i32), c_int(n_chunks),
                                 c_int(batch.n_seqs), c_int(n_tiles), c_int(heads), c_int(dk), c_int(dv), _stream()))
+
+
+def _retention_args(q, k, v, gate, table, heads: int, dk: int, dv: int, pairing: str, who: str):
+    T = q.shape[0]
+    for t, n, name in ((q, dk, "q"), (k, dk, "k"), (v, dv, "v")):
+        if tuple(t.shape) != (T, heads * n):
+            raise KernelError(f"{who}: {name} must be [{T}, {heads * n}], got {tuple(t.shape)}")
+    if gate is not None and tuple(gate.shape) != (T, heads * dv):
+        raise KernelError(f"{who}: the gate must be [{T}, {heads * dv}]")
+    n = 0 if table is None else table.shape[1]
+    if table is not None and (tuple(table.shape) != (T, n, 2) or not table.is_contiguous() or table.dtype != torch.float32):
+        raise KernelError(f"{who}: a table of cosines and sines [{T}, n, 2]")
+    if pairing not in PAIRINGS:
+        raise KernelError(f"{who}: unknown pairing '{pairing}'")
+    ga = _f32_rows(gate, "gate") if gate is not None else (c_void_p(0), c_longlong(0))
+    return (*_f32_rows(q, "q"), *_f32_rows(k, "k"), *_f32_rows(v, "v"), *ga), \
+        (_ptr(table, "table", allow_none=True), c_int(n), c_int(PAIRINGS[pairing]))
+
+
+def retention_step(y, q, k, v, gate, table, decay, state, batch, heads: int, dk: int, dv: int, key_scale: float, eps: float,
+                   pairing: str = "half", magnitude: float = 1.0, gate_act: str = "silu") -> None:
+    """A step of single tokens, one a sequence: q and k (float32 rows [T, heads * dk], column sections allowed) rotated
+    by ``table`` (float32 [T, n, 2] or None, times ``magnitude``), S <- decay[h] S + k v^T in ``state`` (float32 [slots,
+    heads, dv, dk]), y = o / sqrt(mean over the head of o^2 + eps) * act(gate) with o = key_scale S^T q, in y's dtype."""
+    T = y.shape[0]
+    if tuple(y.shape) != (T, heads * dv) or not y.is_contiguous() or batch.n_seqs != T or q.shape[0] != T or gate is None:
+        raise KernelError(f"retention_step: y contiguous [{batch.n_seqs}, {heads * dv}], a row a sequence, and a gate")
+    if state.dtype != torch.float32 or tuple(state.shape[1:]) != (heads, dv, dk) or not state.is_contiguous() \
+            or decay.numel() != heads:
+        raise KernelError(f"retention_step: state contiguous float32 [slots, {heads}, {dv}, {dk}], one decay a head")
+    rows, turn = _retention_args(q, k, v, gate, table, heads, dk, dv, pairing, "retention_step")
+    i32 = torch.int32
+    _check(_lib().af_retention_step(_ptr(y), c_int(dtype_code(y.dtype)), *rows, c_int(GATE_ACTS[gate_act]), *turn,
+                                    c_float(magnitude), _ptr(decay, "decay", torch.float32), _ptr(state, "state"),
+                                    _ptr(batch.slots, "slots", i32), _ptr(batch.seq_starts, "seq_starts", i32),
+                                    c_int(batch.n_seqs), c_int(heads), c_int(dk), c_int(dv), c_float(key_scale), c_float(eps),
+                                    _stream()))
+
+
+RETENTION_TILE = 64        # tokens of a tile of the prompt's kernels
+RETENTION_CHUNK = 128      # tokens of a chunk (whole tiles, at most 256)
+
+
+def retention_prompt_supported(dk: int, dv: int) -> bool:
+    """Whether :func:`retention_prompt` takes heads of these sizes."""
+    return bool(_lib().af_retention_prompt_supported(c_int(dk), c_int(dv)))
+
+
+def _retention_chunks(batch, chunk: int):
+    """The chunks and tiles of a prefill step's sequences (made on the host once a step, kept in ``batch.aux``): device
+    tensors chunk_starts [n_chunks + 1], seq_first_chunk [n_seqs + 1], tiles [n_tiles, 4] = (first row, rows, chunk, the
+    tile's first token in its chunk), and the counts."""
+    key = ("retention_chunks", chunk)
+    if key not in batch.aux:
+        starts, first, tiles, row = [], [0], [], 0
+        for n in batch.seq_lens:
+            for c0 in range(0, n, chunk):
+                rows = min(chunk, n - c0)
+                for t0 in range(0, rows, RETENTION_TILE):
+                    tiles.append((row + c0 + t0, min(RETENTION_TILE, rows - t0), len(starts), t0))
+                starts.append(row + c0)
+            row += n
+            first.append(len(starts))
+        starts.append(row)
+        flat = starts + first + [x for t in tiles for x in t]
+        dev = torch.tensor(flat, dtype=torch.int32).to(batch.tokens.device)
+        a, b = len(starts), len(starts) + len(first)
+        batch.aux[key] = (dev[:a], dev[a:b], dev[b:], len(starts) - 1, len(tiles))
+    return batch.aux[key]
+
+
+def retention_prompt(out, q, k, v, gate, table, powers, state, batch, heads: int, dk: int, dv: int, key_scale: float,
+                     eps: float, pairing: str = "half", magnitude: float = 1.0, gate_act: str = "silu",
+                     chunk: int = RETENTION_CHUNK) -> None:
+    """The same for a prefill step on the tensor cores, the sequences cut into chunks of ``chunk`` tokens: ``powers``
+    float32 [heads, chunk + 1] = decay^0 .. decay^chunk.  ``out`` bfloat16 with the norm and the gate (``dv`` <= 128), or with
+    ``gate`` None float32 key_scale o.  32-bit sums; the operands are pairs of bfloat16 (16 bits of mantissa)."""
+    T = out.shape[0]
+    if tuple(out.shape) != (T, heads * dv) or not out.is_contiguous() \
+            or out.dtype != (torch.float32 if gate is None else torch.bfloat16):
+        raise KernelError(f"retention_prompt: out contiguous [{T}, {heads * dv}], bfloat16 with a gate, float32 without")
+    if state.dtype != torch.float32 or tuple(state.shape[1:]) != (heads, dv, dk) or not state.is_contiguous() \
+            or tuple(powers.shape) != (heads, chunk + 1) or not powers.is_contiguous():
+        raise KernelError(f"retention_prompt: state float32 [slots, {heads}, {dv}, {dk}], powers [{heads}, {chunk + 1}]")
+    rows, turn = _retention_args(q, k, v, gate, table, heads, dk, dv, pairing, "retention_prompt")
+    starts, seq_first, tiles, n_chunks, n_tiles = _retention_chunks(batch, chunk)
+    local = torch.empty(n_chunks, heads, dv, dk, dtype=torch.float32, device=out.device)
+    i32 = torch.int32
+    _check(_lib().af_retention_prompt(_ptr(out), *rows, c_int(GATE_ACTS[gate_act]), *turn, c_float(magnitude),
+                                      _ptr(powers, "powers", torch.float32), c_int(chunk), _ptr(local), _ptr(state, "state"),
+                                      _ptr(starts, "chunk_starts", i32), _ptr(seq_first, "seq_first", i32),
+                                      _ptr(tiles, "tiles", i32), _ptr(batch.slots, "slots", i32), c_int(n_chunks),
+                                      c_int(batch.n_seqs), c_int(n_tiles), c_int(heads), c_int(dk), c_int(dv),
+                                      c_float(key_scale), c_float(eps), _stream()))
 
 
 def conv_pack(qkv, proj, batch, H: int, G: int, d: int, dv: int, pk: int, pv: int, bias=None, taps_w=None, history=None,

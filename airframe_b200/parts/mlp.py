@@ -24,7 +24,9 @@ may be of one matrix and an activation, E(h) = W_down gelu(W_up h) with the exac
 *output* (it is applied behind the activation, in front of the linear down product).
 
 There may be no router at all: a table of integers then names the ``top`` experts of every token id, each with the
-weight 1 / top on its output, which the residual sum applies.  Which experts a step's tokens use is then known before its
+weight 1 / top on its output, which the residual sum applies.  A shared expert of the same form is then, where its size
+comes in whole experts (or nearly), so many more experts that every token uses: its features fall apart into
+groups, E(h) = sum over groups of W_down,g act(W_gate,g h, W_up,g h), and the one sum over experts holds them all.  Which experts a step's tokens use is then known before its
 first layer runs: the pairs of all such layers are sorted by one kernel, at the first of them.
 """
 from __future__ import annotations
@@ -110,6 +112,7 @@ class RoutedExperts(FeedForward):
     ``limit``).  Optional ``router``: {``correction_weight`` (tensor name, [experts]), ``groups``: {``count``,
     ``keep``}, ``normalise`` (bool), ``scale``}.  The result is a sum of 32-bit terms that the residual kernel takes."""
     graph_safe = True
+    JOIN_MOST = 1.25      # a shared expert is padded with zeros to whole experts if that makes it no larger than this
 
     def __init__(self, params, ctx):
         super().__init__(params, ctx)
@@ -151,6 +154,11 @@ class RoutedExperts(FeedForward):
         self.mixed = self.shared is not None and bool(self.shared.get("mix_weight"))
         if self.mixed and self.table_name:
             raise ConfigError("routed_experts: a shared expert's 'mix_weight' rides with the router, which a table replaces")
+        self.joined = 0                      # experts that the shared one adds to the routed ones (0: it runs by itself)
+        if self.table_name and self.shared is not None:
+            pieces = -(-int(self.shared["intermediate_size"]) // self.inter)
+            if pieces * self.inter <= self.JOIN_MOST * int(self.shared["intermediate_size"]):
+                self.joined = pieces
 
     def _name(self, e: int, role: str) -> str:
         return self.pattern.format(e=e, role=role)
@@ -187,7 +195,9 @@ class RoutedExperts(FeedForward):
         rows = [] if self.table_name else [weights[self.router_name]]
         if self.mixed:
             rows.append(weights[self.shared["mix_weight"]].reshape(1, self.hidden))       # the shared expert's gate rides with the router
-        if self.shared is not None:
+        if self.joined:
+            self._join_shared(weights)
+        elif self.shared is not None:
             sh = self.shared
             self.s_gate = weights[sh["gate_weight"]].to(dt).unsqueeze(0).contiguous()
             self.s_up = weights[sh["up_weight"]].to(dt).unsqueeze(0).contiguous()
@@ -197,14 +207,31 @@ class RoutedExperts(FeedForward):
             self.table = weights[self.table_name].to(torch.int32).contiguous()
             if not 0 <= int(self.table.min()) <= int(self.table.max()) < self.n_experts:
                 raise ConfigError(f"routed_experts: {self.table_name} names an expert outside 0 .. {self.n_experts - 1}")
+            if self.joined:
+                more = torch.arange(self.n_experts, self.n_experts + self.joined, dtype=torch.int32, device=self.table.device)
+                self.table = torch.cat([self.table, more.expand(self.vocab, -1)], dim=1).contiguous()
             self.tables = self.table.unsqueeze(0)
+
+    def _join_shared(self, weights) -> None:
+        """The shared expert's matrices behind the routed ones', in pieces of an expert's size (zeros behind the last)."""
+        sh, n, f = self.shared, self.joined, self.inter
+        pad = n * f - int(sh["intermediate_size"])
+
+        def rows(name):
+            w = torch.nn.functional.pad(weights[name].to(self.w_up.dtype), (0, 0, 0, pad))
+            return w.view(n, f, self.hidden)
+
+        down = torch.nn.functional.pad(weights[sh["down_weight"]].to(self.w_up.dtype), (0, pad))
+        self.w_gate = torch.cat([self.w_gate, rows(sh["gate_weight"])]).contiguous()
+        self.w_up = torch.cat([self.w_up, rows(sh["up_weight"])]).contiguous()
+        self.w_down = torch.cat([self.w_down, down.view(self.hidden, n, f).permute(1, 0, 2)]).contiguous()
 
     @classmethod
     def link(cls, parts) -> None:
         groups: dict = {}
         for p in parts:
             if p.table is not None:
-                groups.setdefault((p.n_experts, p.top, p.vocab), []).append(p)
+                groups.setdefault((p.n_experts, p.top, p.joined, p.vocab), []).append(p)
         for same in groups.values():
             tables = torch.stack([p.table for p in same]).contiguous()
             for i, p in enumerate(same):
@@ -234,15 +261,16 @@ class RoutedExperts(FeedForward):
     def _plan(self, x, batch, tile: int):
         """(perm, plan, weights of the pairs or None, the shared expert's factor or None): the step's (token, choice)
         pairs sorted by expert."""
-        T, top, dev, i32 = x.shape[0], self.top, x.device, torch.int32
-        cells = 1 + 3 * kernels.expert_max_tiles(T * top, self.n_experts, tile)
+        T, top, dev, i32 = x.shape[0], self.top + self.joined, x.device, torch.int32
+        n_experts = self.n_experts + self.joined
+        cells = 1 + 3 * kernels.expert_max_tiles(T * top, n_experts, tile)
         if self.table is not None:       # known from the tokens: the plans of all layers that choose alike, made once a step
             key = ("expert_plans", self.tables.data_ptr(), tile)
             if key not in batch.aux:
                 n = self.tables.shape[0]
                 perms = torch.empty(n, T * top, dtype=i32, device=dev)
                 plans = torch.empty(n, cells, dtype=i32, device=dev)
-                kernels.expert_table_plan(perms, plans, batch.tokens, self.tables, self.n_experts, tile)
+                kernels.expert_table_plan(perms, plans, batch.tokens, self.tables, n_experts, tile)
                 batch.aux[key] = (perms, plans)
             perms, plans = batch.aux[key]
             return perms[self.table_index], plans[self.table_index], None, None
@@ -257,13 +285,14 @@ class RoutedExperts(FeedForward):
         return perm, plan, wts, mix
 
     def forward(self, x, batch):
-        T, top, dev = x.shape[0], self.top, x.device
+        T, top, dev = x.shape[0], self.top + self.joined, x.device
         # bfloat16 with sizes the tensor-core products take: the rows in sorted order, then grouped products;
         # else the products on the CUDA cores (32-bit, or odd sizes), which fetch their rows themselves
         fast = (kernels.expert_rows_tc_supported(x, self.w_up) and self.inter % 8 == 0)
         act = None if self.gated else "gelu_erf"
-        tile = kernels.expert_tc_tile(T * top, self.n_experts) if fast else kernels.EXPERT_TILE
+        tile = kernels.expert_tc_tile(T * top, self.n_experts + self.joined) if fast else kernels.EXPERT_TILE
         perm, plan, wts, mix = self._plan(x, batch, tile)
+        second = (self.n_experts, float(self.shared["limit"])) if self.joined else None
         mid = torch.empty(T * top, self.inter, dtype=x.dtype, device=dev)
         out = torch.empty(top, T, self.hidden, dtype=torch.float32, device=dev)
         if fast:
@@ -271,7 +300,7 @@ class RoutedExperts(FeedForward):
             kernels.expert_gather(rows, x, perm, top)
             if self.gated:
                 kernels.expert_rows_tc(mid, rows, self.w_gate, self.w_up, perm=perm, plan=plan, pair_weight=wts,
-                                       n_tokens=T, top=top, limit=self.limit, tile=tile)
+                                       n_tokens=T, top=top, limit=self.limit, tile=tile, second=second)
             else:
                 kernels.expert_rows_tc(mid, rows, self.w_up, perm=perm, plan=plan, pair_weight=wts, n_tokens=T, top=top,
                                        tile=tile, act=act)
@@ -279,10 +308,12 @@ class RoutedExperts(FeedForward):
         else:
             if self.gated:
                 kernels.expert_rows(mid, x, self.w_gate, self.w_up, perm=perm, plan=plan, pair_weight=wts, n_tokens=T,
-                                    top=top, limit=self.limit)
+                                    top=top, limit=self.limit, second=second)
             else:
                 kernels.expert_rows(mid, x, self.w_up, perm=perm, plan=plan, pair_weight=wts, n_tokens=T, top=top, act=act)
             kernels.expert_rows(out, mid, self.w_down, perm=perm, plan=plan, n_tokens=T, top=top)
+        if self.joined:
+            return WeightedSum([(PartialSums(out[: self.top]), 1.0 / self.top), (PartialSums(out[self.top:]), 1.0)])
         terms = [(PartialSums(out), 1.0 / top if self.table is not None else 1.0)]
         if self.shared is not None:
             sf = int(self.shared["intermediate_size"])

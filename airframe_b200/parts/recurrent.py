@@ -229,6 +229,7 @@ class Retention(_StateMixer):
         if not isinstance(decay, (list, tuple)) or len(decay) != self.heads:
             raise ConfigError(f"retention: 'decay' must list one factor for each of the {self.heads} heads")
         self.decay_host = torch.tensor([float(d) for d in decay], dtype=torch.float64).to(torch.float32)
+        self.powers = None               # [heads, chunk + 1]: the decay to the powers 0 .. chunk
         self.key_scale = float(self.params.get("key_scale", self.dk ** -0.5))
         self.gate = self.params.get("gate", "silu")
         if self.gate not in kernels.GATE_ACTS:
@@ -261,18 +262,44 @@ class Retention(_StateMixer):
         return 2 * T * (self.w_in.numel() + self.w_o.numel()) + T * self.heads * 4 * self.dk * self.dv
 
     def forward(self, x, batch, view):
-        T, off, pos = x.shape[0], self.off, self.position
-        nk, nv = self.heads * self.dk, self.heads * self.dv
+        T, off, pos, H, dk, dv = x.shape[0], self.off, self.position, self.heads, self.dk, self.dv
+        nk, nv = H * dk, H * dv
         proj = linear(x, self.w_in, out_dtype=torch.float32)
-        q, k, v = (proj[:, off[n]: off[n] + w] for n, w in (("q", nk), ("k", nk), ("v", nv)))
-        if pos.rotary_dim:
-            kernels.rotate_rows(q, k, pos.step_table(batch), self.heads, self.dk, pairing=pos.pairing, magnitude=pos.magnitude)
-        o = torch.empty(T, nv, dtype=torch.float32, device=x.device)
-        kernels.state_scan("decay", o, q, k, v, view.state, batch, self.heads, self.dk, self.dv, decay=self.decay)
+        q, k, v, g = (proj[:, off[n]: off[n] + w] for n, w in (("q", nk), ("k", nk), ("v", nv), ("g", nv)))
+        table = pos.step_table(batch) if pos.rotary_dim else None
+        turn = {"pairing": pos.pairing, "magnitude": pos.magnitude}
         y = torch.empty(T, nv, dtype=x.dtype, device=x.device)
-        kernels.gated_group_norm(y, o, None, proj[:, off["g"]: off["g"] + nv], self.dv, self.eps, gate_act=self.gate,
-                                 in_scale=self.key_scale)
+        if T == batch.n_seqs:            # single tokens: rotation, state, norm and gate in one kernel
+            kernels.retention_step(y, q, k, v, g, table, self.decay, view.state, batch, H, dk, dv, self.key_scale, self.eps,
+                                   gate_act=self.gate, **turn)
+            return linear_split(y, self.w_o, wide=self.wide)
+        scale = self.key_scale
+        if self._on_tensor_cores(x, batch):
+            fused = dv <= 128            # (a head's values in one block: its norm and gate there too)
+            o = y if fused else torch.empty(T, nv, dtype=torch.float32, device=x.device)
+            kernels.retention_prompt(o, q, k, v, g if fused else None, table, self._powers(), view.state, batch, H, dk, dv,
+                                     scale, self.eps, gate_act=self.gate, **turn)
+            if fused:
+                return linear_split(y, self.w_o, wide=self.wide)
+            scale = 1.0
+        else:                            # token after token, in 32 bits
+            if table is not None:
+                kernels.rotate_rows(q, k, table, H, dk, **turn)
+            o = torch.empty(T, nv, dtype=torch.float32, device=x.device)
+            kernels.state_scan("decay", o, q, k, v, view.state, batch, H, dk, dv, decay=self.decay)
+        kernels.gated_group_norm(y, o, None, g, dv, self.eps, gate_act=self.gate, in_scale=scale)
         return linear_split(y, self.w_o, wide=self.wide)
+
+    def _on_tensor_cores(self, x, batch) -> bool:
+        """A bfloat16 prompt whose tokens fill a tile, cut into chunks on the tensor cores."""
+        return (x.dtype == torch.bfloat16 and batch.max_len >= kernels.RETENTION_TILE
+                and kernels.retention_prompt_supported(self.dk, self.dv))
+
+    def _powers(self):
+        if self.powers is None:
+            n = torch.arange(kernels.RETENTION_CHUNK + 1, dtype=torch.float64)
+            self.powers = (self.decay_host.double()[:, None] ** n).to(torch.float32).to(self.ctx.device).contiguous()
+        return self.powers
 
 
 @register_part("mixer", "mingru")

@@ -35,6 +35,9 @@ for Fiferax and one for Gemma-2 of equal width, depth, feed-forward and vocabula
 every layer, dense and routed feed-forwards in turn).
 ``--tarorax all|w1024|w2304|w4096`` does the same for Tarorax (four residual streams; gated linear attention in
 three layers of four and differential attention in the fourth; dense and routed feed-forwards in turn).
+``--teselix all|w1024|w2304|w4096`` does the same for Teselix (retention and latent attention in turn, experts looked
+up by token in every layer) beside the two models that have the like layers: Tarorax with one stream, gated linear
+attention and routed experts of equal size in every layer, and Banitar with latent attention of equal size in every layer.
 """
 from __future__ import annotations
 
@@ -600,9 +603,53 @@ def tarorax_points(args) -> None:
     side_by_side(args, args.tarorax, TARORAX_POINTS, _tarorax_sizes, "tarorax")
 
 
-def side_by_side(args, which, points, make, arm_name) -> None:
-    """Prefill and decode of a design at the named points, each beside the Gemma-2 model that `make` pairs it
-    with.  One JSON line a model."""
+def _teselix_sizes(width, layers, heads, dim, lat_heads, lat_dim, rot_dim, vdim, kv_rank, q_rank, experts, top, expert_ff,
+                   shared_ff, vocab):
+    """A Teselix model of `layers` layers (retention and latent attention in turn, every feed-forward a table of
+    experts with a shared one), and two models of equal width and vocabulary that have its like layers: Tarorax with one
+    stream (gated linear attention of the same heads, as many experts, of one matrix and an activation), and Banitar with
+    latent attention of the same heads and a dense feed-forward of what a Teselix token uses."""
+    ret = {"heads": heads, "dim": dim, "vdim": dim, "rot": {"base": 10000.0, "dims": dim},
+           "decay": [1.0 - 2.0 ** (-5 - 4 * h / max(heads - 1, 1)) for h in range(heads)]}
+    rot = {"base": 10000.0, "dims": rot_dim}
+    lat = {"heads": lat_heads, "dim": lat_dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank,
+           "scale": (lat_dim + rot_dim) ** -0.5}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff, "limit": 7.0}, "router": {"experts": experts, "top": top},
+           "shared": {"ff": shared_ff, "limit": 7.0}}
+    stretched = dict(rot, scaling={"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0})
+    tx = {"architecture": "Teselix", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "postln_alpha": 2.0,
+          "layers": [{"type": "retention", "mixer": ret, "mlp": moe} if i % 2 == 0 else
+                     {"type": "latent_attention", "mixer": dict(lat, q_rank=q_rank, rot=stretched), "mlp": moe}
+                     for i in range(layers)]}
+    tarorax = {"architecture": "Tarorax", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+               "layers": [{"type": "gla", "mixer": {"heads": heads, "dim": dim, "vdim": dim, "tau": 8.0, "rank": 64},
+                           "mlp": {"kind": "moe", "expert": {"ff": expert_ff},
+                                   "router": {"experts": experts, "top": top, "scale": 1.0}}} for _ in range(layers)]}
+    banitar = {"architecture": "Banitar", "vocab": vocab, "width": width, "embedding": {"scale": 1.0},
+               "norm": {"eps": 1e-6},
+               "layers": [{"type": "latent_attention", "mixer": dict(lat, mask={"size": CONTEXT}, rot=rot),
+                           "mlp": {"kind": "dense", "ff": top * expert_ff + shared_ff}} for _ in range(layers)]}
+    return tx, tarorax, banitar
+
+
+TESELIX_POINTS = {
+    "w1024": dict(width=1024, layers=8, heads=16, dim=64, lat_heads=16, lat_dim=32, rot_dim=32, vdim=64, kv_rank=96,
+                  q_rank=256, experts=16, top=2, expert_ff=1024, shared_ff=1024, vocab=32000),
+    "w2304": dict(width=2304, layers=8, heads=18, dim=128, lat_heads=18, lat_dim=64, rot_dim=64, vdim=128, kv_rank=192,
+                  q_rank=768, experts=16, top=2, expert_ff=2304, shared_ff=2304, vocab=32000),
+    "w4096": dict(width=4096, layers=8, heads=32, dim=128, lat_heads=32, lat_dim=128, rot_dim=64, vdim=128, kv_rank=512,
+                  q_rank=1536, experts=32, top=4, expert_ff=2048, shared_ff=2048, vocab=32000),
+}
+
+
+def teselix_points(args) -> None:
+    """The same figures for Teselix, beside the models that have its like layers."""
+    side_by_side(args, args.teselix, TESELIX_POINTS, _teselix_sizes, "teselix", ("tarorax", "banitar"))
+
+
+def side_by_side(args, which, points, make, arm_name, beside=("gemma2",)) -> None:
+    """Prefill and decode of a design at the named points, each beside the models that `make` pairs it
+    with (named by `beside`).  One JSON line a model."""
     import torch
     sys.path.insert(0, str(ROOT))
     from torch.profiler import ProfilerActivity, profile
@@ -645,7 +692,7 @@ def side_by_side(args, which, points, make, arm_name) -> None:
     for tag, sizes in points.items():
         if which not in ("all", tag):
             continue
-        for arm, cfg_dict in zip((arm_name, "gemma2"), make(**sizes)):
+        for arm, cfg_dict in zip((arm_name, *beside), make(**sizes)):
             cfg = config_from_dict(cfg_dict)
             V = cfg_dict.get("vocab") or cfg_dict["vocab_size"]
             budget = B * ((P + K + W + 8 + 63) // 64 * 64)
@@ -724,6 +771,8 @@ def main() -> int:
                     help="the same for Zatasun (not the default run)")
     ap.add_argument("--tarorax", default="", choices=["", "all", *sorted(TARORAX_POINTS)],
                     help="the same for Tarorax (not the default run)")
+    ap.add_argument("--teselix", default="", choices=["", "all", *sorted(TESELIX_POINTS)],
+                    help="the same for Teselix, beside Tarorax and Banitar (not the default run)")
     args = ap.parse_args()
     if args.impl == "reference":
         print(json.dumps({"impl": "reference", "unavailable":
@@ -747,6 +796,9 @@ def main() -> int:
         return 0
     if args.tarorax:
         tarorax_points(args)
+        return 0
+    if args.teselix:
+        teselix_points(args)
         return 0
     line = run_ours(args)
     if line is not None:
