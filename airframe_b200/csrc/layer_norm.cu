@@ -270,6 +270,39 @@ token_shift_kernel(TY* __restrict__ hs, TY* __restrict__ y, const float* __restr
   }
 }
 
+constexpr int LN_MAX_ROW = 16384;
+
+// Rows that do not fit the default limit of shared memory: raised once a device.
+template <typename K>
+int ln_raise(K kernel, bool* flags, int hidden) {
+  if (hidden * sizeof(float) <= 40 * 1024) return 0;
+  const int dev = af_current_device();
+  if (dev < 0) return -1;
+  if (af_first_on_device(flags, dev)) {
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, LN_MAX_ROW * (int)sizeof(float));
+    if (e != cudaSuccess) return af_fail((int)e, "af_layer_norm: %s", cudaGetErrorString(e));
+  }
+  return 0;
+}
+
+template <typename TY>
+int ln_launch(void* y, const float* x, const float* w, const float* b, const int* rows, int n_rows, int hidden, float eps,
+              cudaStream_t stream) {
+  static bool raised[AF_MAX_DEVICES];
+  if (int e = ln_raise(layer_norm_kernel<TY>, raised, hidden)) return e;
+  af_launch(layer_norm_kernel<TY>, dim3(n_rows), dim3(256), (size_t)hidden * sizeof(float), stream, (TY*)y, x, w, b, rows,
+            hidden, eps);
+  AF_CHECK_LAUNCH("af_layer_norm");
+}
+
+template <typename TY>
+int ln_launch_sum(const LnSumArgs& p, cudaStream_t stream) {
+  static bool raised[AF_MAX_DEVICES];
+  if (int e = ln_raise(norm_of_sum_kernel<TY>, raised, p.hidden)) return e;
+  af_launch(norm_of_sum_kernel<TY>, dim3(p.n_rows), dim3(256), (size_t)p.hidden * sizeof(float), stream, p);
+  AF_CHECK_LAUNCH("af_norm_of_sum");
+}
+
 int ln_term_check(const LnTerm& t, const char* who, const char* what) {
   AF_REQUIRE(t.p == nullptr || (t.parts >= 1 && (t.dtype == AF_F32 || (t.dtype == AF_BF16 && t.parts == 1))),
              "%s: %s must be floats, or one tensor of bfloat16", who, what);
@@ -285,11 +318,9 @@ bool ln_term_vec(const LnTerm& t) {
 AF_EXPORT int af_layer_norm(void* y, int y_dtype, const float* x, const float* w, const float* b, const int* rows,
                             int n_rows, int hidden, float eps, cudaStream_t stream) {
   if (n_rows == 0) return 0;
-  AF_REQUIRE(n_rows > 0 && hidden > 0 && hidden <= 12288, "af_layer_norm: rows of 1 to 12288 values");
-  AF_DISPATCH_DTYPE(y_dtype, TY,
-                    af_launch(layer_norm_kernel<TY>, dim3(n_rows), dim3(256), (size_t)hidden * sizeof(float), stream,
-                              (TY*)y, x, w, b, rows, hidden, eps));
-  AF_CHECK_LAUNCH("af_layer_norm");
+  AF_REQUIRE(n_rows > 0 && hidden > 0 && hidden <= LN_MAX_ROW, "af_layer_norm: rows of 1 to %d values", LN_MAX_ROW);
+  AF_DISPATCH_DTYPE(y_dtype, TY, return ln_launch<TY>(y, x, w, b, rows, n_rows, hidden, eps, stream));
+  return 0;
 }
 
 // y_dtype: of y and hs.  The terms' partial sums lie n_rows * hidden elements apart.
@@ -298,7 +329,7 @@ AF_EXPORT int af_norm_of_sum(float* x, const void* a, int a_dtype, int a_parts, 
                              float alpha, const float* w, const float* bias, float eps, void* y, void* hs, int y_dtype,
                              const float* mu, float* prev, const int* slots, int n_rows, int hidden, cudaStream_t stream) {
   if (n_rows == 0) return 0;
-  AF_REQUIRE(n_rows > 0 && hidden > 0 && hidden <= 12288, "af_norm_of_sum: rows of 1 to 12288 values");
+  AF_REQUIRE(n_rows > 0 && hidden > 0 && hidden <= LN_MAX_ROW, "af_norm_of_sum: rows of 1 to %d values", LN_MAX_ROW);
   AF_REQUIRE(x != nullptr && a != nullptr && w != nullptr && bias != nullptr && (z == nullptr || z_bias != nullptr),
              "af_norm_of_sum: a stream, a term, the norm's weight and bias, a bias with a gate");
   AF_REQUIRE(hs == nullptr || (mu != nullptr && prev != nullptr && slots != nullptr),
@@ -330,9 +361,8 @@ AF_EXPORT int af_norm_of_sum(float* x, const void* a, int a_dtype, int a_parts, 
 #undef LN_LAUNCH
     AF_CHECK_LAUNCH("af_norm_of_sum");
   }
-  AF_DISPATCH_DTYPE(y_dtype, TY,
-                    af_launch(norm_of_sum_kernel<TY>, dim3(n_rows), dim3(256), (size_t)hidden * sizeof(float), stream, p));
-  AF_CHECK_LAUNCH("af_norm_of_sum");
+  AF_DISPATCH_DTYPE(y_dtype, TY, return ln_launch_sum<TY>(p, stream));
+  return 0;
 }
 
 AF_EXPORT int af_token_shift(void* hs, void* y, int dtype, const float* x, const float* mu, float* prev,

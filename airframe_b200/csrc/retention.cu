@@ -18,7 +18,6 @@
 namespace {
 
 constexpr int RT_TILE = 64;        // tokens of a tile
-constexpr int RT_PIECE = 64;       // key channels of a carried state staged at a time
 
 __device__ __forceinline__ uint32_t rt_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void rt_ldm4(uint32_t* r, const void* p) {
@@ -50,10 +49,13 @@ struct RtArgs {
   float magnitude;
   const float* powers;               // [heads][chunk + 1]: decay^0 .. decay^chunk
   int chunk;                         // tokens of a chunk (a multiple of RT_TILE)
-  float* local;                      // [chunks][heads][dv][dk]: B(c), then S_in(c)
+  float* local;                      // [chunks][heads][dv][dk]: B(c)
+  __nv_bfloat16 *k_hi, *k_lo;        // [tokens][heads][dkp]: the rotated keys in two parts
+  __nv_bfloat16 *v_hi, *v_lo;        // [tokens][heads][dvp]: the values
+  __nv_bfloat16 *s_hi, *s_lo;        // [chunks][heads][dv][dkp]: S_in(c)
   const int* chunk_starts;           // [chunks + 1] first rows
   const int* tiles;                  // [tiles][4]: first row, rows, chunk, the tile's first token in its chunk
-  int heads, dk, dv, dkp;            // dkp: dk rounded up to whole groups of 16
+  int heads, dk, dv, dkp, dvp;       // dkp, dvp: rounded up to whole groups of 16
   const float* gate;                 // float rows [tokens][heads * dv] (null: plain float outputs)
   long long gate_ts;
   int gate_act;                      // 0: sigmoid, 1: x sigmoid(x)
@@ -61,6 +63,7 @@ struct RtArgs {
   void* out;                         // [tokens][heads * dv]
   long long out_ts;
   int vec;                           // rows may be read in 16-byte pieces
+  int vec2;                          // gates and outputs may be read and written in pairs
 };
 
 // Four neighbouring channels c .. c + 3 of a head's query or key row of token t, rotated.
@@ -144,7 +147,7 @@ __global__ void __launch_bounds__(256)
 retention_step_kernel(RtStep p) {
   pdl_launch_dependents();
   namespace cg = cooperative_groups;
-  extern __shared__ float o_s[];     // [cols]
+  extern __shared__ __align__(16) float o_s[];     // [cols rounded up to 4], then the rotated query and key
   __shared__ float scratch[33];
   __shared__ float part_s;
   RtArgs a = p.a;
@@ -160,7 +163,10 @@ retention_step_kernel(RtStep p) {
     return;                          // (the whole cluster)
   }
   float* st = p.state + (((size_t)slot * a.heads + h) * a.dv + first) * a.dk + c0;
-  float S[R], qv[R], kv[R];
+  float S[R];
+  constexpr int RP = R + (R == 4 ? 0 : 4);   // (a lane's run of channels, apart from the next one's in the banks)
+  float* q_s = o_s + (p.cols + 3) / 4 * 4;
+  float* k_s = q_s + P * RP;
   auto read_state = [&](int j) {
     const float* src = st + (size_t)j * a.dk;
     if (a.vec) {
@@ -181,16 +187,16 @@ retention_step_kernel(RtStep p) {
   a.q = pdl_fresh(a.q), a.k = pdl_fresh(a.k), a.v = pdl_fresh(a.v), a.table = pdl_fresh(a.table), a.gate = pdl_fresh(a.gate);
   const float* qr = a.q + (size_t)t * a.q_ts + (size_t)h * a.dk;
   const float* kr = a.k + (size_t)t * a.k_ts + (size_t)h * a.dk;
-#pragma unroll
-  for (int i = 0; i < R; i += 4) {
-    if (c0 + i < a.dk) {
-      rt_rotated4(a, qr, t, c0 + i, qv + i);
-      rt_rotated4(a, kr, t, c0 + i, kv + i);
-    } else {
-#pragma unroll
-      for (int u = 0; u < 4; ++u) qv[i + u] = kv[i + u] = 0.f;
-    }
+  for (int i = tid; i < P * R / 2; i += 256) {     // four channels of the query or of the key a thread
+    const bool key = i >= P * R / 4;
+    const int c = (key ? i - P * R / 4 : i) * 4;
+    float y[4] = {0.f, 0.f, 0.f, 0.f};
+    if (c < a.dk) rt_rotated4(a, key ? kr : qr, t, c, y);
+    *reinterpret_cast<float4*>((key ? k_s : q_s) + (c / R) * RP + c % R) = make_float4(y[0], y[1], y[2], y[3]);
   }
+  __syncthreads();
+  const float* qv = q_s + part * RP;
+  const float* kv = k_s + part * RP;
   const float* vr = a.v + (size_t)t * a.v_ts + (size_t)h * a.dv + first;
   float ss = 0.f;
   for (int j0 = 0; j0 < n_cols; j0 += per) {
@@ -199,11 +205,16 @@ retention_step_kernel(RtStep p) {
     const float vj = j < n_cols ? vr[j] : 0.f;
     float o0 = 0.f, o1 = 0.f;
 #pragma unroll
-    for (int i = 0; i < R; i += 2) {
-      S[i] = dec * S[i] + kv[i] * vj;
-      S[i + 1] = dec * S[i + 1] + kv[i + 1] * vj;
-      o0 += qv[i] * S[i];
-      o1 += qv[i + 1] * S[i + 1];
+    for (int i = 0; i < R; i += 4) {
+      const float4 kq = *reinterpret_cast<const float4*>(kv + i), qq = *reinterpret_cast<const float4*>(qv + i);
+      S[i] = dec * S[i] + kq.x * vj;
+      S[i + 1] = dec * S[i + 1] + kq.y * vj;
+      S[i + 2] = dec * S[i + 2] + kq.z * vj;
+      S[i + 3] = dec * S[i + 3] + kq.w * vj;
+      o0 += qq.x * S[i];
+      o1 += qq.y * S[i + 1];
+      o0 += qq.z * S[i + 2];
+      o1 += qq.w * S[i + 3];
     }
     float o = o0 + o1;
     for (int w = 1; w < P; w <<= 1) o += __shfl_xor_sync(0xffffffffu, o, w);
@@ -245,7 +256,7 @@ int rt_launch_step(const RtStep& p, int blocks, int heads, int n_seqs, cudaStrea
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(blocks, heads, n_seqs);
   cfg.blockDim = dim3(256);
-  cfg.dynamicSmemBytes = (size_t)p.cols * sizeof(float);
+  cfg.dynamicSmemBytes = ((size_t)(p.cols + 3) / 4 * 4 + (size_t)2 * p.lanes * (R + 4)) * sizeof(float);
   cfg.stream = stream;
   cudaLaunchAttribute attr[2];
   attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
@@ -263,7 +274,7 @@ int rt_launch_step(const RtStep& p, int blocks, int heads, int n_seqs, cudaStrea
 // Block (chunk, head, value slice x key slice), 256 threads: S[v][c] = sum_t decay^(last - t) v_t[v] k_t[c] for a slice of
 // DVT value columns and DKT key channels; 8 warps as 4 (value rows) x 2 (key channels).
 template <int DVT, int DKT>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 2)
 retention_states_kernel(RtArgs a) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) unsigned char raw[];
@@ -289,25 +300,61 @@ retention_states_kernel(RtArgs a) {
       for (int e = 0; e < 4; ++e) acc[m][n][e] = 0.f;
   pdl_wait();
   a.q = pdl_fresh(a.q), a.k = pdl_fresh(a.k), a.v = pdl_fresh(a.v), a.table = pdl_fresh(a.table);
+  // (the keys of a slice are kept by the blocks of the first value slice, the values by those of the first key slice)
+  const bool keep_k = j0 == 0, keep_v = c0 == 0;
   for (int t0 = first; t0 < last; t0 += RT_TILE) {
     const int rows = min(RT_TILE, last - t0);
     __syncthreads();
-    for (int i = tid; i < RT_TILE * (DKT / 4); i += 256) {
-      const int r = i / (DKT / 4), c = (i - r * (DKT / 4)) * 4;
-      float y[4] = {0.f, 0.f, 0.f, 0.f};
-      if (r < rows && c0 + c < a.dk) {
-        rt_rotated4(a, a.k + (size_t)(t0 + r) * a.k_ts + (size_t)h * a.dk, t0 + r, c0 + c, y);
-        const float w = pw[last - 1 - t0 - r];
+    // four groups of four values at a time: their loads are in flight together
+    constexpr int KQ = DKT / 4, VQ = DVT / 4;
+#pragma unroll 1
+    for (int i0 = 0; i0 < RT_TILE * KQ; i0 += 1024) {
+      float y[4][4];
 #pragma unroll
-        for (int u = 0; u < 4; ++u) y[u] *= w;
+      for (int u = 0; u < 4; ++u) {
+        const int i = i0 + u * 256 + tid, r = min(i / KQ, rows - 1), c = c0 + (i % KQ) * 4;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) y[u][e] = 0.f;
+        if (c < a.dk) rt_rotated4(a, a.k + (size_t)(t0 + r) * a.k_ts + (size_t)h * a.dk, t0 + r, c, y[u]);
       }
-      rt_put4(k_hi + r * PK + c, k_lo + r * PK + c, y);
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const int i = i0 + u * 256 + tid, r = i / KQ, c = (i % KQ) * 4;
+        const bool on = r < rows;
+        if (on && keep_k && c0 + c < a.dkp) {
+          const size_t dst = ((size_t)(t0 + r) * a.heads + h) * a.dkp + c0 + c;
+          rt_put4(a.k_hi + dst, a.k_lo + dst, y[u]);
+        }
+        const float w = on ? pw[last - 1 - t0 - r] : 0.f;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) y[u][e] *= w;
+        rt_put4(k_hi + r * PK + c, k_lo + r * PK + c, y[u]);
+      }
     }
-    for (int i = tid; i < RT_TILE * (DVT / 4); i += 256) {
-      const int r = i / (DVT / 4), c = (i - r * (DVT / 4)) * 4;
-      float y[4] = {0.f, 0.f, 0.f, 0.f};
-      if (r < rows && j0 + c < a.dv) rt_plain4(a.v + (size_t)(t0 + r) * a.v_ts + (size_t)h * a.dv, j0 + c, a.dv, a.vec, y);
-      rt_put4(v_hi + r * PV + c, v_lo + r * PV + c, y);
+#pragma unroll 1
+    for (int i0 = 0; i0 < RT_TILE * VQ; i0 += 1024) {
+      float y[4][4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const int i = i0 + u * 256 + tid, r = min(i / VQ, rows - 1), c = j0 + (i % VQ) * 4;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) y[u][e] = 0.f;
+        if (c < a.dv) rt_plain4(a.v + (size_t)(t0 + r) * a.v_ts + (size_t)h * a.dv, c, a.dv, a.vec, y[u]);
+      }
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const int i = i0 + u * 256 + tid, r = i / VQ, c = (i % VQ) * 4;
+        if (r < rows) {
+          if (keep_v && j0 + c < a.dvp) {
+            const size_t dst = ((size_t)(t0 + r) * a.heads + h) * a.dvp + j0 + c;
+            rt_put4(a.v_hi + dst, a.v_lo + dst, y[u]);
+          }
+        } else {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) y[u][e] = 0.f;
+        }
+        rt_put4(v_hi + r * PV + c, v_lo + r * PV + c, y[u]);
+      }
     }
     __syncthreads();
 #pragma unroll
@@ -362,22 +409,24 @@ retention_states_kernel(RtArgs a) {
 
 // ---------------------------------------------------------------- states from chunk to chunk
 
-// One thread V state elements of a (sequence, head); the loads of four chunks are in flight at a time.
+// One thread V state elements of a (sequence, head); the loads of four chunks are in flight at a time.  The state that
+// enters a chunk goes out in two bfloat16 parts.
 template <int V>
 __global__ void __launch_bounds__(256)
-retention_carry_kernel(float* __restrict__ local, float* __restrict__ state, const float* __restrict__ powers,
-                       const int* __restrict__ chunk_starts, const int* __restrict__ seq_first_chunk,
-                       const int* __restrict__ slots, int heads, int per_head, int chunk) {
+retention_carry_kernel(RtArgs a, float* __restrict__ state, const int* __restrict__ seq_first_chunk,
+                       const int* __restrict__ slots) {
   pdl_launch_dependents();
+  const int per_head = a.dv * a.dk;
   const int e = (blockIdx.x * 256 + threadIdx.x) * V, h = blockIdx.y, b = blockIdx.z;
   const int slot = slots[b], ch0 = seq_first_chunk[b], ch1 = seq_first_chunk[b + 1];
-  const float* pw = powers + (size_t)h * (chunk + 1);
+  const float* pw = a.powers + (size_t)h * (a.chunk + 1);
+  const size_t at16 = (size_t)(e / a.dk) * a.dkp + e % a.dk;
   pdl_wait();
   if (e >= per_head || slot < 0) return;
-  local = pdl_fresh(local);
-  float* st = state + ((size_t)slot * heads + h) * per_head + e;
-  const size_t step = (size_t)heads * per_head;
-  float* p = local + (size_t)ch0 * step + (size_t)h * per_head + e;
+  float* st = state + ((size_t)slot * a.heads + h) * per_head + e;
+  const size_t step = (size_t)a.heads * per_head, step16 = (size_t)a.heads * a.dv * a.dkp;
+  const float* p = pdl_fresh(a.local) + (size_t)ch0 * step + (size_t)h * per_head + e;
+  size_t o = (size_t)ch0 * step16 + (size_t)h * a.dv * a.dkp + at16;
   float S[V];
   auto get = [](const float* src, float* dst) {
     if constexpr (V == 4) {
@@ -386,10 +435,6 @@ retention_carry_kernel(float* __restrict__ local, float* __restrict__ state, con
     } else {
       dst[0] = src[0];
     }
-  };
-  auto put = [](float* dst, const float* src) {
-    if constexpr (V == 4) *reinterpret_cast<float4*>(dst) = make_float4(src[0], src[1], src[2], src[3]);
-    else dst[0] = src[0];
   };
   get(st, S);
   for (int c = ch0; c < ch1; c += 4) {
@@ -400,87 +445,116 @@ retention_carry_kernel(float* __restrict__ local, float* __restrict__ state, con
 #pragma unroll
     for (int u = 0; u < 4; ++u) {
       if (c + u >= ch1) continue;
-      put(p + (size_t)u * step, S);
-      const float w = pw[chunk_starts[c + u + 1] - chunk_starts[c + u]];
+      const float w = pw[a.chunk_starts[c + u + 1] - a.chunk_starts[c + u]];
+      if constexpr (V == 4) {
+        rt_put4(a.s_hi + o + (size_t)u * step16, a.s_lo + o + (size_t)u * step16, S);
+      } else {
+        const __nv_bfloat16 hi = __float2bfloat16_rn(S[0]);
+        a.s_hi[o + (size_t)u * step16] = hi;
+        a.s_lo[o + (size_t)u * step16] = __float2bfloat16_rn(S[0] - __bfloat162float(hi));
+      }
 #pragma unroll
       for (int i = 0; i < V; ++i) S[i] = fmaf(w, S[i], B[u][i]);
     }
     p += 4 * step;
+    o += 4 * step16;
   }
-  put(st, S);
+  if constexpr (V == 4) *reinterpret_cast<float4*>(st) = make_float4(S[0], S[1], S[2], S[3]);
+  else st[0] = S[0];
 }
 
 // ---------------------------------------------------------------- outputs
 
-// Block (tile, head, value slice), four warps of 16 tokens each.
+__device__ __forceinline__ void rt_cp16(void* dst, const void* src, bool on) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(rt_smem(dst)), "l"(src), "r"(on ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void rt_cp_wait() {
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+}
+
+// Block (tile, head, value slice), eight warps: four groups of 16 tokens by two halves of the slice's value columns (both
+// halves work the scores out for themselves).  Keys, values and the entering state come in two parts as the kernels
+// in front left them, in whole 16-byte pieces without a register in between; the queries are rotated here.
 template <int DVT, typename TO, bool NORM>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256, 2)
 retention_outputs_kernel(RtArgs a) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) unsigned char raw[];
   const int PQ = a.dkp + 8;
-  constexpr int PV = DVT + 8, PS = RT_PIECE + 8;
+  constexpr int PV = DVT + 8;
   __nv_bfloat16* q_hi = reinterpret_cast<__nv_bfloat16*>(raw);
   __nv_bfloat16* q_lo = q_hi + RT_TILE * PQ;
   __nv_bfloat16* work = q_lo + RT_TILE * PQ;
-  __nv_bfloat16 *s_hi = work, *s_lo = work + DVT * PS;                                  // a piece of the carried state, or
+  __nv_bfloat16 *s_hi = work, *s_lo = work + DVT * PQ;                                  // the entering state, or
   __nv_bfloat16 *k_hi = work, *k_lo = work + RT_TILE * PQ;                              // a tile of keys and
   __nv_bfloat16 *v_hi = work + 2 * RT_TILE * PQ, *v_lo = v_hi + RT_TILE * PV;           // values
   __shared__ float pw[257];                        // decay^0 .. decay^chunk (chunks of up to 256 tokens)
+  __shared__ float sq[2][RT_TILE];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+  const int rg = warp & 3, half = warp >> 2;
   const int h = blockIdx.y, j0 = blockIdx.z * DVT;
   const int row0 = a.tiles[4 * blockIdx.x], rows = a.tiles[4 * blockIdx.x + 1], ch = a.tiles[4 * blockIdx.x + 2];
   const int at = a.tiles[4 * blockIdx.x + 3];      // the tile's first token in its chunk
-  for (int i = tid; i <= a.chunk; i += 128) pw[i] = a.powers[(size_t)h * (a.chunk + 1) + i];
+  for (int i = tid; i <= a.chunk; i += 256) pw[i] = a.powers[(size_t)h * (a.chunk + 1) + i];
   pdl_wait();
-  a.q = pdl_fresh(a.q), a.k = pdl_fresh(a.k), a.v = pdl_fresh(a.v), a.table = pdl_fresh(a.table);
-  a.local = pdl_fresh(a.local), a.gate = pdl_fresh(a.gate);
-  const int quads = a.dkp / 4;
-  for (int i = tid; i < RT_TILE * quads; i += 128) {
-    const int r = i / quads, c = (i - r * quads) * 4;
-    float y[4] = {0.f, 0.f, 0.f, 0.f};
-    if (r < rows && c < a.dk) rt_rotated4(a, a.q + (size_t)(row0 + r) * a.q_ts + (size_t)h * a.dk, row0 + r, c, y);
-    rt_put4(q_hi + r * PQ + c, q_lo + r * PQ + c, y);
+  a.q = pdl_fresh(a.q), a.table = pdl_fresh(a.table), a.gate = pdl_fresh(a.gate);
+  const int pieces = a.dkp / 8, quads = a.dkp / 4;
+  {
+    const size_t base = ((size_t)ch * a.heads + h) * a.dv;
+    for (int i = tid; i < DVT * pieces; i += 256) {
+      const int v = i / pieces, c = (i - v * pieces) * 8;
+      const bool on = j0 + v < a.dv;
+      const size_t src = (base + (on ? j0 + v : 0)) * a.dkp + c;
+      rt_cp16(s_hi + v * PQ + c, a.s_hi + src, on);
+      rt_cp16(s_lo + v * PQ + c, a.s_lo + src, on);
+    }
   }
-  constexpr int NT = DVT / 8;
+  for (int i0 = 0; i0 < RT_TILE * quads; i0 += 1024) {      // (RT_TILE * quads is a multiple of 256)
+    float y[4][4];
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      const int i = min(i0 + u * 256 + tid, RT_TILE * quads - 1), r = min(i / quads, rows - 1), c = (i % quads) * 4;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) y[u][e] = 0.f;
+      if (c < a.dk) rt_rotated4(a, a.q + (size_t)(row0 + r) * a.q_ts + (size_t)h * a.dk, row0 + r, c, y[u]);
+    }
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      const int i = i0 + u * 256 + tid, r = i / quads, c = (i % quads) * 4;
+      if (i < RT_TILE * quads) rt_put4(q_hi + r * PQ + c, q_lo + r * PQ + c, y[u]);
+    }
+  }
+  constexpr int NT = DVT / 16;                     // n8 tiles of a warp
+  const int n0 = half * (DVT / 2);
   float o[NT][4];
 #pragma unroll
   for (int n = 0; n < NT; ++n)
 #pragma unroll
     for (int e = 0; e < 4; ++e) o[n][e] = 0.f;
+  rt_cp_wait();
+  __syncthreads();
   // ---- what the state that enters the chunk gives
-  const float* S = a.local + ((size_t)ch * a.heads + h) * a.dv * a.dk;
-  for (int p0 = 0; p0 < a.dkp; p0 += RT_PIECE) {
-    const int width = min(RT_PIECE, a.dkp - p0);
-    __syncthreads();
-    for (int i = tid; i < DVT * (RT_PIECE / 4); i += 128) {
-      const int v = i / (RT_PIECE / 4), c = (i - v * (RT_PIECE / 4)) * 4;
-      float y[4] = {0.f, 0.f, 0.f, 0.f};
-      if (j0 + v < a.dv && p0 + c < a.dk) rt_plain4(S + (size_t)(j0 + v) * a.dk, p0 + c, a.dk, a.vec, y);
-      rt_put4(s_hi + v * PS + c, s_lo + v * PS + c, y);
-    }
-    __syncthreads();
-    for (int kk = 0; kk < width; kk += 16) {
-      uint32_t ah[4], al[4];
-      const int qa = (warp * 16 + (lane & 15)) * PQ + p0 + kk + (lane >> 4) * 8;
-      rt_ldm4(ah, q_hi + qa);
-      rt_ldm4(al, q_lo + qa);
+  for (int kk = 0; kk < a.dkp; kk += 16) {
+    uint32_t ah[4], al[4];
+    const int qa = (rg * 16 + (lane & 15)) * PQ + kk + (lane >> 4) * 8;
+    rt_ldm4(ah, q_hi + qa);
+    rt_ldm4(al, q_lo + qa);
 #pragma unroll
-      for (int n2 = 0; n2 < NT / 2; ++n2) {
-        uint32_t bh[4], bl[4];
-        const int sa = (n2 * 16 + (lane & 7) + (lane >> 4) * 8) * PS + kk + ((lane >> 3) & 1) * 8;
-        rt_ldm4(bh, s_hi + sa);
-        rt_ldm4(bl, s_lo + sa);
-        rt_mma(o[2 * n2], ah, bh[0], bh[1]);
-        rt_mma(o[2 * n2 + 1], ah, bh[2], bh[3]);
-        rt_mma(o[2 * n2], ah, bl[0], bl[1]);
-        rt_mma(o[2 * n2 + 1], ah, bl[2], bl[3]);
-        rt_mma(o[2 * n2], al, bh[0], bh[1]);
-        rt_mma(o[2 * n2 + 1], al, bh[2], bh[3]);
-      }
+    for (int n2 = 0; n2 < NT / 2; ++n2) {
+      uint32_t bh[4], bl[4];
+      const int sa = (n0 + n2 * 16 + (lane & 7) + (lane >> 4) * 8) * PQ + kk + ((lane >> 3) & 1) * 8;
+      rt_ldm4(bh, s_hi + sa);
+      rt_ldm4(bl, s_lo + sa);
+      rt_mma(o[2 * n2], ah, bh[0], bh[1]);
+      rt_mma(o[2 * n2 + 1], ah, bh[2], bh[3]);
+      rt_mma(o[2 * n2], ah, bl[0], bl[1]);
+      rt_mma(o[2 * n2 + 1], ah, bl[2], bl[3]);
+      rt_mma(o[2 * n2], al, bh[0], bh[1]);
+      rt_mma(o[2 * n2 + 1], al, bh[2], bh[3]);
     }
   }
-  const int lr0 = warp * 16 + g, lr1 = lr0 + 8;    // this lane's rows of the tile
+  const int lr0 = rg * 16 + g, lr1 = lr0 + 8;      // this lane's rows of the tile
   {
     const float w0 = pw[min(at + lr0 + 1, a.chunk)], w1 = pw[min(at + lr1 + 1, a.chunk)];
 #pragma unroll
@@ -491,21 +565,24 @@ retention_outputs_kernel(RtArgs a) {
     const int krow0 = row0 - at + kt;
     const bool own = kt == at;
     const int krows = own ? rows : RT_TILE;
-    __syncthreads();
-    for (int i = tid; i < RT_TILE * quads; i += 128) {
-      const int r = i / quads, c = (i - r * quads) * 4;
-      float y[4] = {0.f, 0.f, 0.f, 0.f};
-      if (r < krows && c < a.dk) rt_rotated4(a, a.k + (size_t)(krow0 + r) * a.k_ts + (size_t)h * a.dk, krow0 + r, c, y);
-      rt_put4(k_hi + r * PQ + c, k_lo + r * PQ + c, y);
+    __syncthreads();                               // (what lay in the work area is done with)
+    for (int i = tid; i < RT_TILE * pieces; i += 256) {
+      const int r = i / pieces, c = (i - r * pieces) * 8;
+      const bool on = r < krows;
+      const size_t src = ((size_t)(krow0 + (on ? r : 0)) * a.heads + h) * a.dkp + c;
+      rt_cp16(k_hi + r * PQ + c, a.k_hi + src, on);
+      rt_cp16(k_lo + r * PQ + c, a.k_lo + src, on);
     }
-    for (int i = tid; i < RT_TILE * (DVT / 4); i += 128) {
-      const int r = i / (DVT / 4), c = (i - r * (DVT / 4)) * 4;
-      float y[4] = {0.f, 0.f, 0.f, 0.f};
-      if (r < krows && j0 + c < a.dv) rt_plain4(a.v + (size_t)(krow0 + r) * a.v_ts + (size_t)h * a.dv, j0 + c, a.dv, a.vec, y);
-      rt_put4(v_hi + r * PV + c, v_lo + r * PV + c, y);
+    for (int i = tid; i < RT_TILE * (DVT / 8); i += 256) {
+      const int r = i / (DVT / 8), c = (i - r * (DVT / 8)) * 8;
+      const bool on = r < krows && j0 + c < a.dvp;
+      const size_t src = ((size_t)(krow0 + (on ? r : 0)) * a.heads + h) * a.dvp + (on ? j0 + c : 0);
+      rt_cp16(v_hi + r * PV + c, a.v_hi + src, on);
+      rt_cp16(v_lo + r * PV + c, a.v_lo + src, on);
     }
+    rt_cp_wait();
     __syncthreads();
-    const int groups = own ? warp + 1 : RT_TILE / 16;      // groups of 16 keys that this warp's tokens see
+    const int groups = own ? rg + 1 : RT_TILE / 16;        // groups of 16 keys that this warp's tokens see
     float s[RT_TILE / 8][4];
 #pragma unroll
     for (int n = 0; n < RT_TILE / 8; ++n)
@@ -513,7 +590,7 @@ retention_outputs_kernel(RtArgs a) {
       for (int e = 0; e < 4; ++e) s[n][e] = 0.f;
     for (int kk = 0; kk < a.dkp; kk += 16) {
       uint32_t ah[4], al[4];
-      const int qa = (warp * 16 + (lane & 15)) * PQ + kk + (lane >> 4) * 8;
+      const int qa = (rg * 16 + (lane & 15)) * PQ + kk + (lane >> 4) * 8;
       rt_ldm4(ah, q_hi + qa);
       rt_ldm4(al, q_lo + qa);
 #pragma unroll
@@ -531,7 +608,7 @@ retention_outputs_kernel(RtArgs a) {
         rt_mma(s[2 * n2 + 1], al, bh[2], bh[3]);
       }
     }
-    // the weights decay^(t - s); keys behind the token (and rows behind the tile's end) get none
+    // the weights decay^(t - s); keys behind the token get none
     const int d0 = at + lr0 - kt, d1 = d0 + 8;
 #pragma unroll
     for (int n = 0; n < RT_TILE / 8; ++n)
@@ -552,7 +629,7 @@ retention_outputs_kernel(RtArgs a) {
 #pragma unroll
       for (int n2 = 0; n2 < NT / 2; ++n2) {
         uint32_t bh[4], bl[4];
-        const int va = (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PV + n2 * 16 + (lane >> 4) * 8;
+        const int va = (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PV + n0 + n2 * 16 + (lane >> 4) * 8;
         rt_ldm4t(bh, v_hi + va);
         rt_ldm4t(bl, v_lo + va);
         rt_mma(o[2 * n2], ph, bh[0], bh[1]);
@@ -576,9 +653,19 @@ retention_outputs_kernel(RtArgs a) {
     for (int r = 0; r < 2; ++r) {
       ss[r] += __shfl_xor_sync(0xffffffffu, ss[r], 1);
       ss[r] += __shfl_xor_sync(0xffffffffu, ss[r], 2);
-      inv[r] *= rsqrtf(ss[r] / (float)a.dv + a.eps);
+      if (t4 == 0) sq[half][r ? lr1 : lr0] = ss[r];
+    }
+    __syncthreads();
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int lr = r ? lr1 : lr0;
+      inv[r] *= rsqrtf((sq[0][lr] + sq[1][lr]) / (float)a.dv + a.eps);
     }
   }
+  auto gated = [&](float y, float z) {
+    const float sg = 1.f / (1.f + expf(-z));
+    return y * (a.gate_act ? z * sg : sg);
+  };
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
     const int lr = r ? lr1 : lr0;
@@ -588,16 +675,19 @@ retention_outputs_kernel(RtArgs a) {
     const float* gr = NORM ? a.gate + tok * a.gate_ts + (size_t)h * a.dv : nullptr;
 #pragma unroll
     for (int n = 0; n < NT; ++n) {
-      const int c = j0 + n * 8 + 2 * t4;
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        if (c + e >= a.dv) continue;
-        float y = o[n][2 * r + e] * inv[r];
+      const int c = j0 + n0 + n * 8 + 2 * t4;
+      float y0 = o[n][2 * r] * inv[r], y1 = o[n][2 * r + 1] * inv[r];
+      if (a.vec2) {                                // (dv is even: a pair lies inside or outside)
+        if (c >= a.dv) continue;
         if (NORM) {
-          const float z = gr[c + e], sg = 1.f / (1.f + expf(-z));
-          y *= a.gate_act ? z * sg : sg;
+          const float2 z = *reinterpret_cast<const float2*>(gr + c);
+          y0 = gated(y0, z.x), y1 = gated(y1, z.y);
         }
-        dst[c + e] = from_f32<TO>(y);
+        if constexpr (sizeof(TO) == 2) *reinterpret_cast<__nv_bfloat162*>(dst + c) = __floats2bfloat162_rn(y0, y1);
+        else *reinterpret_cast<float2*>(dst + c) = make_float2(y0, y1);
+      } else {
+        if (c < a.dv) dst[c] = from_f32<TO>(NORM ? gated(y0, gr[c]) : y0);
+        if (c + 1 < a.dv) dst[c + 1] = from_f32<TO>(NORM ? gated(y1, gr[c + 1]) : y1);
       }
     }
   }
@@ -605,7 +695,7 @@ retention_outputs_kernel(RtArgs a) {
 
 size_t rt_outputs_smem(int dkp, int dvt) {
   const size_t q = (size_t)2 * RT_TILE * (dkp + 8), kv = (size_t)2 * RT_TILE * (dkp + 8) + (size_t)2 * RT_TILE * (dvt + 8);
-  const size_t s = (size_t)2 * dvt * (RT_PIECE + 8);
+  const size_t s = (size_t)2 * dvt * (dkp + 8);
   return (q + (kv > s ? kv : s)) * sizeof(__nv_bfloat16);
 }
 
@@ -635,7 +725,7 @@ template <int DVT, typename TO, bool NORM>
 int rt_launch_outputs(const RtArgs& a, int n_tiles, cudaStream_t stream) {
   static bool raised[AF_MAX_DEVICES];
   if (int e = rt_raise(retention_outputs_kernel<DVT, TO, NORM>, raised, rt_outputs_smem(256, DVT))) return e;
-  af_launch(retention_outputs_kernel<DVT, TO, NORM>, dim3(n_tiles, a.heads, (a.dv + DVT - 1) / DVT), dim3(128),
+  af_launch(retention_outputs_kernel<DVT, TO, NORM>, dim3(n_tiles, a.heads, (a.dv + DVT - 1) / DVT), dim3(256),
             rt_outputs_smem(a.dkp, DVT), stream, a);
   AF_COUNT_LAUNCH("af_retention_prompt (outputs)");
   return 0;
@@ -647,13 +737,15 @@ int rt_launch_outputs(const RtArgs& a, int n_tiles, cudaStream_t stream) {
 AF_EXPORT int af_retention_prompt_supported(int dk, int dv) { return dk >= 1 && dk <= 256 && dv >= 1 ? 1 : 0; }
 
 // y (bfloat16, contiguous [tokens][heads * dv]) = norm per head (key_scale o) * gate, for dv <= 128; with gate null, out is
-// float [tokens][heads * dv] = key_scale o.  local: scratch [n_chunks][heads][dv][dk].
+// float [tokens][heads * dv] = key_scale o.  Scratch: local float [n_chunks][heads][dv][dk]; with the head sizes rounded
+// up to 16, kv16 bfloat16 2 x [n_tokens][heads][dkp] (keys) then 2 x [n_tokens][heads][dvp] (values), s16 2 x
+// [n_chunks][heads][dv][dkp] (zeros behind dk on entry).
 AF_EXPORT int af_retention_prompt(void* out, const float* q, long long q_ts, const float* k, long long k_ts, const float* v,
                                   long long v_ts, const float* gate, long long gate_ts, int gate_act, const float* table,
                                   int n_rot, int adjacent, float magnitude, const float* powers, int chunk, float* local,
-                                  float* state, const int* chunk_starts, const int* seq_first_chunk, const int* tiles,
-                                  const int* slots, int n_chunks, int n_seqs, int n_tiles, int heads, int dk, int dv,
-                                  float key_scale, float eps, cudaStream_t stream) {
+                                  void* kv16, void* s16, float* state, const int* chunk_starts, const int* seq_first_chunk, const int* tiles,
+                                  const int* slots, int n_tokens, int n_chunks, int n_seqs, int n_tiles, int heads,
+                                  int dk, int dv, float key_scale, float eps, cudaStream_t stream) {
   if (n_tiles == 0) return 0;
   AF_REQUIRE(n_chunks > 0 && n_seqs > 0 && heads > 0 && heads < 65536 && n_seqs < 65536, "af_retention_prompt: bad sizes");
   AF_REQUIRE(af_retention_prompt_supported(dk, dv), "af_retention_prompt: heads of %d keys and %d values", dk, dv);
@@ -666,6 +758,12 @@ AF_EXPORT int af_retention_prompt(void* out, const float* q, long long q_ts, con
   a.chunk_starts = chunk_starts, a.tiles = tiles, a.heads = heads, a.dk = dk, a.dv = dv, a.dkp = (dk + 15) / 16 * 16;
   a.gate = gate, a.gate_ts = gate_ts, a.gate_act = gate_act, a.key_scale = key_scale, a.eps = eps, a.out = out;
   a.out_ts = (long long)heads * dv;
+  a.dvp = (dv + 15) / 16 * 16;
+  const size_t nk = (size_t)n_tokens * heads * a.dkp, nv = (size_t)n_tokens * heads * a.dvp;
+  a.k_hi = (__nv_bfloat16*)kv16, a.k_lo = a.k_hi + nk, a.v_hi = a.k_lo + nk, a.v_lo = a.v_hi + nv;
+  a.s_hi = (__nv_bfloat16*)s16, a.s_lo = a.s_hi + (size_t)n_chunks * heads * dv * a.dkp;
+  AF_REQUIRE((((uintptr_t)kv16 | (uintptr_t)s16) & 15) == 0, "af_retention_prompt: 16-byte aligned scratch");
+  a.vec2 = dv % 2 == 0 && (gate_ts & 1) == 0 && (((uintptr_t)gate | (uintptr_t)out) & 7) == 0;
   a.vec = dk % 4 == 0 && dv % 4 == 0 && n_rot % 4 == 0 && ((q_ts | k_ts | v_ts) & 3) == 0 &&
           (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)table | (uintptr_t)local | (uintptr_t)state) & 15) == 0;
   int e = 0;
@@ -673,13 +771,12 @@ AF_EXPORT int af_retention_prompt(void* out, const float* q, long long q_ts, con
   else e = dk <= 64 ? rt_launch_states<128, 64>(a, n_chunks, stream) : rt_launch_states<128, 128>(a, n_chunks, stream);
   if (e) return e;
   const int per_head = dk * dv;
-  if (a.vec) {
-    af_launch(retention_carry_kernel<4>, dim3((per_head / 4 + 255) / 256, heads, n_seqs), dim3(256), 0, stream, local, state,
-              powers, chunk_starts, seq_first_chunk, slots, heads, per_head, chunk);
-  } else {
-    af_launch(retention_carry_kernel<1>, dim3((per_head + 255) / 256, heads, n_seqs), dim3(256), 0, stream, local, state,
-              powers, chunk_starts, seq_first_chunk, slots, heads, per_head, chunk);
-  }
+  if (a.vec)
+    af_launch(retention_carry_kernel<4>, dim3((per_head / 4 + 255) / 256, heads, n_seqs), dim3(256), 0, stream, a, state,
+              seq_first_chunk, slots);
+  else
+    af_launch(retention_carry_kernel<1>, dim3((per_head + 255) / 256, heads, n_seqs), dim3(256), 0, stream, a, state,
+              seq_first_chunk, slots);
   AF_COUNT_LAUNCH("af_retention_prompt (carry)");
   if (gate != nullptr)
     return dv <= 64 ? rt_launch_outputs<64, __nv_bfloat16, true>(a, n_tiles, stream)

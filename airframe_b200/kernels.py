@@ -1749,14 +1749,18 @@ def retention_prompt(out, q, k, v, gate, table, powers, state, batch, heads: int
         raise KernelError(f"retention_prompt: state float32 [slots, {heads}, {dv}, {dk}], powers [{heads}, {chunk + 1}]")
     rows, turn = _retention_args(q, k, v, gate, table, heads, dk, dv, pairing, "retention_prompt")
     starts, seq_first, tiles, n_chunks, n_tiles = _retention_chunks(batch, chunk)
-    local = torch.empty(n_chunks, heads, dv, dk, dtype=torch.float32, device=out.device)
+    dev, bf16 = out.device, torch.bfloat16
+    dkp, dvp = -(-dk // 16) * 16, -(-dv // 16) * 16
+    local = torch.empty(n_chunks, heads, dv, dk, dtype=torch.float32, device=dev)
+    kv16 = torch.empty(2 * T * heads * (dkp + dvp), dtype=bf16, device=dev)
+    s16 = (torch.empty if dkp == dk else torch.zeros)(2 * n_chunks * heads * dv * dkp, dtype=bf16, device=dev)
     i32 = torch.int32
     _check(_lib().af_retention_prompt(_ptr(out), *rows, c_int(GATE_ACTS[gate_act]), *turn, c_float(magnitude),
-                                      _ptr(powers, "powers", torch.float32), c_int(chunk), _ptr(local), _ptr(state, "state"),
-                                      _ptr(starts, "chunk_starts", i32), _ptr(seq_first, "seq_first", i32),
-                                      _ptr(tiles, "tiles", i32), _ptr(batch.slots, "slots", i32), c_int(n_chunks),
-                                      c_int(batch.n_seqs), c_int(n_tiles), c_int(heads), c_int(dk), c_int(dv),
-                                      c_float(key_scale), c_float(eps), _stream()))
+                                      _ptr(powers, "powers", torch.float32), c_int(chunk), _ptr(local), _ptr(kv16), _ptr(s16),
+                                      _ptr(state, "state"), _ptr(starts, "chunk_starts", i32), _ptr(seq_first, "seq_first", i32),
+                                      _ptr(tiles, "tiles", i32), _ptr(batch.slots, "slots", i32), c_int(T),
+                                      c_int(n_chunks), c_int(batch.n_seqs), c_int(n_tiles), c_int(heads), c_int(dk),
+                                      c_int(dv), c_float(key_scale), c_float(eps), _stream()))
 
 
 def conv_pack(qkv, proj, batch, H: int, G: int, d: int, dv: int, pk: int, pv: int, bias=None, taps_w=None, history=None,
@@ -1821,7 +1825,7 @@ __all__ = [n for n in dir() if not n.startswith("_")]
 
 # ---------------------------------------------------------------- a norm behind the residual sum, the token shift
 
-LAYER_NORM_MAX = 12288     # values a row of these kernels
+LAYER_NORM_MAX = 16384     # values a row of these kernels
 
 
 def layer_norm(y, x, w, b, eps: float, rows=None) -> None:
