@@ -12,6 +12,7 @@ from ctypes import c_float, c_int, c_longlong, c_void_p
 
 import torch
 
+from . import transfers
 from .csrc import KernelLibraryError, load_library
 from .kernels_const import PAGE
 
@@ -1727,8 +1728,9 @@ def _retention_chunks(batch, chunk: int):
             row += n
             first.append(len(starts))
         starts.append(row)
-        flat = starts + first + [x for t in tiles for x in t]
-        dev = torch.tensor(flat, dtype=torch.int32).to(batch.tokens.device)
+        host = torch.tensor(starts + first + [x for t in tiles for x in t], dtype=torch.int32).pin_memory()
+        dev = host.to(batch.tokens.device, non_blocking=True)
+        transfers.count_h2d(host)
         a, b = len(starts), len(starts) + len(first)
         batch.aux[key] = (dev[:a], dev[a:b], dev[b:], len(starts) - 1, len(tiles))
     return batch.aux[key]

@@ -335,7 +335,7 @@ def _loud(name, t):
         t = t.clone()
         t[0] *= 5.0
     if name.endswith("mix.uq"):
-        t = t * 25.0
+        t = t * 4.0
     return t
 
 

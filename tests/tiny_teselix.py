@@ -117,8 +117,10 @@ def make_folder(cfg_dict, seed=0, store_dtype="bfloat16", root=None, edit=None):
                     t = t * (6.0 if ".mlp." in d.name else 3.0)
                 if d.kind == "table":
                     t = t * 20.0
+                if d.name.endswith(("mix.uq", "mix.uv", "mix.o")):
+                    t = t * (6.0 if d.name.endswith("uq") else 3.0)
                 if d.kind == "norm":
-                    t = t * (8.0 if d.name.endswith("sink") else 3.0)
+                    t = t * 8.0 + 2.0 if d.name.endswith("sink") else t * 3.0
                 if edit is not None:
                     t = edit(d.name, t)
                 return t.to(dt)
