@@ -100,6 +100,51 @@ layer_norm_kernel(TY* __restrict__ y, const float* __restrict__ x, const float* 
     y[r * hidden + i] = from_f32<TY>((row[i] - mean) * inv * w[i] + b[i]);
 }
 
+// Rows of whole groups of four: a thread keeps NV groups in registers, the weights are asked for before the wait (they
+// are cold in a decode step: the step's other weights have pushed them out of L2).
+template <typename TY, int NV>
+__global__ void __launch_bounds__(1024)
+layer_norm_row_kernel(TY* __restrict__ y, const float* __restrict__ x, const float* __restrict__ w,
+                      const float* __restrict__ b, const int* __restrict__ rows, int hidden, float eps) {
+  pdl_launch_dependents();
+  __shared__ float scratch[33];
+  const size_t r = blockIdx.x;
+  float4 wv[NV], bv[NV], v[NV];
+#pragma unroll
+  for (int n = 0; n < NV; ++n) {
+    const int i = (threadIdx.x + n * blockDim.x) * 4;
+    wv[n] = bv[n] = v[n] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < hidden) wv[n] = *reinterpret_cast<const float4*>(w + i), bv[n] = *reinterpret_cast<const float4*>(b + i);
+  }
+  const size_t src = rows != nullptr ? (size_t)rows[r] : r;
+  pdl_wait();
+  x = pdl_fresh(x);
+  float s = 0.f;
+#pragma unroll
+  for (int n = 0; n < NV; ++n) {
+    const int i = (threadIdx.x + n * blockDim.x) * 4;
+    if (i < hidden) v[n] = *reinterpret_cast<const float4*>(x + src * hidden + i);
+    s += v[n].x + v[n].y + v[n].z + v[n].w;
+  }
+  const float mean = block_sum(s, scratch) / (float)hidden;
+  float ss = 0.f;
+#pragma unroll
+  for (int n = 0; n < NV; ++n) {
+    v[n].x -= mean, v[n].y -= mean, v[n].z -= mean, v[n].w -= mean;
+    if ((threadIdx.x + n * blockDim.x) * 4 < hidden)
+      ss += v[n].x * v[n].x + v[n].y * v[n].y + v[n].z * v[n].z + v[n].w * v[n].w;
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)hidden + eps);
+#pragma unroll
+  for (int n = 0; n < NV; ++n) {
+    const int i = (threadIdx.x + n * blockDim.x) * 4;
+    if (i >= hidden) continue;
+    const float o[4] = {v[n].x * inv * wv[n].x + bv[n].x, v[n].y * inv * wv[n].y + bv[n].y,
+                        v[n].z * inv * wv[n].z + bv[n].z, v[n].w * inv * wv[n].w + bv[n].w};
+    ln_store4(y + r * hidden + i, o);
+  }
+}
+
 // ---------------------------------------------------------------- the norm of the residual sum
 
 // Any row size: the row waits in shared memory between the passes.
@@ -288,6 +333,14 @@ int ln_raise(K kernel, bool* flags, int hidden) {
 template <typename TY>
 int ln_launch(void* y, const float* x, const float* w, const float* b, const int* rows, int n_rows, int hidden, float eps,
               cudaStream_t stream) {
+  if (hidden % 4 == 0 && hidden <= 8192 && (((uintptr_t)y | (uintptr_t)x | (uintptr_t)w | (uintptr_t)b) & 15) == 0) {
+    const int nv = hidden > 4096 ? 2 : 1, threads = ((hidden / 4 + nv - 1) / nv + 31) / 32 * 32;
+    if (nv == 2)
+      af_launch(layer_norm_row_kernel<TY, 2>, dim3(n_rows), dim3(threads), 0, stream, (TY*)y, x, w, b, rows, hidden, eps);
+    else
+      af_launch(layer_norm_row_kernel<TY, 1>, dim3(n_rows), dim3(threads), 0, stream, (TY*)y, x, w, b, rows, hidden, eps);
+    AF_CHECK_LAUNCH("af_layer_norm");
+  }
   static bool raised[AF_MAX_DEVICES];
   if (int e = ln_raise(layer_norm_kernel<TY>, raised, hidden)) return e;
   af_launch(layer_norm_kernel<TY>, dim3(n_rows), dim3(256), (size_t)hidden * sizeof(float), stream, (TY*)y, x, w, b, rows,
