@@ -715,10 +715,11 @@ def side_by_side(args, which, points, make, arm_name, beside=("gemma2",)) -> Non
             pf_kernels = kernels_of(prefill_once)
             slots = [eng.take_slot() for _ in range(B)]
             eng.step([StepEntry(s, p, [P - 1]) for s, p in zip(slots, ps)])
-            tok = [1] * B
+            # every step other tokens (experts that are looked up by token would otherwise be the same few for the whole batch)
+            toks = iter(torch.randint(0, V, (2 + W + K, B), generator=g).tolist())
 
             def one():
-                eng.step([StepEntry(s, [t], [0]) for s, t in zip(slots, tok)], borrow=True)
+                eng.step([StepEntry(s, [t], [0]) for s, t in zip(slots, next(toks))], borrow=True)
 
             one()
             eng.repeat_last_decode(SETTLE)
