@@ -136,11 +136,11 @@ class Model:
             blk = self.blocks[e.layer]
             if e.enter is not None:
                 normed = self.junctions[e.enter].forward(x, x0, e.enter_index, batch,
-                                                         then=blk.reader(cache.views[i], batch), out_dtype=self.ctx.compute_dtype)
+                                                         then=blk.first_read(cache.views[i], batch), out_dtype=self.ctx.compute_dtype)
             # the last kernel of a run also makes the next run's first norm, unless a junction rewrites the stream first
             nxt = None
             if i + 1 < len(sched) and sched[i + 1].enter is None:
-                nxt = self.blocks[sched[i + 1].layer].reader(cache.views[i + 1], batch)
+                nxt = self.blocks[sched[i + 1].layer].first_read(cache.views[i + 1], batch)
             normed = blk.forward(x, batch, cache.views[i], normed=normed, next_pre=nxt)
             if probe is not None:
                 probe.after(i, e.layer, self._sum_streams(x) if self.streams > 1 else x, batch)

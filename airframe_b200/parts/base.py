@@ -283,7 +283,7 @@ class Block(Part):
         ``block_state``)."""
         return None
 
-    def reader(self, view, batch):
+    def first_read(self, view, batch):
         """What a run of this block with the cache view ``view`` reads first in the step ``batch``: something with a
         ``forward(x, out_dtype)`` that the run before may compute in its last kernel (the first norm, for most blocks)."""
         return self.first_norm()

@@ -203,9 +203,9 @@ class NormedSumBlock(Block):
         return super().prefill_flops(lens) + 2 * sum(lens) * self._gate_numel()
 
     def first_norm(self):
-        raise ConfigError("normed_sum: what a run reads first depends on its state (see Block.reader)")
+        raise ConfigError("normed_sum: what a run reads first depends on its state (see Block.first_read)")
 
-    def reader(self, view, batch):
+    def first_read(self, view, batch):
         return ShiftedReader(self, view, batch)
 
     def _gate(self, which: int, y):
