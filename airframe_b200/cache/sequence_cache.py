@@ -7,7 +7,8 @@ owns K and V pages ``[runs, pages, kv_heads, PAGE, head_dim]`` (value rows may
 have a size of their own, or be left out when a mixer keeps them inside its key rows) and a page
 table ``[slots, pages per sequence]``.  A group with a window keeps rows
 modulo ``ring_rows`` (the window rounded up to whole pages), so a sequence
-never holds more than ``ring_rows`` rows there.  Pages are taken as a
+never holds more than ``ring_rows`` rows there; where the window keeps the sequence's
+first tokens in sight, their pages come before the ring's and stay.  Pages are taken as a
 sequence grows and given back, with the slot, when it ends; both are used
 again by later sequences.
 
@@ -50,7 +51,8 @@ class KVGroup:
         self.run_ids = list(run_ids)
         self.index_of = {r: i for i, r in enumerate(self.run_ids)}
         self.ring_rows = pages_for(need.window) * PAGE if need.window else 0
-        cap_rows = min(self.ring_rows, max_context) if self.ring_rows else max_context
+        self.kept_rows = pages_for(need.keep_first) * PAGE if need.window else 0      # (before the ring)
+        cap_rows = min(self.kept_rows + self.ring_rows, max_context) if self.ring_rows else max_context
         self.pages_per_seq = max(1, pages_for(cap_rows))
         self.n_pages = n_pages
         self.pages = IndexPool(n_pages, "cache page")
@@ -66,7 +68,7 @@ class KVGroup:
             self.table = torch.full((n_slots, self.pages_per_seq), -1, dtype=torch.int32, device=device)
 
     def rows_held(self, length: int) -> int:
-        return min(length, self.ring_rows) if self.ring_rows else length
+        return min(length, self.kept_rows + self.ring_rows) if self.ring_rows else length
 
     def pages_missing(self, slot: int, new_len: int) -> int:
         return max(0, pages_for(self.rows_held(new_len)) - len(self.held[slot]))
@@ -74,7 +76,7 @@ class KVGroup:
     def room(self, slot: int) -> int:
         """Tokens the sequence may hold before this group needs another page."""
         held = len(self.held[slot])
-        if self.ring_rows and held * PAGE >= self.ring_rows:
+        if self.ring_rows and held * PAGE >= self.kept_rows + self.ring_rows:
             return 1 << 62                  # the ring is complete: it never grows again
         return held * PAGE
 
@@ -122,8 +124,9 @@ class KVView:
     k: Optional[torch.Tensor]           # [pages, kv_heads, PAGE, head_dim]
     v: Optional[torch.Tensor]
     page_table: Optional[torch.Tensor]  # [slots, pages per sequence] int32
-    ring_rows: int                      # 0: rows are positions; else rows are positions modulo this
+    ring_rows: int                      # 0: rows are positions; else rows behind the kept pages are a ring of this many
     need: KVNeed
+    keep_first: int = 0                 # the first tokens that stay beside a window: their pages come before the ring
 
 
 @dataclass
@@ -133,7 +136,7 @@ class LayerCacheView:
     writes: bool                        # False: the run reads another run's keys and values
     keep_step_kv: bool                  # a later run reads this run's keys and values
     kv: Optional[KVView]
-    state: Optional[torch.Tensor]       # [slots, *shape]: the mixer's
+    state: Optional[torch.Tensor]       # [slots, *shape]: the mixer's (a tuple of them for a mixer that asked for several)
     block_state: Optional[torch.Tensor] = None      # [slots, *shape]: what the layer's arrangement keeps
 
 
@@ -176,7 +179,7 @@ class SequenceCache:
         for need, runs in by_need.items():
             n_pages = self.total_pages
             if need.window:
-                ring_pages = pages_for(min(pages_for(need.window) * PAGE, self.max_context))
+                ring_pages = pages_for(min((pages_for(need.keep_first) + pages_for(need.window)) * PAGE, self.max_context))
                 n_pages = min(n_pages, self.n_slots * ring_pages)
             self.groups[need] = KVGroup(need, runs, self.n_slots, n_pages, self.max_context, dtype, device)
         for run, (kv_need, state_need, cache_from, block_need) in enumerate(needs):
@@ -186,23 +189,30 @@ class SequenceCache:
             if kv_need is not None:
                 if src_need is None:
                     raise ValueError(f"run {run} reads keys and values of run {src}, which keeps none")
-                if (src_need.num_kv_heads, src_need.head_dim, src_need.value_size) != \
-                        (kv_need.num_kv_heads, kv_need.head_dim, kv_need.value_size):
-                    raise ValueError(f"run {run} reads the cache of run {src} with other head sizes")
+                if (src_need.num_kv_heads, src_need.head_dim, src_need.value_size, src_need.keep_first) != \
+                        (kv_need.num_kv_heads, kv_need.head_dim, kv_need.value_size, kv_need.keep_first):
+                    raise ValueError(f"run {run} reads the cache of run {src} with other head sizes or kept tokens")
                 g = self.groups[src_need]
                 i = g.index_of[src]
                 kv_view = KVView(g.k[i] if g.k is not None else None, g.v[i] if g.v is not None else None,
-                                 g.table, g.ring_rows, src_need)
-            held = []
-            for key, need in ((run, state_need), ((run, "block"), block_need)):
-                state = None
-                if need is not None:
-                    if device is not None:
-                        state = torch.zeros((self.n_slots, *need.shape), dtype=_STATE_DTYPES[need.dtype], device=device)
-                    self.states[key] = state
-                held.append(state)
+                                 g.table, g.ring_rows, src_need, src_need.keep_first if g.ring_rows else 0)
+            if isinstance(state_need, tuple):
+                state = tuple(self._new_state((run, i), need) for i, need in enumerate(state_need))
+            else:
+                state = self._new_state(run, state_need)
+            held = [state, self._new_state((run, "block"), block_need)]
             self.views.append(LayerCacheView(cache_id=src, writes=cache_from is None,
                                              keep_step_kv=run in readers, kv=kv_view, state=held[0], block_state=held[1]))
+
+    def _new_state(self, key, need):
+        """A state of fixed size per slot under ``key``, or None when nothing is asked for (or only bookkeeping exists)."""
+        if need is None:
+            return None
+        state = None
+        if self.device is not None:
+            state = torch.zeros((self.n_slots, *need.shape), dtype=_STATE_DTYPES[need.dtype], device=self.device)
+        self.states[key] = state
+        return state
 
     # ------------------------------------------------------------------ slots
 

@@ -67,6 +67,7 @@ struct DecodeArgs {
   int nq, nkv;
   float scale, cap;
   int window, ring_rows;
+  int keep;        // a window's sequence keeps its first `keep` tokens in sight
   int n_splits;    // at most this many splits of a sequence's keys (the stride of the partial results)
   int batch, n_sms;
   float* part_o;   // [batch, nq, splits, HD]
@@ -107,20 +108,25 @@ __device__ __forceinline__ int da_lo(int pos, int window) {
   return window > 0 ? max(0, pos - window + 1) : (window < 0 ? pos - pos % (-window) : 0);
 }
 
-// Pages of the cache that sequence b's new token attends to: [first, last].
-__device__ __forceinline__ int da_pages(const int* slots, const int* lens, int b, int window, int* first_pp, int* last_pp) {
+// The pages of a sequence that its token at `pos` attends to: the pages of the kept first tokens, then the window's up to
+// the token's own.  The pages count through; `skip` of them lie between the two parts.
+struct DaList {
+  int kept, skip, n;
+};
+__device__ __forceinline__ DaList da_list(int pos, int window, int keep) {
+  DaList l;
+  l.kept = af_kept_pages(keep);
+  l.skip = max(0, da_lo(pos, window) / AF_PAGE - l.kept);
+  l.n = pos / AF_PAGE + 1 - l.skip;
+  return l;
+}
+__device__ __forceinline__ int da_page_of(int kept, int skip, int x) { return x >= kept ? x + skip : x; }
+
+// How many pages of the cache sequence b's new token attends to.
+__device__ __forceinline__ int da_pages(const int* slots, const int* lens, int b, int window, int keep) {
   const int slot = slots[b], len_b = lens[b];   // (both loads at once: neither waits for the other)
   const int len = slot >= 0 ? len_b : 0;
-  if (len <= 0) {
-    *first_pp = 0;
-    *last_pp = -1;
-    return 0;
-  }
-  const int pos = len - 1;
-  const int lo = da_lo(pos, window);
-  *first_pp = lo / AF_PAGE;
-  *last_pp = pos / AF_PAGE;
-  return *last_pp - *first_pp + 1;
+  return len > 0 ? da_list(len - 1, window, keep).n : 0;
 }
 
 template <int HD>
@@ -165,14 +171,14 @@ struct DaPlan {
 // The plan, by one whole warp (every lane returns the same).  32-bit arithmetic all through: the launcher has
 // checked that batch x pages x units stays below 2^31.  If `pages_s` is given it gets the pages of the sequences
 // before b, and `splits_s` their splits in the even cut (b = 0 .. batch).
-__device__ __forceinline__ DaPlan da_plan(const int* slots, const int* lens, int batch, int window, int units_per_seq,
+__device__ __forceinline__ DaPlan da_plan(const int* slots, const int* lens, int batch, int window, int keep, int units_per_seq,
                                           int grid_blocks, int room, int b_query, int* pages_s, int* splits_s) {
   const int lane = threadIdx.x & 31;
-  int carry = 0, most = 0, before = 0, f, l, P_first = 0;
+  int carry = 0, most = 0, before = 0, P_first = 0;
   if (pages_s && lane == 0) pages_s[0] = 0;
   for (int base = 0; base < batch; base += 32) {
     const int i = base + lane;
-    const int P = i < batch ? da_pages(slots, lens, i, window, &f, &l) : 0;
+    const int P = i < batch ? da_pages(slots, lens, i, window, keep) : 0;
     if (base == 0) P_first = P;
     most = max(most, P);
     if (i < b_query) before += P;
@@ -195,7 +201,7 @@ __device__ __forceinline__ DaPlan da_plan(const int* slots, const int* lens, int
   int items1 = 0, worst1 = 0, items2 = 0, worst2 = 0;
   for (int base = 0; base < batch; base += 32) {
     const int i = base + lane;
-    const int P = base == 0 ? P_first : (i < batch ? da_pages(slots, lens, i, window, &f, &l) : 0);
+    const int P = base == 0 ? P_first : (i < batch ? da_pages(slots, lens, i, window, keep) : 0);
     const int sp1 = da_even_splits(P, pl.share, room, 1), sp2 = da_even_splits(P, pl.share, room, 2);
     if (P > 0) {
       worst1 = max(worst1, (P + sp1 - 1) / sp1);
@@ -218,7 +224,7 @@ __device__ __forceinline__ DaPlan da_plan(const int* slots, const int* lens, int
     if (lane == 0) splits_s[0] = 0;
     for (int base = 0; base < batch; base += 32) {
       const int i = base + lane;
-      const int P = base == 0 ? P_first : (i < batch ? da_pages(slots, lens, i, window, &f, &l) : 0);
+      const int P = base == 0 ? P_first : (i < batch ? da_pages(slots, lens, i, window, keep) : 0);
       int v = da_even_splits(P, pl.share, room, pl.even);
 #pragma unroll
       for (int o = 1; o < 32; o <<= 1) {
@@ -306,7 +312,7 @@ __host__ __device__ inline long long da_plan_records_at(int batch, int units_per
 __global__ void __launch_bounds__(256)
 attn_decode_plan_kernel(int* __restrict__ plan, const int* __restrict__ slots, const int* __restrict__ lens,
                         const int* __restrict__ page_table, int max_pages, int batch, int nq, int nkv, int window,
-                        int ring_rows, int room, int grid_blocks) {
+                        int keep, int ring_rows, int room, int grid_blocks) {
   extern __shared__ int dp_smem[];
   int* pages_s = dp_smem;                 // [batch + 1]
   int* splits_s = dp_smem + batch + 1;    // [batch + 1]
@@ -314,7 +320,7 @@ attn_decode_plan_kernel(int* __restrict__ plan, const int* __restrict__ slots, c
   pdl_wait();
   const int group = nq / nkv, tiles = (group + 15) / 16, units_per_seq = nkv * tiles;
   if (threadIdx.x < 32) {
-    const DaPlan pl = da_plan(slots, lens, batch, window, units_per_seq, grid_blocks, room, 0, pages_s, splits_s);
+    const DaPlan pl = da_plan(slots, lens, batch, window, keep, units_per_seq, grid_blocks, room, 0, pages_s, splits_s);
     if (threadIdx.x == 0) plan_s = pl;
   }
   __syncthreads();
@@ -342,7 +348,6 @@ attn_decode_plan_kernel(int* __restrict__ plan, const int* __restrict__ slots, c
     plan[DA_PLAN_HEAD + u] = n;
   }
   int* recs = plan + da_plan_records_at(batch, units_per_seq);
-  const int ring_pages = ring_rows / AF_PAGE;
   for (int w = threadIdx.x; w < grid_blocks; w += blockDim.x) {
     const DaFirst fs = da_first_segment(pl, pages_s, splits_s, batch, units_per_seq, w);
     int* r = recs + (size_t)w * DA_PLAN_REC;
@@ -350,10 +355,9 @@ attn_decode_plan_kernel(int* __restrict__ plan, const int* __restrict__ slots, c
     if (fs.n_pages >= 0) {
       pos = lens[fs.b] - 1;
       slot = slots[fs.b];
-      const int lo = da_lo(pos, window);
+      const DaList l = da_list(pos, window, keep);
       for (int i = 0; i < 4 && i < fs.n_pages; ++i) {
-        const int pp = lo / AF_PAGE + fs.p_in + i;
-        const int entry = ring_pages > 0 ? pp % ring_pages : pp;
+        const int entry = af_cache_row(da_page_of(l.kept, l.skip, fs.p_in + i) * AF_PAGE, ring_rows, keep) / AF_PAGE;
         int page = AF_INDEX_OK(entry < max_pages, entry) ? page_table[(size_t)slot * max_pages + entry] : 0;
         if (!AF_INDEX_OK(page >= 0, page)) page = 0;
         ids[i] = page;
@@ -423,7 +427,7 @@ attn_decode_split_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
     __syncthreads();     // (the barriers are set up)
   } else {
     if (warp == 0) {
-      const DaPlan pl = da_plan(a.slots, a.lens, a.batch, a.window, units_per_seq, (int)gridDim.x, a.n_splits, 0,
+      const DaPlan pl = da_plan(a.slots, a.lens, a.batch, a.window, a.keep, units_per_seq, (int)gridDim.x, a.n_splits, 0,
                                 pages_s, splits_s);
       if (lane == 0) plan_s = pl;
     }
@@ -436,13 +440,12 @@ attn_decode_split_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
   }
   if (fs.n_pages < 0) return;                          // (nothing of the block's is in flight yet)
   int left = fs.run_pages;                             // pages the block has still to work
-  const int ring_pages = a.ring_rows / AF_PAGE;
   const float cs = a.cap > 0.f ? a.scale / a.cap : a.scale * LOG2E;
   const float cap2 = a.cap * LOG2E;
 
   // A segment: some of the pages of one unit.
   struct Segment {
-    int b, y, kvh, row_head0, n_rows, z, n_pages, pp_begin, last_pp, lo, pos;
+    int b, y, kvh, row_head0, n_rows, z, n_pages, x_begin, kept, skip, last_pp, lo, pos;
     const int* pt;
   };
   auto of_unit = [&](Segment& sg, int b, int y, int p_in, int pos, int slot) {
@@ -454,7 +457,9 @@ attn_decode_split_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
     sg.pos = pos;
     sg.lo = da_lo(pos, a.window);
     sg.last_pp = pos / AF_PAGE;        // the page of the new token, which the kernel in front wrote
-    sg.pp_begin = sg.lo / AF_PAGE + p_in;
+    const DaList l = da_list(pos, a.window, a.keep);
+    sg.kept = l.kept, sg.skip = l.skip;
+    sg.x_begin = p_in;                 // (pages of the list; page_of(x) says which of the sequence's)
     sg.pt = a.page_table + (size_t)slot * a.max_pages;
   };
   // the run cut goes on with the unit behind sg's: the same sequence's next, or the first of the next sequence
@@ -464,20 +469,18 @@ attn_decode_split_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
     int b = sg.b, y = sg.y + 1;
     if (y >= units_per_seq) {
       y = 0;
-      int f, l;
-      do ++b; while (b < a.batch - 1 && da_pages(a.slots, a.lens, b, a.window, &f, &l) == 0);
+      do ++b; while (b < a.batch - 1 && da_pages(a.slots, a.lens, b, a.window, a.keep) == 0);
     }
-    int f, l;
-    const int P = da_pages(a.slots, a.lens, b, a.window, &f, &l);
+    const int P = da_pages(a.slots, a.lens, b, a.window, a.keep);
     nx.z = 0;
     nx.n_pages = min(P, left);
     of_unit(nx, b, y, 0, a.lens[b] - 1, a.slots[b]);
     return nx;
   };
   // the cache page that holds page i of segment sg (a load from the page table: asked for ahead of its use)
+  auto page_of = [&](const Segment& sg, int i) { return da_page_of(sg.kept, sg.skip, sg.x_begin + i); };
   auto page_id = [&](const Segment& sg, int i) {
-    const int pp = sg.pp_begin + i;
-    const int entry = ring_pages > 0 ? pp % ring_pages : pp;
+    const int entry = af_cache_row(page_of(sg, i) * AF_PAGE, a.ring_rows, a.keep) / AF_PAGE;
     int page = AF_INDEX_OK(entry < a.max_pages, entry) ? sg.pt[entry] : 0;
     if (!AF_INDEX_OK(page >= 0, page)) page = 0;   // (the copy must still be made: the stage's barrier expects its bytes)
     return page;
@@ -503,7 +506,7 @@ attn_decode_split_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
     int i = from;
 #pragma unroll
     for (int k = 0; k < STAGES; ++k)
-      if (k == i && k < to && !(skip_last && sg.pp_begin + k == sg.last_pp)) {
+      if (k == i && k < to && !(skip_last && page_of(sg, k) == sg.last_pp)) {
         issue(sg.kvh, ids[k], ii0 + k);
         ++i;
       }
@@ -523,7 +526,7 @@ attn_decode_split_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
       // (the plan holds the first pages' ids: no load from the page table stands before the copies)
 #pragma unroll
       for (int k = 0; k < STAGES; ++k)
-        if (k == issued && k < sg.n_pages && sg.pp_begin + k != sg.last_pp) {
+        if (k == issued && k < sg.n_pages && page_of(sg, k) != sg.last_pp) {
           issue(sg.kvh, ids0[k], k);
           ++issued;
         }
@@ -534,7 +537,7 @@ attn_decode_split_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
   pdl_wait();
   while (true) {
     const int b = sg.b, n_pages = sg.n_pages, n_rows = sg.n_rows, row_head0 = sg.row_head0, z = sg.z;
-    const int pp_begin = sg.pp_begin, lo = sg.lo, pos = sg.pos;
+    const int lo = sg.lo, pos = sg.pos;
     if (tid == 0) issued = issue_first(sg, issued, min(STAGES, n_pages), i_base, false);
 
     // the query heads as A fragments: rows g and g + 8 of the tile
@@ -601,7 +604,7 @@ attn_decode_split_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
           sc[n][e] = v;
         }
       // ---- scale, softcap, mask, online softmax (base 2)
-      const int j0 = (pp_begin + i) * AF_PAGE + wq * 16;
+      const int j0 = page_of(sg, i) * AF_PAGE + wq * 16;
       float new_max[2] = {mx[0], mx[1]};
       if (a.cap > 0.f) {
 #pragma unroll
@@ -619,7 +622,7 @@ attn_decode_split_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int j = j0 + n * 8 + 2 * t + (e & 1);
-          const float v = (j >= lo && j <= pos) ? sc[n][e] : -INFINITY;
+          const float v = ((j >= lo || j < a.keep) && j <= pos) ? sc[n][e] : -INFINITY;
           sc[n][e] = v;
           new_max[e >> 1] = fmaxf(new_max[e >> 1], v);
         }
@@ -747,7 +750,7 @@ template <int HD>
 __global__ void attn_decode_merge_kernel(__nv_bfloat16* __restrict__ out, long long out_stride,
                                          const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                          int nq, int nkv, int max_splits, const int* __restrict__ slots,
-                                         const int* __restrict__ lens, int window, int grid_blocks,
+                                         const int* __restrict__ lens, int window, int keep, int grid_blocks,
                                          const int* __restrict__ plan, const float* __restrict__ sinks) {
   pdl_launch_dependents();
   const int b = blockIdx.x, h = blockIdx.y, batch = gridDim.x;
@@ -764,12 +767,12 @@ __global__ void attn_decode_merge_kernel(__nv_bfloat16* __restrict__ out, long l
     n_splits = ld_keep_int(plan + DA_PLAN_HEAD + b * units_per_seq + (h / group) * tiles + (h % group) / 16, l2_policy_keep());
   } else {
     if (threadIdx.x < 32) {
-      const DaPlan pl = da_plan(slots, lens, batch, window, units_per_seq, grid_blocks, max_splits, b, nullptr, nullptr);
+      const DaPlan pl = da_plan(slots, lens, batch, window, keep, units_per_seq, grid_blocks, max_splits, b, nullptr,
+                                nullptr);
       if (threadIdx.x == 0) plan_s = pl;
     }
     __syncthreads();
-    int first_pp, last_pp;
-    const int P = da_pages(slots, lens, b, window, &first_pp, &last_pp);
+    const int P = da_pages(slots, lens, b, window, keep);
     if (plan_s.even) {
       n_splits = da_even_splits(P, plan_s.share, max_splits, plan_s.even);
     } else {
@@ -933,7 +936,7 @@ int launch_decode(DecodeArgs a, int batch, long long n_pages, cudaStream_t strea
   const int merge_threads = a.n_splits > DA_MERGE_FEW && batch * a.nq <= 32 ? DA_MERGE_THREADS : (HD < 128 ? HD : 128);
   af_launch(attn_decode_merge_kernel<HD>, dim3(batch, a.nq), dim3(merge_threads), 0, stream, a.out, a.out_stride,
             (const float*)a.part_o, (const float*)a.part_ml, a.nq, a.nkv, a.n_splits, a.slots, a.lens, a.window,
-            n_blocks, a.plan, a.sinks);
+            a.keep, n_blocks, a.plan, a.sinks);
   AF_CHECK_LAUNCH("af_attn_decode (merge)");
 }
 
@@ -955,9 +958,10 @@ AF_EXPORT long long af_attn_decode_scratch(int batch, int nq, int hd, int n_spli
 static int attn_decode_impl(const float* sinks, void* out, long long out_stride, const void* q, long long q_stride,
                              const void* kcache, const void* vcache, long long n_pages, const int* page_table,
                              int max_pages, const int* slots, const int* lens, int batch, int nq, int nkv, int hd,
-                             float scale, float cap, int window, int ring_rows, int n_splits, float* scratch,
+                             float scale, float cap, int window, int keep, int ring_rows, int n_splits, float* scratch,
                              const int* plan, int* err, cudaStream_t stream) {
   if (batch == 0) return 0;
+  AF_REQUIRE(keep >= 0 && (keep == 0 || window != 0), "af_attn_decode: %d kept tokens with window %d", keep, window);
   AF_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0, "af_attn_decode: heads %d, groups %d", nq, nkv);
   AF_REQUIRE(af_attn_decode_supported(hd), "af_attn_decode: head_dim %d (takes 64, 128, 256)", hd);
   AF_REQUIRE(ring_rows % AF_PAGE == 0 && (ring_rows == 0 || (window != 0 && abs(window) <= ring_rows)),
@@ -980,6 +984,7 @@ static int attn_decode_impl(const float* sinks, void* out, long long out_stride,
   a.cap = cap;
   a.window = window;
   a.ring_rows = ring_rows;
+  a.keep = keep;
   a.n_splits = n_splits;
   a.batch = batch;
   a.n_sms = af_sm_count();
@@ -1003,7 +1008,7 @@ AF_EXPORT int af_attn_decode(void* out, long long out_stride, const void* q, lon
                              float cap, int window, int ring_rows, int n_splits, float* scratch, const int* plan,
                              int* err, cudaStream_t stream) {
   return attn_decode_impl(nullptr, out, out_stride, q, q_stride, kcache, vcache, n_pages, page_table, max_pages, slots,
-                          lens, batch, nq, nkv, hd, scale, cap, window, ring_rows, n_splits, scratch, plan, err, stream);
+                          lens, batch, nq, nkv, hd, scale, cap, window, 0, ring_rows, n_splits, scratch, plan, err, stream);
 }
 
 // The same with a learned sink per head (float [nq], or null): exp(sink) joins the head's softmax denominator
@@ -1014,7 +1019,17 @@ AF_EXPORT int af_attn_decode_sinks(void* out, long long out_stride, const void* 
                                    float scale, float cap, int window, int ring_rows, int n_splits, float* scratch,
                                    const int* plan, const float* sinks, int* err, cudaStream_t stream) {
   return attn_decode_impl(sinks, out, out_stride, q, q_stride, kcache, vcache, n_pages, page_table, max_pages, slots,
-                          lens, batch, nq, nkv, hd, scale, cap, window, ring_rows, n_splits, scratch, plan, err, stream);
+                          lens, batch, nq, nkv, hd, scale, cap, window, 0, ring_rows, n_splits, scratch, plan, err, stream);
+}
+
+// The same with a window (or chunk) beside which the first `keep` tokens of a sequence stay visible.
+AF_EXPORT int af_attn_decode_kept(void* out, long long out_stride, const void* q, long long q_stride,
+                                  const void* kcache, const void* vcache, long long n_pages, const int* page_table,
+                                  int max_pages, const int* slots, const int* lens, int batch, int nq, int nkv, int hd,
+                                  float scale, float cap, int window, int keep, int ring_rows, int n_splits,
+                                  float* scratch, const int* plan, const float* sinks, int* err, cudaStream_t stream) {
+  return attn_decode_impl(sinks, out, out_stride, q, q_stride, kcache, vcache, n_pages, page_table, max_pages, slots,
+                          lens, batch, nq, nkv, hd, scale, cap, window, keep, ring_rows, n_splits, scratch, plan, err, stream);
 }
 
 // ---------------------------------------------------------------- the plan of a step
@@ -1031,13 +1046,14 @@ AF_EXPORT long long af_attn_decode_plan_ints(int batch, int nq, int nkv) {
 // Works out, once for a step, how af_attn_decode cuts the work of the layers that read the same caches the same
 // way (the same slots, lengths, page table, heads, window, ring and n_splits): pass `plan` to each of their calls.
 // It holds for these lengths alone: a step later it is made again.
-AF_EXPORT int af_attn_decode_plan(int* plan, long long plan_ints, const int* page_table, int max_pages,
+AF_EXPORT int af_attn_decode_plan_kept(int* plan, long long plan_ints, const int* page_table, int max_pages,
                                   const int* slots, const int* lens, int batch, int nq, int nkv, int window,
-                                  int ring_rows, int n_splits, cudaStream_t stream) {
+                                  int keep, int ring_rows, int n_splits, cudaStream_t stream) {
   if (batch == 0) return 0;
   AF_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0, "af_attn_decode_plan: heads %d, groups %d", nq, nkv);
   AF_REQUIRE(plan != nullptr && ((uintptr_t)plan & 15) == 0 && plan_ints >= af_attn_decode_plan_ints(batch, nq, nkv),
              "af_attn_decode_plan: a plan of %lld integers, 16-byte aligned, wanted", af_attn_decode_plan_ints(batch, nq, nkv));
+  AF_REQUIRE(keep >= 0 && (keep == 0 || window != 0), "af_attn_decode_plan: %d kept tokens with window %d", keep, window);
   AF_REQUIRE(n_splits >= 1 && ring_rows % AF_PAGE == 0, "af_attn_decode_plan: splits %d, ring rows %d", n_splits, ring_rows);
   const int units_per_seq = nkv * ((nq / nkv + 15) / 16);
   AF_REQUIRE(batch <= DA_MAX_BATCH && (long long)batch * (max_pages + 1) * units_per_seq < (1ll << 31),
@@ -1045,8 +1061,15 @@ AF_EXPORT int af_attn_decode_plan(int* plan, long long plan_ints, const int* pag
   const int sms = af_sm_count();
   if (sms <= 0) return -1;
   af_launch(attn_decode_plan_kernel, dim3(1), dim3(256), (size_t)2 * (batch + 1) * sizeof(int), stream, plan, slots,
-            lens, page_table, max_pages, batch, nq, nkv, window, ring_rows, n_splits, sms);
+            lens, page_table, max_pages, batch, nq, nkv, window, keep, ring_rows, n_splits, sms);
   AF_CHECK_LAUNCH("af_attn_decode_plan");
+}
+
+AF_EXPORT int af_attn_decode_plan(int* plan, long long plan_ints, const int* page_table, int max_pages,
+                                  const int* slots, const int* lens, int batch, int nq, int nkv, int window,
+                                  int ring_rows, int n_splits, cudaStream_t stream) {
+  return af_attn_decode_plan_kept(plan, plan_ints, page_table, max_pages, slots, lens, batch, nq, nkv, window, 0, ring_rows,
+                                  n_splits, stream);
 }
 
 // ---------------------------------------------------------------- no allocation

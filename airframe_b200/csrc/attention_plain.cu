@@ -4,7 +4,8 @@
 //
 // Cache of one layer: pages [n_pages][n_kv_heads][AF_PAGE][head_dim] for K and
 // for V.  A sequence's page table maps row / AF_PAGE to a page.  A layer with
-// a window keeps rows modulo `ring_rows` (a multiple of AF_PAGE, >= window).
+// a window keeps rows modulo `ring_rows` (a multiple of AF_PAGE, >= window), behind the pages of the sequence's
+// first `keep` tokens if the window keeps those in sight.
 #include "common.cuh"
 
 #define AF_MAX_HD 640
@@ -39,7 +40,7 @@ __global__ void rope_cache_kernel(T* __restrict__ qkv, int row_stride, const flo
                                   const int* __restrict__ len_after, const float* __restrict__ inv_freq,
                                   int nq, int nkv, int hd, int rot_dim, int pairing,
                                   T* __restrict__ kcache, T* __restrict__ vcache,
-                                  const int* __restrict__ page_table, int max_pages, int ring_rows) {
+                                  const int* __restrict__ page_table, int max_pages, int ring_rows, int keep) {
   pdl_launch_dependents();
   // Positions, slots, lengths, the page table and the frequencies are inputs of the step, not
   // results of the kernel before: the row's place in the cache and the first pair's sine and
@@ -55,8 +56,8 @@ __global__ void rope_cache_kernel(T* __restrict__ qkv, int row_stride, const flo
     const int seq = seq_of_token[t];
     const int slot = slots[seq];
     // of the tokens of this step that share a ring row only the last is kept; padding rows are skipped
-    if (slot >= 0 && !(ring_rows > 0 && pos + ring_rows < len_after[seq])) {
-      const int r = ring_rows > 0 ? pos % ring_rows : pos;
+    if (slot >= 0 && af_cache_stores(pos, len_after[seq], ring_rows, keep)) {
+      const int r = af_cache_row(pos, ring_rows, keep);
       if (AF_INDEX_OK(pos >= 0 && r / AF_PAGE < max_pages, r)) {
         const int page = page_table[(size_t)slot * max_pages + r / AF_PAGE];
         const bool is_v = head >= nq + nkv;
@@ -112,7 +113,7 @@ rope_cache_vec_kernel(__nv_bfloat16* __restrict__ qkv, long long row_stride, con
                       const int* __restrict__ len_after, const float* __restrict__ inv_freq,
                       const float2* __restrict__ table, int nq, int nkv, int hd,
                       __nv_bfloat16* __restrict__ kcache, __nv_bfloat16* __restrict__ vcache,
-                      const int* __restrict__ page_table, int max_pages, int ring_rows) {
+                      const int* __restrict__ page_table, int max_pages, int ring_rows, int keep) {
   pdl_launch_dependents();
   // (positions, slots, lengths, page table and frequencies are inputs of the step: the row's place in
   // the cache and the sines and cosines are worked out before the wait for the kernel in front)
@@ -128,8 +129,8 @@ rope_cache_vec_kernel(__nv_bfloat16* __restrict__ qkv, long long row_stride, con
   if (kcache != nullptr) {
     const int seq = seq_of_token[t];
     const int slot = slots[seq];
-    if (slot >= 0 && !(ring_rows > 0 && pos + ring_rows < len_after[seq])) {
-      const int r = ring_rows > 0 ? pos % ring_rows : pos;
+    if (slot >= 0 && af_cache_stores(pos, len_after[seq], ring_rows, keep)) {
+      const int r = af_cache_row(pos, ring_rows, keep);
       if (AF_INDEX_OK(pos >= 0 && r / AF_PAGE < max_pages, r)) {
         const int page = page_table[(size_t)slot * max_pages + r / AF_PAGE];
         dst_row = ((size_t)page * nkv) * AF_PAGE + r % AF_PAGE;   // + h * AF_PAGE rows for kv head h
@@ -202,7 +203,7 @@ AF_EXPORT int af_rope_cache_write(void* qkv, int dtype, int row_stride, const fl
                                   const int* seq_of_token, const int* slots, const int* len_after,
                                   const float* inv_freq, const float* table, int n_tokens, int nq, int nkv, int hd,
                                   int rot_dim, int pairing, void* kcache, void* vcache,
-                                  const int* page_table, int max_pages, int ring_rows,
+                                  const int* page_table, int max_pages, int ring_rows, int keep,
                                   cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   AF_REQUIRE(n_tokens > 0 && nq > 0 && nkv > 0 && hd > 0, "af_rope_cache_write: bad sizes");
@@ -217,7 +218,7 @@ AF_EXPORT int af_rope_cache_write(void* qkv, int dtype, int row_stride, const fl
     af_launch(rope_cache_vec_kernel, dim3(n_tokens), dim3(256), 0, stream, (__nv_bfloat16*)qkv, (long long)row_stride,
               positions, seq_of_token, slots, len_after, inv_freq,
               ((uintptr_t)table & 15) == 0 ? reinterpret_cast<const float2*>(table) : nullptr, nq, nkv, hd, (__nv_bfloat16*)kcache,
-              (__nv_bfloat16*)vcache, page_table, max_pages, ring_rows);
+              (__nv_bfloat16*)vcache, page_table, max_pages, ring_rows, keep);
     AF_CHECK_LAUNCH("af_rope_cache_write");
   }
   AF_DISPATCH_DTYPE(dtype, T,
@@ -225,7 +226,7 @@ AF_EXPORT int af_rope_cache_write(void* qkv, int dtype, int row_stride, const fl
                         (T*)qkv, row_stride, parts, n_parts, (size_t)part_stride, positions, seq_of_token,
                         slots, len_after, inv_freq, nq,
                         nkv, hd, rot_dim, pairing, (T*)kcache, (T*)vcache, page_table, max_pages,
-                        ring_rows));
+                        ring_rows, keep));
   AF_CHECK_LAUNCH("af_rope_cache_write");
 }
 
@@ -285,15 +286,15 @@ AF_EXPORT int af_rope_table(float* table, const int* positions, const float* inv
 __global__ void kv_rows_kernel(int* __restrict__ rows, const int* __restrict__ positions,
                                const int* __restrict__ seq_of_token, const int* __restrict__ slots,
                                const int* __restrict__ len_after, const int* __restrict__ page_table, int max_pages,
-                               int ring_rows, int nkv, int n_tokens) {
+                               int ring_rows, int keep, int nkv, int n_tokens) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x * blockDim.x + threadIdx.x;
   if (t >= n_tokens) return;
   const int pos = positions[t], seq = seq_of_token[t], slot = slots[seq];
   int row = -1;
-  if (slot >= 0 && !(ring_rows > 0 && pos + ring_rows < len_after[seq])) {
-    const int r = ring_rows > 0 ? pos % ring_rows : pos;
+  if (slot >= 0 && af_cache_stores(pos, len_after[seq], ring_rows, keep)) {
+    const int r = af_cache_row(pos, ring_rows, keep);
     if (AF_INDEX_OK(pos >= 0 && r / AF_PAGE < max_pages, r)) {
       const int page = page_table[(size_t)slot * max_pages + r / AF_PAGE];
       if (AF_INDEX_OK(page >= 0, page)) row = page * nkv * AF_PAGE + r % AF_PAGE;
@@ -303,12 +304,12 @@ __global__ void kv_rows_kernel(int* __restrict__ rows, const int* __restrict__ p
 }
 
 AF_EXPORT int af_kv_rows(int* rows, const int* positions, const int* seq_of_token, const int* slots,
-                         const int* len_after, const int* page_table, int max_pages, int ring_rows, int nkv,
+                         const int* len_after, const int* page_table, int max_pages, int ring_rows, int keep, int nkv,
                          int n_tokens, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   AF_REQUIRE(n_tokens > 0 && nkv > 0 && ring_rows % AF_PAGE == 0, "af_kv_rows: bad sizes");
   af_launch(kv_rows_kernel, dim3((n_tokens + 127) / 128), dim3(128), 0, stream, rows, positions, seq_of_token, slots,
-            len_after, page_table, max_pages, ring_rows, nkv, n_tokens);
+            len_after, page_table, max_pages, ring_rows, keep, nkv, n_tokens);
   AF_CHECK_LAUNCH("af_kv_rows");
 }
 
@@ -382,7 +383,7 @@ __device__ __forceinline__ float gate_factor(const float* gate, long long gate_s
 
 // Prompts that start at position 0: keys and values are the step's own rows.
 // Warp w of the grid handles (token, head) = (w / nq, w % nq).  `hd` is the key size, `dv` the value
-// size; `sinks` (float [nq]) and `gate` (float logits, row t and column h at gate[t * gate_stride + h]:
+// size; the first `keep` positions stay visible whatever the window; `sinks` (float [nq]) and `gate` (float logits, row t and column h at gate[t * gate_stride + h]:
 // the head's output is multiplied by their sigmoid) may be null.
 template <typename T>
 __global__ void attn_prefill_plain_kernel(T* __restrict__ out, int out_stride, const T* __restrict__ q,
@@ -390,7 +391,7 @@ __global__ void attn_prefill_plain_kernel(T* __restrict__ out, int out_stride, c
                                           const T* __restrict__ v, int v_stride,
                                           const int* __restrict__ positions,
                                           int n_tokens, int nq, int nkv, int hd, int dv, float scale, float cap,
-                                          int window, int mask_kind, const float* __restrict__ slopes,
+                                          int window, int mask_kind, int keep, const float* __restrict__ slopes,
                                           const float* __restrict__ sinks, const float* __restrict__ gate,
                                           long long gate_stride) {
   pdl_launch_dependents();
@@ -406,7 +407,9 @@ __global__ void attn_prefill_plain_kernel(T* __restrict__ out, int out_stride, c
   attn_load_q(st, q + (size_t)t * q_stride + (size_t)h * hd, hd, lane, sinks ? sinks[h] : -INFINITY);
   const int lo = first_visible(pos, window, mask_kind);
   const float slope = slopes ? slopes[h] : 0.f;
-  for (int j = lo; j <= pos; ++j) {
+  const int kept = min(keep, lo);         // the first tokens that stay visible before the window
+  for (int x = 0; x < kept + pos - lo + 1; ++x) {
+    const int j = x < kept ? x : lo + x - kept;
     const size_t r = (size_t)(first_row + j);
     attn_key(st, k + r * k_stride + (size_t)g * hd, v + r * v_stride + (size_t)g * dv, hd, dv, lane, scale,
              cap, slope * (float)(j - pos));
@@ -417,7 +420,7 @@ __global__ void attn_prefill_plain_kernel(T* __restrict__ out, int out_stride, c
 AF_EXPORT int af_attn_prefill_plain(void* out, int out_stride, const void* q, int q_stride,
                                     const void* k, int k_stride, const void* v, int v_stride, int dtype,
                                     const int* positions, int n_tokens, int nq, int nkv, int hd, int dv,
-                                    float scale, float cap, int window, int mask_kind, const float* slopes,
+                                    float scale, float cap, int window, int mask_kind, int keep, const float* slopes,
                                     const float* sinks, const float* gate, long long gate_stride,
                                     cudaStream_t stream) {
   if (n_tokens == 0) return 0;
@@ -425,6 +428,7 @@ AF_EXPORT int af_attn_prefill_plain(void* out, int out_stride, const void* q, in
   AF_REQUIRE(hd > 0 && hd <= AF_MAX_HD && dv > 0 && dv <= AF_MAX_HD,
              "af_attn_prefill_plain: key size %d or value size %d beyond %d", hd, dv, AF_MAX_HD);
   AF_REQUIRE(mask_kind == AF_MASK_WINDOW || mask_kind == AF_MASK_CHUNK, "af_attn_prefill_plain: mask kind %d", mask_kind);
+  AF_REQUIRE(keep >= 0, "af_attn_prefill_plain: %d kept tokens", keep);
   const long long warps = (long long)n_tokens * nq;
   const int wpb = 4;
   const long long blocks = (warps + wpb - 1) / wpb;
@@ -432,7 +436,7 @@ AF_EXPORT int af_attn_prefill_plain(void* out, int out_stride, const void* q, in
   AF_DISPATCH_DTYPE(dtype, T,
                     af_launch(attn_prefill_plain_kernel<T>, dim3((unsigned)blocks), dim3(wpb * 32), 0, stream, 
                         (T*)out, out_stride, (const T*)q, q_stride, (const T*)k, k_stride, (const T*)v,
-                        v_stride, positions, n_tokens, nq, nkv, hd, dv, scale, cap, window, mask_kind, slopes,
+                        v_stride, positions, n_tokens, nq, nkv, hd, dv, scale, cap, window, mask_kind, keep, slopes,
                         sinks, gate, gate_stride));
   AF_CHECK_LAUNCH("af_attn_prefill_plain");
 }
@@ -442,13 +446,14 @@ AF_EXPORT int af_attn_prefill_plain(void* out, int out_stride, const void* q, in
 // value pages rows of `dv`; with no value pages (vcache null) a value is the first `dv` elements of its key row.
 // A warp per (sequence, head, split): with n_splits > 1 the visible keys are cut into that many equal runs and
 // a warp leaves its run's unnormalised output, maximum and sum in part_o / part_ml for the merge kernel.
+// The visible keys: the first `keep` ones where the window does not reach back to them, then the window's.
 template <typename T>
 __global__ void attn_decode_plain_kernel(T* __restrict__ out, int out_stride, const T* __restrict__ q,
                                          int q_stride, const T* __restrict__ kcache,
                                          const T* __restrict__ vcache, const int* __restrict__ page_table,
                                          int max_pages, const int* __restrict__ slots,
                                          const int* __restrict__ lens, int batch, int nq, int nkv, int hd, int dv,
-                                         float scale, float cap, int window, int mask_kind, int ring_rows,
+                                         float scale, float cap, int window, int mask_kind, int ring_rows, int keep,
                                          const float* __restrict__ slopes, const float* __restrict__ sinks,
                                          const float* __restrict__ gate, long long gate_stride, int n_splits,
                                          float* __restrict__ part_o, float* __restrict__ part_ml) {
@@ -474,16 +479,18 @@ __global__ void attn_decode_plain_kernel(T* __restrict__ out, int out_stride, co
   WarpAttn st;
   // (with splits the sink joins in the merge)
   attn_load_q(st, q + (size_t)b * q_stride + (size_t)h * hd, hd, lane, sinks && n_splits == 1 ? sinks[h] : -INFINITY);
-  int lo = first_visible(pos, window, mask_kind), hi = pos;
+  const int lo = first_visible(pos, window, mask_kind), kept = min(keep, lo), n_vis = kept + pos - lo + 1;
+  int x0 = 0, x1 = n_vis;                                   // this warp's run of them
   if (n_splits > 1) {
-    const int per = (pos - lo + n_splits) / n_splits;       // ceil((pos - lo + 1) / n_splits)
-    lo += split * per;
-    hi = min(pos, lo + per - 1);
+    const int per = (n_vis + n_splits - 1) / n_splits;
+    x0 = split * per;
+    x1 = min(n_vis, x0 + per);
   }
   const int* pt = page_table + (size_t)slot * max_pages;
   const float slope = slopes ? slopes[h] : 0.f;
-  for (int j = lo; j <= hi; ++j) {
-    const int r = ring_rows > 0 ? j % ring_rows : j;
+  for (int x = x0; x < x1; ++x) {
+    const int j = x < kept ? x : lo + x - kept;
+    const int r = af_cache_row(j, ring_rows, keep);
     if (!AF_INDEX_OK(r / AF_PAGE < max_pages && pt[r / AF_PAGE] >= 0, r)) continue;
     const size_t row = ((size_t)pt[r / AF_PAGE] * nkv + g) * AF_PAGE + r % AF_PAGE;
     const T* kr = kcache + row * hd;
@@ -559,7 +566,7 @@ AF_EXPORT int af_attn_decode_plain(void* out, int out_stride, const void* q, int
                                    const void* kcache, const void* vcache, int dtype,
                                    const int* page_table, int max_pages, const int* slots,
                                    const int* lens, int batch, int nq, int nkv, int hd, int dv, float scale,
-                                   float cap, int window, int mask_kind, int ring_rows, const float* slopes,
+                                   float cap, int window, int mask_kind, int ring_rows, int keep, const float* slopes,
                                    const float* sinks, const float* gate, long long gate_stride, int n_splits,
                                    float* scratch, cudaStream_t stream) {
   if (batch == 0) return 0;
@@ -570,6 +577,7 @@ AF_EXPORT int af_attn_decode_plain(void* out, int out_stride, const void* q, int
   AF_REQUIRE(mask_kind == AF_MASK_WINDOW || mask_kind == AF_MASK_CHUNK, "af_attn_decode_plain: mask kind %d", mask_kind);
   AF_REQUIRE(ring_rows % AF_PAGE == 0 && (ring_rows == 0 || window > 0) && (window <= ring_rows || ring_rows == 0),
              "af_attn_decode_plain: window %d, ring rows %d", window, ring_rows);
+  AF_REQUIRE(keep >= 0, "af_attn_decode_plain: %d kept tokens", keep);
   AF_REQUIRE(n_splits >= 1 && (n_splits == 1 || scratch != nullptr) && batch < 65536 && nq < 65536,
              "af_attn_decode_plain: %d splits need scratch memory", n_splits);
   const long long warps = (long long)batch * nq * n_splits;
@@ -582,7 +590,7 @@ AF_EXPORT int af_attn_decode_plain(void* out, int out_stride, const void* q, int
                     af_launch(attn_decode_plain_kernel<T>, dim3((unsigned)blocks), dim3(wpb * 32), 0, stream, 
                         (T*)out, out_stride, (const T*)q, q_stride, (const T*)kcache, (const T*)vcache,
                         page_table, max_pages, slots, lens, batch, nq, nkv, hd, dv, scale, cap, window, mask_kind,
-                        ring_rows, slopes, sinks, gate, gate_stride, n_splits, part_o, part_ml));
+                        ring_rows, keep, slopes, sinks, gate, gate_stride, n_splits, part_o, part_ml));
   if (n_splits == 1) AF_CHECK_LAUNCH("af_attn_decode_plain");
   AF_COUNT_LAUNCH("af_attn_decode_plain");
   AF_DISPATCH_DTYPE(dtype, T,
@@ -605,11 +613,12 @@ AF_EXPORT int af_attn_decode_merge_runs(void* out, int out_stride, int dtype, co
   AF_CHECK_LAUNCH("af_attn_decode_merge_runs");
 }
 
-// An output gate behind an attention kernel that has none of its own: x[t, h, :] *= sigmoid(gate[t, h]).
+// An output gate behind an attention kernel that has none of its own: x[t, h, d] *= sigmoid(gate[t, h]) for d < dv, or
+// with per_value sigmoid(gate[t, h dv + d]); the heads of x lie `pitch` apart.
 template <typename T>
 __global__ void __launch_bounds__(256)
 head_gate_kernel(T* __restrict__ x, long long x_stride, const float* __restrict__ gate, long long gate_stride,
-                 int nq, int dv, size_t total) {
+                 int nq, int dv, int pitch, int per_value, size_t total) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t at = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -617,20 +626,21 @@ head_gate_kernel(T* __restrict__ x, long long x_stride, const float* __restrict_
   const int per_row = nq * dv;
   const size_t t = at / per_row;
   const int i = (int)(at - t * per_row);
-  T* p = x + t * x_stride + i;
-  *p = from_f32<T>(to_f32(*p) * gate_factor(gate, gate_stride, (int)t, i / dv));
+  const int h = i / dv;
+  T* p = x + t * x_stride + (size_t)h * pitch + (i - h * dv);
+  *p = from_f32<T>(to_f32(*p) * gate_factor(gate, gate_stride, (int)t, per_value ? i : h));
 }
 
 AF_EXPORT int af_head_gate(void* x, long long x_stride, int dtype, const float* gate, long long gate_stride, int n_rows,
-                           int nq, int dv, cudaStream_t stream) {
+                           int nq, int dv, int pitch, int per_value, cudaStream_t stream) {
   if (n_rows == 0) return 0;
-  AF_REQUIRE(n_rows > 0 && nq > 0 && dv > 0 && gate != nullptr, "af_head_gate: bad sizes");
+  AF_REQUIRE(n_rows > 0 && nq > 0 && dv > 0 && pitch >= dv && gate != nullptr, "af_head_gate: bad sizes");
   const size_t total = (size_t)n_rows * nq * dv;
   const size_t blocks = (total + 255) / 256;
   AF_REQUIRE(blocks < (1ull << 31), "af_head_gate: too many rows");
   AF_DISPATCH_DTYPE(dtype, T,
                     af_launch(head_gate_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, stream, (T*)x, x_stride, gate,
-                              gate_stride, nq, dv, total));
+                              gate_stride, nq, dv, pitch, per_value, total));
   AF_CHECK_LAUNCH("af_head_gate");
 }
 
@@ -653,14 +663,14 @@ AF_EXPORT int af_head_gate(void* x, long long x_stride, int dtype, const float* 
 template <typename T>
 __device__ __forceinline__ void qk_cache_rows(T* kcache, T* vcache, const int* __restrict__ seq_of_token,
                                               const int* __restrict__ slots, const int* __restrict__ len_after,
-                                              const int* __restrict__ page_table, int max_pages, int ring_rows, int nkv,
+                                              const int* __restrict__ page_table, int max_pages, int ring_rows, int keep, int nkv,
                                               int t, int pos, int g, int pk, int pv, T** kdst, T** vdst) {
   *kdst = nullptr, *vdst = nullptr;
   if (kcache == nullptr) return;
   const int seq = seq_of_token[t];
   const int slot = slots[seq];
-  if (slot >= 0 && !(ring_rows > 0 && pos + ring_rows < len_after[seq])) {
-    const int r = ring_rows > 0 ? pos % ring_rows : pos;
+  if (slot >= 0 && af_cache_stores(pos, len_after[seq], ring_rows, keep)) {
+    const int r = af_cache_row(pos, ring_rows, keep);
     if (AF_INDEX_OK(pos >= 0 && r / AF_PAGE < max_pages, r)) {
       const int page = page_table[(size_t)slot * max_pages + r / AF_PAGE];
       if (AF_INDEX_OK(page >= 0, page)) {
@@ -765,7 +775,7 @@ qk_norm_rope_store_kernel(T* __restrict__ qkv, long long out_stride, const float
                           const float* __restrict__ inv_freq, const float2* __restrict__ table, int n_tokens, int nq,
                           int nkv, int hd, int dv, int rot_dim,
                           int pairing, T* __restrict__ kcache, T* __restrict__ vcache,
-                          const int* __restrict__ page_table, int max_pages, int ring_rows, int pitch) {
+                          const int* __restrict__ page_table, int max_pages, int ring_rows, int keep, int pitch) {
   pdl_launch_dependents();
   const int lane = threadIdx.x & 31;
   const long long wi = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -775,7 +785,7 @@ qk_norm_rope_store_kernel(T* __restrict__ qkv, long long out_stride, const float
   const int pk = pitch > 0 ? pitch : hd, pv = pitch > 0 ? pitch : dv;      // elements between heads (and of a cache row)
   T *kdst = nullptr, *vdst = nullptr;
   if (head >= nq)
-    qk_cache_rows(kcache, vcache, seq_of_token, slots, len_after, page_table, max_pages, ring_rows, nkv, t, pos,
+    qk_cache_rows(kcache, vcache, seq_of_token, slots, len_after, page_table, max_pages, ring_rows, keep, nkv, t, pos,
                   head - nq, pk, pv, &kdst, &vdst);
   pdl_wait();
   qk_pack_head(qkv, out_stride, proj, ld, bias, head >= nq ? k_weight : q_weight, false, 1.f, eps, norm_after, magnitude,
@@ -794,7 +804,7 @@ qk_whole_norm_rope_store_kernel(T* __restrict__ qkv, long long out_stride, const
                                 const float* __restrict__ inv_freq, const float2* __restrict__ table, int nq, int nkv,
                                 int hd, int dv, int rot_dim,
                                 int pairing, T* __restrict__ kcache, T* __restrict__ vcache,
-                                const int* __restrict__ page_table, int max_pages, int ring_rows, int pitch) {
+                                const int* __restrict__ page_table, int max_pages, int ring_rows, int keep, int pitch) {
   pdl_launch_dependents();
   __shared__ float scratch[33];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
@@ -816,7 +826,7 @@ qk_whole_norm_rope_store_kernel(T* __restrict__ qkv, long long out_stride, const
     const bool is_k = head >= nq;
     T *kdst = nullptr, *vdst = nullptr;
     if (is_k)
-      qk_cache_rows(kcache, vcache, seq_of_token, slots, len_after, page_table, max_pages, ring_rows, nkv, t, pos,
+      qk_cache_rows(kcache, vcache, seq_of_token, slots, len_after, page_table, max_pages, ring_rows, keep, nkv, t, pos,
                     head - nq, pk, pv, &kdst, &vdst);
     const float* w = is_k ? k_weight + (size_t)(head - nq) * hd : q_weight + (size_t)head * hd;
     qk_pack_head(qkv, out_stride, proj, ld, bias, w, true, is_k ? inv_k : inv_q, eps, norm_after, magnitude, v_from_k,
@@ -836,7 +846,7 @@ qk_whole_norm_rope_row_kernel(T* __restrict__ qkv, long long out_stride, const f
                               const int* __restrict__ slots, const int* __restrict__ len_after,
                               const float* __restrict__ inv_freq, const float2* __restrict__ table, int nq, int nkv,
                               int hd, int dv, int rot_dim, int pairing, T* __restrict__ kcache, T* __restrict__ vcache,
-                              const int* __restrict__ page_table, int max_pages, int ring_rows, int pitch) {
+                              const int* __restrict__ page_table, int max_pages, int ring_rows, int keep, int pitch) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) float srow[];          // q | k | v of the token, biases added
   __shared__ float red[2][8];
@@ -847,7 +857,7 @@ qk_whole_norm_rope_row_kernel(T* __restrict__ qkv, long long out_stride, const f
   const int pk = pitch > 0 ? pitch : hd, pv = pitch > 0 ? pitch : dv;
   if (threadIdx.x == 0) {                                // (the step's tables are there before the step begins)
     T *k0 = nullptr, *v0 = nullptr;
-    qk_cache_rows(kcache, vcache, seq_of_token, slots, len_after, page_table, max_pages, ring_rows, nkv, t, pos, 0, pk,
+    qk_cache_rows(kcache, vcache, seq_of_token, slots, len_after, page_table, max_pages, ring_rows, keep, nkv, t, pos, 0, pk,
                   pv, &k0, &v0);
     cache_rows[0] = k0, cache_rows[1] = v0;
   }
@@ -925,7 +935,7 @@ AF_EXPORT int af_qk_norm_rope_store(void* qkv, int dtype, long long out_stride, 
                                     const int* len_after, const float* inv_freq, const float* table, int n_tokens,
                                     int nq, int nkv, int hd,
                                     int dv, int rot_dim, int pairing, void* kcache, void* vcache, const int* page_table,
-                                    int max_pages, int ring_rows, int pitch, int whole_norm, cudaStream_t stream) {
+                                    int max_pages, int ring_rows, int keep, int pitch, int whole_norm, cudaStream_t stream) {
   const float2* tab = reinterpret_cast<const float2*>(table);
   AF_REQUIRE(((uintptr_t)table & 7) == 0, "af_qk_norm_rope_store: the table of cosines and sines lies on 8 bytes");
   if (n_tokens == 0) return 0;
@@ -946,7 +956,7 @@ AF_EXPORT int af_qk_norm_rope_store(void* qkv, int dtype, long long out_stride, 
                       af_launch(qk_whole_norm_rope_row_kernel<T>, dim3((unsigned)n_tokens), dim3(256), row_bytes, stream,
                                 (T*)qkv, out_stride, proj, ld, bias, q_weight, k_weight, eps, magnitude, positions,
                                 seq_of_token, slots, len_after, inv_freq, tab, nq, nkv, hd, dv, rot_dim, pairing,
-                                (T*)kcache, (T*)vcache, page_table, max_pages, ring_rows, pitch));
+                                (T*)kcache, (T*)vcache, page_table, max_pages, ring_rows, keep, pitch));
     AF_CHECK_LAUNCH("af_qk_norm_rope_store");
   }
   if (whole_norm) {
@@ -954,7 +964,7 @@ AF_EXPORT int af_qk_norm_rope_store(void* qkv, int dtype, long long out_stride, 
                       af_launch(qk_whole_norm_rope_store_kernel<T>, dim3((unsigned)n_tokens), dim3(256), 0, stream, (T*)qkv,
                                 out_stride, proj, ld, bias, q_weight, k_weight, eps, norm_after, magnitude, v_from_k,
                                 positions, seq_of_token, slots, len_after, inv_freq, tab, nq, nkv, hd, dv, rot_dim, pairing,
-                                (T*)kcache, (T*)vcache, page_table, max_pages, ring_rows, pitch));
+                                (T*)kcache, (T*)vcache, page_table, max_pages, ring_rows, keep, pitch));
     AF_CHECK_LAUNCH("af_qk_norm_rope_store");
   }
   const long long warps = (long long)n_tokens * (nq + nkv);
@@ -964,7 +974,7 @@ AF_EXPORT int af_qk_norm_rope_store(void* qkv, int dtype, long long out_stride, 
                     af_launch(qk_norm_rope_store_kernel<T>, dim3((unsigned)blocks), dim3(128), 0, stream, (T*)qkv,
                               out_stride, proj, ld, bias, q_weight, k_weight, eps, norm_after, magnitude, v_from_k,
                               positions, seq_of_token, slots, len_after, inv_freq, tab, n_tokens, nq, nkv, hd, dv, rot_dim,
-                              pairing, (T*)kcache, (T*)vcache, page_table, max_pages, ring_rows, pitch));
+                              pairing, (T*)kcache, (T*)vcache, page_table, max_pages, ring_rows, keep, pitch));
   AF_CHECK_LAUNCH("af_qk_norm_rope_store");
 }
 
@@ -1138,14 +1148,16 @@ AF_EXPORT int af_latent_prep(void* q, long long q_stride, const float* q_src, lo
 // out[t, h, n] = sum_d x[t, h, d] * w[h, d, n] for d < D, n < N (32-bit sums), and the
 // `extra` elements that follow a head's D inputs copied behind its N outputs.  x rows: heads `x_pitch`
 // elements apart (at least D + extra), rows `x_stride` apart; out rows: heads of (N + extra), `out_stride` apart;
-// w [heads, D, N].
+// w [heads, D, N].  With `gate` (float logits [t, h N + n], rows gate_stride apart) the outputs are multiplied by their
+// sigmoid.
 // One block of 256 threads per (token, head); the head's inputs wait in shared memory.  With fewer than 256
 // outputs the threads form 256 / cols groups that each take a stretch of the inputs (a long sum is then several
 // short chains side by side); the groups' sums are added in group order.
 template <typename T>
 __global__ void __launch_bounds__(256)
 head_project_kernel(T* __restrict__ out, long long out_stride, const T* __restrict__ x, long long x_stride,
-                    const T* __restrict__ w, int D, int N, int extra, int x_pitch, int cols) {
+                    const T* __restrict__ w, int D, int N, int extra, int x_pitch, int cols,
+                    const float* __restrict__ gate, long long gate_stride) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float xs[];                     // D inputs, then [groups][cols] partial sums
@@ -1167,7 +1179,7 @@ head_project_kernel(T* __restrict__ out, long long out_stride, const T* __restri
       for (int d = d0; d < d1; ++d) acc += xs[d] * to_f32(wh[(size_t)d * N + n]);
     }
     if (groups == 1) {
-      if (n < N) o[n] = from_f32<T>(acc);
+      if (n < N) o[n] = from_f32<T>(acc * gate_factor(gate, gate_stride, t, h * N + n));
       continue;
     }
     if (grp < groups) red[grp * cols + col] = acc;
@@ -1175,7 +1187,7 @@ head_project_kernel(T* __restrict__ out, long long out_stride, const T* __restri
     if (grp == 0 && n < N) {
       float sum = red[col];
       for (int g2 = 1; g2 < groups; ++g2) sum += red[g2 * cols + col];
-      o[n] = from_f32<T>(sum);
+      o[n] = from_f32<T>(sum * gate_factor(gate, gate_stride, t, h * N + n));
     }
   }
 }
@@ -1186,7 +1198,8 @@ head_project_kernel(T* __restrict__ out, long long out_stride, const T* __restri
 template <typename T>
 __global__ void __launch_bounds__(256)
 head_project_few_kernel(T* __restrict__ out, long long out_stride, const T* __restrict__ x, long long x_stride,
-                        const T* __restrict__ w, int D, int N, int extra, int x_pitch, int n_tokens) {
+                        const T* __restrict__ w, int D, int N, int extra, int x_pitch, int n_tokens,
+                        const float* __restrict__ gate, long long gate_stride) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float xs[];                     // [8 tokens][D] inputs, then [8 groups][8 tokens][32] partial sums
@@ -1223,13 +1236,14 @@ head_project_few_kernel(T* __restrict__ out, long long out_stride, const T* __re
     float sum = 0.f;
 #pragma unroll
     for (int g2 = 0; g2 < 8; ++g2) sum += red[(g2 * 8 + u) * 32 + (threadIdx.x & 31)];
-    out[(size_t)(t0 + u) * out_stride + (size_t)h * (N + extra) + n] = from_f32<T>(sum);
+    out[(size_t)(t0 + u) * out_stride + (size_t)h * (N + extra) + n] =
+        from_f32<T>(sum * gate_factor(gate, gate_stride, t0 + u, h * N + n));
   }
 }
 
 AF_EXPORT int af_head_project(void* out, long long out_stride, const void* x, long long x_stride, const void* w,
                               int dtype, int n_tokens, int heads, int D, int N, int extra, int x_pitch,
-                              cudaStream_t stream) {
+                              const float* gate, long long gate_stride, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   AF_REQUIRE(n_tokens > 0 && heads > 0 && heads < 65536 && D > 0 && N > 0 && extra >= 0 && x_pitch >= D + extra,
              "af_head_project: bad sizes");
@@ -1238,12 +1252,12 @@ AF_EXPORT int af_head_project(void* out, long long out_stride, const void* x, lo
     AF_DISPATCH_DTYPE(dtype, T,
                       af_launch(head_project_few_kernel<T>, dim3(heads, (N + 31) / 32, (n_tokens + 7) / 8), dim3(256),
                                 (size_t)(8 * D + 2048) * sizeof(float), stream, (T*)out, out_stride, (const T*)x, x_stride,
-                                (const T*)w, D, N, extra, x_pitch, n_tokens));
+                                (const T*)w, D, N, extra, x_pitch, n_tokens, gate, gate_stride));
     AF_CHECK_LAUNCH("af_head_project");
   }
   const int cols = N >= 256 ? 256 : ((N + 31) / 32) * 32;          // outputs a round; 256 / cols groups share the inputs
   AF_DISPATCH_DTYPE(dtype, T,
                     af_launch(head_project_kernel<T>, dim3(n_tokens, heads), dim3(256), (size_t)(D + 256) * sizeof(float),
-                              stream, (T*)out, out_stride, (const T*)x, x_stride, (const T*)w, D, N, extra, x_pitch, cols));
+                              stream, (T*)out, out_stride, (const T*)x, x_stride, (const T*)w, D, N, extra, x_pitch, cols, gate, gate_stride));
   AF_CHECK_LAUNCH("af_head_project");
 }

@@ -70,7 +70,7 @@ struct PrefillArgs {
   const int* seq_starts;  // [n_seqs + 1] first row of each sequence
   int nq, nkv;
   float scale, cap;
-  int window;
+  int window, keep;        // (the first `keep` positions stay visible whatever the window)
   const float* sinks;      // [nq] or null: exp(sink) joins a head's softmax denominator (no key, no value)
   const float* gate;       // float logits or null: row t, head h at gate[t * gate_stride + h]; the head's output times their sigmoid
   long long gate_stride;
@@ -127,11 +127,14 @@ attn_prefill_mma_kernel(PrefillArgs a) {
 
   const int m_last = min(m0 + PF_BM, len) - 1;                               // last query row of the block
   const int j_lo = a.window > 0 ? max(0, m0 - a.window + 1) : 0;             // first key any row sees
-  const int kb_lo = j_lo / PF_BN, kb_hi = m_last / PF_BN;                    // key tiles [kb_lo, kb_hi]
+  // the key tiles: those of the kept first positions, then the window's up to m_last's (`skip` tiles between the two)
+  const int kb_keep = (a.keep + PF_BN - 1) / PF_BN, skip = max(0, j_lo / PF_BN - kb_keep);
+  const int n_kb = m_last / PF_BN + 1 - skip;
+  auto tile_of = [&](int x) { return x >= kb_keep ? x + skip : x; };
 
   pf_load_tile<HD, PF_BM>(q_s, qb, a.q_stride, m0, len);
-  pf_load_tile<HD, PF_BN>(kv_s, kb, a.k_stride, kb_lo * PF_BN, len);
-  pf_load_tile<HD, PF_BN>(kv_s + TILE_KV, vb, a.v_stride, kb_lo * PF_BN, len);
+  pf_load_tile<HD, PF_BN>(kv_s, kb, a.k_stride, tile_of(0) * PF_BN, len);
+  pf_load_tile<HD, PF_BN>(kv_s + TILE_KV, vb, a.v_stride, tile_of(0) * PF_BN, len);
   asm volatile("cp.async.commit_group;" ::: "memory");
 
   float o[ONT][4];
@@ -142,14 +145,14 @@ attn_prefill_mma_kernel(PrefillArgs a) {
   const float cs = a.cap > 0.f ? a.scale / a.cap : a.scale * LOG2E;           // scale into tanh, or straight to base 2
   const float cap2 = a.cap * LOG2E;
 
-  for (int kt = kb_lo; kt <= kb_hi; ++kt) {
-    const int st = (kt - kb_lo) & 1;
+  for (int x = 0; x < n_kb; ++x) {
+    const int kt = tile_of(x), st = x & 1;
     unsigned char* k_s = kv_s + (size_t)st * 2 * TILE_KV;
     unsigned char* v_s = k_s + TILE_KV;
-    if (kt < kb_hi) {  // next tile into the other stage
+    if (x + 1 < n_kb) {  // next tile into the other stage
       unsigned char* nk = kv_s + (size_t)(st ^ 1) * 2 * TILE_KV;
-      pf_load_tile<HD, PF_BN>(nk, kb, a.k_stride, (kt + 1) * PF_BN, len);
-      pf_load_tile<HD, PF_BN>(nk + TILE_KV, vb, a.v_stride, (kt + 1) * PF_BN, len);
+      pf_load_tile<HD, PF_BN>(nk, kb, a.k_stride, tile_of(x + 1) * PF_BN, len);
+      pf_load_tile<HD, PF_BN>(nk + TILE_KV, vb, a.v_stride, tile_of(x + 1) * PF_BN, len);
       asm volatile("cp.async.commit_group;" ::: "memory");
       asm volatile("cp.async.wait_group 1;" ::: "memory");
     } else {
@@ -200,7 +203,7 @@ attn_prefill_mma_kernel(PrefillArgs a) {
         for (int e = 0; e < 4; ++e) {
           const int j = j0 + n * 8 + 2 * t + (e & 1);
           const int i = qrow[e >> 1];
-          const bool ok = j <= i && j < len && (a.window <= 0 || i - j < a.window);
+          const bool ok = j <= i && j < len && (a.window <= 0 || i - j < a.window || j < a.keep);
           s[n][e] = ok ? s[n][e] : -INFINITY;
         }
       }
@@ -301,11 +304,11 @@ int launch_prefill(const PrefillArgs& a, int n_seqs, int max_len, cudaStream_t s
 AF_EXPORT int af_attn_prefill_supported(int hd) { return hd == 64 || hd == 128 || hd == 256 ? 1 : 0; }
 
 // out [T, nq * hd] = attention of sequences that start at position 0 over
-// their own keys.  q, k, v, out: bfloat16 rows with the given strides
+// their own keys; with a window the first `keep` ones stay visible.  q, k, v, out: bfloat16 rows with the given strides
 // (elements, multiples of 8; bases 16-byte aligned); seq_starts [n_seqs + 1].
 AF_EXPORT int af_attn_prefill(void* out, long long out_stride, const void* q, long long q_stride, const void* k,
                               long long k_stride, const void* v, long long v_stride, const int* seq_starts,
-                              int n_seqs, int max_len, int nq, int nkv, int hd, float scale, float cap, int window,
+                              int n_seqs, int max_len, int nq, int nkv, int hd, float scale, float cap, int window, int keep,
                               const float* sinks, const float* gate, long long gate_stride, cudaStream_t stream) {
   if (n_seqs == 0 || max_len == 0) return 0;
   AF_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0, "af_attn_prefill: heads %d, groups %d", nq, nkv);
@@ -314,9 +317,10 @@ AF_EXPORT int af_attn_prefill(void* out, long long out_stride, const void* q, lo
              "af_attn_prefill: row strides must be multiples of 8");
   AF_REQUIRE((((uintptr_t)q | (uintptr_t)k | (uintptr_t)v) & 15) == 0 && ((uintptr_t)out & 3) == 0,
              "af_attn_prefill: operands must be 16-byte aligned");
+  AF_REQUIRE(keep >= 0, "af_attn_prefill: %d kept tokens", keep);
   AF_REQUIRE(n_seqs <= 65535 && nq <= 65535, "af_attn_prefill: too many sequences or heads");
   PrefillArgs a{(__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)k,
-                k_stride, (const __nv_bfloat16*)v, v_stride, seq_starts, nq, nkv, scale, cap, window, sinks, gate, gate_stride};
+                k_stride, (const __nv_bfloat16*)v, v_stride, seq_starts, nq, nkv, scale, cap, window, keep, sinks, gate, gate_stride};
   if (hd == 64) return launch_prefill<64>(a, n_seqs, max_len, stream);
   if (hd == 128) return launch_prefill<128>(a, n_seqs, max_len, stream);
   return launch_prefill<256>(a, n_seqs, max_len, stream);

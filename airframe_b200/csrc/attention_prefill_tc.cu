@@ -61,7 +61,7 @@ struct TaArgs {
   const int* seq_starts;
   int nq, nkv;
   float scale, cap;
-  int window;
+  int window, keep;        // (the first `keep` positions stay visible whatever the window)
   int* err;
   const float* sinks;      // [nq] or null: exp(sink) joins a head's softmax denominator (no key, no value)
   const float* gate;       // float logits or null: row t, head h at gate[t * gate_stride + h]; the head's output times their sigmoid
@@ -143,8 +143,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
   const bool active = m0 < len;
   const int m_last = min(m0 + TA_BM, len) - 1;
   const int j_lo = a.window > 0 ? max(0, m0 - a.window + 1) : 0;
-  const int kt_lo = j_lo / TA_KT, kt_hi = active ? m_last / TA_KT : -1;
-  const int n_tiles = active ? kt_hi - kt_lo + 1 : 0;   // 64-key tiles this block needs
+  // 64-key tiles this block needs: those of the kept first positions, then the window's up to m_last's (`skip` tiles
+  // lie between the two)
+  const int kt_keep = (a.keep + TA_KT - 1) / TA_KT, skip = max(0, j_lo / TA_KT - kt_keep);
+  const int n_tiles = active ? m_last / TA_KT + 1 - skip : 0;
+  auto tile_of = [&](int x) { return x >= kt_keep ? x + skip : x; };
   const int np = (n_tiles + 1) / 2;                     // steps: pairs of tiles (the last may hold one masked tile)
 
   if (warp == 0) {
@@ -159,12 +162,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         if (j >= 2 && !mbar_wait(&k_empty[b], ((j >> 1) & 1) ^ 1, give_up)) break;
         unsigned char* kb = k_s + (size_t)b * K_BYTES;
         mbar_expect_tx(&k_full[b], K_BYTES);
-        const int r = row0 + (kt_lo + 2 * j) * TA_KT;
+        const int r = row0 + tile_of(2 * j) * TA_KT, r2 = row0 + tile_of(2 * j + 1) * TA_KT;
 #pragma unroll
         for (int c = 0; c < SUB; ++c) {
           // rows past the packed rows read as zeros; rows of the next sequence are masked by position
           tma_load_2d(kb + c * K_SUB, &map_k, kvh * HD + c * 64, r, &k_full[b]);
-          tma_load_2d(kb + c * K_SUB + TA_KT * 128, &map_k, kvh * HD + c * 64, r + TA_KT, &k_full[b]);
+          tma_load_2d(kb + c * K_SUB + TA_KT * 128, &map_k, kvh * HD + c * 64, r2, &k_full[b]);
         }
       }
       if (*give_up) grace_period();
@@ -176,7 +179,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         if (!mbar_wait(&v_empty[s], ((t >> 1) & 1) ^ 1, give_up)) break;
         unsigned char* st = v_s + (size_t)s * V_BYTES;
         mbar_expect_tx(&v_full[s], V_BYTES);
-        const int r = row0 + (kt_lo + t) * TA_KT;
+        const int r = row0 + tile_of(t) * TA_KT;
 #pragma unroll
         for (int c = 0; c < SUB; ++c) tma_load_2d(st + c * V_SUB, &map_v, kvh * HD + c * 64, r, &v_full[s]);
       }
@@ -279,7 +282,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&s_empty);                   // the S buffer may be overwritten
-      const int j0 = (kt_lo + 2 * j + grp) * TA_KT + part * W;
+      const int j0 = tile_of(2 * j + grp) * TA_KT + part * W;
       const bool edge = (j0 + W - 1 > i) || (j0 + W > len) || (a.window > 0 && i - j0 >= a.window);
       // (the tests on the cap and on the edge stand outside the loops: inside, the compiler kept
       // them as a branch per element)
@@ -293,8 +296,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
       if (edge) {
         const int hi = min(i, len - 1) - j0;                       // last visible key of this part
         const int lo = a.window > 0 ? i - a.window + 1 - j0 : -1;  // first visible key
+        const int kept = a.keep - j0;                              // keys before this one stay visible
 #pragma unroll
-        for (int c = 0; c < W; ++c) s[c] = (c <= hi && c >= lo) ? s[c] : -INFINITY;
+        for (int c = 0; c < W; ++c) s[c] = (c <= hi && (c >= lo || c < kept)) ? s[c] : -INFINITY;
       }
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -451,14 +455,14 @@ int launch_ta(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& m
 AF_EXPORT int af_attn_prefill_tc_supported(int hd) { return hd == 128 || hd == 256 ? 1 : 0; }
 
 // out [T, nq * hd] = attention of sequences that start at position 0 over
-// their own keys, on tcgen05.  q [T, nq * hd], k and v [T, nkv * hd]:
+// their own keys, on tcgen05 (with a window the first `keep` keys stay visible).  q [T, nq * hd], k and v [T, nkv * hd]:
 // bfloat16 rows with the given strides (elements, multiples of 8; bases
 // 16-byte aligned); n_tokens rows in all; seq_starts [n_seqs + 1].
 AF_EXPORT int af_attn_prefill_tc(void* out, long long out_stride, const void* q, long long q_stride, const void* k,
                                  long long k_stride, const void* v, long long v_stride, const int* seq_starts,
                                  int n_seqs, int n_tokens, int max_len, int nq, int nkv, int hd, float scale,
-                                 float cap, int window, const float* sinks, const float* gate, long long gate_stride,
-                                 int* err, cudaStream_t stream) {
+                                 float cap, int window, int keep, const float* sinks, const float* gate,
+                                 long long gate_stride, int* err, cudaStream_t stream) {
   if (n_seqs == 0 || max_len == 0) return 0;
   AF_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0, "af_attn_prefill_tc: heads %d, groups %d", nq, nkv);
   AF_REQUIRE(af_attn_prefill_tc_supported(hd), "af_attn_prefill_tc: head_dim %d (takes 128, 256)", hd);
@@ -466,6 +470,7 @@ AF_EXPORT int af_attn_prefill_tc(void* out, long long out_stride, const void* q,
              "af_attn_prefill_tc: row strides must be multiples of 8");
   AF_REQUIRE((((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)out) & 15) == 0,
              "af_attn_prefill_tc: operands must be 16-byte aligned");
+  AF_REQUIRE(keep >= 0, "af_attn_prefill_tc: %d kept tokens", keep);
   AF_REQUIRE(n_seqs <= 65535 && nq <= 65535, "af_attn_prefill_tc: too many sequences or heads");
   CUtensorMap mq, mk, mv;
   int rc = af_make_map_bf16(&mq, q, n_tokens, (long long)nq * hd, q_stride, TA_BM);
@@ -474,7 +479,7 @@ AF_EXPORT int af_attn_prefill_tc(void* out, long long out_stride, const void* q,
   if (rc) return rc;
   rc = af_make_map_bf16(&mv, v, n_tokens, (long long)nkv * hd, v_stride, TA_KT);
   if (rc) return rc;
-  TaArgs a{(__nv_bfloat16*)out, out_stride, seq_starts, nq, nkv, scale, cap, window, err, sinks, gate, gate_stride};
+  TaArgs a{(__nv_bfloat16*)out, out_stride, seq_starts, nq, nkv, scale, cap, window, keep, err, sinks, gate, gate_stride};
   if (hd == 128) return launch_ta<128>(mq, mk, mv, a, n_seqs, max_len, stream);
   return launch_ta<256>(mq, mk, mv, a, n_seqs, max_len, stream);
 }

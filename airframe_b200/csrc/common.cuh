@@ -57,6 +57,20 @@ __host__ __device__ __forceinline__ int af_tile_group(int tiles_m, int sms) {
 }
 #endif
 
+// The cache row of a position.  ring_rows 0: its own.  Else the pages of the sequence's first `keep` tokens (tokens that
+// a window keeps in sight; whole pages, none for 0) stay, and the rows behind them are a ring of `ring_rows`.
+#ifdef __CUDACC__
+__host__ __device__ __forceinline__ int af_kept_pages(int keep) { return (keep + AF_PAGE - 1) / AF_PAGE; }
+__device__ __forceinline__ int af_cache_row(int pos, int ring_rows, int keep) {
+  const int kept = af_kept_pages(keep) * AF_PAGE;
+  return ring_rows > 0 && pos >= kept ? kept + (pos - kept) % ring_rows : pos;
+}
+// Of the tokens of a step that share a ring row only the last is stored.
+__device__ __forceinline__ bool af_cache_stores(int pos, int len_after, int ring_rows, int keep) {
+  return !(ring_rows > 0 && pos >= af_kept_pages(keep) * AF_PAGE && pos + ring_rows < len_after);
+}
+#endif
+
 // Records a message that af_last_error() returns and yields the error code.
 int af_fail(int code, const char* fmt, ...);
 

@@ -432,6 +432,61 @@ AF_EXPORT int af_gated_act(void* out, const void* gu, int dtype, int n_rows, int
   AF_CHECK_LAUNCH("af_gated_act");
 }
 
+// out[t, c] = act(z[t, c]) * table[ids[t]][off + c] for c < dim: a token's own row of a table (columns off .. of it) gated
+// by a product, z float rows or `parts` partial sums of them (added in order).  A thread takes V neighbours.
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+token_gate_kernel(T* __restrict__ out, const float* __restrict__ z, int parts, size_t part_stride,
+                  const T* __restrict__ table, size_t ld, int off, const int* __restrict__ ids, int vocab, int n_rows,
+                  int dim, int act) {
+  pdl_launch_dependents();
+  const size_t at = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * V;
+  if (at >= (size_t)n_rows * dim) return;
+  const int t = (int)(at / dim), c = (int)(at - (size_t)t * dim);
+  const int id = ids[t];
+  // (the step's tokens and the table are there before the kernel in front: the row is asked for before the wait)
+  const bool known = AF_INDEX_OK(id >= 0 && id < vocab, id);
+  float e[V];
+#pragma unroll
+  for (int u = 0; u < V; ++u) e[u] = known ? to_f32(table[(size_t)id * ld + off + c + u]) : 0.f;
+  pdl_wait();
+  z = pdl_fresh(z);
+  float g[V];
+#pragma unroll
+  for (int u = 0; u < V; ++u) g[u] = z[at + u];
+  for (int p0 = 1; p0 < parts; p0 += 8) {
+    float q[8][V];
+#pragma unroll
+    for (int p = 0; p < 8; ++p)
+#pragma unroll
+      for (int u = 0; u < V; ++u) q[p][u] = p0 + p < parts ? z[(size_t)(p0 + p) * part_stride + at + u] : 0.f;
+#pragma unroll
+    for (int p = 0; p < 8; ++p)
+#pragma unroll
+      for (int u = 0; u < V; ++u) g[u] += q[p][u];
+  }
+#pragma unroll
+  for (int u = 0; u < V; ++u) out[at + u] = from_f32<T>(act_f32(g[u], act) * e[u]);
+}
+
+AF_EXPORT int af_token_gate(void* out, int dtype, const float* z, int parts, const void* table, long long ld, int off,
+                            const int* ids, int vocab, int n_rows, int dim, int act, cudaStream_t stream) {
+  if (n_rows == 0) return 0;
+  AF_REQUIRE(n_rows > 0 && dim > 0 && parts >= 1 && vocab > 0 && off >= 0 && off + dim <= ld, "af_token_gate: bad sizes");
+  AF_REQUIRE(act == AF_ACT_GELU_TANH || act == AF_ACT_SILU, "af_token_gate: unknown activation %d", act);
+  const size_t n = (size_t)n_rows * dim;
+  const int v = dim % 2 == 0 ? 2 : 1;
+  const size_t blocks = (n / v + 255) / 256;
+  AF_REQUIRE(blocks < (1ull << 31), "af_token_gate: too many rows");
+#define TG_LAUNCH(T, V)                                                                                             \
+  af_launch(token_gate_kernel<T, V>, dim3((unsigned)blocks), dim3(256), 0, stream, (T*)out, z, parts, n, (const T*)table, \
+            (size_t)ld, off, ids, vocab, n_rows, dim, act)
+  if (v == 2) AF_DISPATCH_DTYPE(dtype, T, TG_LAUNCH(T, 2));
+  else AF_DISPATCH_DTYPE(dtype, T, TG_LAUNCH(T, 1));
+#undef TG_LAUNCH
+  AF_CHECK_LAUNCH("af_token_gate");
+}
+
 // ---------------------------------------------------------------- residual sum
 
 template <typename T>

@@ -2,10 +2,10 @@
 //   expert_route   per token the router's logits in 32 bits, a score per expert (the sigmoid of its logit), the `top`
 //                  experts with the largest scores (equal scores: the lower index) and their scores (optionally: a
 //                  correction added to the scores for the choice only, a choice among the best groups of experts,
-//                  weights divided by their sum and scaled); also the
+//                  weights divided by their sum and scaled; or the softmax of the logits as the scores); also the
 //                  sigmoid of one more row of the router matrix when there is one (the gate of a shared expert);
 //   expert_plan    the (token, choice) pairs sorted by expert: a permutation, and a table of tiles of up to 32
-//                  pairs of one expert each;
+//                  pairs of one expert each (pairs of identity experts, which have no matrices, come last and in no tile);
 //   expert_rows    a tile's rows times its expert's matrices on the CUDA cores, 32-bit sums in index order:
 //                  either gate and up with the activation behind them, or down.
 // The order of the pairs of an expert depends on the order in which blocks arrive, but every row of a tile is
@@ -35,10 +35,11 @@ __device__ __forceinline__ void load4_f32<__nv_bfloat16>(float* v, const __nv_bf
 // Scores first, the choice behind them.  A warp of the scores' kernel takes one row of the router (an expert, or
 // the shared expert's gate) and TM tokens, and adds a token's products in one fixed order whatever TM is, so that a
 // prompt and a decode step choose alike; the warps of a block share their tokens.  scores: [tokens, rows].
+// With `raw` the logits themselves are left there.
 template <typename TX, int TM>
 __global__ void __launch_bounds__(256)
 expert_score_kernel(float* __restrict__ scores, const TX* __restrict__ h, const float* __restrict__ router, int n_tokens,
-                    int hidden, int rows) {
+                    int hidden, int rows, int raw) {
   pdl_launch_dependents();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const long long job = (long long)blockIdx.x * (blockDim.x >> 5) + warp;
@@ -84,20 +85,22 @@ expert_score_kernel(float* __restrict__ scores, const TX* __restrict__ h, const 
 #pragma unroll
   for (int m = 0; m < TM; ++m) {
     const float zs = warp_sum(z[m]);
-    if (lane == 0 && t0 + m < n_tokens) scores[(size_t)(t0 + m) * rows + e] = 1.f / (1.f + expf(-zs));
+    if (lane == 0 && t0 + m < n_tokens) scores[(size_t)(t0 + m) * rows + e] = raw ? zs : 1.f / (1.f + expf(-zs));
   }
 }
 
 // A warp a token: the `top` largest choice scores in turn (equal scores: the lower index), each struck out once
 // chosen.  The choice score is the score plus `correction[e]` (none: the score); the weight is always the score
 // itself.  With `groups` > 1 the experts form that many equal groups of neighbours, a group's score is the sum of its
-// two largest choice scores (of its only one, in groups of one), and only experts of the `keep` best groups (equal
-// scores: the lower group) can be chosen.  With `normalise` the chosen weights are divided by their sum + 1e-20;
+// two largest choice scores (of its only one, in groups of one; with `group_max` its largest alone), and only experts of
+// the `keep` best groups (equal scores: the lower group) can be chosen.  With `softmax` the kernel finds logits and the
+// scores are their softmax over all experts.  With `normalise` the chosen weights are divided by their sum + 1e-20;
 // all weights are multiplied by `out_scale`.
 __global__ void __launch_bounds__(128)
 expert_choose_kernel(int* __restrict__ ids, float* __restrict__ wts, float* __restrict__ shared_gate,
                      const float* __restrict__ scores, const float* __restrict__ correction, int n_tokens,
-                     int n_experts, int rows, int top, int groups, int keep, int normalise, float out_scale) {
+                     int n_experts, int rows, int top, int groups, int keep, int normalise, float out_scale, int softmax,
+                     int group_max) {
   pdl_launch_dependents();
   extern __shared__ float score_all[];              // a warp: n_experts choice scores, n_experts scores, `groups` group scores
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -110,12 +113,24 @@ expert_choose_kernel(int* __restrict__ ids, float* __restrict__ wts, float* __re
   float* gscore = score + n_experts;
   const float OUT = -3.0e38f;                       // an expert of a group that is not kept (it still beats a struck one)
   const float STRUCK = -INFINITY;
+  float most = 0.f, inv = 1.f;
+  if (softmax) {
+    float m = -INFINITY, sum = 0.f;
+    for (int e = lane; e < n_experts; e += 32) m = fmaxf(m, scores[(size_t)t * rows + e]);
+    most = warp_max(m);
+    for (int e = lane; e < n_experts; e += 32) sum += expf(scores[(size_t)t * rows + e] - most);
+    inv = 1.f / warp_sum(sum);
+  }
   for (int e = lane; e < n_experts; e += 32) {
-    const float sc = scores[(size_t)t * rows + e];
+    const float z = scores[(size_t)t * rows + e];
+    const float sc = softmax ? expf(z - most) * inv : z;
     score[e] = sc;
     choice[e] = sc + (correction != nullptr ? correction[e] : 0.f);
   }
-  if (shared_gate != nullptr && lane == 0) shared_gate[t] = scores[(size_t)t * rows + n_experts];
+  if (shared_gate != nullptr && lane == 0) {
+    const float z = scores[(size_t)t * rows + n_experts];
+    shared_gate[t] = softmax ? 1.f / (1.f + expf(-z)) : z;
+  }
   __syncwarp();
   if (groups > 1 && keep < groups) {
     const int per = n_experts / groups;
@@ -126,7 +141,7 @@ expert_choose_kernel(int* __restrict__ ids, float* __restrict__ wts, float* __re
         if (c > a) b = a, a = c;
         else if (c > b) b = c;
       }
-      gscore[g] = per > 1 ? a + b : a;
+      gscore[g] = per > 1 && !group_max ? a + b : a;
     }
     __syncwarp();
     for (int k = 0; k < keep; ++k) {                // the best groups in turn, marked by +infinity
@@ -178,8 +193,8 @@ expert_choose_kernel(int* __restrict__ ids, float* __restrict__ wts, float* __re
 // scores: room for n_tokens x (n_experts + 1) floats.
 AF_EXPORT int af_expert_route(int* ids, float* wts, float* shared_gate, float* scores, const void* h, int h_dtype,
                               const float* router, int n_tokens, int hidden, int n_experts, int top,
-                              const float* correction, int groups, int keep, int normalise, float out_scale,
-                              cudaStream_t stream) {
+                              const float* correction, int groups, int keep, int normalise, float out_scale, int softmax,
+                              int group_max, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   AF_REQUIRE(n_tokens > 0 && hidden > 0 && n_experts > 0 && top >= 1 && top <= n_experts && scores != nullptr,
              "af_expert_route: %d of %d experts", top, n_experts);
@@ -197,17 +212,17 @@ AF_EXPORT int af_expert_route(int* ids, float* wts, float* shared_gate, float* s
   if (tm == 4) {
     AF_DISPATCH_DTYPE(h_dtype, TX,
                       af_launch(expert_score_kernel<TX, 4>, dim3((unsigned)blocks), dim3(256), 0, stream, scores,
-                                (const TX*)h, router, n_tokens, hidden, rows));
+                                (const TX*)h, router, n_tokens, hidden, rows, softmax));
   } else {
     AF_DISPATCH_DTYPE(h_dtype, TX,
                       af_launch(expert_score_kernel<TX, 1>, dim3((unsigned)blocks), dim3(256), 0, stream, scores,
-                                (const TX*)h, router, n_tokens, hidden, rows));
+                                (const TX*)h, router, n_tokens, hidden, rows, softmax));
   }
   AF_COUNT_LAUNCH("af_expert_route");
   const int warps = n_experts <= 1024 ? 4 : 1;
   af_launch(expert_choose_kernel, dim3((n_tokens + warps - 1) / warps), dim3(32 * warps),
             (size_t)warps * (2 * n_experts + groups) * sizeof(float), stream, ids, wts, shared_gate, (const float*)scores,
-            correction, n_tokens, n_experts, rows, top, groups, keep, normalise, out_scale);
+            correction, n_tokens, n_experts, rows, top, groups, keep, normalise, out_scale, softmax, group_max);
   AF_CHECK_LAUNCH("af_expert_route");
 }
 
@@ -216,16 +231,18 @@ AF_EXPORT int af_expert_route(int* ids, float* wts, float* shared_gate, float* s
 // One block a plan.  plan: [0] tiles in use; then per tile (expert, first sorted row, rows).  perm[sorted row] = pair.
 // The experts of pair p come from `ids`, or with `table` (rows of `top` expert numbers, one row a token id) from the
 // token that the pair belongs to: expert = table[tokens[p / top]][p % top].  Block b takes the b-th table of
-// [blocks][vocab][top] and writes the b-th perm [n_pairs] and plan.
+// [blocks][vocab][top] and writes the b-th perm [n_pairs] and plan.  Numbers n_experts .. n_ids - 1 name identity
+// experts: their pairs end the permutation and belong to no tile.
 __global__ void __launch_bounds__(1024)
 expert_plan_kernel(int* __restrict__ perm, int* __restrict__ plan, const int* __restrict__ ids,
-                   const int* __restrict__ table, int vocab, int top, int n_pairs, int n_experts, int max_tiles, int tile) {
+                   const int* __restrict__ table, int vocab, int top, int n_pairs, int n_experts, int n_ids, int max_tiles,
+                   int tile) {
   pdl_launch_dependents();
-  extern __shared__ int sh[];                       // count[E], first[E], cursor[E]
+  extern __shared__ int sh[];                       // count[E + 1], first[E + 1], cursor[E + 1] (the last: identity experts)
   int* count = sh;
-  int* first = sh + n_experts;
-  int* cursor = sh + 2 * n_experts;
-  for (int e = threadIdx.x; e < n_experts; e += blockDim.x) count[e] = 0, cursor[e] = 0;
+  int* first = sh + n_experts + 1;
+  int* cursor = sh + 2 * (n_experts + 1);
+  for (int e = threadIdx.x; e <= n_experts; e += blockDim.x) count[e] = 0, cursor[e] = 0;
   __syncthreads();
   pdl_wait();
   ids = pdl_fresh(ids);
@@ -241,9 +258,9 @@ expert_plan_kernel(int* __restrict__ perm, int* __restrict__ plan, const int* __
   };
   for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
     const int e = expert_of(p);
-    const bool ok = e >= 0 && e < n_experts;
+    const bool ok = e >= 0 && e < n_ids;
     (void)AF_INDEX_OK(ok, e);
-    if (ok) atomicAdd(&count[e], 1);
+    if (ok) atomicAdd(&count[min(e, n_experts)], 1);
   }
   __syncthreads();
   if (threadIdx.x == 0) {
@@ -261,24 +278,25 @@ expert_plan_kernel(int* __restrict__ perm, int* __restrict__ plan, const int* __
       }
       rows += count[e];
     }
+    first[n_experts] = rows;
     plan[0] = tiles;
   }
   __syncthreads();
   for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
-    const int e = expert_of(p);
-    if (e >= 0 && e < n_experts) perm[first[e] + atomicAdd(&cursor[e], 1)] = p;
+    const int id = expert_of(p), e = min(id, n_experts);
+    if (id >= 0 && id < n_ids) perm[first[e] + atomicAdd(&cursor[e], 1)] = p;
   }
 }
 
-AF_EXPORT int af_expert_plan(int* perm, int* plan, const int* ids, int n_pairs, int n_experts, int max_tiles,
-                             int tile, cudaStream_t stream) {
+AF_EXPORT int af_expert_plan(int* perm, int* plan, const int* ids, int n_pairs, int n_experts, int identity,
+                             int max_tiles, int tile, cudaStream_t stream) {
   if (n_pairs == 0) return 0;
-  AF_REQUIRE(n_pairs > 0 && n_experts > 0 && n_experts <= 4096 && tile > 0, "af_expert_plan: bad sizes");
+  AF_REQUIRE(n_pairs > 0 && n_experts > 0 && n_experts < 4096 && identity >= 0 && tile > 0, "af_expert_plan: bad sizes");
   // (every expert may end on a tile that is not full)
   AF_REQUIRE(max_tiles >= n_pairs / tile + n_experts || max_tiles >= n_pairs,
              "af_expert_plan: room for %d tiles is too little", max_tiles);
-  af_launch(expert_plan_kernel, dim3(1), dim3(1024), (size_t)3 * n_experts * sizeof(int), stream, perm, plan, ids,
-            (const int*)nullptr, 0, 1, n_pairs, n_experts, max_tiles, tile);
+  af_launch(expert_plan_kernel, dim3(1), dim3(1024), (size_t)3 * (n_experts + 1) * sizeof(int), stream, perm, plan, ids,
+            (const int*)nullptr, 0, 1, n_pairs, n_experts, n_experts + identity, max_tiles, tile);
   AF_CHECK_LAUNCH("af_expert_plan");
 }
 
@@ -287,24 +305,27 @@ AF_EXPORT int af_expert_plan(int* perm, int* plan, const int* ids, int n_pairs, 
 AF_EXPORT int af_expert_table_plan(int* perm, int* plan, const int* tokens, const int* tables, int n_tables, int vocab,
                                    int top, int n_tokens, int n_experts, int max_tiles, int tile, cudaStream_t stream) {
   if (n_tokens == 0 || n_tables == 0) return 0;
-  AF_REQUIRE(n_tokens > 0 && n_tables > 0 && vocab > 0 && top > 0 && n_experts > 0 && n_experts <= 4096 && tile > 0,
+  AF_REQUIRE(n_tokens > 0 && n_tables > 0 && vocab > 0 && top > 0 && n_experts > 0 && n_experts < 4096 && tile > 0,
              "af_expert_table_plan: bad sizes");
   AF_REQUIRE((long long)n_tokens * top < (1ll << 31), "af_expert_table_plan: too many pairs");
   const int n_pairs = n_tokens * top;
   AF_REQUIRE(max_tiles >= n_pairs / tile + n_experts || max_tiles >= n_pairs,
              "af_expert_table_plan: room for %d tiles is too little", max_tiles);
-  af_launch(expert_plan_kernel, dim3(n_tables), dim3(n_pairs <= 256 ? 256 : 1024), (size_t)3 * n_experts * sizeof(int), stream, perm, plan,
-            tokens, tables, vocab, top, n_pairs, n_experts, max_tiles, tile);
+  af_launch(expert_plan_kernel, dim3(n_tables), dim3(n_pairs <= 256 ? 256 : 1024), (size_t)3 * (n_experts + 1) * sizeof(int), stream, perm, plan,
+            tokens, tables, vocab, top, n_pairs, n_experts, n_experts, max_tiles, tile);
   AF_CHECK_LAUNCH("af_expert_table_plan");
 }
 
 // ---------------------------------------------------------------- the tokens' rows in sorted order
 
-// out[sorted row] = x[perm[sorted row] / top]: the rows a tensor-core product fetches tile by tile.
+// out[sorted row] = x[perm[sorted row] / top]: the rows a tensor-core product fetches tile by tile.  A pair of an
+// identity expert (ids[pair] >= n_experts; `ids` null: there are none) has no product: wts[pair] x goes straight to its
+// place among the down products' results, result[choice][token].  `out` null: the identity experts' rows alone.
 template <typename T>
 __global__ void __launch_bounds__(256)
 expert_gather_kernel(T* __restrict__ out, const T* __restrict__ x, const int* __restrict__ perm, int n_rows, int top,
-                     int H) {
+                     int H, const int* __restrict__ ids, int n_experts, const float* __restrict__ wts,
+                     float* __restrict__ result) {
   pdl_launch_dependents();
   pdl_wait();
   const int warps = blockDim.x >> 5, lane = threadIdx.x & 31;
@@ -313,6 +334,21 @@ expert_gather_kernel(T* __restrict__ out, const T* __restrict__ x, const int* __
   const int pair = __ldcg(perm + r);
   if (!AF_INDEX_OK(pair >= 0 && pair < n_rows, pair)) return;
   const T* src = x + (size_t)(pair / top) * H;
+  if (ids != nullptr && __ldcg(ids + pair) >= n_experts) {
+    const float w = __ldcg(wts + pair);
+    float* to = result + ((size_t)(pair % top) * (n_rows / top) + pair / top) * H;
+    if (H % 4 == 0) {
+      for (int i = lane * 4; i < H; i += 128) {
+        float v[4];
+        load4_f32<T>(v, src + i);
+        *reinterpret_cast<float4*>(to + i) = make_float4(w * v[0], w * v[1], w * v[2], w * v[3]);
+      }
+    } else {
+      for (int i = lane; i < H; i += 32) to[i] = w * to_f32<T>(src[i]);
+    }
+    return;
+  }
+  if (out == nullptr) return;
   T* dst = out + (size_t)r * H;
   if ((H * sizeof(T)) % 16 == 0) {
     const int n16 = H * sizeof(T) / 16;
@@ -323,13 +359,15 @@ expert_gather_kernel(T* __restrict__ out, const T* __restrict__ x, const int* __
 }
 
 AF_EXPORT int af_expert_gather(void* out, const void* x, int dtype, const int* perm, int n_rows, int top, int H,
-                               cudaStream_t stream) {
+                               const int* ids, int n_experts, const float* wts, float* result, cudaStream_t stream) {
   if (n_rows == 0) return 0;
-  AF_REQUIRE(n_rows > 0 && top >= 1 && H > 0 && perm != nullptr, "af_expert_gather: bad sizes");
+  AF_REQUIRE(n_rows > 0 && top >= 1 && n_rows % top == 0 && H > 0 && perm != nullptr, "af_expert_gather: bad sizes");
+  AF_REQUIRE(ids == nullptr ? out != nullptr : wts != nullptr && result != nullptr && ((uintptr_t)result & 15) == 0,
+             "af_expert_gather: identity experts need their weights and the results' rows");
   AF_REQUIRE(((uintptr_t)out & 15) == 0 && ((uintptr_t)x & 15) == 0, "af_expert_gather: rows must be 16-byte aligned");
   AF_DISPATCH_DTYPE(dtype, T,
                     af_launch(expert_gather_kernel<T>, dim3((n_rows + 7) / 8), dim3(256), 0, stream, (T*)out,
-                              (const T*)x, perm, n_rows, top, H));
+                              (const T*)x, perm, n_rows, top, H, ids, n_experts, wts, result));
   AF_CHECK_LAUNCH("af_expert_gather");
 }
 
@@ -346,6 +384,7 @@ __device__ __forceinline__ float clamped_glu(float g, float u, float limit) {
 //       token names, s the pair's weight (a weight on an expert's input goes through its products, which have no
 //       bias), post the token's `scale_out` (1 without); out of the compute dtype, rows of N values.  With split > 0
 //       the experts from there on have the limit limit_b.
+// MODE 3: out[sorted row][n] = silu(x . w0[e][n]) * (x . w1[e][n]) * s * post: the weight on the expert's output.
 // MODE 2: out[sorted row][n] = gelu(x . w0[e][n]) * s * post with the exact (erf) GELU: an expert of one matrix, whose
 //       weight stands behind the activation.
 // else: out[(choice, token)][n] = a[sorted row] . w0[e][n] as floats: [top][tokens][N], partial sums that the
@@ -358,7 +397,7 @@ expert_rows_kernel(void* __restrict__ out_, const T* __restrict__ a, const T* __
                    const float* __restrict__ scale_out, int n_rows, int n_tokens, int top, int N, int K, float limit, int split,
                    float limit_b) {
   pdl_launch_dependents();
-  constexpr bool DUAL = MODE == 1;                  // gate and up with the clamped activation
+  constexpr bool DUAL = MODE == 1 || MODE == 3;     // gate and up with the clamped activation, or with SiLU
   constexpr bool MID = MODE != 0;                   // rows out in sorted order, of the compute dtype (MODE 2: one matrix, exact GELU)
   __shared__ float as[AF_EX_TM][AF_EX_TK];
   __shared__ float w0s[AF_EX_TN][AF_EX_TK + 1];
@@ -427,7 +466,8 @@ expert_rows_kernel(void* __restrict__ out_, const T* __restrict__ a, const T* __
     if (MID) {
       const float s = pair_weight != nullptr ? pair_weight[pair] : 1.f;
       const float post = scale_out != nullptr ? scale_out[pair / top] : 1.f;
-      const float val = DUAL ? clamped_glu(s * acc0[m], s * acc1[m], limit) * post
+      const float val = MODE == 3 ? acc0[m] / (1.f + expf(-acc0[m])) * acc1[m] * s * post
+                        : DUAL ? clamped_glu(s * acc0[m], s * acc1[m], limit) * post
                              : 0.5f * acc0[m] * (1.f + erff(acc0[m] * 0.70710678118654752f)) * s * post;
       static_cast<T*>(out_)[(size_t)(row0 + row) * N + n] = from_f32<T>(val);
     } else {
@@ -449,7 +489,13 @@ AF_EXPORT int af_expert_rows(void* out, const void* a, const void* w0, const voi
   AF_REQUIRE(tiles > 0, "af_expert_rows: no tiles");
   const dim3 grid(tiles, (N + AF_EX_TN - 1) / AF_EX_TN);
   AF_REQUIRE(grid.y < 65536, "af_expert_rows: too many outputs");
-  if (w1 != nullptr) {
+  AF_REQUIRE(act == 0 || (act == 1 && w1 == nullptr) || (act == 2 && w1 != nullptr), "af_expert_rows: activation %d", act);
+  if (w1 != nullptr && act == 2) {
+    AF_DISPATCH_DTYPE(dtype, T,
+                      af_launch(expert_rows_kernel<T, 3>, grid, dim3(256), 0, stream, out, (const T*)a, (const T*)w0,
+                                (const T*)w1, perm, plan, pair_weight, scale_out, n_rows, n_tokens, top, N, K, limit, split,
+                                limit_b));
+  } else if (w1 != nullptr) {
     AF_DISPATCH_DTYPE(dtype, T,
                       af_launch(expert_rows_kernel<T, 1>, grid, dim3(256), 0, stream, out, (const T*)a, (const T*)w0,
                                 (const T*)w1, perm, plan, pair_weight, scale_out, n_rows, n_tokens, top, N, K, limit, split,

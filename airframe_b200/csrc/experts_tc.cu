@@ -2,6 +2,7 @@
 // rows that are sorted by expert.
 //
 //   DUAL   mid[row, f] = act(s (x[row] . gate_e[f]), s (x[row] . up_e[f])) * post     (bfloat16, sorted rows)
+//          or, for experts with a SiLU gate, silu(x[row] . gate_e[f]) (x[row] . up_e[f]) * s * post
 //   else   out[choice, token, f] = mid[row] . down_e[f]                               (float, scattered by pair)
 //
 // A tile is 128 output features of one expert (the tcgen05 "A" operand: the TMEM lanes) by up to BN sorted rows of
@@ -67,8 +68,8 @@ struct ExArgs {
   float limit_b;
 };
 
-enum { EX_DOWN = 0, EX_ACT = 1, EX_GATES = 2, EX_GELU = 3 };
-__host__ __device__ constexpr int ex_accs(int epi) { return epi == EX_ACT || epi == EX_GATES ? 2 : 1; }
+enum { EX_DOWN = 0, EX_ACT = 1, EX_GATES = 2, EX_GELU = 3, EX_SILU = 4 };
+__host__ __device__ constexpr int ex_accs(int epi) { return epi == EX_ACT || epi == EX_GATES || epi == EX_SILU ? 2 : 1; }
 
 __device__ __forceinline__ float ex_act(float g, float u, float limit) {
   g = fminf(g, limit);
@@ -78,6 +79,13 @@ __device__ __forceinline__ float ex_act(float g, float u, float limit) {
   float t;
   asm("tanh.approx.f32 %0, %1;" : "=f"(t) : "f"(0.851f * g));
   return 0.5f * g * (1.f + t) * (u + 1.f);
+}
+
+// silu(g) u, the sigmoid from the tangent as above
+__device__ __forceinline__ float ex_silu(float g, float u) {
+  float t;
+  asm("tanh.approx.f32 %0, %1;" : "=f"(t) : "f"(0.5f * g));
+  return 0.5f * g * (1.f + t) * u;
 }
 
 __device__ __forceinline__ void ex_tile(const ExArgs& a, int row_tile, int bn, int* expert, int* row0, int* rows) {
@@ -300,6 +308,8 @@ expert_rows_tc_kernel(const __grid_constant__ CUtensorMap map_w0, const __grid_c
             if (j >= n || f >= a.N) continue;
             if constexpr (SINGLE)       // (the weight stands behind the activation: it is the expert's output that is weighed)
               o[(size_t)j * a.N] = __float2bfloat16_rn(0.5f * g[j] * (1.f + erff(g[j] * 0.70710678118654752f)) * s * post);
+            else if constexpr (EPI == EX_SILU)      // (likewise)
+              o[(size_t)j * a.N] = __float2bfloat16_rn(ex_silu(g[j], u[j]) * s * post);
             else
               o[(size_t)j * a.N] = __float2bfloat16_rn(ex_act(s * g[j], s * u[j], limit) * post);
           }
@@ -366,7 +376,7 @@ int ex_launch_bn(int bn, const CUtensorMap& m0, const CUtensorMap& m1, const CUt
 // the pairs' tokens name, gathered; else the first product's output); w0, w1 [experts, N, K] bfloat16; tile: the
 // plan's row tile (16, 32, 64, 128 or 256; at most so many rows a plan entry).  K a multiple of 8, bases 16-byte
 // aligned.  act 1 (no w1): out[sorted row] = gelu(a w0[e]^T) * s * post with the exact (erf) GELU, rows of the
-// compute dtype like the two-matrix form's.  Otherwise as af_expert_rows (split > 0: experts from there on have the
+// compute dtype like the two-matrix form's.  act 2 (with w1): silu(a w0[e]^T) * (a w1[e]^T) * s * post.  Otherwise as af_expert_rows (split > 0: experts from there on have the
 // limit limit_b).
 AF_EXPORT int af_expert_rows_tc(void* out, const void* a, const void* w0, const void* w1, int n_experts, const int* perm,
                                 const int* plan, const float* pair_weight, const float* scale_out, int n_rows,
@@ -392,7 +402,9 @@ AF_EXPORT int af_expert_rows_tc(void* out, const void* a, const void* w0, const 
               plan != nullptr ? max_tiles : (n_rows + tile - 1) / tile, perm, plan, pair_weight, scale_out, limit, err};
   args.split = split, args.limit_b = limit_b;
   AF_REQUIRE(args.max_row_tiles > 0, "af_expert_rows_tc: no tiles");
-  AF_REQUIRE(act == 0 || (act == 1 && w1 == nullptr), "af_expert_rows_tc: the exact GELU stands behind one matrix");
+  AF_REQUIRE(act == 0 || (act == 1 && w1 == nullptr) || (act == 2 && w1 != nullptr),
+             "af_expert_rows_tc: the exact GELU stands behind one matrix, SiLU on the first of two");
+  if (act == 2) return ex_launch_bn<EX_SILU>(tile, m0, m1, mx, args, stream);
   if (w1 != nullptr) return ex_launch_bn<EX_ACT>(tile, m0, m1, mx, args, stream);
   if (act == 1) return ex_launch_bn<EX_GELU>(tile, m0, m1, mx, args, stream);
   return ex_launch_bn<EX_DOWN>(tile, m0, m1, mx, args, stream);

@@ -4,6 +4,8 @@
 //   norm_of_sum   x <- layer_norm(alpha x + gate * (scale_a a + scale_b b)), the terms tensors or split-K partial sums,
 //                 gate = sigmoid(z + z_bias) per element or nothing; in the same pass a copy of the new row in the
 //                 compute dtype for the sublayer that reads it next, and, for single tokens, that row shifted;
+//   add_layer_norm  x <- x + layer_norm(scale_a a + scale_b b) (the norm on the sublayer's output alone): the same
+//                 kernels with the stream added behind the norm instead of in front of it;
 //   token_shift   h_t = x_t + (x_(t-1) - x_t) mu, the row before a sequence's first row of the step from its state
 //                 (zeros before the first token), which keeps the sequence's last row.
 #include "common.cuh"
@@ -148,7 +150,8 @@ layer_norm_row_kernel(TY* __restrict__ y, const float* __restrict__ x, const flo
 // ---------------------------------------------------------------- the norm of the residual sum
 
 // Any row size: the row waits in shared memory between the passes.
-template <typename TY>
+// POST: the stream is added to the norm's result, not to its input.
+template <typename TY, bool POST>
 __global__ void __launch_bounds__(256)
 norm_of_sum_kernel(LnSumArgs p) {
   pdl_launch_dependents();
@@ -162,7 +165,7 @@ norm_of_sum_kernel(LnSumArgs p) {
     float v = ln_term1(p.a, base + i);
     if (p.b.p != nullptr) v += ln_term1(p.b, base + i);
     if (p.z.p != nullptr) v *= ln_sigmoid(ln_term1(p.z, base + i) + p.z_bias[i]);
-    v = fmaf(p.alpha, p.x[base + i], v);
+    if (!POST) v = fmaf(p.alpha, p.x[base + i], v);
     row[i] = v;
     s += v;
   }
@@ -172,7 +175,8 @@ norm_of_sum_kernel(LnSumArgs p) {
   const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)hidden + p.eps);
   const int slot = p.hs != nullptr ? p.slots[r] : -1;
   for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
-    const float v = (row[i] - mean) * inv * p.w[i] + p.bias[i];
+    float v = (row[i] - mean) * inv * p.w[i] + p.bias[i];
+    if (POST) v += p.x[base + i];
     p.x[base + i] = v;
     if (p.y != nullptr) reinterpret_cast<TY*>(p.y)[base + i] = from_f32<TY>(v);
     if (p.hs != nullptr) {
@@ -186,14 +190,14 @@ norm_of_sum_kernel(LnSumArgs p) {
 // Rows of whole groups of four: a thread keeps NV groups in registers and every load of a group is in flight before
 // the first sum.  Few rows (a decode step): one group a thread, the weights and the state asked for before the wait for
 // the kernel in front; many rows (MANY): two groups a thread, the weights read where they are used (L1 holds them).
-template <typename TY, int NV, bool MANY>
+template <typename TY, int NV, bool MANY, bool POST>
 __global__ void __launch_bounds__(MANY ? 512 : 1024, MANY ? 3 : 1)
 norm_of_sum_row_kernel(LnSumArgs p) {
   pdl_launch_dependents();
   __shared__ float scratch[33];
   const int r = blockIdx.x, hidden = p.hidden;
   const size_t base = (size_t)r * hidden;
-  float v[NV][4], wv[NV][4], bv[NV][4], zb[NV][4], mu[NV][4], pv[NV][4];
+  float v[NV][4], wv[NV][4], bv[NV][4], zb[NV][4], mu[NV][4], pv[NV][4], xs[POST ? NV : 1][4];
   const int slot = p.hs != nullptr ? p.slots[r] : -1;
   auto get4 = [](const float* src, float* dst) {
     const float4 q = *reinterpret_cast<const float4*>(src);
@@ -231,7 +235,8 @@ norm_of_sum_row_kernel(LnSumArgs p) {
     for (int u = 0; u < 4; ++u) {
       float t = v[n][u] + bt[u];
       if (p.z.p != nullptr) t *= ln_sigmoid(zt[u] + zb[n][u]);
-      v[n][u] = fmaf(p.alpha, xv[u], t);
+      if (POST) xs[n][u] = xv[u], v[n][u] = t;
+      else v[n][u] = fmaf(p.alpha, xv[u], t);
       s += v[n][u];
     }
   }
@@ -253,7 +258,7 @@ norm_of_sum_row_kernel(LnSumArgs p) {
     if (i >= hidden) continue;
     if (MANY) get4(p.w + i, wv[n]), get4(p.bias + i, bv[n]);
 #pragma unroll
-    for (int u = 0; u < 4; ++u) v[n][u] = v[n][u] * inv * wv[n][u] + bv[n][u];
+    for (int u = 0; u < 4; ++u) v[n][u] = v[n][u] * inv * wv[n][u] + bv[n][u] + (POST ? xs[n][u] : 0.f);
     ln_store4(p.x + base + i, v[n]);
     if (p.y != nullptr) ln_store4(reinterpret_cast<TY*>(p.y) + base + i, v[n]);
     if (p.hs != nullptr) {
@@ -348,11 +353,11 @@ int ln_launch(void* y, const float* x, const float* w, const float* b, const int
   AF_CHECK_LAUNCH("af_layer_norm");
 }
 
-template <typename TY>
+template <typename TY, bool POST>
 int ln_launch_sum(const LnSumArgs& p, cudaStream_t stream) {
   static bool raised[AF_MAX_DEVICES];
-  if (int e = ln_raise(norm_of_sum_kernel<TY>, raised, p.hidden)) return e;
-  af_launch(norm_of_sum_kernel<TY>, dim3(p.n_rows), dim3(256), (size_t)p.hidden * sizeof(float), stream, p);
+  if (int e = ln_raise(norm_of_sum_kernel<TY, POST>, raised, p.hidden)) return e;
+  af_launch(norm_of_sum_kernel<TY, POST>, dim3(p.n_rows), dim3(256), (size_t)p.hidden * sizeof(float), stream, p);
   AF_CHECK_LAUNCH("af_norm_of_sum");
 }
 
@@ -376,12 +381,15 @@ AF_EXPORT int af_layer_norm(void* y, int y_dtype, const float* x, const float* w
   return 0;
 }
 
-// y_dtype: of y and hs.  The terms' partial sums lie n_rows * hidden elements apart.
+// y_dtype: of y and hs.  The terms' partial sums lie n_rows * hidden elements apart.  `post`: the stream is added
+// behind the norm (alpha, the gate and the shift belong to the other form).
 AF_EXPORT int af_norm_of_sum(float* x, const void* a, int a_dtype, int a_parts, float scale_a, const void* b, int b_dtype,
                              int b_parts, float scale_b, const void* z, int z_dtype, int z_parts, const float* z_bias,
                              float alpha, const float* w, const float* bias, float eps, void* y, void* hs, int y_dtype,
-                             const float* mu, float* prev, const int* slots, int n_rows, int hidden, cudaStream_t stream) {
+                             const float* mu, float* prev, const int* slots, int n_rows, int hidden, int post,
+                             cudaStream_t stream) {
   if (n_rows == 0) return 0;
+  AF_REQUIRE(!post || (z == nullptr && hs == nullptr), "af_norm_of_sum: a norm in front of the sum has no gate and no shift");
   AF_REQUIRE(n_rows > 0 && hidden > 0 && hidden <= LN_MAX_ROW, "af_norm_of_sum: rows of 1 to %d values", LN_MAX_ROW);
   AF_REQUIRE(x != nullptr && a != nullptr && w != nullptr && bias != nullptr && (z == nullptr || z_bias != nullptr),
              "af_norm_of_sum: a stream, a term, the norm's weight and bias, a bias with a gate");
@@ -404,17 +412,19 @@ AF_EXPORT int af_norm_of_sum(float* x, const void* a, int a_dtype, int a_parts, 
     const bool many = n_rows >= 256 && hidden >= 1024 && hidden <= 4096;
     const int nv = many || hidden > 4096 ? 2 : 1;
     const int threads = ((hidden / 4 + nv - 1) / nv + 31) / 32 * 32;
-#define LN_LAUNCH(TY)                                                                                              \
-  do {                                                                                                             \
-    if (many) af_launch(norm_of_sum_row_kernel<TY, 2, true>, dim3(n_rows), dim3(threads), 0, stream, p);           \
-    else if (nv == 2) af_launch(norm_of_sum_row_kernel<TY, 2, false>, dim3(n_rows), dim3(threads), 0, stream, p);  \
-    else af_launch(norm_of_sum_row_kernel<TY, 1, false>, dim3(n_rows), dim3(threads), 0, stream, p);               \
+#define LN_LAUNCH(TY, P)                                                                                              \
+  do {                                                                                                                \
+    if (many) af_launch(norm_of_sum_row_kernel<TY, 2, true, P>, dim3(n_rows), dim3(threads), 0, stream, p);           \
+    else if (nv == 2) af_launch(norm_of_sum_row_kernel<TY, 2, false, P>, dim3(n_rows), dim3(threads), 0, stream, p);  \
+    else af_launch(norm_of_sum_row_kernel<TY, 1, false, P>, dim3(n_rows), dim3(threads), 0, stream, p);               \
   } while (0)
-    AF_DISPATCH_DTYPE(y_dtype, TY, LN_LAUNCH(TY));
+    if (post) AF_DISPATCH_DTYPE(y_dtype, TY, LN_LAUNCH(TY, true));
+    else AF_DISPATCH_DTYPE(y_dtype, TY, LN_LAUNCH(TY, false));
 #undef LN_LAUNCH
     AF_CHECK_LAUNCH("af_norm_of_sum");
   }
-  AF_DISPATCH_DTYPE(y_dtype, TY, return ln_launch_sum<TY>(p, stream));
+  if (post) AF_DISPATCH_DTYPE(y_dtype, TY, return (ln_launch_sum<TY, true>(p, stream)));
+  AF_DISPATCH_DTYPE(y_dtype, TY, return (ln_launch_sum<TY, false>(p, stream)));
   return 0;
 }
 

@@ -80,7 +80,7 @@ AF_EXPORT int af_delta_prep(float* out, const float* proj, long long ld, int off
 
 // ---------------------------------------------------------------- the scan over a matrix state
 
-enum AfScanMode { AF_SCAN_DECAY = 0, AF_SCAN_DELTA = 1, AF_SCAN_CHANNEL = 3 };
+enum AfScanMode { AF_SCAN_DECAY = 0, AF_SCAN_DELTA = 1, AF_SCAN_CHANNEL = 3, AF_SCAN_GATED = 4 };
 // (inside the library: the decay recurrence whose r, k and v pass through SiLU as they are read; a kernel of
 // its own, so that the others carry no exponentials)
 #define AF_SCAN_DECAY_SILU 2
@@ -90,11 +90,15 @@ enum AfScanMode { AF_SCAN_DECAY = 0, AF_SCAN_DELTA = 1, AF_SCAN_CHANNEL = 3 };
 //   DECAY:  S <- decay[h] S + k v^T                          o = S^T q     (q = `r`)
 //   DELTA:  S <- diag(w) S - au (u^T S) + k v^T              o = S^T r     (decay and removal act on the S before the token)
 //   CHANNEL: S <- diag(w) S + k v^T                          o = S^T q     (a decay per key channel and token, no removal)
-// With `silu` the r, k and v values go through x / (1 + exp(-x)) as they are read.
+//   GATED:  S <- diag(w) S, then S <- S + beta k (v - S^T k)^T  o = S^T q     (the delta rule behind a decay per key channel)
+// r and k may belong to fewer heads than v (`rep` heads share one).  With `silu` the r, k and v values go through x / (1 + exp(-x)) as they are read.
 struct AfScanArgs {
   const float *r, *k, *v, *w, *u, *au;
   long long r_ts, k_ts, v_ts, w_ts, u_ts, au_ts;
   const float* decay;          // [heads] (DECAY)
+  const float* beta;           // GATED: one number per token and head, tokens beta_ts apart
+  long long beta_ts;
+  int rep;                     // heads that share an r and k head
   float* state;                // [slots][heads][dv][dk]
   float* out;                  // [tokens][heads * dv]
   long long out_ts;
@@ -134,13 +138,14 @@ state_scan_kernel(AfScanArgs a) {
   constexpr bool SILU = MODE == AF_SCAN_DECAY_SILU;
   extern __shared__ __align__(16) float smem[];
   const int P = a.lanes, CT = a.cols, CH = a.chunk, dk = a.dk, dv = a.dv;
-  const int NV = MODE == AF_SCAN_DELTA ? 5 : MODE == AF_SCAN_CHANNEL ? 3 : 2;   // staged key-sized vectors: r, k (, w (, u, au))
+  constexpr bool GATED = MODE == AF_SCAN_GATED;
+  const int NV = MODE == AF_SCAN_DELTA ? 5 : (MODE == AF_SCAN_CHANNEL || GATED) ? 3 : 2;   // staged key-sized vectors: r, k (, w (, u, au))
   const int dkp = P * (R + AF_SCAN_PAD(R));
   const int tok_floats = NV * dkp + CT;                     // a token's staged floats: the vectors, then its v tile
   const int buf_floats = CH * tok_floats;
   const int tid = threadIdx.x, nthr = blockDim.x;
   const int part = tid % P, col = tid / P;
-  const int h = blockIdx.y, b = blockIdx.z;
+  const int h = blockIdx.y, b = blockIdx.z, hk = h / a.rep;
   const int j0 = blockIdx.x * CT, j = j0 + col;
   const bool col_on = j < dv;
   // a token's values in the order they are fetched: NV key vectors of dk, then CT values of v
@@ -190,6 +195,8 @@ state_scan_kernel(AfScanArgs a) {
   constexpr int FE = VEC ? AF_SCAN_VEC_ITEMS : AF_SCAN_PREFETCH;   // key-vector items a thread fetches (per vector if VEC)
   constexpr int FV = VEC ? AF_SCAN_VEC_ITEMS : 1;                  // value-tile items
   float4 pq[VEC ? 5 : 1][VEC ? FE : 1], pvq[FV];
+  float pbeta = 0.f;                                         // GATED: thread tt's token's (CH <= 16 threads)
+  float* beta_s = smem + 2 * buf_floats;                     // [buffer][CH]
   float pf[VEC ? 1 : AF_SCAN_PREFETCH];
   int ftt[VEC ? FE : 1], fgo[VEC ? FE : 1], fso[VEC ? FE : 1], vtt[FV], vgo[FV], vso[FV];
   if constexpr (VEC) {
@@ -199,7 +206,7 @@ state_scan_kernel(AfScanArgs a) {
       const int idx = tid + e * nthr;
       const int tt = idx / dkq, c = (idx - tt * dkq) * 4;
       ftt[e] = idx < CH * dkq ? tt : CH;                     // (CH: never among a chunk's tokens)
-      fgo[e] = h * dk + c;
+      fgo[e] = c;
       fso[e] = tt * tok_floats + (c / R) * (R + AF_SCAN_PAD(R)) + c % R;
     }
 #pragma unroll
@@ -217,6 +224,8 @@ state_scan_kernel(AfScanArgs a) {
     return q;
   };
   auto fetch = [&](int t0, int n) {                          // tokens t0 .. t0 + n - 1 into registers
+    if constexpr (GATED)
+      if (tid < n) pbeta = a.beta[(size_t)(t0 + tid) * a.beta_ts + h];
     if constexpr (VEC) {
 #pragma unroll
       for (int v = 0; v < NV; ++v) {
@@ -224,7 +233,8 @@ state_scan_kernel(AfScanArgs a) {
         const long long ts = v == 0 ? a.r_ts : v == 1 ? a.k_ts : v == 2 ? a.w_ts : v == 3 ? a.u_ts : a.au_ts;
 #pragma unroll
         for (int e = 0; e < FE; ++e)
-          if (ftt[e] < n) pq[v][e] = *reinterpret_cast<const float4*>(p + (size_t)(t0 + ftt[e]) * ts + fgo[e]);
+          if (ftt[e] < n)
+            pq[v][e] = *reinterpret_cast<const float4*>(p + (size_t)(t0 + ftt[e]) * ts + (v < 2 ? hk : h) * dk + fgo[e]);
       }
 #pragma unroll
       for (int e = 0; e < FV; ++e)
@@ -241,7 +251,7 @@ state_scan_kernel(AfScanArgs a) {
             const int vec = x / dk, c = x - vec * dk;
             const float* p = vec == 0 ? a.r + t * a.r_ts : vec == 1 ? a.k + t * a.k_ts
                            : vec == 2 ? a.w + t * a.w_ts : vec == 3 ? a.u + t * a.u_ts : a.au + t * a.au_ts;
-            val = p[h * dk + c];
+            val = p[(vec < 2 ? hk : h) * dk + c];
           } else {
             const int jj = j0 + x - NV * dk;
             if (jj < dv) val = a.v[t * a.v_ts + h * dv + jj];
@@ -252,6 +262,8 @@ state_scan_kernel(AfScanArgs a) {
     }
   };
   auto stage = [&](float* buf, int n) {                      // registers into a shared-memory buffer
+    if constexpr (GATED)
+      if (tid < n) beta_s[(buf == smem ? 0 : CH) + tid] = pbeta;
     if constexpr (VEC) {
 #pragma unroll
       for (int v = 0; v < NV; ++v)
@@ -329,6 +341,20 @@ state_scan_kernel(AfScanArgs a) {
           *reinterpret_cast<float4*>(wv + i) = *reinterpret_cast<const float4*>(tk + 2 * dkp + i);
 #pragma unroll
         for (int i = 0; i < R; ++i) S[i] = wv[i] * S[i] + kv[i] * vj;
+      } else if (GATED) {
+        float wv[R], d0 = 0.f, d1 = 0.f;
+#pragma unroll
+        for (int i = 0; i < R; i += 4)
+          *reinterpret_cast<float4*>(wv + i) = *reinterpret_cast<const float4*>(tk + 2 * dkp + i);
+#pragma unroll
+        for (int i = 0; i < R; i += 2) {
+          S[i] *= wv[i], S[i + 1] *= wv[i + 1];
+          d0 = fmaf(kv[i], S[i], d0);
+          d1 = fmaf(kv[i + 1], S[i + 1], d1);
+        }
+        const float u = beta_s[which * CH + tt] * (vj - lanes_sum(d0 + d1, P));
+#pragma unroll
+        for (int i = 0; i < R; ++i) S[i] = fmaf(kv[i], u, S[i]);
       } else {
 #pragma unroll
         for (int i = 0; i < R; ++i) S[i] = dec * S[i] + kv[i] * vj;
@@ -360,7 +386,7 @@ state_step_kernel(AfScanArgs a, int vec) {
   const int P = a.lanes, CT = a.cols, dk = a.dk, dv = a.dv;
   const int tid = threadIdx.x;
   const int part = tid % P, col = tid / P;
-  const int h = blockIdx.y, b = blockIdx.z;
+  const int h = blockIdx.y, b = blockIdx.z, hk = h / a.rep;
   const int j = blockIdx.x * CT + col;
   const bool col_on = j < dv;
   const int slot = a.slots[b];
@@ -387,8 +413,8 @@ state_step_kernel(AfScanArgs a, int vec) {
   }
   const float dec = (MODE == AF_SCAN_DECAY || MODE == AF_SCAN_DECAY_SILU) ? a.decay[h] : 0.f;
   pdl_wait();
-  auto piece = [&](const float* p, float* dst, bool act) {
-    p += h * dk + c0;
+  auto piece = [&](const float* p, float* dst, bool act, int head) {
+    p += head * dk + c0;
     if (vec) {
 #pragma unroll
       for (int i = 0; i < R; i += 4) {
@@ -406,15 +432,15 @@ state_step_kernel(AfScanArgs a, int vec) {
     }
   };
   float rv[R], kv[R];
-  piece(a.r + t * a.r_ts, rv, SILU);
-  piece(a.k + t * a.k_ts, kv, SILU);
+  piece(a.r + t * a.r_ts, rv, SILU, hk);
+  piece(a.k + t * a.k_ts, kv, SILU, hk);
   float vj = col_on ? a.v[t * a.v_ts + h * dv + j] : 0.f;
   if (SILU) vj = vj / (1.f + expf(-vj));
   if (MODE == AF_SCAN_DELTA) {
     float wv[R], uv[R], av[R];
-    piece(a.w + t * a.w_ts, wv, false);
-    piece(a.u + t * a.u_ts, uv, false);
-    piece(a.au + t * a.au_ts, av, false);
+    piece(a.w + t * a.w_ts, wv, false, h);
+    piece(a.u + t * a.u_ts, uv, false, h);
+    piece(a.au + t * a.au_ts, av, false, h);
     float d0 = 0.f, d1 = 0.f;
 #pragma unroll
     for (int i = 0; i < R; i += 2) d0 += uv[i] * S[i], d1 += uv[i + 1] * S[i + 1];
@@ -423,9 +449,21 @@ state_step_kernel(AfScanArgs a, int vec) {
     for (int i = 0; i < R; ++i) S[i] = wv[i] * S[i] - av[i] * dot + kv[i] * vj;
   } else if (MODE == AF_SCAN_CHANNEL) {
     float wv[R];
-    piece(a.w + t * a.w_ts, wv, false);
+    piece(a.w + t * a.w_ts, wv, false, h);
 #pragma unroll
     for (int i = 0; i < R; ++i) S[i] = wv[i] * S[i] + kv[i] * vj;
+  } else if (MODE == AF_SCAN_GATED) {
+    float wv[R], d0 = 0.f, d1 = 0.f;
+    piece(a.w + t * a.w_ts, wv, false, h);
+#pragma unroll
+    for (int i = 0; i < R; i += 2) {
+      S[i] *= wv[i], S[i + 1] *= wv[i + 1];
+      d0 = fmaf(kv[i], S[i], d0);
+      d1 = fmaf(kv[i + 1], S[i + 1], d1);
+    }
+    const float u = a.beta[t * a.beta_ts + h] * (vj - lanes_sum(d0 + d1, P));
+#pragma unroll
+    for (int i = 0; i < R; ++i) S[i] = fmaf(kv[i], u, S[i]);
   } else {
 #pragma unroll
     for (int i = 0; i < R; ++i) S[i] = dec * S[i] + kv[i] * vj;
@@ -451,6 +489,7 @@ template <int R>
 static int launch_step(const AfScanArgs& a, int mode, int vec, dim3 grid, int threads, cudaStream_t stream) {
   if (mode == AF_SCAN_DELTA) af_launch(state_step_kernel<R, AF_SCAN_DELTA>, grid, dim3(threads), 0, stream, a, vec);
   else if (mode == AF_SCAN_CHANNEL) af_launch(state_step_kernel<R, AF_SCAN_CHANNEL>, grid, dim3(threads), 0, stream, a, vec);
+  else if (mode == AF_SCAN_GATED) af_launch(state_step_kernel<R, AF_SCAN_GATED>, grid, dim3(threads), 0, stream, a, vec);
   else if (a.silu) af_launch(state_step_kernel<R, AF_SCAN_DECAY_SILU>, grid, dim3(threads), 0, stream, a, vec);
   else af_launch(state_step_kernel<R, AF_SCAN_DECAY>, grid, dim3(threads), 0, stream, a, vec);
   AF_CHECK_LAUNCH("af_state_scan");
@@ -458,24 +497,26 @@ static int launch_step(const AfScanArgs& a, int mode, int vec, dim3 grid, int th
 
 template <int R, bool VEC>
 static int launch_scan(const AfScanArgs& a, int mode, dim3 grid, int threads, size_t smem, cudaStream_t stream) {
-  static bool raised[4][AF_MAX_DEVICES];
+  static bool raised[5][AF_MAX_DEVICES];
   auto k0 = state_scan_kernel<R, AF_SCAN_DECAY, VEC>;
   auto k1 = state_scan_kernel<R, AF_SCAN_DELTA, VEC>;
   auto k2 = state_scan_kernel<R, AF_SCAN_DECAY_SILU, VEC>;
   auto k3 = state_scan_kernel<R, AF_SCAN_CHANNEL, VEC>;
-  const int which = mode == AF_SCAN_DELTA ? 1 : mode == AF_SCAN_CHANNEL ? 3 : (a.silu ? 2 : 0);
+  auto k4 = state_scan_kernel<R, AF_SCAN_GATED, VEC>;
+  const int which = mode == AF_SCAN_DELTA ? 1 : mode == AF_SCAN_CHANNEL ? 3 : mode == AF_SCAN_GATED ? 4 : (a.silu ? 2 : 0);
   if (smem > 48 * 1024) {
     const int dev = af_current_device();
     if (dev < 0) return -1;
     if (af_first_on_device(raised[which], dev)) {
-      cudaError_t e = cudaFuncSetAttribute(which == 1 ? k1 : which == 2 ? k2 : which == 3 ? k3 : k0, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                           96 * 1024);
+      cudaError_t e = cudaFuncSetAttribute(which == 1 ? k1 : which == 2 ? k2 : which == 3 ? k3 : which == 4 ? k4 : k0, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                           97 * 1024);
       if (e != cudaSuccess) return af_fail((int)e, "af_state_scan: %s", cudaGetErrorString(e));
     }
   }
   if (which == 1) af_launch(k1, grid, dim3(threads), smem, stream, a);
   else if (which == 2) af_launch(k2, grid, dim3(threads), smem, stream, a);
   else if (which == 3) af_launch(k3, grid, dim3(threads), smem, stream, a);
+  else if (which == 4) af_launch(k4, grid, dim3(threads), smem, stream, a);
   else af_launch(k0, grid, dim3(threads), smem, stream, a);
   AF_CHECK_LAUNCH("af_state_scan");
 }
@@ -497,7 +538,7 @@ static void scan_cut(int mode, int dk, int dv, bool vec, long long units, int wa
   // (few blocks a head, many warps a block) cost less than narrow ones, also where that leaves SMs without a block
   int ct = 256 / p;
   while (ct > 4 && ct / 2 >= dv && (ct / 2) * p >= 32) ct /= 2;   // (no wider than the state's columns need; whole warps)
-  const int nv = mode == AF_SCAN_DELTA ? 5 : mode == AF_SCAN_CHANNEL ? 3 : 2;
+  const int nv = mode == AF_SCAN_DELTA ? 5 : mode == AF_SCAN_CHANNEL || mode == AF_SCAN_GATED ? 3 : 2;
   const int tok_vals = nv * dk + ct, tok_floats = nv * p * (r + AF_SCAN_PAD(r)) + ct;
   const int threads = ct * p;
   int ch = 16;
@@ -512,11 +553,15 @@ static void scan_cut(int mode, int dk, int dv, bool vec, long long units, int wa
 
 AF_EXPORT int af_state_scan(int mode, const float* r, long long r_ts, const float* k, long long k_ts, const float* v,
                             long long v_ts, const float* w, long long w_ts, const float* u, long long u_ts,
-                            const float* au, long long au_ts, const float* decay, float* state, float* out,
+                            const float* au, long long au_ts, const float* decay, const float* beta, long long beta_ts,
+                            int rep, float* state, float* out,
                             long long out_ts, const int* seq_starts, const int* slots, int n_seqs, int n_tokens, int heads,
                             int dk, int dv, int silu, cudaStream_t stream) {
   if (n_seqs == 0) return 0;
-  AF_REQUIRE(mode == AF_SCAN_DECAY || mode == AF_SCAN_DELTA || mode == AF_SCAN_CHANNEL, "af_state_scan: mode %d", mode);
+  AF_REQUIRE(mode == AF_SCAN_DECAY || mode == AF_SCAN_DELTA || mode == AF_SCAN_CHANNEL || mode == AF_SCAN_GATED,
+             "af_state_scan: mode %d", mode);
+  AF_REQUIRE(rep >= 1 && heads % rep == 0 && (mode != AF_SCAN_GATED || beta != nullptr),
+             "af_state_scan: %d heads share a key head of %d, or no step sizes", rep, heads);
   AF_REQUIRE(!(mode != AF_SCAN_DECAY && silu), "af_state_scan: only the plain decay takes its vectors through SiLU");
   AF_REQUIRE(n_seqs > 0 && heads > 0 && dk > 0 && dv > 0 && dk <= 1024, "af_state_scan: bad sizes (key size up to 1024)");
   AF_REQUIRE(n_seqs < 65536 && heads < 65536, "af_state_scan: too many sequences or heads for one grid");
@@ -524,11 +569,12 @@ AF_EXPORT int af_state_scan(int mode, const float* r, long long r_ts, const floa
   a.r = r, a.k = k, a.v = v, a.w = w, a.u = u, a.au = au;
   a.r_ts = r_ts, a.k_ts = k_ts, a.v_ts = v_ts, a.w_ts = w_ts, a.u_ts = u_ts, a.au_ts = au_ts;
   a.decay = decay, a.state = state, a.out = out, a.out_ts = out_ts, a.seq_starts = seq_starts, a.slots = slots;
+  a.beta = beta, a.beta_ts = beta_ts, a.rep = rep;
   a.heads = heads, a.dk = dk, a.dv = dv, a.silu = silu;
   // whole 16-byte pieces: sizes and strides in multiples of four floats, bases on 16 bytes
   bool vec = dk % 4 == 0 && dv % 4 == 0 && ((r_ts | k_ts | v_ts) & 3) == 0 &&
              (((uintptr_t)r | (uintptr_t)k | (uintptr_t)v) & 15) == 0;
-  if (mode == AF_SCAN_CHANNEL) vec = vec && (w_ts & 3) == 0 && ((uintptr_t)w & 15) == 0;
+  if (mode == AF_SCAN_CHANNEL || mode == AF_SCAN_GATED) vec = vec && (w_ts & 3) == 0 && ((uintptr_t)w & 15) == 0;
   if (mode == AF_SCAN_DELTA)
     vec = vec && ((w_ts | u_ts | au_ts) & 3) == 0 && (((uintptr_t)w | (uintptr_t)u | (uintptr_t)au) & 15) == 0;
   const int sms = af_sm_count();
@@ -536,7 +582,7 @@ AF_EXPORT int af_state_scan(int mode, const float* r, long long r_ts, const floa
   int R, P, CT, CH;
   scan_cut(mode, dk, dv, vec, (long long)heads * n_seqs, sms, &R, &P, &CT, &CH);
   AF_REQUIRE(P * R >= dk, "af_state_scan: key size %d does not fit %d lanes of %d", dk, P, R);
-  const int nv = mode == AF_SCAN_DELTA ? 5 : mode == AF_SCAN_CHANNEL ? 3 : 2;
+  const int nv = mode == AF_SCAN_DELTA ? 5 : mode == AF_SCAN_CHANNEL || mode == AF_SCAN_GATED ? 3 : 2;
   if (vec)
     AF_REQUIRE(CH * (dk / 4) <= AF_SCAN_VEC_ITEMS * CT * P && CH * (CT / 4) <= AF_SCAN_VEC_ITEMS * CT * P,
                "af_state_scan: a token of %d values is too long to stage", nv * dk + CT);
@@ -553,7 +599,8 @@ AF_EXPORT int af_state_scan(int mode, const float* r, long long r_ts, const floa
       default: return launch_step<32>(a, mode, vec ? 1 : 0, grid, CT * P, stream);
     }
   }
-  const size_t smem = (size_t)2 * CH * (nv * P * (R + AF_SCAN_PAD(R)) + CT) * sizeof(float);
+  const size_t smem = (size_t)2 * CH * (nv * P * (R + AF_SCAN_PAD(R)) + CT) * sizeof(float) +
+                      (mode == AF_SCAN_GATED ? 2 * CH * sizeof(float) : 0);
   const dim3 grid((dv + CT - 1) / CT, heads, n_seqs);
   const int threads = CT * P;
   if (vec) {
@@ -749,6 +796,8 @@ AF_EXPORT int af_gated_scan(void* y, int y_dtype, const float* proj, long long l
 
 // ---------------------------------------------------------------- decays of gated linear attention
 
+// What becomes of z: AF_CD_SIGMOID: sigmoid(z)^(1 / tau); AF_CD_SOFTPLUS: exp(-rate[c] softplus(z)), its factor of
+// softplus per channel; AF_CD_LOGIT: z itself (a gate's logits).  For the first:
 // alpha[t][c] = sigmoid(z)^(1 / tau), z = b[c] + sum_r w2t[r][c] * low[t][r], with low the `rank` columns of the packed
 // float32 projection rows that begin at off_low (the first factor of a low-rank pair, applied with the other
 // projections), w2t [rank, n] the second factor transposed.  Worked out as exp(log(sigmoid(z)) / tau) with
@@ -762,9 +811,13 @@ AF_EXPORT int af_gated_scan(void* y, int y_dtype, const float* proj, long long l
 #define AF_CD_TOK 16
 #define AF_CD_SLICES 8
 
-__device__ __forceinline__ float decay_of(float z, float inv_tau) {
-  const float ls = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
-  return expf(ls * inv_tau);
+enum AfDecayKind { AF_CD_SIGMOID = 0, AF_CD_SOFTPLUS = 1, AF_CD_LOGIT = 2 };
+
+// `p`: 1 / tau, or the channel's rate
+__device__ __forceinline__ float decay_of(float z, float p, int kind) {
+  if (kind == AF_CD_LOGIT) return z;
+  const float l = log1pf(expf(-fabsf(z)));
+  return kind == AF_CD_SOFTPLUS ? expf(-p * (fmaxf(z, 0.f) + l)) : expf((fminf(z, 0.f) - l) * p);
 }
 
 // z[.] += w2t[r][c] * low[r][.] for r in [r0, r1): the partial sum of one run, from zero
@@ -789,13 +842,14 @@ __device__ __forceinline__ void decay_run(float* p, const float* __restrict__ w2
 
 __global__ void __launch_bounds__(128)
 channel_decay_kernel(float* __restrict__ alpha, const float* __restrict__ proj, long long ld, int off_low,
-                     const float* __restrict__ w2t, const float* __restrict__ bias, int rank, int n, int n_tokens,
-                     float inv_tau) {
+                     const float* __restrict__ w2t, const float* __restrict__ bias, const float* __restrict__ rate,
+                     int rank, int n, int n_tokens, float inv_tau, int kind) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) float low[];                // [rank][AF_CD_TOK]
   const int t0 = blockIdx.y * AF_CD_TOK;
   const int c = blockIdx.x * 128 + threadIdx.x;
-  const float b = c < n ? bias[c] : 0.f;
+  const float b = c < n && bias != nullptr ? bias[c] : 0.f;
+  const float f = kind == AF_CD_SOFTPLUS ? (c < n ? rate[c] : 0.f) : inv_tau;
   pdl_wait();
   proj = pdl_fresh(proj);
   for (int i = threadIdx.x; i < rank * AF_CD_TOK; i += 128) {
@@ -817,21 +871,22 @@ channel_decay_kernel(float* __restrict__ alpha, const float* __restrict__ proj, 
 #pragma unroll
   for (int tt = 0; tt < AF_CD_TOK; ++tt) {
     if (t0 + tt >= n_tokens) break;
-    alpha[(size_t)(t0 + tt) * n + c] = decay_of(z[tt] + b, inv_tau);
+    alpha[(size_t)(t0 + tt) * n + c] = decay_of(z[tt] + b, f, kind);
   }
 }
 
 // Up to AF_CD_TOK tokens: block = 32 channels x AF_CD_SLICES runs (warp s takes run s).
 __global__ void __launch_bounds__(32 * AF_CD_SLICES)
 channel_decay_few_kernel(float* __restrict__ alpha, const float* __restrict__ proj, long long ld, int off_low,
-                         const float* __restrict__ w2t, const float* __restrict__ bias, int rank, int n, int n_tokens,
-                         float inv_tau) {
+                         const float* __restrict__ w2t, const float* __restrict__ bias, const float* __restrict__ rate,
+                         int rank, int n, int n_tokens, float inv_tau, int kind) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) float low[];                // [rank][AF_CD_TOK], then the runs' sums [runs][tokens][32]
   float* sums = low + (size_t)rank * AF_CD_TOK;
   const int lane = threadIdx.x & 31, s = threadIdx.x >> 5;
   const int c = blockIdx.x * 32 + lane;
-  const float b = c < n ? bias[c] : 0.f;
+  const float b = c < n && bias != nullptr ? bias[c] : 0.f;
+  const float f = kind == AF_CD_SOFTPLUS ? (c < n ? rate[c] : 0.f) : inv_tau;
   pdl_wait();
   proj = pdl_fresh(proj);
   for (int i = threadIdx.x; i < rank * AF_CD_TOK; i += blockDim.x) {
@@ -850,24 +905,27 @@ channel_decay_few_kernel(float* __restrict__ alpha, const float* __restrict__ pr
     float z = 0.f;
 #pragma unroll
     for (int q = 0; q < AF_CD_SLICES; ++q) z += sums[(q * AF_CD_TOK + tt) * 32 + lane];
-    alpha[(size_t)tt * n + c] = decay_of(z + b, inv_tau);
+    alpha[(size_t)tt * n + c] = decay_of(z + b, f, kind);
   }
 }
 
 AF_EXPORT int af_channel_decay(float* alpha, const float* proj, long long ld, int off_low, const float* w2t,
-                               const float* bias, int rank, int n_tokens, int n, float tau, cudaStream_t stream) {
+                               const float* bias, const float* rate, int rank, int n_tokens, int n, float tau, int kind,
+                               cudaStream_t stream) {
   if (n_tokens == 0) return 0;
+  AF_REQUIRE(kind >= AF_CD_SIGMOID && kind <= AF_CD_LOGIT && (kind != AF_CD_SOFTPLUS || rate != nullptr),
+             "af_channel_decay: kind %d, a rate per channel with softplus", kind);
   AF_REQUIRE(n_tokens > 0 && n > 0 && rank > 0 && rank <= 512 && tau > 0.f, "af_channel_decay: bad sizes (rank up to 512)");
   if (n_tokens <= AF_CD_TOK) {
     const size_t smem = ((size_t)rank * AF_CD_TOK + AF_CD_SLICES * AF_CD_TOK * 32) * sizeof(float);
     af_launch(channel_decay_few_kernel, dim3((n + 31) / 32), dim3(32 * AF_CD_SLICES), smem, stream, alpha, proj, ld, off_low,
-              w2t, bias, rank, n, n_tokens, 1.f / tau);
+              w2t, bias, rate, rank, n, n_tokens, 1.f / tau, kind);
     AF_CHECK_LAUNCH("af_channel_decay");
   }
   const dim3 grid((n + 127) / 128, (n_tokens + AF_CD_TOK - 1) / AF_CD_TOK);
   AF_REQUIRE(grid.y < 65536, "af_channel_decay: too many tokens for one grid");
   af_launch(channel_decay_kernel, grid, dim3(128), (size_t)rank * AF_CD_TOK * sizeof(float), stream, alpha, proj, ld,
-            off_low, w2t, bias, rank, n, n_tokens, 1.f / tau);
+            off_low, w2t, bias, rate, rank, n, n_tokens, 1.f / tau, kind);
   AF_CHECK_LAUNCH("af_channel_decay");
 }
 

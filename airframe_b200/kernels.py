@@ -166,6 +166,19 @@ def gated_act(out, gu, activation: str) -> None:
                                c_int(ACTIVATIONS[activation]), _stream()))
 
 
+def token_gate(out, z, table, off: int, ids, activation: str) -> None:
+    """out[t, c] = act(z[t, c]) * table[ids[t], off + c]: z float32 [T, dim], or partial sums [n, T, dim] added in index
+    order; out and ``table`` [vocab, >= off + dim] of the compute dtype."""
+    T, dim = out.shape
+    if tuple(z.shape[-2:]) != (T, dim) or not z.is_contiguous() or not out.is_contiguous() or table.dtype != out.dtype \
+            or off + dim > table.shape[1] or activation not in ACTIVATIONS:
+        raise KernelError("token_gate: contiguous float32 rows, a table of the rows' dtype that holds the columns, a known activation")
+    _check(_lib().af_token_gate(_ptr(out), c_int(dtype_code(out.dtype)), _ptr(z, "z", torch.float32),
+                                c_int(z.shape[0] if z.dim() == 3 else 1), _ptr(table), c_longlong(_rows(table, "table")),
+                                c_int(off), _ptr(ids, "ids", torch.int32), c_int(table.shape[0]), c_int(T), c_int(dim),
+                                c_int(ACTIVATIONS[activation]), _stream()))
+
+
 def softcap_(z, cap: float) -> None:
     if not z.is_contiguous():
         raise KernelError("softcap_: tensor must be contiguous")
@@ -189,18 +202,24 @@ def gemm_plain(out, x, w, cap: float = 0.0) -> None:
 
 # ---------------------------------------------------------------- attention
 
+def kv_keep(kv) -> int:
+    """The first tokens of a sequence whose pages lie before the ring of a layer's view of its cache."""
+    return int(getattr(kv, "keep_first", 0))
+
+
 ROPE_TABLE_ROWS = 64     # from this many rows on, the rotary kernel for bfloat16 rows takes the step's table
 
 
 def rope_cache_write(qkv, positions, inv_freq, nq: int, nkv: int, hd: int, rot_dim: int, pairing: str,
                      seq_of_token=None, slots=None, len_after=None, kcache=None, vcache=None,
-                     page_table=None, ring_rows: int = 0, parts=None, table=None) -> None:
+                     page_table=None, ring_rows: int = 0, parts=None, table=None, keep: int = 0) -> None:
     """Rotate the q and k heads of the packed rows [q | k | v] in place and,
     when a cache is given, store k and v at each token's row of its page.
     ``parts`` (float32 [S, T, width] split-K partial sums) are added into qkv first.
     ``table``: the step's cosines and sines (:func:`rope_table` of these positions and
     frequencies); the kernel for many bfloat16 rows reads them instead of working them
-    out for every layer again (the same 32-bit values)."""
+    out for every layer again (the same 32-bit values).  ``keep``: the sequence's first tokens whose pages lie before
+    the ring (:class:`~airframe_b200.cache.KVView`)."""
     T = qkv.shape[0]
     if qkv.shape[1] != (nq + 2 * nkv) * hd:
         raise KernelError(f"rope_cache_write: row width {qkv.shape[1]} is not (nq + 2 nkv) * head_dim")
@@ -228,7 +247,7 @@ def rope_cache_write(qkv, positions, inv_freq, nq: int, nkv: int, hd: int, rot_d
         c_int(T), c_int(nq), c_int(nkv), c_int(hd), c_int(rot_dim),
         c_int(PAIRINGS[pairing]), _ptr(kcache, allow_none=True), _ptr(vcache, allow_none=True),
         _ptr(page_table, "page_table", torch.int32, allow_none=True), c_int(max_pages), c_int(ring_rows),
-        _stream()))
+        c_int(keep), _stream()))
 
 
 _EMPTY_F32 = {}
@@ -253,7 +272,8 @@ def store_kv(qkv, batch, nq: int, nkv: int, hd: int, kv, parts=None) -> None:
     ``qkv`` first.  Nothing is rotated."""
     rope_cache_write(qkv, batch.positions, _no_frequencies(qkv.device), nq, nkv, hd, 0, "half",
                      seq_of_token=batch.seq_of_token, slots=batch.slots, len_after=batch.len_after,
-                     kcache=kv.k, vcache=kv.v, page_table=kv.page_table, ring_rows=kv.ring_rows, parts=parts)
+                     kcache=kv.k, vcache=kv.v, page_table=kv.page_table, ring_rows=kv.ring_rows, parts=parts,
+                     keep=kv_keep(kv))
 
 
 def sum_parts(qkv, parts, batch, nq: int, nkv: int, hd: int) -> None:
@@ -272,11 +292,12 @@ def _gate_args(gate, rows: int, nq: int, who: str):
 
 
 def attn_prefill_plain(out, q, k, v, positions, nq: int, nkv: int, hd: int, scale: float, cap: float,
-                       window: int, slopes=None, dv=None, mask: str = "window", sinks=None, gate=None) -> None:
+                       window: int, slopes=None, dv=None, mask: str = "window", sinks=None, gate=None,
+                       keep: int = 0) -> None:
     """Attention of prompts that start at position 0 over the step's own keys.
     q [T, nq*hd], k [T, nkv*hd], v [T, nkv*dv] are row views (any row stride; ``dv`` = hd by default).
     ``window`` > 0 with ``mask`` "window": a position sees the last ``window`` ones; "chunk": those of its
-    own chunk of ``window`` positions.  ``slopes`` (float32 [nq]): slope[h] * (key position - query position)
+    own chunk of ``window`` positions; with either the sequence's first ``keep`` positions stay visible.  ``slopes`` (float32 [nq]): slope[h] * (key position - query position)
     is added to head h's scores after scale and cap (a position encoding that biases scores).  ``sinks``
     (float32 [nq]): exp(sink[h]) joins head h's softmax denominator without a key or a value.  ``gate``
     (float32 [T, nq] logits): head h's output is multiplied by their sigmoid."""
@@ -292,7 +313,7 @@ def attn_prefill_plain(out, q, k, v, positions, nq: int, nkv: int, hd: int, scal
         _ptr(out), c_int(_rows(out, "out")), _ptr(q), c_int(_rows(q, "q")), _ptr(k), c_int(_rows(k, "k")),
         _ptr(v), c_int(_rows(v, "v")), c_int(dtype_code(q.dtype)), _ptr(positions, "positions", torch.int32),
         c_int(T), c_int(nq), c_int(nkv), c_int(hd), c_int(dv or hd), c_float(scale), c_float(cap), c_int(window),
-        c_int(MASKS[mask]), _ptr(slopes, "slopes", torch.float32, allow_none=True),
+        c_int(MASKS[mask]), c_int(keep), _ptr(slopes, "slopes", torch.float32, allow_none=True),
         _ptr(sinks, "sinks", torch.float32, allow_none=True), gp, gs, _stream()))
 
 
@@ -305,7 +326,7 @@ def plain_decode_splits(batch: int, nq: int, most_keys: int) -> int:
 
 def attn_decode_plain(out, q, kcache, vcache, page_table, slots, lens, nq: int, nkv: int, hd: int,
                       scale: float, cap: float, window: int, ring_rows: int, slopes=None, dv=None,
-                      mask: str = "window", sinks=None, gate=None, n_splits: int = 1) -> None:
+                      mask: str = "window", sinks=None, gate=None, n_splits: int = 1, keep: int = 0) -> None:
     """Attention of one new token per sequence over the cache pages (options as in
     :func:`attn_prefill_plain`).  ``vcache`` None: a value is the first ``dv`` elements of its key row.
     ``n_splits`` > 1: a sequence's visible keys are cut into that many runs, a warp each, joined by a
@@ -330,7 +351,7 @@ def attn_decode_plain(out, q, kcache, vcache, page_table, slots, lens, nq: int, 
         c_int(dtype_code(q.dtype)), _ptr(page_table, "page_table", torch.int32), c_int(page_table.shape[1]),
         _ptr(slots, "slots", torch.int32), _ptr(lens, "lens", torch.int32), c_int(B), c_int(nq), c_int(nkv),
         c_int(hd), c_int(dv), c_float(scale), c_float(cap), c_int(window), c_int(MASKS[mask]), c_int(ring_rows),
-        _ptr(slopes, "slopes", torch.float32, allow_none=True), _ptr(sinks, "sinks", torch.float32, allow_none=True),
+        c_int(keep), _ptr(slopes, "slopes", torch.float32, allow_none=True), _ptr(sinks, "sinks", torch.float32, allow_none=True),
         gp, gs, c_int(n_splits), _ptr(scratch, "scratch", torch.float32, allow_none=True), _stream()))
 
 
@@ -510,7 +531,7 @@ def kv_rows(batch, kv, nkv: int) -> torch.Tensor:
                              _ptr(batch.seq_of_token, "seq_of_token", torch.int32),
                              _ptr(batch.slots, "slots", torch.int32), _ptr(batch.len_after, "len_after", torch.int32),
                              _ptr(kv.page_table, "page_table", torch.int32), c_int(kv.page_table.shape[1]),
-                             c_int(kv.ring_rows), c_int(nkv), c_int(T), _stream()))
+                             c_int(kv.ring_rows), c_int(kv_keep(kv)), c_int(nkv), c_int(T), _stream()))
     return rows
 
 
@@ -614,9 +635,9 @@ def interleave_gate_up(w_gate, w_up):
     return out
 
 def attn_prefill_mma(out, q, k, v, seq_starts, n_seqs: int, max_len: int, nq, nkv, hd, scale, cap, window,
-                     sinks=None, gate=None) -> None:
+                     sinks=None, gate=None, keep: int = 0) -> None:
     """bfloat16 prefill attention on the tensor cores; sequences packed row
-    after row, ``seq_starts`` int32 [n_seqs + 1].  ``sinks`` and ``gate`` as in :func:`attn_prefill_plain`."""
+    after row, ``seq_starts`` int32 [n_seqs + 1].  ``sinks``, ``gate`` and ``keep`` as in :func:`attn_prefill_plain`."""
     gp, gs = _gate_args(gate, q.shape[0], nq, "attn_prefill_mma")
     if q.dtype != torch.bfloat16 or k.dtype != torch.bfloat16 or v.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
         raise KernelError("attn_prefill_mma: bfloat16 only")
@@ -624,13 +645,13 @@ def attn_prefill_mma(out, q, k, v, seq_starts, n_seqs: int, max_len: int, nq, nk
         _ptr(out), c_longlong(_rows(out, "out")), _ptr(q), c_longlong(_rows(q, "q")), _ptr(k),
         c_longlong(_rows(k, "k")), _ptr(v), c_longlong(_rows(v, "v")), _ptr(seq_starts, "seq_starts", torch.int32),
         c_int(n_seqs), c_int(max_len), c_int(nq), c_int(nkv), c_int(hd), c_float(scale), c_float(cap), c_int(window),
-        _ptr(sinks, "sinks", torch.float32, allow_none=True), gp, gs, _stream()))
+        c_int(keep), _ptr(sinks, "sinks", torch.float32, allow_none=True), gp, gs, _stream()))
 
 
 def attn_prefill_tc(out, q, k, v, seq_starts, n_seqs: int, max_len: int, nq, nkv, hd, scale, cap, window,
-                    sinks=None, gate=None) -> None:
+                    sinks=None, gate=None, keep: int = 0) -> None:
     """bfloat16 prefill attention on tcgen05 (S and O in TMEM); sequences packed
-    row after row, ``seq_starts`` int32 [n_seqs + 1].  ``sinks`` and ``gate`` as in :func:`attn_prefill_plain`."""
+    row after row, ``seq_starts`` int32 [n_seqs + 1].  ``sinks``, ``gate`` and ``keep`` as in :func:`attn_prefill_plain`."""
     gp, gs = _gate_args(gate, q.shape[0], nq, "attn_prefill_tc")
     if q.dtype != torch.bfloat16 or k.dtype != torch.bfloat16 or v.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
         raise KernelError("attn_prefill_tc: bfloat16 only")
@@ -640,17 +661,17 @@ def attn_prefill_tc(out, q, k, v, seq_starts, n_seqs: int, max_len: int, nq, nkv
         _ptr(out), c_longlong(_rows(out, "out")), _ptr(q), c_longlong(_rows(q, "q")), _ptr(k),
         c_longlong(_rows(k, "k")), _ptr(v), c_longlong(_rows(v, "v")), _ptr(seq_starts, "seq_starts", torch.int32),
         c_int(n_seqs), c_int(q.shape[0]), c_int(max_len), c_int(nq), c_int(nkv), c_int(hd), c_float(scale),
-        c_float(cap), c_int(window), _ptr(sinks, "sinks", torch.float32, allow_none=True), gp, gs,
+        c_float(cap), c_int(window), c_int(keep), _ptr(sinks, "sinks", torch.float32, allow_none=True), gp, gs,
         _ptr(error_word(q.device), "err", torch.int32), _stream()))
 
 
-def head_gate(x, gate, nq: int, dv: int) -> None:
-    """x[t, h, :] *= sigmoid(gate[t, h]) for rows x [T, nq dv] (an output gate behind an attention kernel that
-    has none of its own)."""
+def head_gate(x, gate, nq: int, dv: int, per_value: bool = False, pitch: int = 0) -> None:
+    """x[t, h, :dv] *= sigmoid(gate[t, h]) for rows x [T, nq pitch] (``pitch`` = dv by default; an output gate behind an
+    attention kernel that has none of its own).  ``per_value``: a factor an element, gate [T, nq dv]."""
     T = x.shape[0]
-    gp, gs = _gate_args(gate, T, nq, "head_gate")
+    gp, gs = _gate_args(gate, T, nq * dv if per_value else nq, "head_gate")
     _check(_lib().af_head_gate(_ptr(x), c_longlong(_rows(x, "x")), c_int(dtype_code(x.dtype)), gp, gs, c_int(T),
-                               c_int(nq), c_int(dv), _stream()))
+                               c_int(nq), c_int(dv), c_int(pitch or dv), c_int(1 if per_value else 0), _stream()))
 
 
 def _chunk_starts(batch, size: int):
@@ -670,19 +691,21 @@ def _chunk_starts(batch, size: int):
 
 
 def attn_prefill(out, q, k, v, batch, nq, nkv, hd, scale, cap, window, slopes=None, dv=None, mask: str = "window",
-                 sinks=None, gate=None) -> None:
+                 sinks=None, gate=None, keep: int = 0) -> None:
     """Attention of a prefill step: for bfloat16 the tcgen05 kernel (head sizes
     128, 256) or the mma.sync kernel (64), else the plain kernel (which also
     serves scores with a per-head slope and values of another size than the keys).  A chunked mask
-    reaches the fast kernels as what it is: causal attention within chunks that know nothing of one another."""
-    fast = q.dtype == torch.bfloat16 and slopes is None and (dv or hd) == hd
+    reaches the fast kernels as what it is: causal attention within chunks that know nothing of one another (with
+    first tokens that stay visible it goes to the plain kernel)."""
+    keep = keep if window else 0         # (without a window everything stays visible)
+    fast = q.dtype == torch.bfloat16 and slopes is None and (dv or hd) == hd and not (keep and mask == "chunk")
     aligned = all(t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0 for t in (q, k, v, out))
     use_tc = fast and aligned and bool(_lib().af_attn_prefill_tc_supported(c_int(hd)))
     use_mma = fast and not use_tc and bool(_lib().af_attn_prefill_supported(c_int(hd))) \
         and all(t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0 for t in (q, k, v))
     if not (use_tc or use_mma):
         attn_prefill_plain(out, q, k, v, batch.positions, nq, nkv, hd, scale, cap, window, slopes, dv=dv, mask=mask,
-                           sinks=sinks, gate=gate)
+                           sinks=sinks, gate=gate, keep=keep)
         return
     starts, n_seqs, max_len, size = batch.seq_starts, batch.n_seqs, batch.max_len, window
     if mask == "chunk" and window:
@@ -690,14 +713,15 @@ def attn_prefill(out, q, k, v, batch, nq, nkv, hd, scale, cap, window, slopes=No
         window = 0
     if n_seqs > 65535:          # (more sequences than a grid's second axis takes)
         attn_prefill_plain(out, q, k, v, batch.positions, nq, nkv, hd, scale, cap, size, slopes, dv=dv, mask=mask,
-                           sinks=sinks, gate=gate)
+                           sinks=sinks, gate=gate, keep=keep)
     elif use_tc:
-        attn_prefill_tc(out, q, k, v, starts, n_seqs, max_len, nq, nkv, hd, scale, cap, window, sinks, gate)
+        attn_prefill_tc(out, q, k, v, starts, n_seqs, max_len, nq, nkv, hd, scale, cap, window, sinks, gate, keep)
     else:
-        attn_prefill_mma(out, q, k, v, starts, n_seqs, max_len, nq, nkv, hd, scale, cap, window, sinks, gate)
+        attn_prefill_mma(out, q, k, v, starts, n_seqs, max_len, nq, nkv, hd, scale, cap, window, sinks, gate, keep)
 
 
-def attn_decode_max_splits(batch: int, nkv: int, max_len: int, window: int, blocks: int = 0, nq: int = 0) -> int:
+def attn_decode_max_splits(batch: int, nkv: int, max_len: int, window: int, blocks: int = 0, nq: int = 0,
+                           keep: int = 0) -> int:
     """The most splits the decode kernel may give one (sequence, kv head) unit:
     the room its partial results need.  The kernel's blocks (one an SM) each
     take an equal share of all units' cache pages, so a unit lies in at most
@@ -706,12 +730,13 @@ def attn_decode_max_splits(batch: int, nkv: int, max_len: int, window: int, bloc
     blocks = blocks or sm_count()
     window = abs(window)            # (negative: a chunk of that many positions)
     rows = min(max_len, window) if window else max_len
-    pages = max(1, (rows + PAGE - 1) // PAGE + (1 if window else 0))
+    pages = max(1, (rows + PAGE - 1) // PAGE + (1 if window else 0) + (keep + PAGE - 1) // PAGE)
     tiles = ((nq // nkv) + 15) // 16 if nq else 1
     return max(1, min(blocks // max(1, nkv * tiles) + 2, pages + 1))
 
 
-def attn_decode_plan(page_table, slots, lens, nq: int, nkv: int, window: int, ring_rows: int, n_splits: int):
+def attn_decode_plan(page_table, slots, lens, nq: int, nkv: int, window: int, ring_rows: int, n_splits: int,
+                     keep: int = 0):
     """The plan of a decode step for :func:`attn_decode_split`: how the work is
     cut among the blocks, worked out by one small kernel for all layers that
     read the same caches the same way (these slots, lengths, page table, heads,
@@ -723,20 +748,20 @@ def attn_decode_plan(page_table, slots, lens, nq: int, nkv: int, window: int, ri
     if n <= 0:
         raise KernelError(f"attn_decode_plan: {B} sequences, {nq} heads in {nkv} groups")
     plan = torch.empty(n, dtype=torch.int32, device=slots.device)
-    _check(lib.af_attn_decode_plan(
+    _check(lib.af_attn_decode_plan_kept(
         _ptr(plan, "plan", torch.int32), c_longlong(n), _ptr(page_table, "page_table", torch.int32),
         c_int(page_table.shape[1]), _ptr(slots, "slots", torch.int32), _ptr(lens, "lens", torch.int32), c_int(B),
-        c_int(nq), c_int(nkv), c_int(window), c_int(ring_rows), c_int(n_splits), _stream()))
+        c_int(nq), c_int(nkv), c_int(window), c_int(keep), c_int(ring_rows), c_int(n_splits), _stream()))
     return plan
 
 
 def attn_decode_split(out, q, kcache, vcache, page_table, slots, lens, nq, nkv, hd, scale, cap, window, ring_rows,
-                      n_splits: int, scratch=None, plan=None, sinks=None) -> None:
+                      n_splits: int, scratch=None, plan=None, sinks=None, keep: int = 0) -> None:
     """bfloat16 decode attention, split over the keys (two kernels: partial
     results into ``scratch``, then their merge).  ``n_splits`` is the most
     splits a (sequence, kv head) unit gets: the kernel cuts the units' pages so
     that all blocks get about the same number of them (with less room than
-    :func:`attn_decode_max_splits` fewer blocks work)."""
+    :func:`attn_decode_max_splits` fewer blocks work).  ``keep``: with a window, the first tokens that stay visible."""
     B = q.shape[0]
     lib = _lib()
     lib.af_attn_decode_scratch.restype = ctypes.c_longlong
@@ -749,12 +774,12 @@ def attn_decode_split(out, q, kcache, vcache, page_table, slots, lens, nq, nkv, 
         raise KernelError("attn_decode_split: bfloat16 only")
     if sinks is not None and sinks.numel() != nq:
         raise KernelError(f"attn_decode_split: {sinks.numel()} sinks for {nq} heads")
-    _check(lib.af_attn_decode_sinks(
+    _check(lib.af_attn_decode_kept(
         _ptr(out), c_longlong(_rows(out, "out")), _ptr(q), c_longlong(_rows(q, "q")), _ptr(kcache), _ptr(vcache),
         c_longlong(kcache.shape[0]), _ptr(page_table, "page_table", torch.int32), c_int(page_table.shape[1]),
         _ptr(slots, "slots", torch.int32),
         _ptr(lens, "lens", torch.int32), c_int(B), c_int(nq), c_int(nkv), c_int(hd), c_float(scale), c_float(cap),
-        c_int(window), c_int(ring_rows), c_int(n_splits), _ptr(scratch, "scratch", torch.float32),
+        c_int(window), c_int(keep), c_int(ring_rows), c_int(n_splits), _ptr(scratch, "scratch", torch.float32),
         _ptr(plan, "plan", torch.int32) if plan is not None else ctypes.c_void_p(0),
         _ptr(sinks, "sinks", torch.float32, allow_none=True),
         _ptr(error_word(q.device), "err", torch.int32), _stream()))
@@ -808,29 +833,30 @@ def attn_decode(out, q, kv, batch, nq, nkv, hd, scale, cap, window, slopes=None,
     # values that lie inside their key rows: the split kernel takes the key pages for the value pages too and gives
     # whole key-sized rows back, of which the caller (who asked for it with an `out` that wide) reads the values' part
     wide = kv.v is None and out.shape[1] == nq * hd
+    keep = kv_keep(kv)
     special = slopes is not None or (not wide and ((dv or hd) != hd or kv.v is None))
     if (not special and q.dtype == torch.bfloat16 and _lib().af_attn_decode_supported(c_int(hd))
             and batch.n_seqs <= ATTN_DECODE_MAX_SEQS):
         if mask == "chunk":
             window = -window
-        n = attn_decode_max_splits(batch.n_seqs, nkv, batch.max_len_after, window, nq=nq)
+        n = attn_decode_max_splits(batch.n_seqs, nkv, batch.max_len_after, window, nq=nq, keep=keep)
         # the plan of the step, shared by the layers that read this group of caches alike (a batch without a
         # place for the step's tables gets none: every block then works the cut out itself)
         plan, aux = None, getattr(batch, "aux", None)
         if aux is not None:
-            key = ("attn_decode_plan", kv.page_table.data_ptr(), kv.ring_rows, nq, nkv, window, n)
+            key = ("attn_decode_plan", kv.page_table.data_ptr(), kv.ring_rows, nq, nkv, window, keep, n)
             if key not in aux:
                 aux[key] = attn_decode_plan(kv.page_table, batch.slots, batch.len_after, nq, nkv, window,
-                                            kv.ring_rows, n)
+                                            kv.ring_rows, n, keep)
             plan = aux[key]
         attn_decode_split(out, q, kv.k, kv.k if wide else kv.v, kv.page_table, batch.slots, batch.len_after, nq, nkv,
-                          hd, scale, cap, window, kv.ring_rows, n, plan=plan, sinks=sinks)
+                          hd, scale, cap, window, kv.ring_rows, n, plan=plan, sinks=sinks, keep=keep)
         if gate is not None:
             head_gate(out, gate, nq, hd)
         return
     # (a captured step sizes its cut for the longest context; the keys a token sees are bounded by its window or chunk)
-    most = min(batch.max_len_after, window) if window else batch.max_len_after
-    if (kv.v is None and slopes is None and cap == 0.0 and attn_decode_latent_supported(q.dtype, hd, dv or hd)
+    most = min(batch.max_len_after, window + keep) if window else batch.max_len_after
+    if (kv.v is None and not keep and slopes is None and cap == 0.0 and attn_decode_latent_supported(q.dtype, hd, dv or hd)
             and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and batch.n_seqs < 65536):
         # wide rows with the values inside: the tensor-core kernel, runs of at least 64 keys, some two blocks an SM
         units = batch.n_seqs * nkv * ((nq // nkv + 15) // 16)
@@ -840,12 +866,12 @@ def attn_decode(out, q, kv, batch, nq, nkv, hd, scale, cap, window, slopes=None,
         return
     attn_decode_plain(out, q, kv.k, kv.v, kv.page_table, batch.slots, batch.len_after, nq, nkv, hd,
                       scale, cap, window, kv.ring_rows, slopes, dv=dv, mask=mask, sinks=sinks, gate=gate,
-                      n_splits=plain_decode_splits(batch.n_seqs, nq, most))
+                      n_splits=plain_decode_splits(batch.n_seqs, nq, most), keep=keep)
 
 
 # ---------------------------------------------------------------- mixers with a state of fixed size
 
-SCAN_MODES = {"decay": 0, "delta": 1, "channel": 3}
+SCAN_MODES = {"decay": 0, "delta": 1, "channel": 3, "gated": 4}
 
 
 def _f32_rows(t, name):
@@ -878,13 +904,15 @@ def delta_prep(out, proj, off_k: int, off_a: int, off_w1: int, a_bias, w0, w2t, 
 
 
 def state_scan(mode: str, out, r, k, v, state, batch, heads: int, dk: int, dv: int, w=None, u=None, au=None,
-               decay=None, silu: bool = False) -> None:
+               decay=None, silu: bool = False, beta=None) -> None:
     """The recurrence of a matrix state per head over the step's tokens, sequence by sequence, from
     the state that earlier steps left in ``state`` (float32 [slots, heads, dv, dk]; left updated):
 
     ``decay``: S <- decay[h] S + k v^T, o = S^T r;
     ``delta``: S <- diag(w) S - au (u^T S) + k v^T, o = S^T r (the decay and the removal act on the state before the token);
-    ``channel``: S <- diag(w) S + k v^T, o = S^T r (a decay per key channel and token, no removal).
+    ``channel``: S <- diag(w) S + k v^T, o = S^T r (a decay per key channel and token, no removal);
+    ``gated``: S <- diag(w) S, then S <- S + beta k (v - S^T k)^T, o = S^T r (``beta`` float32 [T, heads]; r and k may have
+    fewer heads than v, [T, G * dk]: head h reads theirs h // (heads / G)).
 
     r, k, w, u, au: float32 rows [T, heads * dk] (column sections allowed), v [T, heads * dv], out float32
     [T, heads * dv].  ``silu``: r, k and v pass through x * sigmoid(x) as they are read.  A step in which
@@ -894,16 +922,19 @@ def state_scan(mode: str, out, r, k, v, state, batch, heads: int, dk: int, dv: i
     T = out.shape[0]
     if state.dtype != torch.float32 or tuple(state.shape[1:]) != (heads, dv, dk) or not state.is_contiguous():
         raise KernelError(f"state_scan: state must be contiguous float32 [slots, {heads}, {dv}, {dk}]")
-    for t, name, n in ((r, "r", dk), (k, "k", dk), (v, "v", dv), (out, "out", dv)):
-        if tuple(t.shape) != (T, heads * n):
-            raise KernelError(f"state_scan: {name} must be [{T}, {heads * n}], got {tuple(t.shape)}")
+    key_heads = r.shape[1] // dk if mode == "gated" else heads
+    if key_heads < 1 or heads % key_heads:
+        raise KernelError(f"state_scan: {heads} heads over {key_heads} key heads")
+    for t, name, n in ((r, "r", key_heads * dk), (k, "k", key_heads * dk), (v, "v", heads * dv), (out, "out", heads * dv)):
+        if tuple(t.shape) != (T, n):
+            raise KernelError(f"state_scan: {name} must be [{T}, {n}], got {tuple(t.shape)}")
     null = (ctypes.c_void_p(0), c_longlong(0))
     if mode == "delta":
         if w is None or u is None or au is None:
             raise KernelError("state_scan: the delta rule needs w, u and au")
         extra = [_f32_rows(t, n) for t, n in ((w, "w"), (u, "u"), (au, "au"))]
         dec = ctypes.c_void_p(0)
-    elif mode == "channel":
+    elif mode in ("channel", "gated"):
         if w is None or tuple(w.shape) != (T, heads * dk):
             raise KernelError(f"state_scan: a decay per key channel and token, [{T}, {heads * dk}]")
         extra = [_f32_rows(w, "w"), null, null]
@@ -913,9 +944,14 @@ def state_scan(mode: str, out, r, k, v, state, batch, heads: int, dk: int, dv: i
             raise KernelError("state_scan: one decay per head")
         extra = [null, null, null]
         dec = _ptr(decay, "decay", torch.float32)
+    bp = null
+    if mode == "gated":
+        if beta is None or tuple(beta.shape) != (T, heads):
+            raise KernelError(f"state_scan: one step size per token and head, [{T}, {heads}]")
+        bp = _f32_rows(beta, "beta")
     rp, kp, vp, op = (_f32_rows(t, n) for t, n in ((r, "r"), (k, "k"), (v, "v"), (out, "out")))
     _check(_lib().af_state_scan(c_int(SCAN_MODES[mode]), *rp, *kp, *vp, *extra[0], *extra[1], *extra[2], dec,
-                                _ptr(state, "state", torch.float32), *op,
+                                *bp, c_int(heads // key_heads), _ptr(state, "state", torch.float32), *op,
                                 _ptr(batch.seq_starts, "seq_starts", torch.int32), _ptr(batch.slots, "slots", torch.int32),
                                 c_int(batch.n_seqs), c_int(T), c_int(heads), c_int(dk), c_int(dv), c_int(1 if silu else 0),
                                 _stream()))
@@ -1008,9 +1044,9 @@ def qk_norm_rope_store(qkv, proj, batch, nq: int, nkv: int, hd: int, inv_freq, r
     if bias is not None and bias.numel() < width_in:
         raise KernelError(f"qk_norm_rope_store: a bias of {width_in} values")
     kc = vc = pt = None
-    max_pages = ring = 0
+    max_pages = ring = keep = 0
     if kv is not None:
-        kc, vc, pt, ring = kv.k, kv.v, kv.page_table, kv.ring_rows
+        kc, vc, pt, ring, keep = kv.k, kv.v, kv.page_table, kv.ring_rows, kv_keep(kv)
         if kc.dtype != qkv.dtype or tuple(kc.shape[1:]) != (nkv, PAGE, pk) or vc is None \
                 or tuple(vc.shape[1:]) != (nkv, PAGE, pv) or not kc.is_contiguous() or not vc.is_contiguous():
             raise KernelError(f"qk_norm_rope_store: cache pages must be [pages, {nkv}, {PAGE}, {pk}] (values {pv}) "
@@ -1028,7 +1064,7 @@ def qk_norm_rope_store(qkv, proj, batch, nq: int, nkv: int, hd: int, inv_freq, r
         _ptr(inv_freq, "inv_freq", torch.float32), _ptr(table, "table", torch.float32, allow_none=True),
         c_int(T), c_int(nq), c_int(nkv), c_int(hd), c_int(dv), c_int(rot_dim),
         c_int(PAIRINGS[pairing]), _ptr(kc, allow_none=True), _ptr(vc, allow_none=True),
-        _ptr(pt, "page_table", torch.int32, allow_none=True), c_int(max_pages), c_int(ring), c_int(pitch),
+        _ptr(pt, "page_table", torch.int32, allow_none=True), c_int(max_pages), c_int(ring), c_int(keep), c_int(pitch),
         c_int(1 if whole_norm else 0), _stream()))
 
 
@@ -1103,10 +1139,11 @@ def latent_prep(batch, heads: int, dim: int, rot: int, rank: int, eps: float, in
         _ptr(pt, "page_table", torch.int32, allow_none=True), c_int(max_pages), c_int(ring), _stream()))
 
 
-def head_project(out, x, w, heads: int, D: int, N: int, extra: int = 0, x_pitch: int = 0) -> None:
+def head_project(out, x, w, heads: int, D: int, N: int, extra: int = 0, x_pitch: int = 0, gate=None) -> None:
     """out[t, h, :N] = x[t, h, :D] @ w[h] for w [heads, D, N] (32-bit sums), and the ``extra`` elements behind a
     head's D inputs copied behind its N outputs.  x [T, heads x_pitch] (``x_pitch`` = D + extra by default: what
-    else a head holds is skipped), out [T, heads (N + extra)]: row views of one dtype, which is w's too."""
+    else a head holds is skipped), out [T, heads (N + extra)]: row views of one dtype, which is w's too.
+    ``gate`` (float32 logits [T, heads N]; a column section is fine): the N outputs are multiplied by their sigmoid."""
     T = x.shape[0]
     x_pitch = x_pitch or D + extra
     if tuple(x.shape) != (T, heads * x_pitch) or tuple(out.shape) != (T, heads * (N + extra)) \
@@ -1114,7 +1151,7 @@ def head_project(out, x, w, heads: int, D: int, N: int, extra: int = 0, x_pitch:
         raise KernelError("head_project: shapes or dtypes do not fit")
     _check(_lib().af_head_project(_ptr(out), c_longlong(_rows(out, "out")), _ptr(x), c_longlong(_rows(x, "x")), _ptr(w),
                                   c_int(dtype_code(x.dtype)), c_int(T), c_int(heads), c_int(D), c_int(N), c_int(extra),
-                                  c_int(x_pitch), _stream()))
+                                  c_int(x_pitch), *_gate_args(gate, T, heads * N, "head_project"), _stream()))
 
 
 # ---------------------------------------------------------------- the norm without statistics, and re-entry
@@ -1372,13 +1409,16 @@ def expert_tc_tile(n_pairs: int, n_experts: int) -> int:
 
 
 def expert_route(ids, wts, shared_gate, h, router, n_experts: int, correction=None, groups: int = 1, keep: int = 1,
-                 normalise: bool = False, out_scale: float = 1.0) -> None:
+                 normalise: bool = False, out_scale: float = 1.0, score: str = "sigmoid", group_score: str = "top2") -> None:
     """Per row of h [T, H]: scores = sigmoid(router[:n_experts] h) in 32 bits; ids, wts [T, top] = the experts
     with the largest scores (equal scores: the lower index) and their scores; ``shared_gate`` float32 [T], when
     given, = sigmoid(router[n_experts] h).  ``correction`` (float32 [experts]) is added to the scores for the
     choice only.  ``groups`` > 1: the experts form so many equal groups of neighbours, a group's score is the sum
     of its two largest choice scores, and only experts of the ``keep`` best groups can be chosen.  ``normalise``:
-    the chosen scores are divided by their sum + 1e-20; ``out_scale`` multiplies the weights."""
+    the chosen scores are divided by their sum + 1e-20; ``out_scale`` multiplies the weights.  ``score`` "softmax": the
+    scores are the softmax of the logits over all experts; ``group_score`` "max": a group's score is its largest alone."""
+    if score not in ROUTER_SCORES or group_score not in GROUP_SCORES:
+        raise KernelError(f"expert_route: score '{score}' or group score '{group_score}'")
     T, H = h.shape
     top = ids.shape[1]
     rows = n_experts + (1 if shared_gate is not None else 0)
@@ -1395,20 +1435,26 @@ def expert_route(ids, wts, shared_gate, h, router, n_experts: int, correction=No
                                   c_int(dtype_code(h.dtype)), _ptr(router), c_int(T), c_int(H), c_int(n_experts),
                                   c_int(top), _ptr(correction, "correction", torch.float32, allow_none=True),
                                   c_int(groups), c_int(keep if groups > 1 else 1), c_int(1 if normalise else 0),
-                                  c_float(out_scale), _stream()))
+                                  c_float(out_scale), c_int(ROUTER_SCORES[score]), c_int(GROUP_SCORES[group_score]),
+                                  _stream()))
 
 
-def expert_plan(perm, plan, ids, n_experts: int, tile: int = EXPERT_TILE) -> None:
+ROUTER_SCORES = {"sigmoid": 0, "softmax": 1}
+GROUP_SCORES = {"top2": 0, "max": 1}
+
+
+def expert_plan(perm, plan, ids, n_experts: int, tile: int = EXPERT_TILE, identity: int = 0) -> None:
     """The (token, choice) pairs of ``ids`` [T, top] sorted by expert: perm int32 [T * top] (sorted row -> pair),
     plan int32 [1 + 3 * expert_max_tiles]: tiles in use, then (expert, first sorted row, rows) per tile; a tile
-    holds up to ``tile`` rows, and an expert's tiles are of equal size."""
+    holds up to ``tile`` rows, and an expert's tiles are of equal size.  Ids from n_experts on name ``identity`` experts
+    without matrices: their pairs end the permutation and lie in no tile."""
     n_pairs = ids.numel()
     max_tiles = (plan.numel() - 1) // 3
     if perm.numel() != n_pairs or not (perm.is_contiguous() and plan.is_contiguous() and ids.is_contiguous()):
         raise KernelError("expert_plan: one entry of perm per pair")
     _check(_lib().af_expert_plan(_ptr(perm, "perm", torch.int32), _ptr(plan, "plan", torch.int32),
-                                 _ptr(ids, "ids", torch.int32), c_int(n_pairs), c_int(n_experts), c_int(max_tiles),
-                                 c_int(tile), _stream()))
+                                 _ptr(ids, "ids", torch.int32), c_int(n_pairs), c_int(n_experts), c_int(identity),
+                                 c_int(max_tiles), c_int(tile), _stream()))
 
 
 def expert_table_plan(perm, plan, tokens, tables, n_experts: int, tile: int = EXPERT_TILE) -> None:
@@ -1435,7 +1481,7 @@ def _second_limit(second):
     return c_int(second[0]), c_float(second[1])
 
 
-EXPERT_ACTS = {None: 0, "gelu_erf": 1}
+EXPERT_ACTS = {None: 0, "gelu_erf": 1, "silu_glu": 2}      # gelu_erf: behind one matrix; silu_glu: gate and up
 
 
 def expert_rows(out, a, w0, w1=None, perm=None, plan=None, pair_weight=None, scale_out=None, n_tokens: int = 0,
@@ -1447,13 +1493,14 @@ def expert_rows(out, a, w0, w1=None, perm=None, plan=None, pair_weight=None, sca
     that limit.  Without: out float32 [top, tokens, N] with
     out[choice, token] = a[sorted row] w0[e]^T.  Without ``w1`` but with ``act`` = "gelu_erf": an expert of one
     matrix, out[sorted row] = gelu(x w0[e]^T) * s * post with the exact GELU (the weight stands behind the
-    activation).  w0, w1: [experts, N, K].  Without a plan: one expert, the rows in order."""
+    activation).  With ``w1`` and ``act`` = "silu_glu": silu(x w0[e]^T) * (x w1[e]^T) * s * post, the weight likewise
+    behind the activation.  w0, w1: [experts, N, K].  Without a plan: one expert, the rows in order."""
     n_rows = n_tokens * top
     E, N, K = w0.shape
     if not (a.is_contiguous() and out.is_contiguous() and w0.is_contiguous()) or a.shape[1] != K or a.dtype != w0.dtype:
         raise KernelError("expert_rows: contiguous rows of the matrices' dtype and row size")
-    if act not in EXPERT_ACTS or (act is not None and w1 is not None):
-        raise KernelError(f"expert_rows: activation '{act}' (known: gelu_erf, behind one matrix)")
+    if act not in EXPERT_ACTS or (act is not None and (w1 is not None) != (act == "silu_glu")):
+        raise KernelError(f"expert_rows: activation '{act}' (known: gelu_erf behind one matrix, silu_glu on two)")
     if w1 is not None or act is not None:
         if w1 is not None and (w1.shape != w0.shape or w1.dtype != w0.dtype or not w1.is_contiguous()):
             raise KernelError("expert_rows: gate and up matrices alike")
@@ -1473,14 +1520,23 @@ def expert_rows(out, a, w0, w1=None, perm=None, plan=None, pair_weight=None, sca
                                  *_second_limit(second), c_int(EXPERT_ACTS[act]), _stream()))
 
 
-def expert_gather(out, x, perm, top: int) -> None:
-    """out[sorted row] = x[perm[sorted row] // top]: the tokens' rows in the order of the plan."""
-    n_rows, H = out.shape
-    if not (out.is_contiguous() and x.is_contiguous()) or x.shape[1] != H or out.dtype != x.dtype \
-            or perm.numel() != n_rows or x.shape[0] * top != n_rows:
+def expert_gather(out, x, perm, top: int, ids=None, n_experts: int = 0, wts=None, result=None) -> None:
+    """out[sorted row] = x[perm[sorted row] // top]: the tokens' rows in the order of the plan.  With ``ids`` and ``wts``
+    [T, top]: a pair whose id is ``n_experts`` or more belongs to an identity expert, and its weight times its token's row
+    goes to ``result`` (float32 [top, T, H], the down products' results) at [choice, token].  ``out`` None: those rows alone."""
+    T, H = x.shape
+    n_rows = T * top
+    if not x.is_contiguous() or perm.numel() != n_rows or (out is None and ids is None) \
+            or (out is not None and (tuple(out.shape) != (n_rows, H) or not out.is_contiguous() or out.dtype != x.dtype)):
         raise KernelError("expert_gather: contiguous rows of one size and dtype, one entry of perm a row")
-    _check(_lib().af_expert_gather(_ptr(out), _ptr(x), c_int(dtype_code(x.dtype)), _ptr(perm, "perm", torch.int32),
-                                   c_int(n_rows), c_int(top), c_int(H), _stream()))
+    if ids is not None and (tuple(ids.shape) != (T, top) or tuple(wts.shape) != (T, top) or tuple(result.shape) != (top, T, H)
+                            or not (ids.is_contiguous() and wts.is_contiguous() and result.is_contiguous())):
+        raise KernelError(f"expert_gather: ids and weights [{T}, {top}], results [{top}, {T}, {H}]")
+    i32, f32 = torch.int32, torch.float32
+    _check(_lib().af_expert_gather(_ptr(out, allow_none=True), _ptr(x), c_int(dtype_code(x.dtype)), _ptr(perm, "perm", i32),
+                                   c_int(n_rows), c_int(top), c_int(H), _ptr(ids, "ids", i32, allow_none=True),
+                                   c_int(n_experts), _ptr(wts if ids is not None else None, "wts", f32, allow_none=True),
+                                   _ptr(result if ids is not None else None, "result", f32, allow_none=True), _stream()))
 
 
 def expert_rows_tc_supported(a, w0) -> bool:
@@ -1499,8 +1555,8 @@ def expert_rows_tc(out, a, w0, w1=None, perm=None, plan=None, pair_weight=None, 
     E, N, K = w0.shape
     if not expert_rows_tc_supported(a, w0) or tuple(a.shape) != (n_rows, K) or not out.is_contiguous():
         raise KernelError("expert_rows_tc: contiguous bfloat16 rows [rows, K], K a multiple of 8, 16-byte aligned")
-    if act not in EXPERT_ACTS or (act is not None and w1 is not None):
-        raise KernelError(f"expert_rows_tc: activation '{act}' (known: gelu_erf, behind one matrix)")
+    if act not in EXPERT_ACTS or (act is not None and (w1 is not None) != (act == "silu_glu")):
+        raise KernelError(f"expert_rows_tc: activation '{act}' (known: gelu_erf behind one matrix, silu_glu on two)")
     if w1 is not None or act is not None:
         if w1 is not None and (w1.shape != w0.shape or w1.dtype != w0.dtype or not w1.is_contiguous() or w1.data_ptr() % 16):
             raise KernelError("expert_rows_tc: gate and up matrices alike")
@@ -1596,18 +1652,25 @@ def stream_sum(out, x, S: int) -> None:
 
 # ---------------------------------------------------------------- gated linear attention, differential attention
 
-def channel_decay(alpha, proj, off_low: int, w2t, bias, tau: float) -> None:
-    """alpha [T, n] float32 = sigmoid(bias + low w2t)^(1 / tau), ``low`` the ``rank`` columns of the packed float32
-    projection rows at ``off_low``, w2t float32 [rank, n]."""
+DECAY_KINDS = {"sigmoid": 0, "softplus": 1, "logit": 2}
+
+
+def channel_decay(alpha, proj, off_low: int, w2t, bias, tau: float = 1.0, kind: str = "sigmoid", rate=None) -> None:
+    """alpha [T, n] float32 = f(bias + low w2t), ``low`` the ``rank`` columns of the packed float32 projection rows at
+    ``off_low``, w2t float32 [rank, n] (``bias`` None: 0); f(z) = sigmoid(z)^(1 / tau), or by ``kind`` "softplus":
+    exp(-rate softplus(z)) with ``rate`` float32 [n], or "logit": z."""
     T, n = alpha.shape
     rank = w2t.shape[0]
+    if kind not in DECAY_KINDS or (kind == "softplus" and (rate is None or rate.numel() != n)):
+        raise KernelError("channel_decay: a known kind, and a rate per channel with softplus")
     if alpha.dtype != torch.float32 or not alpha.is_contiguous() or tuple(w2t.shape) != (rank, n) or not w2t.is_contiguous() \
-            or bias.numel() != n or off_low + rank > proj.shape[1] or proj.shape[0] != T:
+            or (bias is not None and bias.numel() != n) or off_low + rank > proj.shape[1] or proj.shape[0] != T:
         raise KernelError("channel_decay: alpha float32 [T, n], w2t [rank, n], bias [n], the low-rank section inside the row")
     pp, ld = _f32_rows(proj, "proj")
     _check(_lib().af_channel_decay(_ptr(alpha), pp, ld, c_int(off_low), _ptr(w2t, "w2t", torch.float32),
-                                   _ptr(bias, "bias", torch.float32), c_int(rank), c_int(T), c_int(n), c_float(tau),
-                                   _stream()))
+                                   _ptr(bias, "bias", torch.float32, allow_none=True),
+                                   _ptr(rate, "rate", torch.float32, allow_none=True), c_int(rank), c_int(T), c_int(n),
+                                   c_float(tau), c_int(DECAY_KINDS[kind]), _stream()))
 
 
 SCAN_CHUNK = 128     # tokens of a chunk when a long prompt's scan is cut into chunks that run side by side
@@ -1822,6 +1885,34 @@ def diff_join(y, ctx, gate, H: int, G: int, dv: int, pv: int, lam: float, eps: f
                                c_float(lam), c_float(eps), c_float(post), c_int(ones), _stream()))
 
 
+def delta_conv(out, proj, offsets, taps_w, history, batch, key_heads: int, heads: int, dk: int, dv: int, key_eps: float,
+               query_scale: float) -> None:
+    """From float32 projection rows with the sections q, k (``key_heads`` heads of dk), v (``heads`` of dv) and b (a logit
+    per head) at ``offsets``: silu of a causal convolution over time on every channel of q, k and v (``taps_w`` float32
+    [taps, C], C = 2 key_heads dk + heads dv, the last tap on the token itself; inputs before the step from ``history``
+    float32 [slots, taps - 1, C], which is left holding each sequence's last inputs), q and k heads over
+    sqrt(sum of squares + key_eps), q times ``query_scale``; and sigmoid(b): out float32 [T, C + heads] = [q | k | v | beta]."""
+    T = proj.shape[0]
+    C = 2 * key_heads * dk + heads * dv
+    taps = taps_w.shape[0]
+    if tuple(out.shape) != (T, C + heads) or tuple(taps_w.shape) != (taps, C) or not taps_w.is_contiguous() or heads % key_heads:
+        raise KernelError(f"delta_conv: out [{T}, {C + heads}], taps [taps, {C}]")
+    if taps > 1 and (history is None or history.dtype != torch.float32 or tuple(history.shape[1:]) != (taps - 1, C)
+                     or not history.is_contiguous()):
+        raise KernelError(f"delta_conv: a history float32 [slots, {taps - 1}, {C}]")
+    ends = [o + n for o, n in zip(offsets, (key_heads * dk, key_heads * dk, heads * dv, heads))]
+    if len(offsets) != 4 or max(ends) > proj.shape[1] or min(offsets) < 0:
+        raise KernelError("delta_conv: a section lies outside the projection row")
+    op, pp = _f32_rows(out, "out"), _f32_rows(proj, "proj")
+    i32 = torch.int32
+    _check(_lib().af_delta_conv(
+        *op, *pp, *(c_int(o) for o in offsets), _ptr(taps_w, "taps_w", torch.float32),
+        _ptr(history if taps > 1 else None, "history", torch.float32, allow_none=True),
+        _ptr(batch.positions, "positions", i32), _ptr(batch.seq_of_token, "seq_of_token", i32), _ptr(batch.slots, "slots", i32),
+        _ptr(batch.seq_starts, "seq_starts", i32), c_int(T), c_int(batch.n_seqs), c_int(taps), c_int(key_heads), c_int(heads),
+        c_int(dk), c_int(dv), c_float(key_eps), c_float(query_scale), _stream()))
+
+
 __all__ = [n for n in dir() if not n.startswith("_")]
 
 
@@ -1857,8 +1948,25 @@ def norm_of_sum(x, terms, alpha: float, w, bias, eps: float, gate=None, gate_bia
     if shifted is not None and (shift is None or shift.numel() != H or prev is None or prev.dtype != torch.float32
                                 or prev.shape[1:] != (H,) or not prev.is_contiguous() or slots.shape[0] != n):
         raise KernelError("norm_of_sum: a shifted row needs factors [H], float32 state [slots, H] and one slot a row")
+    _norm_of_sum(x, terms, alpha, w, bias, eps, outs, gate, gate_bias, y, shifted, shift, prev, slots, 0, "norm_of_sum")
+
+
+def add_layer_norm(x, terms, w, bias, eps: float, y=None) -> None:
+    """x += layer_norm(sum of scale * term) in place (float32 [rows, H]; all sums 32-bit): ``terms`` as in
+    :func:`norm_of_sum`.  ``y``: the new row in y's dtype."""
+    n, H = x.shape
+    if not x.is_contiguous() or (y is not None and (tuple(y.shape) != (n, H) or not y.is_contiguous())) \
+            or w.numel() != H or bias.numel() != H:
+        raise KernelError("add_layer_norm: contiguous rows of one size, weight and bias of that size")
+    _norm_of_sum(x, terms, 1.0, w, bias, eps, [y] if y is not None else [], None, None, y, None, None, None, None, 1,
+                 "add_layer_norm")
+
+
+def _norm_of_sum(x, terms, alpha, w, bias, eps, outs, gate, gate_bias, y, shifted, shift, prev, slots, post: int,
+                 who: str) -> None:
+    n, H = x.shape
     if not terms:
-        raise KernelError("norm_of_sum: at least one term")
+        raise KernelError(f"{who}: at least one term")
     if len(terms) > 2:
         total = torch.zeros(n, H, dtype=torch.float32, device=x.device)
         add_scaled_rmsnorm(total, terms)
@@ -1866,16 +1974,16 @@ def norm_of_sum(x, terms, alpha: float, w, bias, eps: float, gate=None, gate_bia
     none = (c_void_p(0), c_int(F32), c_int(1))
     a, sa = terms[0]
     b, sb = terms[1] if len(terms) > 1 else (None, 0.0)
-    barg = _term_arg(b, n, H, "norm_of_sum") if b is not None else none
-    zarg = _term_arg(gate, n, H, "norm_of_sum") if gate is not None else none
+    barg = _term_arg(b, n, H, who) if b is not None else none
+    zarg = _term_arg(gate, n, H, who) if gate is not None else none
     f32 = torch.float32
     _check(_lib().af_norm_of_sum(
-        _ptr(x, "x", f32), *_term_arg(a, n, H, "norm_of_sum"), c_float(sa), *barg, c_float(sb), *zarg,
+        _ptr(x, "x", f32), *_term_arg(a, n, H, who), c_float(sa), *barg, c_float(sb), *zarg,
         _ptr(gate_bias if gate is not None else None, "gate_bias", f32, allow_none=True), c_float(alpha), _ptr(w, "w", f32),
         _ptr(bias, "bias", f32), c_float(eps), _ptr(y, "y", allow_none=True), _ptr(shifted, "shifted", allow_none=True),
         c_int(dtype_code(outs[0].dtype) if outs else F32), _ptr(shift, "shift", f32, allow_none=True),
         _ptr(prev, "prev", f32, allow_none=True), _ptr(slots, "slots", torch.int32, allow_none=True), c_int(n), c_int(H),
-        _stream()))
+        c_int(post), _stream()))
 
 
 def token_shift(shifted, x, shift, prev, batch, y=None) -> None:

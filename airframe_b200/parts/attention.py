@@ -22,7 +22,8 @@ position sees the earlier positions of its own chunk of ``window`` positions, ch
 counted from position 0) instead of the sliding one; a learned sink per head in the
 softmax's denominator; an output gate, one number per head and token (the sigmoid of
 a projection of the mixer's input), that multiplies the head's output before the
-output projection; and ``qk_norm`` taken over a token's whole q (and whole k)
+output projection; first tokens of a sequence that stay visible beside a window
+(``keep_first``; their keys are rotated by their true positions as ever); and ``qk_norm`` taken over a token's whole q (and whole k)
 projection, all heads at once, with weights of that size.
 """
 from __future__ import annotations
@@ -46,7 +47,8 @@ class Attention(Mixer):
     projected); optional ``qk_norm``: {``q_weight``, ``k_weight`` (tensor names of head_dim
     values each), ``eps``}; optional ``wide_output`` (default false): the output projection's
     result stays float32 on its way into the residual sum; optional ``value_dim`` (default ``head_dim``);
-    optional ``mask`` ("window", the default, or "chunk") that says what ``window`` means; optional ``q_bias``,
+    optional ``mask`` ("window", the default, or "chunk") that says what ``window`` means; optional ``keep_first`` (with
+    a window: so many first positions stay visible); optional ``q_bias``,
     ``k_bias``, ``v_bias`` (tensor names; all or none); ``qk_norm`` may instead be {``after_rotation``: true,
     ``eps``} (no weights: q and k over their root mean square once they are rotated), or carry ``whole``: true
     (the mean square is taken over all heads of the token's q, and of its k, and the two weights hold
@@ -94,6 +96,9 @@ class Attention(Mixer):
                 raise ConfigError(f"attention: 'qk_norm' needs {missing}")
         self.dv = int(self.params.get("value_dim") or self.hd)
         self.mask = self.params.get("mask") or "window"
+        self.keep = int(self.params.get("keep_first") or 0) if self.window else 0
+        if self.keep < 0:
+            raise ConfigError(f"attention: keep_first {self.keep} is negative")
         if self.mask not in kernels.MASKS:
             raise ConfigError(f"attention: unknown mask '{self.mask}' (known: {sorted(kernels.MASKS)})")
         self.bias_names = [self.params.get(k) for k in ("q_bias", "k_bias", "v_bias")]
@@ -128,8 +133,8 @@ class Attention(Mixer):
     def kv_need(self):
         # (a chunk's keys all lie within the last ``window`` positions: the ring of a window serves it)
         if self.pad:
-            return KVNeed(self.nkv, self.pad, self.window)
-        return KVNeed(self.nkv, self.hd, self.window, None if self.dv == self.hd else self.dv)
+            return KVNeed(self.nkv, self.pad, self.window, keep_first=self.keep)
+        return KVNeed(self.nkv, self.hd, self.window, None if self.dv == self.hd else self.dv, self.keep)
 
     def weight_decls(self):
         q, k, v, o = self.names
@@ -196,7 +201,8 @@ class Attention(Mixer):
         """Keys that the token at ``pos`` sees."""
         if not self.window:
             return pos + 1
-        return pos % self.window + 1 if self.mask == "chunk" else min(pos + 1, self.window)
+        near = pos % self.window + 1 if self.mask == "chunk" else min(pos + 1, self.window)
+        return near + min(self.keep, pos + 1 - near)
 
     def score_flops(self, lens) -> int:
         """The part of :meth:`prefill_flops` that is scores and their products with v."""
@@ -208,6 +214,9 @@ class Attention(Mixer):
                 pairs += full * (w * (w + 1) // 2) + rest * (rest + 1) // 2
             else:
                 pairs += n * (n + 1) // 2 if not w or n <= w else w * (w + 1) // 2 + (n - w) * w
+            if w and self.keep:
+                pairs += sum(self._visible(i) for i in range(n)) - sum(min(i + 1, w) if self.mask == "window" else i % w + 1
+                                                                       for i in range(n))
         return 2 * pairs * self.nq * (self.hd + self.dv)
 
     def prefill_flops(self, lens) -> int:
@@ -296,7 +305,8 @@ class Attention(Mixer):
                 k, v = batch.step_kv[view.cache_id]
             elif view.keep_step_kv:
                 batch.step_kv[view.cache_id] = (k.clone(), v.clone())
-            kernels.attn_prefill(ctx, q, k, v, batch, nq, nkv, hd, self.scale, self.softcap, window, slopes, **more)
+            kernels.attn_prefill(ctx, q, k, v, batch, nq, nkv, hd, self.scale, self.softcap, window, slopes,
+                                 keep=self.keep, **more)
         else:
             kernels.attn_decode(ctx, q, kv, batch, nq, nkv, hd, self.scale, self.softcap, window, slopes, **more)
         return linear_split(ctx, self.w_o, wide=bool(self.params.get("wide_output", False)))

@@ -69,11 +69,13 @@ class KVNeed:
     """Keys and values per token.  ``window`` None: all of them are kept;
     otherwise the last ``window`` rows (a ring).  ``value_dim``: the size of a
     value row (None: ``head_dim``, as the keys; 0: no value pages, the mixer finds
-    its values inside the key rows)."""
+    its values inside the key rows).  ``keep_first``: beside the window's rows those of
+    the sequence's first tokens are kept (their pages never belong to the ring)."""
     num_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     value_dim: Optional[int] = None
+    keep_first: int = 0
 
     @property
     def value_size(self) -> int:
@@ -207,7 +209,8 @@ class Mixer(Part):
     def kv_need(self) -> Optional[KVNeed]:
         return None
 
-    def state_need(self) -> Optional[StateNeed]:
+    def state_need(self):
+        """None, a :class:`StateNeed`, or a tuple of them (the run's view then has a tuple of tensors)."""
         return None
 
     def forward(self, x, batch, view):

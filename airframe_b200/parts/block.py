@@ -13,7 +13,8 @@ first).
 stream itself and the only norms stand behind them (each on the sublayer's output,
 not on the sum); a layer whose feed-forward is of the kind ``none`` has the first
 half only.  On the 16-bit path the kernel of a residual sum also writes the new
-stream in 16 bits for the sublayer that reads it next.
+stream in 16 bits for the sublayer that reads it next.  A third sublayer of the
+feed-forward kind (``side``) may follow, with its own norm behind it.
 ``normed_sum``: x <- norm1(alpha x + mixer(x)); x <- norm2(alpha x + ff(x)): the norm is
 taken of the residual sum, so the stream itself is a norm's output; the sublayers read it as it stands.
 Each sublayer's result may be multiplied element by element by sigmoid(W x + b) first, and what the
@@ -91,25 +92,33 @@ class PreNormBlock(Block):
 
 @register_part("block", "postnorm")
 class PostNormBlock(Block):
+    """Optional parameter ``side``: a PartSpec of category ``feed_forward``, run last (norm role ``post_side``)."""
     roles = ("post_mixer", "post_feed_forward")
 
     def __init__(self, params, ctx, mixer, feed_forward, norms):
-        if not feed_forward.present:
-            self.roles = ("post_mixer",)
+        side = params.get("side")
+        self.roles = ("post_mixer", *(("post_feed_forward",) if feed_forward.present else ()),
+                      *(("post_side",) if side is not None else ()))
         super().__init__(params, ctx, mixer, feed_forward, norms)
+        self.side = build_part("feed_forward", side, ctx) if side is not None else None
         # "the norm in front of a sublayer" is none: the stream as it stands, in the compute dtype
         self.reader = build_part("norm", PartSpec("as_is", {"size": norms["post_mixer"].size}), ctx)
 
+    def children(self):
+        return [*super().children(), *([self.side] if self.side is not None else [])]
+
     def forward(self, x, batch, view, normed=None, next_pre=None):
-        n = self.norms
         dt = self.ctx.compute_dtype
         h = normed if normed is not None else self.reader.forward(x, dt)
-        a = self.mixer.forward(h, batch, view)
-        if not self.feed_forward.present:
-            return n["post_mixer"].add_normed(x, a, then=next_pre, out_dtype=dt)
-        h = n["post_mixer"].add_normed(x, a, then=self.reader, out_dtype=dt)
-        f = self.feed_forward.forward(h, batch)
-        return n["post_feed_forward"].add_normed(x, f, then=next_pre, out_dtype=dt)
+        run = [("post_mixer", lambda h: self.mixer.forward(h, batch, view))]
+        if self.feed_forward.present:
+            run.append(("post_feed_forward", lambda h: self.feed_forward.forward(h, batch)))
+        if self.side is not None:
+            run.append(("post_side", lambda h: self.side.forward(h, batch)))
+        for i, (role, sublayer) in enumerate(run):
+            then = self.reader if i + 1 < len(run) else next_pre
+            h = self.norms[role].add_normed(x, sublayer(h), then=then, out_dtype=dt)
+        return h
 
     def first_norm(self):
         return self.reader

@@ -9,7 +9,7 @@ elements; the queries may be made from a latent of their own (``q_rank``:
 q = W_uq (W_dq h / rms * w_q)).  score = (q_plain . k_plain + q_rot . r) * scale
 over all earlier keys or a sliding window, softmax (with a learned sink per head in
 the denominator when the model has one), each head's output times a gate
-sigmoid(W_g h) when the model has one, output projection over the concatenated heads.
+sigmoid(W_g h) when the model has one (a factor per head, or one per element of the heads' values), output projection over the concatenated heads.
 
 The products with W_uk and W_uv are moved to the query's side, where they
 cost one small product per new token instead of one per cached token:
@@ -47,7 +47,8 @@ class LatentAttention(Mixer):
     ``dq_norm_weight`` [q_rank] and ``uq_weight`` [heads (head_dim + rot_dim), q_rank]; ``dkv_weight``
     [kv_rank + rot_dim, hidden], ``dkv_norm_weight`` [kv_rank], ``uk_weight`` [heads head_dim, kv_rank],
     ``uv_weight`` [heads value_dim, kv_rank], ``o_weight`` [hidden, heads value_dim]; optional ``sink_weight``
-    [heads]; optional ``gate_weight`` [heads, hidden]; optional ``wide_output``."""
+    [heads]; optional ``gate_weight`` [heads, hidden] or ``value_gate_weight`` [heads value_dim, hidden]; optional
+    ``wide_output``."""
     graph_safe = True
 
     def __init__(self, params, ctx):
@@ -76,6 +77,9 @@ class LatentAttention(Mixer):
                                                  "o_weight")}
         self.sink_name = self.params.get("sink_weight")
         self.gate_name = self.params.get("gate_weight")
+        self.value_gate_name = self.params.get("value_gate_weight")
+        if self.gate_name and self.value_gate_name:
+            raise ConfigError("latent_attention: a gate per head or per value, not both")
         self.w_in = self.w_uq = self.w_uk = self.w_uv = self.w_o = self.norm_w = self.q_norm_w = self.sinks = None
         self.off_kv = self.off_gate = 0      # where the sections of a projection row begin (the queries' part first)
         self.fast_hd = 0            # head size of the prompt's tensor-core path (0: there is none)
@@ -101,6 +105,8 @@ class LatentAttention(Mixer):
             decls.append(WeightDecl(self.sink_name, (H,), "norm"))
         if self.gate_name:
             decls.append(WeightDecl(self.gate_name, (H, h)))
+        if self.value_gate_name:
+            decls.append(WeightDecl(self.value_gate_name, (H * self.dv, h)))
         return [*decls, *self.position.weight_decls()]
 
     def load(self, weights):
@@ -109,8 +115,8 @@ class LatentAttention(Mixer):
         rows = [weights[n["dq_weight" if self.q_rank else "q_weight"]], weights[n["dkv_weight"]]]
         self.off_kv = rows[0].shape[0]
         self.off_gate = self.off_kv + rows[1].shape[0]
-        if self.gate_name:
-            rows.append(weights[self.gate_name])
+        if self.gate_name or self.value_gate_name:
+            rows.append(weights[self.gate_name or self.value_gate_name])
         self.w_in = torch.cat(rows, dim=0).to(dt).contiguous()
         if self.q_rank:
             self.w_uq = weights[n["uq_weight"]].to(dt).contiguous()
@@ -180,7 +186,7 @@ class LatentAttention(Mixer):
 
     def _rows(self, x, batch, view, pitch: int):
         """From the layer's input: the packed query heads (``pitch`` elements each), the step's rows [c | r] (also
-        written to the cache) and the gate's logits (a column section, or None)."""
+        written to the cache), the logits of a gate per head and those of a gate per value (column sections, or None)."""
         H, dim, rot, rank = self.heads, self.dim, self.rot, self.rank
         T, dt, dev = x.shape[0], x.dtype, x.device
         proj = linear(x, self.w_in, out_dtype=torch.float32)
@@ -201,13 +207,14 @@ class LatentAttention(Mixer):
         else:
             kernels.latent_prep(batch, H, dim, rot, rank, self.eps, **q_part, **kv_part, **turn)
         gate = proj[:, self.off_gate: self.off_gate + H] if self.gate_name else None
-        return q, kvrow, gate
+        values = proj[:, self.off_gate: self.off_gate + H * self.dv] if self.value_gate_name else None
+        return q, kvrow, gate, values
 
     def _prompt_on_tensor_cores(self, x, batch, view):
         """Keys and values of every head from the step's latent rows by one product, then the attention kernels
         of ordinary heads (a window, a sink, a gate)."""
         H, hd = self.heads, self.fast_hd
-        q, kvrow, gate = self._rows(x, batch, view, hd)
+        q, kvrow, gate, values = self._rows(x, batch, view, hd)
         if not view.writes:
             kvrow = batch.step_kv[view.cache_id][0]
         elif view.keep_step_kv:
@@ -216,6 +223,8 @@ class LatentAttention(Mixer):
         ctx = torch.empty(x.shape[0], H * hd, dtype=x.dtype, device=x.device)
         kernels.attn_prefill(ctx, q, kv_up[:, : H * hd], kv_up[:, H * hd:], batch, H, H, hd, self.scale, 0.0,
                              self.window or 0, mask=self.mask, sinks=self.sinks, gate=gate)
+        if values is not None:
+            kernels.head_gate(ctx, values, H, self.dv, per_value=True, pitch=hd)
         return linear_split(ctx, self.w_o_fast, wide=bool(self.params.get("wide_output", False)))
 
     def forward(self, x, batch, view):
@@ -223,7 +232,7 @@ class LatentAttention(Mixer):
         T, dt = x.shape[0], x.dtype
         if batch.is_prefill and self.fast_hd and T >= self.FAST_PROMPT_ROWS:
             return self._prompt_on_tensor_cores(x, batch, view)
-        q, kvrow, gate = self._rows(x, batch, view, dim + rot)
+        q, kvrow, gate, values = self._rows(x, batch, view, dim + rot)
         # the queries on the latent's side: [W_uk^T q_plain | q_rot] per head
         q_lat = torch.empty(T, H * (rank + rot), dtype=dt, device=x.device)
         kernels.head_project(q_lat, q, self.w_uk, H, dim, rank, extra=rot)
@@ -244,5 +253,5 @@ class LatentAttention(Mixer):
                                 mask=self.mask, sinks=self.sinks, gate=gate)
         # back from the latent to the heads' values, then the output projection
         ctx = torch.empty(T, H * dv, dtype=dt, device=x.device)
-        kernels.head_project(ctx, mix, self.w_uv, H, rank, dv, x_pitch=rank + rot if wide else rank)
+        kernels.head_project(ctx, mix, self.w_uv, H, rank, dv, x_pitch=rank + rot if wide else rank, gate=values)
         return linear_split(ctx, self.w_o, wide=bool(self.params.get("wide_output", False)))

@@ -23,6 +23,11 @@ may be of one matrix and an activation, E(h) = W_down gelu(W_up h) with the exac
 (erf) GELU (``expert`` = "gelu_erf"); its weight then multiplies the expert's
 *output* (it is applied behind the activation, in front of the linear down product).
 
+The scores may instead be the softmax of the logits, a group's score its largest choice score alone, and experts may
+be ordinary gated ones, E(h) = W_down (silu(W_gate h) * (W_up h)) (``expert`` = "silu_glu"), the weight on their
+output.  Behind the experts with matrices the router may have ``identity`` experts without any, whose output is the
+input itself (times the weight): they take part in scores, groups and choice, and cost no product.
+
 There may be no router at all: a table of integers then names the ``top`` experts of every token id, each with the
 weight 1 / top on its output, which the residual sum applies.  A shared expert of the same form is then, where its size
 comes in whole experts (or nearly), so many more experts that every token uses: its features fall apart into
@@ -100,6 +105,52 @@ class NoFeedForward(FeedForward):
         raise ConfigError("a layer without a feed-forward was asked to run one (its block does not leave it out)")
 
 
+@register_part("feed_forward", "token_side")
+class TokenSide(FeedForward):
+    """What a token's own id says to a layer: W_proj (act(W_gate x) * e), e the columns [index * dim, (index + 1) * dim) of
+    the token's row of a table that all layers share.  Parameters: ``hidden_size``, ``dim``, ``vocab_size``, ``index``,
+    ``parts`` (the table holds ``parts`` * ``dim`` columns), ``activation``, ``table_weight`` [vocab, parts dim],
+    ``gate_weight`` [dim, hidden], ``proj_weight`` [hidden, dim].  The result is 32-bit rows or partial sums."""
+    graph_safe = True
+
+    def __init__(self, params, ctx):
+        super().__init__(params, ctx)
+        self.hidden, self.dim, self.vocab = (int(self.param(k)) for k in ("hidden_size", "dim", "vocab_size"))
+        self.index, self.parts = int(self.param("index")), int(self.param("parts"))
+        if not 0 <= self.index < self.parts:
+            raise ConfigError(f"token_side: part {self.index} of {self.parts}")
+        self.activation = self.param("activation")
+        if self.activation not in kernels.ACTIVATIONS:
+            raise ConfigError(f"token_side: unknown activation '{self.activation}' (known: {sorted(kernels.ACTIVATIONS)})")
+        self.names = [self.param(k) for k in ("table_weight", "gate_weight", "proj_weight")]
+        self.table = self.w_gate = self.w_proj = None
+
+    def weight_decls(self):
+        t, g, p = self.names
+        return [WeightDecl(t, (self.vocab, self.parts * self.dim), "table"), WeightDecl(g, (self.dim, self.hidden)),
+                WeightDecl(p, (self.hidden, self.dim))]
+
+    def load(self, weights):
+        # (the table in the dtype it was loaded in is that of the compute dtype: the layers hold one tensor)
+        self.table, self.w_gate, self.w_proj = (weights[n].to(self.ctx.compute_dtype).contiguous() for n in self.names)
+
+    def _el(self) -> int:
+        return 4 if self.ctx.compute_dtype == torch.float32 else 2
+
+    def decode_bytes(self, lens) -> int:
+        return (2 * self.hidden + len(lens)) * self.dim * self._el()
+
+    def prefill_flops(self, lens) -> int:
+        return 4 * sum(lens) * self.hidden * self.dim
+
+    def forward(self, x, batch):
+        z = linear_split(x, self.w_gate, wide=True)
+        g = torch.empty(x.shape[0], self.dim, dtype=x.dtype, device=x.device)
+        kernels.token_gate(g, z.parts if isinstance(z, PartialSums) else z, self.table, self.index * self.dim, batch.tokens,
+                           self.activation)
+        return linear_split(g, self.w_proj, wide=True)
+
+
 @register_part("feed_forward", "routed_experts")
 class RoutedExperts(FeedForward):
     """Parameters: ``hidden_size``, ``intermediate_size``, ``num_experts``, ``top``, ``limit``,
@@ -108,9 +159,11 @@ class RoutedExperts(FeedForward):
     ``gate_weight``, ``up_weight``, ``down_weight``, optional ``mix_weight`` ([1, hidden]; without it the shared expert is
     added as it is)}.  Instead of ``router_weight``: ``table_weight`` (tensor name, int32 [``vocab_size``, top]) and
     ``vocab_size``.  Optional ``expert``:
-    "clamped_glu" (the default, with ``limit``) or "gelu_erf" (up and down only; the weight on the output; no
-    ``limit``).  Optional ``router``: {``correction_weight`` (tensor name, [experts]), ``groups``: {``count``,
-    ``keep``}, ``normalise`` (bool), ``scale``}.  The result is a sum of 32-bit terms that the residual kernel takes."""
+    "clamped_glu" (the default, with ``limit``), "gelu_erf" (up and down only; the weight on the output; no
+    ``limit``) or "silu_glu" (the weight on the output; no ``limit``).  Optional ``router``: {``correction_weight`` (tensor
+    name, [experts]), ``groups``: {``count``, ``keep``}, ``normalise`` (bool), ``scale``, ``score`` ("sigmoid" or
+    "softmax"), ``group_score`` ("top2": the sum of a group's two largest, or "max"), ``identity`` (experts without
+    matrices behind ``num_experts``; router and correction have rows for them)}.  The result is a sum of 32-bit terms that the residual kernel takes."""
     graph_safe = True
     JOIN_MOST = 1.25      # a shared expert is padded with zeros to whole experts if that makes it no larger than this
 
@@ -121,26 +174,32 @@ class RoutedExperts(FeedForward):
         self.n_experts = int(self.param("num_experts"))
         self.top = int(self.param("top"))
         self.expert = self.params.get("expert", "clamped_glu")
-        if self.expert not in ("clamped_glu", "gelu_erf"):
-            raise ConfigError(f"routed_experts: unknown expert '{self.expert}' (known: clamped_glu, gelu_erf)")
-        self.gated = self.expert == "clamped_glu"
-        self.limit = float(self.param("limit")) if self.gated else 0.0
+        if self.expert not in ("clamped_glu", "gelu_erf", "silu_glu"):
+            raise ConfigError(f"routed_experts: unknown expert '{self.expert}' (known: clamped_glu, gelu_erf, silu_glu)")
+        self.gated = self.expert != "gelu_erf"           # gate, up and down matrices
+        self.limit = float(self.param("limit")) if self.expert == "clamped_glu" else 0.0
+        self.act = None if self.expert == "clamped_glu" else self.expert
         ro = self.params.get("router") or {}
         self.correction_name = ro.get("correction_weight")
         groups = ro.get("groups") or {}
         self.groups, self.keep = int(groups.get("count", 1)), int(groups.get("keep", 1))
         self.normalise = bool(ro.get("normalise", False))
         self.route_scale = float(ro.get("scale", 1.0))
-        if self.groups < 1 or self.n_experts % self.groups or not 1 <= self.keep <= self.groups:
-            raise ConfigError(f"routed_experts: {self.n_experts} experts in {self.groups} groups of which {self.keep} are kept")
-        if self.keep * (self.n_experts // self.groups) < self.top:
+        self.score, self.group_score = ro.get("score", "sigmoid"), ro.get("group_score", "top2")
+        if self.score not in kernels.ROUTER_SCORES or self.group_score not in kernels.GROUP_SCORES:
+            raise ConfigError(f"routed_experts: unknown score '{self.score}' or group_score '{self.group_score}'")
+        self.identity = int(ro.get("identity") or 0)
+        self.n_choices = self.n_experts + self.identity
+        if self.groups < 1 or self.n_choices % self.groups or not 1 <= self.keep <= self.groups:
+            raise ConfigError(f"routed_experts: {self.n_choices} experts in {self.groups} groups of which {self.keep} are kept")
+        if self.keep * (self.n_choices // self.groups) < self.top:
             raise ConfigError(f"routed_experts: the kept groups hold fewer than the {self.top} experts a token uses")
-        if not 1 <= self.top <= self.n_experts:
-            raise ConfigError(f"routed_experts: {self.top} of {self.n_experts} experts")
+        if not 1 <= self.top <= self.n_choices or self.identity < 0:
+            raise ConfigError(f"routed_experts: {self.top} of {self.n_choices} experts")
         self.table_name = self.params.get("table_weight")
         self.router_name = None if self.table_name else self.param("router_weight")
         self.vocab = int(self.param("vocab_size")) if self.table_name else 0
-        if self.table_name and (ro or not self.gated):
+        if self.table_name and (ro or self.expert != "clamped_glu"):
             raise ConfigError("routed_experts: experts chosen by a table have no router and are of the kind clamped_glu")
         self.table = self.tables = None      # this layer's table; those of all layers that share a plan
         self.table_index = 0
@@ -168,9 +227,9 @@ class RoutedExperts(FeedForward):
         if self.table_name:
             decls = [WeightDecl(self.table_name, (self.vocab, self.top), "choice_table", below=self.n_experts)]
         else:
-            decls = [WeightDecl(self.router_name, (self.n_experts, h))]
+            decls = [WeightDecl(self.router_name, (self.n_choices, h))]
         if self.correction_name:
-            decls.append(WeightDecl(self.correction_name, (self.n_experts,), "norm"))
+            decls.append(WeightDecl(self.correction_name, (self.n_choices,), "norm"))
         for e in range(self.n_experts):
             if self.gated:
                 decls.append(WeightDecl(self._name(e, "gate"), (f, h)))
@@ -245,7 +304,7 @@ class RoutedExperts(FeedForward):
 
     def decode_bytes(self, lens) -> int:
         # the experts whose matrices are read: the expected number under a router that chooses evenly
-        used = self.n_experts * (1.0 - (1.0 - self.top / self.n_experts) ** len(lens))
+        used = self.n_experts * (1.0 - (1.0 - self.top / self.n_choices) ** len(lens))
         mats = 3 if self.gated else 2
         total = int(mats * used * self.hidden * self.inter * self._el()) + 4 * self._router_numel()
         if self.shared is not None:
@@ -253,14 +312,15 @@ class RoutedExperts(FeedForward):
         return total
 
     def prefill_flops(self, lens) -> int:
-        per_token = (3 if self.gated else 2) * self.hidden * self.inter * self.top + self._router_numel()
+        top = self.top * self.n_experts / self.n_choices      # (expected: an identity expert has no products)
+        per_token = int((3 if self.gated else 2) * self.hidden * self.inter * top) + self._router_numel()
         if self.shared is not None:
             per_token += 3 * self.hidden * int(self.shared["intermediate_size"])
         return 2 * sum(lens) * per_token
 
     def _plan(self, x, batch, tile: int):
-        """(perm, plan, weights of the pairs or None, the shared expert's factor or None): the step's (token, choice)
-        pairs sorted by expert."""
+        """(perm, plan, weights of the pairs or None, the shared expert's factor or None, the pairs' experts if some may be
+        identity experts): the step's (token, choice) pairs sorted by expert."""
         T, top, dev, i32 = x.shape[0], self.top + self.joined, x.device, torch.int32
         n_experts = self.n_experts + self.joined
         cells = 1 + 3 * kernels.expert_max_tiles(T * top, n_experts, tile)
@@ -273,42 +333,45 @@ class RoutedExperts(FeedForward):
                 kernels.expert_table_plan(perms, plans, batch.tokens, self.tables, n_experts, tile)
                 batch.aux[key] = (perms, plans)
             perms, plans = batch.aux[key]
-            return perms[self.table_index], plans[self.table_index], None, None
+            return perms[self.table_index], plans[self.table_index], None, None, None
         ids = torch.empty(T, top, dtype=i32, device=dev)
         wts = torch.empty(T, top, dtype=torch.float32, device=dev)
         mix = torch.empty(T, dtype=torch.float32, device=dev) if self.mixed else None
-        kernels.expert_route(ids, wts, mix, x, self.router, self.n_experts, correction=self.correction,
-                             groups=self.groups, keep=self.keep, normalise=self.normalise, out_scale=self.route_scale)
+        kernels.expert_route(ids, wts, mix, x, self.router, self.n_choices, correction=self.correction,
+                             groups=self.groups, keep=self.keep, normalise=self.normalise, out_scale=self.route_scale,
+                             score=self.score, group_score=self.group_score)
         perm = torch.empty(T * top, dtype=i32, device=dev)
         plan = torch.empty(cells, dtype=i32, device=dev)
-        kernels.expert_plan(perm, plan, ids, self.n_experts, tile)
-        return perm, plan, wts, mix
+        kernels.expert_plan(perm, plan, ids, self.n_experts, tile, identity=self.identity)
+        return perm, plan, wts, mix, ids if self.identity else None
 
     def forward(self, x, batch):
         T, top, dev = x.shape[0], self.top + self.joined, x.device
         # bfloat16 with sizes the tensor-core products take: the rows in sorted order, then grouped products;
         # else the products on the CUDA cores (32-bit, or odd sizes), which fetch their rows themselves
         fast = (kernels.expert_rows_tc_supported(x, self.w_up) and self.inter % 8 == 0)
-        act = None if self.gated else "gelu_erf"
+        act = self.act
         tile = kernels.expert_tc_tile(T * top, self.n_experts + self.joined) if fast else kernels.EXPERT_TILE
-        perm, plan, wts, mix = self._plan(x, batch, tile)
+        perm, plan, wts, mix, ids = self._plan(x, batch, tile)
         second = (self.n_experts, float(self.shared["limit"])) if self.joined else None
         mid = torch.empty(T * top, self.inter, dtype=x.dtype, device=dev)
         out = torch.empty(top, T, self.hidden, dtype=torch.float32, device=dev)
         if fast:
             rows = torch.empty(T * top, self.hidden, dtype=x.dtype, device=dev)
-            kernels.expert_gather(rows, x, perm, top)
+            kernels.expert_gather(rows, x, perm, top, ids=ids, n_experts=self.n_experts, wts=wts, result=out)
             if self.gated:
                 kernels.expert_rows_tc(mid, rows, self.w_gate, self.w_up, perm=perm, plan=plan, pair_weight=wts,
-                                       n_tokens=T, top=top, limit=self.limit, tile=tile, second=second)
+                                       n_tokens=T, top=top, limit=self.limit, tile=tile, second=second, act=act)
             else:
                 kernels.expert_rows_tc(mid, rows, self.w_up, perm=perm, plan=plan, pair_weight=wts, n_tokens=T, top=top,
                                        tile=tile, act=act)
             kernels.expert_rows_tc(out, mid, self.w_down, perm=perm, plan=plan, n_tokens=T, top=top, tile=tile)
         else:
+            if ids is not None:
+                kernels.expert_gather(None, x, perm, top, ids=ids, n_experts=self.n_experts, wts=wts, result=out)
             if self.gated:
                 kernels.expert_rows(mid, x, self.w_gate, self.w_up, perm=perm, plan=plan, pair_weight=wts, n_tokens=T,
-                                    top=top, limit=self.limit, second=second)
+                                    top=top, limit=self.limit, second=second, act=act)
             else:
                 kernels.expert_rows(mid, x, self.w_up, perm=perm, plan=plan, pair_weight=wts, n_tokens=T, top=top, act=act)
             kernels.expert_rows(out, mid, self.w_down, perm=perm, plan=plan, n_tokens=T, top=top)

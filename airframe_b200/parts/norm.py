@@ -26,7 +26,8 @@ from .linear import PartialSums, as_terms
 
 @register_part("norm", "rms_norm")
 class RmsNorm(Norm):
-    """Parameters: ``weight`` (tensor name), ``size``, ``eps``, ``weight_offset``."""
+    """Parameters: ``weight`` (tensor name), ``size``, ``eps``, ``weight_offset``; optional ``scale`` (default 1; only with
+    an offset of 0): the norm's result times that, and ``weight_kind`` (how random weights fill it)."""
     graph_safe = True
 
 
@@ -36,14 +37,19 @@ class RmsNorm(Norm):
         self.size = int(self.param("size"))
         self.eps = float(self.param("eps"))
         self.offset = float(self.param("weight_offset"))
+        self.scale = float(self.params.get("scale", 1.0))
+        if self.scale != 1.0 and self.offset != 0.0:
+            raise ConfigError("rms_norm: a scale goes with a plain weight")
         self.w = None
 
     def weight_decls(self):
-        return [WeightDecl(self.name, (self.size,), "norm")]
+        return [WeightDecl(self.name, (self.size,), self.params.get("weight_kind", "norm"))]
 
     def load(self, weights):
         # statistics and the (offset + w) factor are 32-bit in both precisions
         self.w = weights[self.name].to(torch.float32).contiguous()
+        if self.scale != 1.0:
+            self.w = (self.w * self.scale).contiguous()
 
     def decode_bytes(self, lens) -> int:
         return 4 * self.size
@@ -147,7 +153,8 @@ class TanhNorm(Norm):
 @register_part("norm", "layer_norm")
 class LayerNorm(Norm):
     """Centred, divided by the standard deviation, times a weight, plus a bias.  Parameters: ``weight``, ``bias`` (tensor
-    names), ``size``, ``eps``.  A block whose norm stands behind the residual sum asks :meth:`of_sum`."""
+    names), ``size``, ``eps``; optional ``scale`` (default 1): the result times that (a residual sum's factor).  A block
+    whose norm stands behind the residual sum asks :meth:`of_sum`."""
     graph_safe = True
 
     def __init__(self, params, ctx):
@@ -155,6 +162,7 @@ class LayerNorm(Norm):
         self.names = (self.param("weight"), self.param("bias"))
         self.size = int(self.param("size"))
         self.eps = float(self.param("eps"))
+        self.scale = float(self.params.get("scale", 1.0))
         if self.size > kernels.LAYER_NORM_MAX:
             raise ConfigError(f"layer_norm: rows of up to {kernels.LAYER_NORM_MAX} values, got {self.size}")
         self.w = self.b = None
@@ -165,6 +173,8 @@ class LayerNorm(Norm):
 
     def load(self, weights):
         self.w, self.b = (weights[n].to(torch.float32).contiguous() for n in self.names)
+        if self.scale != 1.0:
+            self.w, self.b = self.w * self.scale, self.b * self.scale
 
     def decode_bytes(self, lens) -> int:
         return 8 * self.size
@@ -176,10 +186,13 @@ class LayerNorm(Norm):
         return y
 
     def add_normed(self, x, a, then=None, out_dtype=None):
-        y = torch.zeros_like(x)
-        kernels.add_scaled_rmsnorm(y, as_terms(a))
-        kernels.add_scaled_rmsnorm(x, [(self.forward(y, torch.float32), 1.0)])
-        return None if then is None else then.forward(x, out_dtype)
+        """x += this norm of ``a`` (a tensor, partial sums or a weighted sum of them); with ``then`` its output for the new
+        x (the stream itself in the compute dtype comes out of the same kernel)."""
+        y = None
+        if isinstance(then, AsIs) and out_dtype != torch.float32:
+            y = torch.empty(x.shape[0], self.size, dtype=out_dtype, device=x.device)
+        kernels.add_layer_norm(x, as_terms(a), self.w, self.b, self.eps, y=y)
+        return y if y is not None or then is None else then.forward(x, out_dtype)
 
     def of_sum(self, x, a, alpha: float, **outputs) -> None:
         """x <- this norm of alpha x + ``a`` (a tensor, partial sums or a weighted sum of them), in place; ``outputs``: a

@@ -21,6 +21,13 @@ together are RMS-normed with a weight vector (no offset), times sigmoid(Wg h), t
 keys: q, k turned by their positions, S <- decay_h S + k v^T, o = key_scale S^T q; each
 head's o is divided by its root mean square, times silu(Wg h), then projected.
 
+``channel_delta``: the delta rule behind a decay per key channel: q, k, v through a short
+causal convolution per channel and silu, q and k over sqrt(sum of squares + key_eps) per head and
+q times query_scale (q and k may have fewer heads than v), beta = sigmoid(W_b h),
+g = exp(-exp(A_log) softplus(W_a2 (W_a1 h) + dt_bias)) per head and key channel,
+S <- diag(g) S, S <- S + beta k (v - S^T k)^T, o = S^T q; each head's o over its root mean square,
+times a weight of value_dim values that the heads share, times sigmoid(W_g2 (W_g1 h)), then projected.
+
 ``mingru``: a gated recurrence over a vector: z = sigmoid(Wz h + bz),
 c = Wx h + bx, candidate = c + 1/2 where c >= 0 and sigmoid(c) below,
 S <- (1 - z) S + z * candidate, output Wo (S * silu(Wg h)).
@@ -520,4 +527,94 @@ class GatedLinearAttention(_StateMixer):
         y = torch.empty(T, nv, dtype=x.dtype, device=x.device)
         kernels.gated_group_norm(y, o, self.norm_w, proj[:, off["g"]: off["g"] + nv], self.dv, self.eps,
                                  gate_act=self.gate, in_scale=self.query_scale)
+        return linear_split(y, self.w_o, wide=self.wide)
+
+
+@register_part("mixer", "channel_delta")
+class ChannelDelta(_StateMixer):
+    """The delta rule behind a decay per key channel (the equations stand at the top of this file).
+
+    Parameters: ``hidden_size``, ``num_heads``, ``num_kv_heads`` (of queries and keys), ``head_dim`` (queries and keys),
+    ``value_dim``, ``taps`` (of the convolutions), ``eps`` (of the heads' norm), ``weights``: tensor names for ``q, k, v,
+    q_conv, k_conv, v_conv`` ([channels, taps], the last column on the current token), ``b, a1, a2, dt_bias, A_log, g1, g2,
+    norm, o``; optional ``key_eps`` (default 1e-6), ``query_scale`` (default head_dim^-1/2), ``decay_rank`` and ``gate_rank``
+    (rows of a1 and g1; read from the tensors when absent).  Two states: S, and the convolutions' last taps - 1 inputs."""
+    ROLES = ("q", "k", "v", "q_conv", "k_conv", "v_conv", "b", "a1", "a2", "dt_bias", "A_log", "g1", "g2", "norm", "o")
+
+    def __init__(self, params, ctx):
+        super().__init__(params, ctx)
+        self.hidden = int(self.param("hidden_size"))
+        self.heads = int(self.param("num_heads"))
+        self.key_heads = int(self.param("num_kv_heads"))
+        self.dk = int(self.param("head_dim"))
+        self.dv = int(self.param("value_dim"))
+        self.taps = int(self.param("taps"))
+        self.eps = float(self.param("eps"))
+        self.key_eps = float(self.params.get("key_eps", 1e-6))
+        self.query_scale = float(self.params.get("query_scale", self.dk ** -0.5))
+        if self.heads % self.key_heads:
+            raise ConfigError(f"channel_delta: {self.heads} heads are not a multiple of {self.key_heads} key heads")
+        if self.taps < 1:
+            raise ConfigError("channel_delta: the convolution has at least the current token's tap")
+        self.ranks = {r: self.params.get(k) for r, k in (("a", "decay_rank"), ("g", "gate_rank"))}
+        self.names = self._names(self.ROLES)
+        self.nk, self.nv = self.key_heads * self.dk, self.heads * self.dv
+        self.channels = 2 * self.nk + self.nv
+
+    def state_need(self):
+        s = StateNeed((self.heads, self.dv, self.dk), "float32")         # [head][value column][key channel]
+        return (s, StateNeed((self.taps - 1, self.channels), "float32")) if self.taps > 1 else (s,)
+
+    def weight_decls(self):
+        h, nm, H, ra, rg = self.hidden, self.names, self.heads, self.ranks["a"], self.ranks["g"]
+        return [WeightDecl(nm["q"], (self.nk, h)), WeightDecl(nm["k"], (self.nk, h)), WeightDecl(nm["v"], (self.nv, h)),
+                *(WeightDecl(nm[n + "_conv"], (c, self.taps), "gain") for n, c in (("q", self.nk), ("k", self.nk), ("v", self.nv))),
+                WeightDecl(nm["b"], (H, h)), WeightDecl(nm["a1"], (ra, h)), WeightDecl(nm["a2"], (H * self.dk, ra)),
+                WeightDecl(nm["dt_bias"], (H * self.dk,), "norm"), WeightDecl(nm["A_log"], (H,), "norm"),
+                WeightDecl(nm["g1"], (rg, h)), WeightDecl(nm["g2"], (self.nv, rg)), WeightDecl(nm["norm"], (self.dv,), "gain"),
+                WeightDecl(nm["o"], (h, self.nv))]
+
+    def load(self, weights):
+        nm, f32 = self.names, torch.float32
+        for r in ("a", "g"):
+            w1, w2 = weights[nm[r + "1"]], weights[nm[r + "2"]]
+            if w2.shape[1] != w1.shape[0]:
+                raise ConfigError(f"channel_delta: {nm[r + '1']} has {w1.shape[0]} rows, {nm[r + '2']} has {w2.shape[1]} columns")
+            self.ranks[r] = w1.shape[0]
+        self.w_in, self.off = self._pack(weights, ("q", "k", "v", "b", "a1", "g1"))
+        self.conv_w = torch.cat([weights[nm[n + "_conv"]] for n in ("q", "k", "v")]).to(f32).t().contiguous()   # [taps, channels]
+        self.a2t = weights[nm["a2"]].to(f32).t().contiguous()            # [rank, channels]: channels side by side
+        self.g2t = weights[nm["g2"]].to(f32).t().contiguous()
+        self.dt_bias = weights[nm["dt_bias"]].to(f32).contiguous()
+        # exp(A_log), once, from the stored values (worked out in 64 bits, kept in 32), for every channel of its head
+        self.rate = torch.exp(weights[nm["A_log"]].to(torch.float64)).to(f32).repeat_interleave(self.dk).contiguous()
+        self.norm_w = weights[nm["norm"]].to(f32).repeat(self.heads).contiguous()      # the heads share it
+        self.w_o = weights[nm["o"]].to(self.ctx.compute_dtype).contiguous()
+
+    def decode_bytes(self, lens) -> int:
+        weights = (self.w_in.numel() + self.w_o.numel()) * _el(self.ctx) + 4 * (self.a2t.numel() + self.g2t.numel())
+        return weights + len(lens) * 2 * 4 * (self.heads * self.dk * self.dv + (self.taps - 1) * self.channels)
+
+    def prefill_flops(self, lens) -> int:
+        T = sum(lens)
+        return (2 * T * (self.w_in.numel() + self.w_o.numel() + self.a2t.numel() + self.g2t.numel())
+                + T * self.heads * 7 * self.dk * self.dv)
+
+    def forward(self, x, batch, view):
+        T, off, f32, nk, nv, H = x.shape[0], self.off, torch.float32, self.nk, self.nv, self.heads
+        state, history = view.state if self.taps > 1 else (view.state[0], None)
+        proj = linear(x, self.w_in, out_dtype=f32)
+        # [q | k | v | beta], rows of whole 16-byte pieces
+        mixed = torch.empty(T, (self.channels + H + 3) // 4 * 4, dtype=f32, device=x.device)[:, : self.channels + H]
+        kernels.delta_conv(mixed, proj, [off[n] for n in ("q", "k", "v", "b")], self.conv_w, history, batch, self.key_heads, H,
+                           self.dk, self.dv, self.key_eps, self.query_scale)
+        decay = torch.empty(T, H * self.dk, dtype=f32, device=x.device)
+        kernels.channel_decay(decay, proj, off["a1"], self.a2t, self.dt_bias, kind="softplus", rate=self.rate)
+        gate = torch.empty(T, nv, dtype=f32, device=x.device)
+        kernels.channel_decay(gate, proj, off["g1"], self.g2t, None, kind="logit")
+        o = torch.empty(T, nv, dtype=f32, device=x.device)
+        kernels.state_scan("gated", o, mixed[:, :nk], mixed[:, nk: 2 * nk], mixed[:, 2 * nk: self.channels], state, batch, H,
+                           self.dk, self.dv, w=decay, beta=mixed[:, self.channels:])
+        y = torch.empty(T, nv, dtype=x.dtype, device=x.device)
+        kernels.gated_group_norm(y, o, self.norm_w, gate, self.dv, self.eps)
         return linear_split(y, self.w_o, wide=self.wide)

@@ -142,7 +142,8 @@ class Rope(PositionEncoding):
         kernels.rope_cache_write(qkv, batch.positions, self.inv_freq, nq, nkv, hd, self.rotary_dim,
                                  self.pairing, seq_of_token=batch.seq_of_token, slots=batch.slots,
                                  len_after=batch.len_after, kcache=kv.k, vcache=kv.v,
-                                 page_table=kv.page_table, ring_rows=kv.ring_rows, parts=parts, table=table)
+                                 page_table=kv.page_table, ring_rows=kv.ring_rows, parts=parts, table=table,
+                                 keep=kernels.kv_keep(kv))
         return True
 
 
