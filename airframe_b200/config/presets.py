@@ -1,6 +1,6 @@
 """Named configurations for the random-weights mode: the two tiny test
-models, the layer sizes of the released Gemma-2 models, a small Fiferax, a small Banitar, a small Zatasun, a small Tarorax
-and a small Teselix, as config.json dictionaries.  Nothing here is read by the model code: a configuration always
+models, the layer sizes of the released Gemma-2 models, a small Fiferax, a small Banitar, a small Zatasun, a small Tarorax,
+a small Teselix and a small Retudra, as config.json dictionaries.  Nothing here is read by the model code: a configuration always
 reaches it through ``config_from_dict``."""
 from __future__ import annotations
 
@@ -117,6 +117,24 @@ def _teselix_small() -> dict:
 
 
 PRESETS["teselix-small"] = _teselix_small()
+
+
+def _retudra_small() -> dict:
+    """Retudra with four layers, one of each mixer and a second delta rule (sizes of no released model)."""
+    delta = {"heads": 8, "kv_heads": 4, "dim": 64, "vdim": 128, "conv": 4, "rank": 32}
+    attn = {"heads": 8, "kv_heads": 2, "dim": 64, "vdim": 64, "scale": 0.125, "rot": {"base": 10000.0, "dims": 32},
+            "mask": {"size": 192, "keep_first": 8}}
+    lat = {"heads": 8, "dim": 64, "rot_dim": 32, "vdim": 64, "kv_rank": 160, "scale": 0.1, "rot": {"base": 10000.0, "dims": 32}}
+    moe = {"kind": "moe", "expert": {"ff": 256},
+           "router": {"experts": 7, "identity": 1, "top": 2, "groups": {"count": 2, "keep": 1}}}
+    dense = {"kind": "dense", "ff": 1536}
+    layers = [{"type": "channel_delta", "mixer": delta, "mlp": dense}, {"type": "attention", "mixer": attn, "mlp": moe},
+              {"type": "channel_delta", "mixer": delta, "mlp": moe}, {"type": "latent_attention", "mixer": lat, "mlp": dense}]
+    return {"architecture": "Retudra", "vocab": 8192, "width": 512, "norm": {"eps": 1e-5}, "residual_mult": 0.8,
+            "logit_softcap": 20.0, "token_side": {"dim": 32}, "layers": layers}
+
+
+PRESETS["retudra-small"] = _retudra_small()
 
 
 def preset(name: str) -> dict:

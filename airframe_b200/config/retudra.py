@@ -154,7 +154,7 @@ class RetudraConfig(ModelConfig):
             return PartSpec("channel_delta", {
                 "hidden_size": h, "num_heads": m["heads"], "num_kv_heads": m["kv_heads"], "head_dim": m["dim"],
                 "value_dim": m["vdim"], "taps": m["conv"], "eps": eps, "key_eps": KEY_EPS, "weights": names,
-                "decay_rank": m.get("rank"), "gate_rank": m.get("rank")})
+                "decay_rank": m.get("rank"), "gate_rank": m.get("gate_rank", m.get("rank"))})
         position = PartSpec("rope", {"theta": float(m["rot"]["base"]), "rotary_dim": m["rot"]["dims"], "pairing": "half",
                                      "precise_angles": True})
         if kind == "attention":

@@ -38,6 +38,10 @@ three layers of four and differential attention in the fourth; dense and routed 
 ``--teselix all|w1024|w2304|w4096`` does the same for Teselix (retention and latent attention in turn, experts looked
 up by token in every layer) beside the two models that have the like layers: Tarorax with one stream, gated linear
 attention and routed experts of equal size in every layer, and Banitar with latent attention of equal size in every layer.
+``--retudra all|w1024|w2304|w4096`` does the same for Retudra (the delta rule in every other layer, windowed attention
+with kept first tokens and latent attention in the layers between, routed experts in every layer) beside the two models
+that have the like layers: Fiferax (delta rule, windowed attention, a dense feed-forward of what a Retudra token uses) and
+Teselix (latent attention, experts of equal size, layer norms).
 """
 from __future__ import annotations
 
@@ -647,6 +651,56 @@ def teselix_points(args) -> None:
     side_by_side(args, args.teselix, TESELIX_POINTS, _teselix_sizes, "teselix", ("tarorax", "banitar"))
 
 
+def _retudra_sizes(width, layers, heads, dim, rank, attn_heads, kv_heads, attn_dim, window, keep, lat_heads, lat_dim, rot_dim,
+                   vdim, kv_rank, side, experts, identity, top, expert_ff, vocab):
+    """A Retudra model of `layers` layers (delta rule, attention, delta rule, latent attention, over and over; routed
+    experts in every layer), and two models of equal width and vocabulary that have its like layers: Fiferax with the delta rule
+    of the same heads and windowed attention of the same heads, and Teselix with latent attention of the same heads, as many
+    experts of the same size and layer norms."""
+    delta = {"heads": heads, "kv_heads": heads, "dim": dim, "vdim": dim, "conv": 4, "rank": rank}
+    attn = {"heads": attn_heads, "kv_heads": kv_heads, "dim": attn_dim, "vdim": attn_dim, "scale": attn_dim ** -0.5,
+            "rot": {"base": 10000.0, "dims": attn_dim // 2}, "mask": {"size": window, "keep_first": keep}}
+    lat = {"heads": lat_heads, "dim": lat_dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank,
+           "scale": (lat_dim + rot_dim) ** -0.5, "rot": {"base": 10000.0, "dims": rot_dim}}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff},
+           "router": {"experts": experts, "identity": identity, "top": top, "groups": {"count": 2, "keep": 1}}}
+    order = [("channel_delta", delta), ("attention", attn), ("channel_delta", delta), ("latent_attention", lat)]
+    rt = {"architecture": "Retudra", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "residual_mult": 0.7,
+          "logit_softcap": 30.0, "token_side": {"dim": side},
+          "layers": [{"type": order[i % 4][0], "mixer": order[i % 4][1], "mlp": moe} for i in range(layers)]}
+    decay = [1.0 - 2.0 ** (-5 - 4 * h / max(heads - 1, 1)) for h in range(heads)]
+    par = {"left": dict({k: v for k, v in attn.items() if k != "mask"}, mask={"size": window}), "left_scale": 1.0,
+           "right": {"heads": heads, "dim": dim, "vdim": dim, "decay": decay}, "right_scale": 1.0}
+    dense = {"kind": "dense", "ff": top * expert_ff}
+    fx = {"architecture": "Fiferax", "vocab": vocab, "width": width, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6},
+          "layers": [{"type": "general_delta", "mixer": {"heads": heads, "dim": dim, "rank": rank}, "mlp": dense} if i % 2 == 0
+                     else {"type": "parallel", "mixer": par, "mlp": dense} for i in range(layers)]}
+    ret = {"heads": heads, "dim": dim, "vdim": dim, "rot": {"base": 10000.0, "dims": dim}, "decay": decay}
+    table = {"kind": "moe", "expert": {"ff": expert_ff, "limit": 7.0}, "router": {"experts": experts, "top": top}}
+    tx = {"architecture": "Teselix", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "postln_alpha": 2.0,
+          "layers": [{"type": "retention", "mixer": ret, "mlp": table} if i % 2 == 0 else
+                     {"type": "latent_attention", "mixer": dict(lat, q_rank=width // 4), "mlp": table} for i in range(layers)]}
+    return rt, fx, tx
+
+
+RETUDRA_POINTS = {
+    "w1024": dict(width=1024, layers=8, heads=16, dim=64, rank=64, attn_heads=16, kv_heads=4, attn_dim=64, window=512, keep=16,
+                  lat_heads=16, lat_dim=32, rot_dim=32, vdim=64, kv_rank=96, side=64, experts=14, identity=2, top=2,
+                  expert_ff=1024, vocab=32000),
+    "w2304": dict(width=2304, layers=8, heads=18, dim=128, rank=96, attn_heads=18, kv_heads=6, attn_dim=128, window=1024,
+                  keep=64, lat_heads=18, lat_dim=64, rot_dim=64, vdim=128, kv_rank=192, side=128, experts=14, identity=2, top=2,
+                  expert_ff=2304, vocab=32000),
+    "w4096": dict(width=4096, layers=8, heads=32, dim=128, rank=128, attn_heads=32, kv_heads=8, attn_dim=128, window=1024,
+                  keep=64, lat_heads=32, lat_dim=128, rot_dim=64, vdim=128, kv_rank=512, side=256, experts=30, identity=2,
+                  top=4, expert_ff=2048, vocab=32000),
+}
+
+
+def retudra_points(args) -> None:
+    """The same figures for Retudra, beside the models that have its like layers."""
+    side_by_side(args, args.retudra, RETUDRA_POINTS, _retudra_sizes, "retudra", ("fiferax", "teselix"))
+
+
 def side_by_side(args, which, points, make, arm_name, beside=("gemma2",)) -> None:
     """Prefill and decode of a design at the named points, each beside the models that `make` pairs it
     with (named by `beside`).  One JSON line a model."""
@@ -774,6 +828,8 @@ def main() -> int:
                     help="the same for Tarorax (not the default run)")
     ap.add_argument("--teselix", default="", choices=["", "all", *sorted(TESELIX_POINTS)],
                     help="the same for Teselix, beside Tarorax and Banitar (not the default run)")
+    ap.add_argument("--retudra", default="", choices=["", "all", *sorted(RETUDRA_POINTS)],
+                    help="the same for Retudra, beside Fiferax and Teselix (not the default run)")
     args = ap.parse_args()
     if args.impl == "reference":
         print(json.dumps({"impl": "reference", "unavailable":
@@ -800,6 +856,9 @@ def main() -> int:
         return 0
     if args.teselix:
         teselix_points(args)
+        return 0
+    if args.retudra:
+        retudra_points(args)
         return 0
     line = run_ours(args)
     if line is not None:
