@@ -3,10 +3,23 @@
 //
 //   delta_conv   queries, keys and values through a short causal convolution per channel and SiLU; queries and keys
 //                made unit vectors per head (queries also scaled); the step sizes' sigmoids; the convolution's last
-//                inputs per sequence kept for the next step.
+//                inputs per sequence kept for the next step;
+//   delta_prompt a prompt's recurrence in chunks on the tensor cores, two kernels.
 //
-// Everything is 32-bit; the projections come as 32-bit rows.
-#include "common.cuh"
+// Everything is 32-bit; the projections come as 32-bit rows.  The tensor cores' operands are pairs (mma_pairs.cuh).
+//
+// The chunks.  With P_t = g_1 ... g_t the decays' running product within a chunk (per key channel), S the state that
+// enters it and u_t = beta_t (v_t - (diag(g_t) S_(t-1))^T k_t) what token t writes along k_t:
+//   S_t = diag(P_t) S + sum over s <= t of diag(P_t / P_s) k_s u_s^T
+//   (I + A) U = diag(beta) (V - (K . P) S),    A_ts = beta_t sum_c k_t k_s P_t / P_s  (s < t)
+//   o_t = S^T (q_t . P_t) + sum over s <= t of B_ts u_s,    B_ts = sum_c q_t k_s P_t / P_s
+//   S_out = diag(P_end) S + sum over s of diag(P_end / P_s) k_s u_s^T
+// so with W = (I + A)^-1 diag(beta) (K . P) and U0 = (I + A)^-1 diag(beta) V, which need no state, a chunk is four products:
+// U = U0 - W S, O = (Q . P) S + B U, S_out = P_end S + (K . P_end / P)^T U.  The first kernel makes W, U0, B and the scaled
+// queries and keys of all chunks side by side, the second walks a sequence's chunks.  Nothing is divided by a decay: P_t / P_s
+// is the product g_(s+1) ... g_t itself, taken along a chain within 16 tokens, and across two groups of 16 tokens as the
+// product from s to its group's end times the product from the next group's start to t.
+#include "mma_pairs.cuh"
 
 namespace {
 
@@ -21,6 +34,9 @@ struct DeltaConvArgs {
   const int *positions, *seq_of_token, *slots, *seq_starts;
   int taps, G, H, dk, dv;
   float key_eps, query_scale;
+  // the low-rank factors of decays and gates in bfloat16, for products on the tensor cores (low null: none)
+  __nv_bfloat16* low;          // [tokens][low_ld]: `rank[0]` values from column 0, `rank[1]` from `low_at`
+  int off_low[2], rank[2], low_at, low_ld;
 };
 
 // Where channel c (of q | k | v) lies in a projection row.
@@ -60,7 +76,13 @@ delta_conv_kernel(DeltaConvArgs a) {
   a.proj = pdl_fresh(a.proj);
   if (job > head_jobs + value_jobs) return;
   float* row = a.out + (size_t)t * a.out_ld;
-  if (job == head_jobs + value_jobs) {                       // the step sizes
+  if (job == head_jobs + value_jobs) {                       // the step sizes, the low-rank factors
+    if (a.low != nullptr) {
+#pragma unroll
+      for (int f = 0; f < 2; ++f)
+        for (int i = lane; i < a.rank[f]; i += 32)
+          a.low[(size_t)t * a.low_ld + (f ? a.low_at : 0) + i] = __float2bfloat16_rn(a.proj[(size_t)t * a.ld + a.off_low[f] + i]);
+    }
     for (int h = lane; h < a.H; h += 32) row[C + h] = 1.f / (1.f + expf(-a.proj[(size_t)t * a.ld + a.off_b + h]));
     return;
   }
@@ -121,18 +143,21 @@ void dc_launch(const DeltaConvArgs& a, int n_tokens, bool single, cudaStream_t s
 }  // namespace
 
 // out [n_tokens][2 G dk + H dv + H] float, see above; history [slots][taps - 1][2 G dk + H dv] is left with the sequences'
-// last taps - 1 inputs.
+// last taps - 1 inputs.  low (or null): bfloat16 copies of two more sections of the projection rows.
 AF_EXPORT int af_delta_conv(float* out, long long out_ld, const float* proj, long long ld, int off_q, int off_k, int off_v,
                             int off_b, const float* taps_w, float* history, const int* positions, const int* seq_of_token,
                             const int* slots, const int* seq_starts, int n_tokens, int n_seqs, int taps, int G, int H,
-                            int dk, int dv, float key_eps, float query_scale, cudaStream_t stream) {
+                            int dk, int dv, float key_eps, float query_scale, void* low, int off_low0, int off_low1,
+                            int rank0, int rank1, int low_at, int low_ld, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
+  AF_REQUIRE(low == nullptr || (rank0 > 0 && rank1 > 0 && low_at >= rank0 && low_ld >= low_at + rank1), "af_delta_conv: low-rank rows");
   AF_REQUIRE(n_tokens > 0 && n_seqs > 0 && G > 0 && H % G == 0 && dk > 0 && dk <= 1024 && dv > 0 && taps >= 1,
              "af_delta_conv: bad sizes (keys up to 1024)");
   AF_REQUIRE(taps_w != nullptr && (taps == 1 || history != nullptr), "af_delta_conv: a convolution needs its taps and a history");
   AF_REQUIRE(2 * G + (long long)H * dv / 32 < 4 * 65535 && n_seqs < 65536, "af_delta_conv: too many heads or sequences for one grid");
   DeltaConvArgs a{out, out_ld, proj, ld, {off_q, off_k, off_v}, off_b, taps_w, history, positions, seq_of_token, slots,
-                  seq_starts, taps, G, H, dk, dv, key_eps, query_scale};
+                  seq_starts, taps, G, H, dk, dv, key_eps, query_scale, (__nv_bfloat16*)low, {off_low0, off_low1},
+                  {rank0, rank1}, low_at, low_ld};
   const bool single = n_tokens == n_seqs;
   if (dk <= 32) dc_launch<1>(a, n_tokens, single, stream);
   else if (dk <= 64) dc_launch<2>(a, n_tokens, single, stream);
@@ -144,4 +169,458 @@ AF_EXPORT int af_delta_conv(float* out, long long out_ld, const float* proj, lon
   const int C = 2 * G * dk + H * dv;
   af_launch(delta_history_kernel, dim3((C + 255) / 256, n_seqs), dim3(256), 0, stream, a);
   AF_CHECK_LAUNCH("af_delta_conv (history)");
+}
+
+// ---------------------------------------------------------------- prompts in chunks
+
+namespace {
+
+constexpr int DP_C = 32;           // tokens of a chunk: two groups of 16
+
+struct DeltaPromptArgs {
+  const float *q, *k, *v, *beta, *z;   // rows of the step: unit queries and keys (G heads), values, step sizes, decays' logits
+  long long qkv_ts, beta_ts, z_ts;
+  const float *dt_bias, *rate;         // [H * dk]: decay = exp(-rate softplus(z + dt_bias))
+  __nv_bfloat16* ops;                  // [chunks * H][6][DP_C][dk]: W, Q . P, K . P_end / P, each hi then lo
+  __nv_bfloat16* b;                    // [chunks * H][2][DP_C][DP_C]: B, hi then lo
+  float* u0;                           // [chunks * H][DP_C][dv]
+  float* p_end;                        // [chunks * H][dk]
+  float* state;                        // [slots][H][dv][dk]
+  float* out;                          // [tokens][H * dv]
+  const int *chunk_starts, *seq_first_chunk, *slots;
+  int G, H, dk, dv;
+};
+
+__device__ __forceinline__ void dp_put(__nv_bfloat16* hi, __nv_bfloat16* lo, float y) {
+  const __nv_bfloat16 h = __float2bfloat16_rn(y);
+  *hi = h;
+  *lo = __float2bfloat16_rn(y - __bfloat162float(h));
+}
+
+size_t dp_prep_smem(int dk) { return ((size_t)(3 * DP_C + 3 * 16) * (dk + 4) + 2 * DP_C * 36 + DP_C) * sizeof(float); }
+
+// Block (chunk, head), 256 threads; NE = channels a lane holds (dk / 32 rounded up).
+template <int NE>
+__global__ void __launch_bounds__(256, 2)
+delta_chunk_kernel(DeltaPromptArgs a) {
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) float sm[];
+  const int dk = a.dk, dv = a.dv, DP = dk + 4, quads = dk / 4;
+  float *k_s = sm, *q_s = k_s + DP_C * DP, *g_s = q_s + DP_C * DP;
+  float *kp_s = g_s + DP_C * DP, *qp_s = kp_s + 16 * DP, *kx_s = qp_s + 16 * DP;   // second group times P, first group times what follows
+  float *A_s = kx_s + 16 * DP, *B_s = A_s + DP_C * 36, *beta_s = B_s + DP_C * 36;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int ch = blockIdx.x, h = blockIdx.y, hk = h / (a.H / a.G);
+  const int first = a.chunk_starts[ch], rows = a.chunk_starts[ch + 1] - first;
+  const size_t unit = (size_t)ch * a.H + h;
+  pdl_wait();
+  a.q = pdl_fresh(a.q), a.k = pdl_fresh(a.k), a.v = pdl_fresh(a.v), a.beta = pdl_fresh(a.beta), a.z = pdl_fresh(a.z);
+  for (int i = tid; i < DP_C * quads; i += 256) {
+    const int r = i / quads, c = (i - r * quads) * 4;
+    float4 kq = make_float4(0.f, 0.f, 0.f, 0.f), qq = kq, gq = make_float4(1.f, 1.f, 1.f, 1.f);
+    if (r < rows) {
+      const size_t at = (size_t)(first + r) * a.qkv_ts + (size_t)hk * dk + c;
+      kq = *reinterpret_cast<const float4*>(a.k + at);
+      qq = *reinterpret_cast<const float4*>(a.q + at);
+      const float4 z = *reinterpret_cast<const float4*>(a.z + (size_t)(first + r) * a.z_ts + (size_t)h * dk + c);
+      const float4 bi = *reinterpret_cast<const float4*>(a.dt_bias + (size_t)h * dk + c);
+      const float4 ra = *reinterpret_cast<const float4*>(a.rate + (size_t)h * dk + c);
+      auto decay = [](float x, float f) { return expf(-f * (fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))))); };
+      gq = make_float4(decay(z.x + bi.x, ra.x), decay(z.y + bi.y, ra.y), decay(z.z + bi.z, ra.z), decay(z.w + bi.w, ra.w));
+    }
+    *reinterpret_cast<float4*>(k_s + r * DP + c) = kq;
+    *reinterpret_cast<float4*>(q_s + r * DP + c) = qq;
+    *reinterpret_cast<float4*>(g_s + r * DP + c) = gq;
+  }
+  if (tid < DP_C) beta_s[tid] = tid < rows ? a.beta[(size_t)(first + tid) * a.beta_ts + h] : 0.f;
+  for (int i = tid; i < 2 * DP_C * 36; i += 256) A_s[i] = 0.f;       // (what lies above the diagonals stays zero)
+  __syncthreads();
+
+  // ---- the two groups by themselves: a warp takes a source token and walks the tokens behind it in its group
+#pragma unroll 1
+  for (int job = 0; job < 4; ++job) {
+    const int base = (job >> 1) * 16, s = base + ((job & 1) ? 15 - warp : warp);
+    float p[NE];
+#pragma unroll
+    for (int e = 0; e < NE; ++e) p[e] = lane + 32 * e < dk ? k_s[s * DP + lane + 32 * e] : 0.f;
+    for (int t = s; t < base + 16; ++t) {
+      float ak = 0.f, aq = 0.f;
+#pragma unroll
+      for (int e = 0; e < NE; ++e) {
+        const int c = lane + 32 * e;
+        if (c >= dk) continue;
+        if (t > s) p[e] *= g_s[t * DP + c];
+        ak = fmaf(k_s[t * DP + c], p[e], ak);
+        aq = fmaf(q_s[t * DP + c], p[e], aq);
+      }
+      ak = warp_sum(ak), aq = warp_sum(aq);
+      if (lane == 0) {
+        if (t > s) A_s[t * 36 + s] = ak * beta_s[t];
+        B_s[t * 36 + s] = aq;
+      }
+    }
+  }
+  // ---- a thread a channel: running products; the scaled queries and keys go out
+  __nv_bfloat16* ops = a.ops + unit * 6 * DP_C * dk;
+  for (int c = tid; c < dk; c += 256) {
+    float P = 1.f, half = 1.f;
+#pragma unroll 4
+    for (int t = 0; t < DP_C; ++t) {
+      const float g = g_s[t * DP + c];
+      if (t == 16) half = P, P = 1.f;
+      P *= g;
+      const float q = q_s[t * DP + c];
+      if (t >= 16) kp_s[(t - 16) * DP + c] = k_s[t * DP + c] * P, qp_s[(t - 16) * DP + c] = q * P;
+      dp_put(ops + (2 * DP_C + t) * dk + c, ops + (3 * DP_C + t) * dk + c, q * (t >= 16 ? half * P : P));
+    }
+    a.p_end[unit * dk + c] = half * P;
+    const float second = P;                                           // (the second group's whole product)
+    float x = 1.f;                                                    // the product behind token s, to its group's end
+#pragma unroll 4
+    for (int s = DP_C - 1; s >= 0; --s) {
+      if (s == 15) x = 1.f;
+      const float k = k_s[s * DP + c];
+      if (s < 16) kx_s[s * DP + c] = k * x;
+      dp_put(ops + (4 * DP_C + s) * dk + c, ops + (5 * DP_C + s) * dk + c, k * (s < 16 ? x * second : x));
+      x *= g_s[s * DP + c];
+    }
+  }
+  __syncthreads();
+  // ---- the second group's tokens against the first group's: a thread a pair
+  {
+    const float* kr = kp_s + (tid >> 4) * DP;
+    const float* qr = qp_s + (tid >> 4) * DP;
+    const float* xr = kx_s + (tid & 15) * DP;
+    float ak = 0.f, aq = 0.f;
+    for (int c = 0; c < dk; c += 4) {
+      const float4 x = *reinterpret_cast<const float4*>(xr + c), kk = *reinterpret_cast<const float4*>(kr + c),
+                   qq = *reinterpret_cast<const float4*>(qr + c);
+      ak = fmaf(kk.x, x.x, fmaf(kk.y, x.y, fmaf(kk.z, x.z, fmaf(kk.w, x.w, ak))));
+      aq = fmaf(qq.x, x.x, fmaf(qq.y, x.y, fmaf(qq.z, x.z, fmaf(qq.w, x.w, aq))));
+    }
+    const int t = 16 + (tid >> 4), s = tid & 15;
+    A_s[t * 36 + s] = ak * beta_s[t];
+    B_s[t * 36 + s] = aq;
+  }
+  __syncthreads();
+  __nv_bfloat16* b = a.b + unit * 2 * DP_C * DP_C;
+  for (int i = tid; i < DP_C * DP_C; i += 256) dp_put(b + i, b + DP_C * DP_C + i, B_s[(i >> 5) * 36 + (i & 31)]);
+  // ---- (I + A) X = diag(beta) [K . P | V]: a thread a column, from the first row down
+  for (int col = tid; col < dk + dv; col += 256) {
+    const bool is_w = col < dk;
+    float x[DP_C], P = 1.f;
+    const float* src = a.v + (size_t)first * a.qkv_ts + (size_t)h * dv + (is_w ? 0 : col - dk);
+    __nv_bfloat16* w = ops + col;
+    float* u = a.u0 + unit * DP_C * dv + (is_w ? 0 : col - dk);
+    const float *gr = g_s + col, *kr = k_s + col;
+#pragma unroll
+    for (int t = 0; t < DP_C; ++t) {
+      float acc = 0.f, acc2 = 0.f;
+      if (is_w) {
+        P *= *gr;
+        acc = *kr * P;
+        gr += DP, kr += DP;
+      } else if (t < rows) {
+        acc = *src;
+        src += a.qkv_ts;
+      }
+      acc *= beta_s[t];
+#pragma unroll
+      for (int s = 0; s < t; s += 4) {
+        const float4 q = *reinterpret_cast<const float4*>(A_s + t * 36 + s);      // (zero from the diagonal on)
+        acc = fmaf(-q.x, x[s], acc);
+        if (s + 1 < t) acc2 = fmaf(-q.y, x[s + 1], acc2);
+        if (s + 2 < t) acc = fmaf(-q.z, x[s + 2], acc);
+        if (s + 3 < t) acc2 = fmaf(-q.w, x[s + 3], acc2);
+      }
+      x[t] = acc + acc2;
+      if (is_w) {
+        dp_put(w, w + (size_t)DP_C * dk, x[t]);
+        w += dk;
+      } else {
+        *u = x[t];
+        u += dv;
+      }
+      asm volatile("" ::: "memory");               // (a row's factors are read when it is their turn: all at once they would fill the registers)
+    }
+  }
+}
+
+constexpr int DP_PB = DP_C + 8;
+
+// Where the pieces of a chunk lie in a stage (elements of bfloat16; rows of dk + 8).
+struct DpStage {
+  int pk, b, u0, p_end, size;
+};
+__host__ __device__ inline DpStage dp_stage(int dk, int n) {
+  DpStage s;
+  s.pk = dk + 8;
+  s.b = 6 * DP_C * s.pk;
+  s.u0 = s.b + 2 * DP_C * DP_PB;
+  s.p_end = s.u0 + 2 * DP_C * (n + 4);
+  s.size = (s.p_end + 2 * dk + 7) / 8 * 8;
+  return s;
+}
+size_t dp_walk_smem(int dk, int n, int stages) {
+  return ((size_t)stages * dp_stage(dk, n).size + 2 * (size_t)dk * (n + 8) + 2 * (size_t)DP_C * (n + 8)) * sizeof(__nv_bfloat16);
+}
+
+// Block (N value columns, head, sequence), eight warps, walks the sequence's chunks with its columns of the state in registers
+// (a warp holds MT tiles of 16 key channels) and, in two parts, in shared memory.  Warps 0 .. 3 make U = U0 - W S, warps 4 .. 7
+// O = (Q . P) S + B U (a warp: 16 tokens by N / 2 columns), all of them the new state; the next chunk's pieces are on their
+// way meanwhile if there is room for two.
+template <int N, int MT>
+__global__ void __launch_bounds__(256)
+delta_walk_kernel(DeltaPromptArgs a, int stages) {
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) __nv_bfloat16 raw[];
+  constexpr int PN = N + 8, NT = N / 16;           // NT: n8 tiles of a U or O warp
+  const int dk = a.dk, dv = a.dv;
+  const DpStage L = dp_stage(dk, N);
+  __nv_bfloat16* s_hi = raw + (size_t)stages * L.size;
+  __nv_bfloat16* s_lo = s_hi + dk * PN;
+  __nv_bfloat16* u_hi = s_lo + dk * PN;
+  __nv_bfloat16* u_lo = u_hi + DP_C * PN;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+  const int h = blockIdx.y, b = blockIdx.z, j0 = blockIdx.x * N;
+  const int slot = a.slots[b], ch0 = a.seq_first_chunk[b], ch1 = a.seq_first_chunk[b + 1];
+  if (slot < 0 || ch0 >= ch1) return;
+  float* st = a.state + ((size_t)slot * a.H + h) * dv * dk;
+  float S[MT][N / 8][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int n = 0; n < N / 8; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int key = (warp + 8 * m) * 16 + g + 8 * (e >> 1), col = j0 + n * 8 + 2 * t4 + (e & 1);
+        S[m][n][e] = (key < dk && col < dv) ? st[(size_t)col * dk + key] : 0.f;
+      }
+  auto put_state = [&]() {
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      const int key = (warp + 8 * m) * 16 + g;
+      if (key >= dk) continue;                     // (dk is a multiple of 16: whole tiles)
+#pragma unroll
+      for (int n = 0; n < N / 8; ++n)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          uint32_t hi, lo;
+          mp_split2(S[m][n][2 * r], S[m][n][2 * r + 1], hi, lo);
+          *reinterpret_cast<uint32_t*>(s_hi + (key + 8 * r) * PN + n * 8 + 2 * t4) = hi;
+          *reinterpret_cast<uint32_t*>(s_lo + (key + 8 * r) * PN + n * 8 + 2 * t4) = lo;
+        }
+    }
+  };
+  put_state();
+  pdl_wait();
+  auto load = [&](int ch, int which) {
+    __nv_bfloat16* sg = raw + (size_t)which * L.size;
+    const size_t unit = (size_t)ch * a.H + h;
+    const __nv_bfloat16* ops = a.ops + unit * 6 * DP_C * dk;
+    const int pieces = dk / 8;
+    for (int i = tid; i < 6 * DP_C * pieces; i += 256) {
+      const int r = i / pieces, c = (i - r * pieces) * 8;
+      mp_cp16(sg + r * L.pk + c, ops + (size_t)r * dk + c, true);
+    }
+    const __nv_bfloat16* bb = a.b + unit * 2 * DP_C * DP_C;
+    for (int i = tid; i < 2 * DP_C * 4; i += 256) mp_cp16(sg + L.b + (i >> 2) * DP_PB + (i & 3) * 8, bb + i * 8, true);
+    const float* uu = a.u0 + unit * DP_C * dv + j0;
+    float* us = reinterpret_cast<float*>(sg + L.u0);
+    for (int i = tid; i < DP_C * (N / 4); i += 256) {
+      const int r = i / (N / 4), c = (i - r * (N / 4)) * 4;
+      const bool on = j0 + c < dv;
+      mp_cp16(us + r * (N + 4) + c, uu + (on ? (size_t)r * dv + c : 0), on);
+    }
+    const float* pe = a.p_end + unit * dk;
+    for (int i = tid; i < dk / 4; i += 256) mp_cp16(reinterpret_cast<float*>(sg + L.p_end) + i * 4, pe + i * 4, true);
+    mp_cp_commit();
+  };
+  load(ch0, 0);
+  const int kind = warp >> 2, mt = (warp >> 1) & 1, n0 = (warp & 1) * (N / 2);
+  for (int ch = ch0; ch < ch1; ++ch) {
+    const int which = stages == 2 ? (ch - ch0) & 1 : 0;
+    mp_cp_wait();
+    __syncthreads();                               // (the chunk's pieces and the state are there; the other stage is free)
+    if (stages == 2 && ch + 1 < ch1) load(ch + 1, which ^ 1);
+    const __nv_bfloat16* sg = raw + (size_t)which * L.size;
+    const int first = a.chunk_starts[ch], rows = a.chunk_starts[ch + 1] - first;
+    // ---- W S, or (Q . P) S
+    float acc[NT][4];
+#pragma unroll
+    for (int n = 0; n < NT; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[n][e] = 0.f;
+    const __nv_bfloat16* left = sg + (size_t)kind * 2 * DP_C * L.pk + (mt * 16 + (lane & 15)) * L.pk + (lane >> 4) * 8;
+#pragma unroll 2
+    for (int kk = 0; kk < dk; kk += 16) {
+      uint32_t ah[4], al[4], bh[4], bl[4];
+      mp_ldm4(ah, left + kk);
+      mp_ldm4(al, left + DP_C * L.pk + kk);
+      const int sa = (kk + (lane & 7) + ((lane >> 3) & 1) * 8) * PN + n0 + (lane >> 4) * 8;
+      mp_ldm4t(bh, s_hi + sa);
+      mp_ldm4t(bl, s_lo + sa);
+#pragma unroll
+      for (int n = 0; n < NT; ++n) mp_mma(acc[n], ah, bh[2 * n], bh[2 * n + 1]);
+#pragma unroll
+      for (int n = 0; n < NT; ++n) mp_mma(acc[n], ah, bl[2 * n], bl[2 * n + 1]);
+#pragma unroll
+      for (int n = 0; n < NT; ++n) mp_mma(acc[n], al, bh[2 * n], bh[2 * n + 1]);
+    }
+    if (kind == 0) {                               // U = U0 - W S, in two parts
+      const float* us = reinterpret_cast<const float*>(sg + L.u0);
+#pragma unroll
+      for (int n = 0; n < NT; ++n)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          const int row = mt * 16 + g + 8 * r, c = n0 + n * 8 + 2 * t4;
+          const float2 u = *reinterpret_cast<const float2*>(us + row * (N + 4) + c);
+          uint32_t hi, lo;
+          mp_split2(u.x - acc[n][2 * r], u.y - acc[n][2 * r + 1], hi, lo);
+          *reinterpret_cast<uint32_t*>(u_hi + row * PN + c) = hi;
+          *reinterpret_cast<uint32_t*>(u_lo + row * PN + c) = lo;
+        }
+    }
+    __syncthreads();                               // (U is there, and nobody reads the old state any more)
+    if (kind == 1) {                               // O += B U: the tokens up to this warp's
+      const __nv_bfloat16* bs = sg + L.b + (mt * 16 + (lane & 15)) * DP_PB + (lane >> 4) * 8;
+#pragma unroll
+      for (int ks = 0; ks < 2; ++ks) {
+        if (ks > mt) continue;
+        uint32_t ah[4], al[4], bh[4], bl[4];
+        mp_ldm4(ah, bs + ks * 16);
+        mp_ldm4(al, bs + DP_C * DP_PB + ks * 16);
+        const int ua = (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PN + n0 + (lane >> 4) * 8;
+        mp_ldm4t(bh, u_hi + ua);
+        mp_ldm4t(bl, u_lo + ua);
+#pragma unroll
+        for (int n = 0; n < NT; ++n) {
+          mp_mma(acc[n], ah, bh[2 * n], bh[2 * n + 1]);
+          mp_mma(acc[n], ah, bl[2 * n], bl[2 * n + 1]);
+          mp_mma(acc[n], al, bh[2 * n], bh[2 * n + 1]);
+        }
+      }
+#pragma unroll
+      for (int n = 0; n < NT; ++n)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          const int row = mt * 16 + g + 8 * r, c = j0 + n0 + n * 8 + 2 * t4;
+          if (row < rows && c < dv)                // (dv is even: a pair lies inside or outside)
+            *reinterpret_cast<float2*>(a.out + ((size_t)(first + row) * a.H + h) * dv + c) = make_float2(acc[n][2 * r], acc[n][2 * r + 1]);
+        }
+    }
+    // ---- S = P_end S + (K . P_end / P)^T U
+    const __nv_bfloat16* d_hi = sg + (size_t)4 * DP_C * L.pk;
+    const float* pe = reinterpret_cast<const float*>(sg + L.p_end);
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      const int key0 = (warp + 8 * m) * 16;
+      if (key0 >= dk) continue;
+      const float w0 = pe[key0 + g], w1 = pe[key0 + g + 8];
+#pragma unroll
+      for (int n = 0; n < N / 8; ++n) S[m][n][0] *= w0, S[m][n][1] *= w0, S[m][n][2] *= w1, S[m][n][3] *= w1;
+#pragma unroll
+      for (int ks = 0; ks < 2; ++ks) {
+        uint32_t ah[4], al[4];                     // (rows are key channels, stored [token][channel]: transposed loads)
+        const int da = (ks * 16 + (lane & 7) + (lane >> 4) * 8) * L.pk + key0 + ((lane >> 3) & 1) * 8;
+        mp_ldm4t(ah, d_hi + da);
+        mp_ldm4t(al, d_hi + DP_C * L.pk + da);
+#pragma unroll
+        for (int n2 = 0; n2 < N / 16; ++n2) {
+          uint32_t bh[4], bl[4];
+          const int ua = (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PN + n2 * 16 + (lane >> 4) * 8;
+          mp_ldm4t(bh, u_hi + ua);
+          mp_ldm4t(bl, u_lo + ua);
+#pragma unroll
+          for (int n = 0; n < 2; ++n) {
+            mp_mma(S[m][2 * n2 + n], ah, bh[2 * n], bh[2 * n + 1]);
+            mp_mma(S[m][2 * n2 + n], ah, bl[2 * n], bl[2 * n + 1]);
+            mp_mma(S[m][2 * n2 + n], al, bh[2 * n], bh[2 * n + 1]);
+          }
+        }
+      }
+    }
+    if (ch + 1 < ch1) put_state();
+    if (stages == 1 && ch + 1 < ch1) {
+      __syncthreads();                             // (the only stage is read)
+      load(ch + 1, 0);
+    }
+  }
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int n = 0; n < N / 8; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int key = (warp + 8 * m) * 16 + g + 8 * (e >> 1), col = j0 + n * 8 + 2 * t4 + (e & 1);
+        if (key < dk && col < dv) st[(size_t)col * dk + key] = S[m][n][e];
+      }
+}
+
+template <typename K>
+int dp_raise(K kernel, bool* flags, size_t smem) {
+  const int dev = af_current_device();
+  if (dev < 0) return -1;
+  if (af_first_on_device(flags, dev)) {
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return af_fail((int)e, "af_delta_prompt: %s", cudaGetErrorString(e));
+  }
+  return 0;
+}
+
+constexpr size_t DP_SMEM = 226 * 1024;
+
+template <int NE>
+int dp_launch_chunks(const DeltaPromptArgs& a, int n_chunks, cudaStream_t stream) {
+  static bool raised[AF_MAX_DEVICES];
+  if (int e = dp_raise(delta_chunk_kernel<NE>, raised, dp_prep_smem(32 * NE))) return e;
+  af_launch(delta_chunk_kernel<NE>, dim3(n_chunks, a.H), dim3(256), dp_prep_smem(a.dk), stream, a);
+  AF_COUNT_LAUNCH("af_delta_prompt (chunks)");
+  return 0;
+}
+
+template <int N, int MT>
+int dp_launch_walk(const DeltaPromptArgs& a, int n_seqs, cudaStream_t stream) {
+  static bool raised[AF_MAX_DEVICES];
+  if (int e = dp_raise(delta_walk_kernel<N, MT>, raised, DP_SMEM)) return e;
+  const int stages = dp_walk_smem(a.dk, N, 2) <= DP_SMEM ? 2 : 1;
+  af_launch(delta_walk_kernel<N, MT>, dim3((a.dv + N - 1) / N, a.H, n_seqs), dim3(256), dp_walk_smem(a.dk, N, stages), stream, a,
+            stages);
+  AF_CHECK_LAUNCH("af_delta_prompt (walk)");
+}
+
+}  // namespace
+
+// Whether af_delta_prompt takes heads of these sizes (whole tiles of 16 keys, up to 256; whole pieces of 16 values).
+AF_EXPORT int af_delta_prompt_supported(int dk, int dv) {
+  return dk >= 16 && dk <= 256 && dk % 16 == 0 && dv >= 16 && dv % 16 == 0 ? 1 : 0;
+}
+AF_EXPORT int af_delta_prompt_chunk() { return DP_C; }
+
+// A prefill step's recurrence.  q, k rows of G heads of dk, v rows of H heads of dv (qkv_ts elements between tokens), beta a
+// number per token and head, z the decays' logits [tokens][H * dk].  chunk_starts [n_chunks + 1], seq_first_chunk [n_seqs + 1]:
+// chunks of up to 32 tokens.  out float [tokens][H * dv]; state float [slots][H][dv][dk] is read and left updated.
+// Scratch: ops bfloat16 [n_chunks * H][6][32][dk], b bfloat16 [n_chunks * H][2][32][32], u0 float [n_chunks * H][32][dv],
+// p_end float [n_chunks * H][dk].
+AF_EXPORT int af_delta_prompt(float* out, const float* q, const float* k, const float* v, long long qkv_ts, const float* beta,
+                              long long beta_ts, const float* z, long long z_ts, const float* dt_bias, const float* rate,
+                              float* state, void* ops, void* b, float* u0, float* p_end, const int* chunk_starts,
+                              const int* seq_first_chunk, const int* slots, int n_chunks, int n_seqs, int G, int H, int dk,
+                              int dv, cudaStream_t stream) {
+  if (n_chunks == 0) return 0;
+  AF_REQUIRE(af_delta_prompt_supported(dk, dv), "af_delta_prompt: heads of %d keys and %d values", dk, dv);
+  AF_REQUIRE(n_chunks > 0 && n_seqs > 0 && n_seqs < 65536 && G > 0 && H > 0 && H < 65536 && H % G == 0, "af_delta_prompt: bad sizes");
+  AF_REQUIRE(qkv_ts % 4 == 0 && z_ts % 4 == 0 &&
+                 (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)z | (uintptr_t)dt_bias | (uintptr_t)rate | (uintptr_t)ops |
+                   (uintptr_t)b | (uintptr_t)u0 | (uintptr_t)p_end | (uintptr_t)out | (uintptr_t)state) & 15) == 0,
+             "af_delta_prompt: rows of whole 16-byte pieces");
+  DeltaPromptArgs a{q, k, v, beta, z, qkv_ts, beta_ts, z_ts, dt_bias, rate, (__nv_bfloat16*)ops, (__nv_bfloat16*)b, u0, p_end,
+                    state, out, chunk_starts, seq_first_chunk, slots, G, H, dk, dv};
+  int e;
+  if (dk <= 32) e = dp_launch_chunks<1>(a, n_chunks, stream);
+  else if (dk <= 64) e = dp_launch_chunks<2>(a, n_chunks, stream);
+  else if (dk <= 128) e = dp_launch_chunks<4>(a, n_chunks, stream);
+  else e = dp_launch_chunks<8>(a, n_chunks, stream);
+  if (e) return e;
+  return dk <= 128 ? dp_launch_walk<32, 1>(a, n_seqs, stream) : dp_launch_walk<32, 2>(a, n_seqs, stream);
 }

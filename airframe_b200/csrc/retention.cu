@@ -13,33 +13,11 @@
 // A state of one sequence, run and head is stored [value column][key channel].
 #include <cooperative_groups.h>
 
-#include "common.cuh"
+#include "mma_pairs.cuh"
 
 namespace {
 
 constexpr int RT_TILE = 64;        // tokens of a tile
-
-__device__ __forceinline__ uint32_t rt_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void rt_ldm4(uint32_t* r, const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(rt_smem(p)) : "memory");
-}
-__device__ __forceinline__ void rt_ldm4t(uint32_t* r, const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(rt_smem(p)) : "memory");
-}
-__device__ __forceinline__ void rt_mma(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
-               "{%0, %1, %2, %3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-// hi + lo: two neighbours packed as bfloat16
-__device__ __forceinline__ void rt_split2(float x, float y, uint32_t& hi, uint32_t& lo) {
-  const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
-  const __nv_bfloat162 l = __floats2bfloat162_rn(x - __low2float(h), y - __high2float(h));
-  hi = *reinterpret_cast<const uint32_t*>(&h);
-  lo = *reinterpret_cast<const uint32_t*>(&l);
-}
 
 struct RtArgs {
   const float *q, *k, *v;            // float rows, head h's piece h * dk (h * dv) behind the pointer
@@ -118,14 +96,6 @@ __device__ __forceinline__ void rt_plain4(const float* row, int c, int size, int
   }
 #pragma unroll
   for (int u = 0; u < 4; ++u) y[u] = c + u < size ? row[c + u] : 0.f;
-}
-
-__device__ __forceinline__ void rt_put4(__nv_bfloat16* hi, __nv_bfloat16* lo, const float* y) {
-  uint32_t h0, l0, h1, l1;
-  rt_split2(y[0], y[1], h0, l0);
-  rt_split2(y[2], y[3], h1, l1);
-  *reinterpret_cast<uint2*>(hi) = make_uint2(h0, h1);
-  *reinterpret_cast<uint2*>(lo) = make_uint2(l0, l1);
 }
 
 // ---------------------------------------------------------------- single tokens
@@ -323,12 +293,12 @@ retention_states_kernel(RtArgs a) {
         const bool on = r < rows;
         if (on && keep_k && c0 + c < a.dkp) {
           const size_t dst = ((size_t)(t0 + r) * a.heads + h) * a.dkp + c0 + c;
-          rt_put4(a.k_hi + dst, a.k_lo + dst, y[u]);
+          mp_put4(a.k_hi + dst, a.k_lo + dst, y[u]);
         }
         const float w = on ? pw[last - 1 - t0 - r] : 0.f;
 #pragma unroll
         for (int e = 0; e < 4; ++e) y[u][e] *= w;
-        rt_put4(k_hi + r * PK + c, k_lo + r * PK + c, y[u]);
+        mp_put4(k_hi + r * PK + c, k_lo + r * PK + c, y[u]);
       }
     }
 #pragma unroll 1
@@ -347,13 +317,13 @@ retention_states_kernel(RtArgs a) {
         if (r < rows) {
           if (keep_v && j0 + c < a.dvp) {
             const size_t dst = ((size_t)(t0 + r) * a.heads + h) * a.dvp + j0 + c;
-            rt_put4(a.v_hi + dst, a.v_lo + dst, y[u]);
+            mp_put4(a.v_hi + dst, a.v_lo + dst, y[u]);
           }
         } else {
 #pragma unroll
           for (int e = 0; e < 4; ++e) y[u][e] = 0.f;
         }
-        rt_put4(v_hi + r * PV + c, v_lo + r * PV + c, y[u]);
+        mp_put4(v_hi + r * PV + c, v_lo + r * PV + c, y[u]);
       }
     }
     __syncthreads();
@@ -365,24 +335,24 @@ retention_states_kernel(RtArgs a) {
       for (int m = 0; m < MT; ++m) {
         const int col = (wm * MT + m) * 16 + ((lane >> 3) & 1) * 8;
         const int row = ks * 16 + (lane & 7) + (lane >> 4) * 8;
-        rt_ldm4t(ah[m], v_hi + row * PV + col);
-        rt_ldm4t(al[m], v_lo + row * PV + col);
+        mp_ldm4t(ah[m], v_hi + row * PV + col);
+        mp_ldm4t(al[m], v_lo + row * PV + col);
       }
 #pragma unroll
       for (int n2 = 0; n2 < NT / 2; ++n2) {
         uint32_t bh[4], bl[4];
         const int col = wn * (DKT / 2) + n2 * 16 + (lane >> 4) * 8;
         const int row = ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8;
-        rt_ldm4t(bh, k_hi + row * PK + col);
-        rt_ldm4t(bl, k_lo + row * PK + col);
+        mp_ldm4t(bh, k_hi + row * PK + col);
+        mp_ldm4t(bl, k_lo + row * PK + col);
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
-          rt_mma(acc[m][2 * n2], ah[m], bh[0], bh[1]);
-          rt_mma(acc[m][2 * n2 + 1], ah[m], bh[2], bh[3]);
-          rt_mma(acc[m][2 * n2], ah[m], bl[0], bl[1]);
-          rt_mma(acc[m][2 * n2 + 1], ah[m], bl[2], bl[3]);
-          rt_mma(acc[m][2 * n2], al[m], bh[0], bh[1]);
-          rt_mma(acc[m][2 * n2 + 1], al[m], bh[2], bh[3]);
+          mp_mma(acc[m][2 * n2], ah[m], bh[0], bh[1]);
+          mp_mma(acc[m][2 * n2 + 1], ah[m], bh[2], bh[3]);
+          mp_mma(acc[m][2 * n2], ah[m], bl[0], bl[1]);
+          mp_mma(acc[m][2 * n2 + 1], ah[m], bl[2], bl[3]);
+          mp_mma(acc[m][2 * n2], al[m], bh[0], bh[1]);
+          mp_mma(acc[m][2 * n2 + 1], al[m], bh[2], bh[3]);
         }
       }
     }
@@ -447,7 +417,7 @@ retention_carry_kernel(RtArgs a, float* __restrict__ state, const int* __restric
       if (c + u >= ch1) continue;
       const float w = pw[a.chunk_starts[c + u + 1] - a.chunk_starts[c + u]];
       if constexpr (V == 4) {
-        rt_put4(a.s_hi + o + (size_t)u * step16, a.s_lo + o + (size_t)u * step16, S);
+        mp_put4(a.s_hi + o + (size_t)u * step16, a.s_lo + o + (size_t)u * step16, S);
       } else {
         const __nv_bfloat16 hi = __float2bfloat16_rn(S[0]);
         a.s_hi[o + (size_t)u * step16] = hi;
@@ -464,14 +434,6 @@ retention_carry_kernel(RtArgs a, float* __restrict__ state, const int* __restric
 }
 
 // ---------------------------------------------------------------- outputs
-
-__device__ __forceinline__ void rt_cp16(void* dst, const void* src, bool on) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(rt_smem(dst)), "l"(src), "r"(on ? 16 : 0) : "memory");
-}
-__device__ __forceinline__ void rt_cp_wait() {
-  asm volatile("cp.async.commit_group;" ::: "memory");
-  asm volatile("cp.async.wait_group 0;" ::: "memory");
-}
 
 // Block (tile, head, value slice), eight warps: four groups of 16 tokens by two halves of the slice's value columns (both
 // halves work the scores out for themselves).  Keys, values and the entering state come in two parts as the kernels
@@ -506,8 +468,8 @@ retention_outputs_kernel(RtArgs a) {
       const int v = i / pieces, c = (i - v * pieces) * 8;
       const bool on = j0 + v < a.dv;
       const size_t src = (base + (on ? j0 + v : 0)) * a.dkp + c;
-      rt_cp16(s_hi + v * PQ + c, a.s_hi + src, on);
-      rt_cp16(s_lo + v * PQ + c, a.s_lo + src, on);
+      mp_cp16(s_hi + v * PQ + c, a.s_hi + src, on);
+      mp_cp16(s_lo + v * PQ + c, a.s_lo + src, on);
     }
   }
   for (int i0 = 0; i0 < RT_TILE * quads; i0 += 1024) {      // (RT_TILE * quads is a multiple of 256)
@@ -522,7 +484,7 @@ retention_outputs_kernel(RtArgs a) {
 #pragma unroll
     for (int u = 0; u < 4; ++u) {
       const int i = i0 + u * 256 + tid, r = i / quads, c = (i % quads) * 4;
-      if (i < RT_TILE * quads) rt_put4(q_hi + r * PQ + c, q_lo + r * PQ + c, y[u]);
+      if (i < RT_TILE * quads) mp_put4(q_hi + r * PQ + c, q_lo + r * PQ + c, y[u]);
     }
   }
   constexpr int NT = DVT / 16;                     // n8 tiles of a warp
@@ -532,26 +494,27 @@ retention_outputs_kernel(RtArgs a) {
   for (int n = 0; n < NT; ++n)
 #pragma unroll
     for (int e = 0; e < 4; ++e) o[n][e] = 0.f;
-  rt_cp_wait();
+  mp_cp_commit();
+  mp_cp_wait();
   __syncthreads();
   // ---- what the state that enters the chunk gives
   for (int kk = 0; kk < a.dkp; kk += 16) {
     uint32_t ah[4], al[4];
     const int qa = (rg * 16 + (lane & 15)) * PQ + kk + (lane >> 4) * 8;
-    rt_ldm4(ah, q_hi + qa);
-    rt_ldm4(al, q_lo + qa);
+    mp_ldm4(ah, q_hi + qa);
+    mp_ldm4(al, q_lo + qa);
 #pragma unroll
     for (int n2 = 0; n2 < NT / 2; ++n2) {
       uint32_t bh[4], bl[4];
       const int sa = (n0 + n2 * 16 + (lane & 7) + (lane >> 4) * 8) * PQ + kk + ((lane >> 3) & 1) * 8;
-      rt_ldm4(bh, s_hi + sa);
-      rt_ldm4(bl, s_lo + sa);
-      rt_mma(o[2 * n2], ah, bh[0], bh[1]);
-      rt_mma(o[2 * n2 + 1], ah, bh[2], bh[3]);
-      rt_mma(o[2 * n2], ah, bl[0], bl[1]);
-      rt_mma(o[2 * n2 + 1], ah, bl[2], bl[3]);
-      rt_mma(o[2 * n2], al, bh[0], bh[1]);
-      rt_mma(o[2 * n2 + 1], al, bh[2], bh[3]);
+      mp_ldm4(bh, s_hi + sa);
+      mp_ldm4(bl, s_lo + sa);
+      mp_mma(o[2 * n2], ah, bh[0], bh[1]);
+      mp_mma(o[2 * n2 + 1], ah, bh[2], bh[3]);
+      mp_mma(o[2 * n2], ah, bl[0], bl[1]);
+      mp_mma(o[2 * n2 + 1], ah, bl[2], bl[3]);
+      mp_mma(o[2 * n2], al, bh[0], bh[1]);
+      mp_mma(o[2 * n2 + 1], al, bh[2], bh[3]);
     }
   }
   const int lr0 = rg * 16 + g, lr1 = lr0 + 8;      // this lane's rows of the tile
@@ -570,17 +533,18 @@ retention_outputs_kernel(RtArgs a) {
       const int r = i / pieces, c = (i - r * pieces) * 8;
       const bool on = r < krows;
       const size_t src = ((size_t)(krow0 + (on ? r : 0)) * a.heads + h) * a.dkp + c;
-      rt_cp16(k_hi + r * PQ + c, a.k_hi + src, on);
-      rt_cp16(k_lo + r * PQ + c, a.k_lo + src, on);
+      mp_cp16(k_hi + r * PQ + c, a.k_hi + src, on);
+      mp_cp16(k_lo + r * PQ + c, a.k_lo + src, on);
     }
     for (int i = tid; i < RT_TILE * (DVT / 8); i += 256) {
       const int r = i / (DVT / 8), c = (i - r * (DVT / 8)) * 8;
       const bool on = r < krows && j0 + c < a.dvp;
       const size_t src = ((size_t)(krow0 + (on ? r : 0)) * a.heads + h) * a.dvp + (on ? j0 + c : 0);
-      rt_cp16(v_hi + r * PV + c, a.v_hi + src, on);
-      rt_cp16(v_lo + r * PV + c, a.v_lo + src, on);
+      mp_cp16(v_hi + r * PV + c, a.v_hi + src, on);
+      mp_cp16(v_lo + r * PV + c, a.v_lo + src, on);
     }
-    rt_cp_wait();
+    mp_cp_commit();
+    mp_cp_wait();
     __syncthreads();
     const int groups = own ? rg + 1 : RT_TILE / 16;        // groups of 16 keys that this warp's tokens see
     float s[RT_TILE / 8][4];
@@ -591,21 +555,21 @@ retention_outputs_kernel(RtArgs a) {
     for (int kk = 0; kk < a.dkp; kk += 16) {
       uint32_t ah[4], al[4];
       const int qa = (rg * 16 + (lane & 15)) * PQ + kk + (lane >> 4) * 8;
-      rt_ldm4(ah, q_hi + qa);
-      rt_ldm4(al, q_lo + qa);
+      mp_ldm4(ah, q_hi + qa);
+      mp_ldm4(al, q_lo + qa);
 #pragma unroll
       for (int n2 = 0; n2 < RT_TILE / 16; ++n2) {
         if (n2 >= groups) continue;
         uint32_t bh[4], bl[4];
         const int ka = (n2 * 16 + (lane & 7) + (lane >> 4) * 8) * PQ + kk + ((lane >> 3) & 1) * 8;
-        rt_ldm4(bh, k_hi + ka);
-        rt_ldm4(bl, k_lo + ka);
-        rt_mma(s[2 * n2], ah, bh[0], bh[1]);
-        rt_mma(s[2 * n2 + 1], ah, bh[2], bh[3]);
-        rt_mma(s[2 * n2], ah, bl[0], bl[1]);
-        rt_mma(s[2 * n2 + 1], ah, bl[2], bl[3]);
-        rt_mma(s[2 * n2], al, bh[0], bh[1]);
-        rt_mma(s[2 * n2 + 1], al, bh[2], bh[3]);
+        mp_ldm4(bh, k_hi + ka);
+        mp_ldm4(bl, k_lo + ka);
+        mp_mma(s[2 * n2], ah, bh[0], bh[1]);
+        mp_mma(s[2 * n2 + 1], ah, bh[2], bh[3]);
+        mp_mma(s[2 * n2], ah, bl[0], bl[1]);
+        mp_mma(s[2 * n2 + 1], ah, bl[2], bl[3]);
+        mp_mma(s[2 * n2], al, bh[0], bh[1]);
+        mp_mma(s[2 * n2 + 1], al, bh[2], bh[3]);
       }
     }
     // the weights decay^(t - s); keys behind the token get none
@@ -622,22 +586,22 @@ retention_outputs_kernel(RtArgs a) {
     for (int ks = 0; ks < RT_TILE / 16; ++ks) {
       if (ks >= groups) continue;
       uint32_t ph[4], pl[4];
-      rt_split2(s[2 * ks][0], s[2 * ks][1], ph[0], pl[0]);
-      rt_split2(s[2 * ks][2], s[2 * ks][3], ph[1], pl[1]);
-      rt_split2(s[2 * ks + 1][0], s[2 * ks + 1][1], ph[2], pl[2]);
-      rt_split2(s[2 * ks + 1][2], s[2 * ks + 1][3], ph[3], pl[3]);
+      mp_split2(s[2 * ks][0], s[2 * ks][1], ph[0], pl[0]);
+      mp_split2(s[2 * ks][2], s[2 * ks][3], ph[1], pl[1]);
+      mp_split2(s[2 * ks + 1][0], s[2 * ks + 1][1], ph[2], pl[2]);
+      mp_split2(s[2 * ks + 1][2], s[2 * ks + 1][3], ph[3], pl[3]);
 #pragma unroll
       for (int n2 = 0; n2 < NT / 2; ++n2) {
         uint32_t bh[4], bl[4];
         const int va = (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PV + n0 + n2 * 16 + (lane >> 4) * 8;
-        rt_ldm4t(bh, v_hi + va);
-        rt_ldm4t(bl, v_lo + va);
-        rt_mma(o[2 * n2], ph, bh[0], bh[1]);
-        rt_mma(o[2 * n2 + 1], ph, bh[2], bh[3]);
-        rt_mma(o[2 * n2], ph, bl[0], bl[1]);
-        rt_mma(o[2 * n2 + 1], ph, bl[2], bl[3]);
-        rt_mma(o[2 * n2], pl, bh[0], bh[1]);
-        rt_mma(o[2 * n2 + 1], pl, bh[2], bh[3]);
+        mp_ldm4t(bh, v_hi + va);
+        mp_ldm4t(bl, v_lo + va);
+        mp_mma(o[2 * n2], ph, bh[0], bh[1]);
+        mp_mma(o[2 * n2 + 1], ph, bh[2], bh[3]);
+        mp_mma(o[2 * n2], ph, bl[0], bl[1]);
+        mp_mma(o[2 * n2 + 1], ph, bl[2], bl[3]);
+        mp_mma(o[2 * n2], pl, bh[0], bh[1]);
+        mp_mma(o[2 * n2 + 1], pl, bh[2], bh[3]);
       }
     }
   }

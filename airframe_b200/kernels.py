@@ -1886,12 +1886,14 @@ def diff_join(y, ctx, gate, H: int, G: int, dv: int, pv: int, lam: float, eps: f
 
 
 def delta_conv(out, proj, offsets, taps_w, history, batch, key_heads: int, heads: int, dk: int, dv: int, key_eps: float,
-               query_scale: float) -> None:
+               query_scale: float, low=None, low_sections=None) -> None:
     """From float32 projection rows with the sections q, k (``key_heads`` heads of dk), v (``heads`` of dv) and b (a logit
     per head) at ``offsets``: silu of a causal convolution over time on every channel of q, k and v (``taps_w`` float32
     [taps, C], C = 2 key_heads dk + heads dv, the last tap on the token itself; inputs before the step from ``history``
     float32 [slots, taps - 1, C], which is left holding each sequence's last inputs), q and k heads over
-    sqrt(sum of squares + key_eps), q times ``query_scale``; and sigmoid(b): out float32 [T, C + heads] = [q | k | v | beta]."""
+    sqrt(sum of squares + key_eps), q times ``query_scale``; and sigmoid(b): out float32 [T, C + heads] = [q | k | v | beta].
+    ``low`` (bfloat16 [T, n]) with ``low_sections`` = ((offset, rank, column), (offset, rank, column)): two more sections of
+    the projection rows, rounded, at these columns."""
     T = proj.shape[0]
     C = 2 * key_heads * dk + heads * dv
     taps = taps_w.shape[0]
@@ -1903,6 +1905,13 @@ def delta_conv(out, proj, offsets, taps_w, history, batch, key_heads: int, heads
     ends = [o + n for o, n in zip(offsets, (key_heads * dk, key_heads * dk, heads * dv, heads))]
     if len(offsets) != 4 or max(ends) > proj.shape[1] or min(offsets) < 0:
         raise KernelError("delta_conv: a section lies outside the projection row")
+    low_args = (c_void_p(0), c_int(0), c_int(0), c_int(0), c_int(0), c_int(0), c_int(0))
+    if low is not None:
+        (o0, r0, at0), (o1, r1, at1) = low_sections
+        if low.dtype != torch.bfloat16 or low.shape[0] != T or at0 != 0 or max(o0 + r0, o1 + r1) > proj.shape[1] \
+                or at1 + r1 > low.shape[1] or at1 < r0:
+            raise KernelError("delta_conv: low-rank rows bfloat16 [T, n], their sections inside the projection row")
+        low_args = (_ptr(low), c_int(o0), c_int(o1), c_int(r0), c_int(r1), c_int(at1), c_int(_rows(low, "low")))
     op, pp = _f32_rows(out, "out"), _f32_rows(proj, "proj")
     i32 = torch.int32
     _check(_lib().af_delta_conv(
@@ -1910,7 +1919,59 @@ def delta_conv(out, proj, offsets, taps_w, history, batch, key_heads: int, heads
         _ptr(history if taps > 1 else None, "history", torch.float32, allow_none=True),
         _ptr(batch.positions, "positions", i32), _ptr(batch.seq_of_token, "seq_of_token", i32), _ptr(batch.slots, "slots", i32),
         _ptr(batch.seq_starts, "seq_starts", i32), c_int(T), c_int(batch.n_seqs), c_int(taps), c_int(key_heads), c_int(heads),
-        c_int(dk), c_int(dv), c_float(key_eps), c_float(query_scale), _stream()))
+        c_int(dk), c_int(dv), c_float(key_eps), c_float(query_scale), *low_args, _stream()))
+
+
+def delta_prompt_supported(dk: int, dv: int) -> bool:
+    """Whether :func:`delta_prompt` takes heads of these sizes."""
+    return bool(_lib().af_delta_prompt_supported(c_int(dk), c_int(dv)))
+
+
+def _delta_chunks(batch):
+    """The chunks of a prefill step's sequences (made on the host once a step, kept in ``batch.aux``): device tensors
+    chunk_starts [n_chunks + 1] and seq_first_chunk [n_seqs + 1], and how many chunks there are."""
+    if "delta_chunks" not in batch.aux:
+        chunk = int(_lib().af_delta_prompt_chunk())
+        starts, first, row = [], [0], 0
+        for n in batch.seq_lens:
+            starts.extend(range(row, row + n, chunk))
+            row += n
+            first.append(len(starts))
+        starts.append(row)
+        host = torch.tensor(starts + first, dtype=torch.int32).pin_memory()
+        dev = host.to(batch.tokens.device, non_blocking=True)
+        transfers.count_h2d(host)
+        batch.aux["delta_chunks"] = (dev[:len(starts)], dev[len(starts):], len(starts) - 1)
+    return batch.aux["delta_chunks"]
+
+
+def delta_prompt(out, q, k, v, beta, z, dt_bias, rate, state, batch, heads: int, dk: int, dv: int) -> None:
+    """:func:`state_scan`'s rule ``gated`` for a prefill step on the tensor cores, the sequences cut into chunks, with the
+    decays exp(-rate softplus(z + dt_bias)) worked out from their logits ``z`` float32 [T, heads * dk]: q, k, v float32
+    sections of one row, out float32 [T, heads * dv].  32-bit sums; the operands are pairs of bfloat16."""
+    T = out.shape[0]
+    key_heads = q.shape[1] // dk
+    if tuple(q.shape) != (T, key_heads * dk) or q.shape != k.shape or tuple(v.shape) != (T, heads * dv) or heads % key_heads \
+            or not (q.stride(0) == k.stride(0) == v.stride(0)) or tuple(beta.shape) != (T, heads) or tuple(z.shape) != (T, heads * dk):
+        raise KernelError(f"delta_prompt: q, k [{T}, G * {dk}] and v [{T}, {heads * dv}] of one row stride, beta [{T}, {heads}], "
+                          f"z [{T}, {heads * dk}]")
+    if tuple(out.shape) != (T, heads * dv) or not out.is_contiguous() or out.dtype != torch.float32 or state.dtype != torch.float32 \
+            or tuple(state.shape[1:]) != (heads, dv, dk) or not state.is_contiguous() or dt_bias.numel() != heads * dk \
+            or rate.numel() != heads * dk:
+        raise KernelError(f"delta_prompt: out contiguous float32 [{T}, {heads * dv}], state float32 [slots, {heads}, {dv}, {dk}]")
+    starts, first, n = _delta_chunks(batch)
+    dev, f32, i32 = out.device, torch.float32, torch.int32
+    chunk = int(_lib().af_delta_prompt_chunk())
+    ops = torch.empty(n * heads * 6 * chunk * dk, dtype=torch.bfloat16, device=dev)
+    b = torch.empty(n * heads * 2 * chunk * chunk, dtype=torch.bfloat16, device=dev)
+    u0 = torch.empty(n * heads * chunk * dv, dtype=f32, device=dev)
+    p_end = torch.empty(n * heads * dk, dtype=f32, device=dev)
+    (qp, ts), (kp, _), (vp, _) = _f32_rows(q, "q"), _f32_rows(k, "k"), _f32_rows(v, "v")
+    _check(_lib().af_delta_prompt(
+        _ptr(out), qp, kp, vp, ts, *_f32_rows(beta, "beta"), *_f32_rows(z, "z"), _ptr(dt_bias, "dt_bias", f32),
+        _ptr(rate, "rate", f32), _ptr(state), _ptr(ops), _ptr(b), _ptr(u0), _ptr(p_end), _ptr(starts, "chunk_starts", i32),
+        _ptr(first, "seq_first_chunk", i32), _ptr(batch.slots, "slots", i32), c_int(n), c_int(batch.n_seqs), c_int(key_heads),
+        c_int(heads), c_int(dk), c_int(dv), _stream()))
 
 
 __all__ = [n for n in dir() if not n.startswith("_")]

@@ -585,6 +585,9 @@ class ChannelDelta(_StateMixer):
         self.conv_w = torch.cat([weights[nm[n + "_conv"]] for n in ("q", "k", "v")]).to(f32).t().contiguous()   # [taps, channels]
         self.a2t = weights[nm["a2"]].to(f32).t().contiguous()            # [rank, channels]: channels side by side
         self.g2t = weights[nm["g2"]].to(f32).t().contiguous()
+        self.a2_16 = self.g2_16 = None
+        if self.ctx.compute_dtype == torch.bfloat16 and self.ranks["a"] % 8 == 0 and self.ranks["g"] % 8 == 0:
+            self.a2_16, self.g2_16 = (weights[nm[n]].to(torch.bfloat16).contiguous() for n in ("a2", "g2"))
         self.dt_bias = weights[nm["dt_bias"]].to(f32).contiguous()
         # exp(A_log), once, from the stored values (worked out in 64 bits, kept in 32), for every channel of its head
         self.rate = torch.exp(weights[nm["A_log"]].to(torch.float64)).to(f32).repeat_interleave(self.dk).contiguous()
@@ -606,15 +609,41 @@ class ChannelDelta(_StateMixer):
         proj = linear(x, self.w_in, out_dtype=f32)
         # [q | k | v | beta], rows of whole 16-byte pieces
         mixed = torch.empty(T, (self.channels + H + 3) // 4 * 4, dtype=f32, device=x.device)[:, : self.channels + H]
+        q, k, v = mixed[:, :nk], mixed[:, nk: 2 * nk], mixed[:, 2 * nk: self.channels]
+        beta = mixed[:, self.channels:]
+        chunked = self._on_tensor_cores(x, batch)
+        ra, rg = self.ranks["a"], self.ranks["g"]
+        low = None
+        if self.a2_16 is not None and T >= self.LOW_TC_ROWS:      # the low-rank factors' second products on the tensor cores
+            low = torch.empty(T, (ra + 7) // 8 * 8 + rg, dtype=x.dtype, device=x.device)
         kernels.delta_conv(mixed, proj, [off[n] for n in ("q", "k", "v", "b")], self.conv_w, history, batch, self.key_heads, H,
-                           self.dk, self.dv, self.key_eps, self.query_scale)
-        decay = torch.empty(T, H * self.dk, dtype=f32, device=x.device)
-        kernels.channel_decay(decay, proj, off["a1"], self.a2t, self.dt_bias, kind="softplus", rate=self.rate)
-        gate = torch.empty(T, nv, dtype=f32, device=x.device)
-        kernels.channel_decay(gate, proj, off["g1"], self.g2t, None, kind="logit")
+                           self.dk, self.dv, self.key_eps, self.query_scale, low=low,
+                           low_sections=((off["a1"], ra, 0), (off["g1"], rg, (ra + 7) // 8 * 8)))
+        if low is not None:
+            gate = linear(low[:, (ra + 7) // 8 * 8:], self.g2_16, out_dtype=f32)
+        else:
+            gate = torch.empty(T, nv, dtype=f32, device=x.device)
+            kernels.channel_decay(gate, proj, off["g1"], self.g2t, None, kind="logit")
         o = torch.empty(T, nv, dtype=f32, device=x.device)
-        kernels.state_scan("gated", o, mixed[:, :nk], mixed[:, nk: 2 * nk], mixed[:, 2 * nk: self.channels], state, batch, H,
-                           self.dk, self.dv, w=decay, beta=mixed[:, self.channels:])
+        if chunked:
+            if low is not None:
+                z = linear(low[:, :ra], self.a2_16, out_dtype=f32)
+            else:
+                z = torch.empty(T, H * self.dk, dtype=f32, device=x.device)
+                kernels.channel_decay(z, proj, off["a1"], self.a2t, None, kind="logit")
+            kernels.delta_prompt(o, q, k, v, beta, z, self.dt_bias, self.rate, state, batch, H, self.dk, self.dv)
+        else:
+            decay = torch.empty(T, H * self.dk, dtype=f32, device=x.device)
+            kernels.channel_decay(decay, proj, off["a1"], self.a2t, self.dt_bias, kind="softplus", rate=self.rate)
+            kernels.state_scan("gated", o, q, k, v, state, batch, H, self.dk, self.dv, w=decay, beta=beta)
         y = torch.empty(T, nv, dtype=x.dtype, device=x.device)
         kernels.gated_group_norm(y, o, self.norm_w, gate, self.dv, self.eps)
         return linear_split(y, self.w_o, wide=self.wide)
+
+    LOW_TC_ROWS = 64           # from so many rows on the low-rank second products go to the tensor cores
+    CHUNKED_FROM = 64          # tokens of the longest prompt of a step that is cut into chunks on the tensor cores
+
+    def _on_tensor_cores(self, x, batch) -> bool:
+        """A bfloat16 prompt that is worth cutting into chunks, with heads of sizes those kernels take."""
+        return (x.dtype == torch.bfloat16 and batch.is_prefill and batch.max_len >= self.CHUNKED_FROM
+                and kernels.delta_prompt_supported(self.dk, self.dv))

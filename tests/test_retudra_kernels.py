@@ -253,6 +253,87 @@ def test_delta_rule_token_by_token(K, G, H, dk, dv):
     assert float(state[1].abs().max()) == 0.0
 
 
+def _chunked_run(K, parts, picks, batch, state, H, dk, dv, G):
+    """:func:`kernels.delta_prompt` on rows whose logits give the parts' decays (rate 1, softplus inverted)."""
+    rows = [torch.cat([p[i][s].flatten(1) for p, s in zip(parts, picks)]) for i in range(5)]
+    q, k, v, w, beta = rows
+    lg = -torch.log(w.double().clamp_min(1e-30))                          # softplus(z + bias) is to be this
+    z = torch.where(lg > 30.0, lg, torch.log(torch.expm1(lg.clamp(1e-9, 60.0)))).float()
+    bias = torch.linspace(-1.0, 1.0, H * dk)
+    mixed = torch.cat([q, k, v, beta, torch.zeros(q.shape[0], (-(q.shape[1] * 2 + v.shape[1] + H)) % 4)], 1).to(DEV)
+    n = q.shape[1]
+    out = torch.full((q.shape[0], H * dv), float("nan"), device=DEV)
+    K.delta_prompt(out, mixed[:, :n], mixed[:, n: 2 * n], mixed[:, 2 * n: 2 * n + H * dv], mixed[:, 2 * n + H * dv: 2 * n + H * dv + H],
+                   (z - bias).to(DEV).contiguous(), bias.to(DEV), torch.ones(H * dk, device=DEV), state, batch, H, dk, dv)
+    return out
+
+
+CHUNK_SHAPES = [(1, 3, 64, 64), (2, 2, 128, 128), (1, 2, 192, 96), (1, 2, 32, 208), (1, 1, 256, 64), (3, 3, 16, 16), (1, 4, 112, 48), (2, 2, 240, 80)]
+
+
+@pytest.mark.parametrize("G,H,dk,dv", CHUNK_SHAPES)
+@pytest.mark.parametrize("keep", [None, 1.0, 0.99])
+def test_delta_rule_in_chunks(K, G, H, dk, dv, keep):
+    """Prompts of one token, of a group and a token, of a chunk and a token, of whole chunks and of many; decays from nothing to
+    everything, none at all, and slow ones; then single tokens from the states the chunks left; slots in any order."""
+    assert K.delta_prompt_supported(dk, dv) and not K.delta_prompt_supported(dk + 1, dv) and not K.delta_prompt_supported(dk, dv + 8)
+    lens, tail = [1, 17, 33, 64, 230, 16, 31], 3
+    full = [n + tail for n in lens]
+    parts = [delta_inputs(n, G, H, dk, dv, 5 * n + dk, keep) for n in full]
+    refs = [ref_scan(*p) for p in parts]
+    slots = [6, 2, 0, 5, 1, 7, 3]
+    state = torch.zeros(8, H, dv, dk, device=DEV)
+    out = _chunked_run(K, parts, [slice(0, n) for n in lens], batch_of(lens, slots), state, H, dk, dv, G)
+    row = 0
+    for n, r in zip(lens, refs):
+        close(out[row: row + n], r[:n].flatten(1), 2e-4, n)
+        row += n
+    assert float(state[4].abs().max()) == 0.0
+    for j in range(tail):
+        rows = [torch.cat([p[i][n + j: n + j + 1].flatten(1) for p, n in zip(parts, lens)]).to(DEV).contiguous() for i in range(5)]
+        step = torch.empty(len(lens), H * dv, device=DEV)
+        K.state_scan("gated", step, rows[0], rows[1], rows[2], state, batch_of([1] * len(lens), slots, [n + j for n in lens]), H, dk, dv,
+                     w=rows[3], beta=rows[4])
+        close(step, torch.cat([r[n + j: n + j + 1].flatten(1) for r, n in zip(refs, lens)]), 2e-4, j)
+
+
+def test_a_prompt_in_two_steps_of_chunks(K):
+    """The second step goes on from the states the first one left (both in chunks that end inside a group)."""
+    G, H, dk, dv = 1, 2, 64, 64
+    p = delta_inputs(150, G, H, dk, dv, 3)
+    ref = ref_scan(*p).flatten(1)
+    state = torch.zeros(3, H, dv, dk, device=DEV)
+    a = _chunked_run(K, [p], [slice(0, 83)], batch_of([83], [1]), state, H, dk, dv, G)
+    b = _chunked_run(K, [p], [slice(83, 150)], batch_of([67], [1]), state, H, dk, dv, G)
+    close(torch.cat([a, b]), ref, 2e-4)
+
+
+@pytest.mark.parametrize("back", [1, 5, 15, 16, 17, 31, 32, 33, 48, 64, 200])
+def test_one_key_stands_out_in_chunks(K, back):
+    """A query asks for one earlier key (orthogonal to all others) ``back`` tokens on: its value comes out, decayed by every
+    channel's product in between, and the query right before the key sees nothing of it."""
+    G, H, dk, dv, T = 1, 1, 64, 32, 260
+    g = torch.Generator().manual_seed(back)
+    at = 230 - back
+    k = torch.zeros(T, G, dk)
+    k[:, :, :32] = torch.randn(T, G, 32, generator=g)
+    q = plain.unit(k.double()).float()
+    k = q.clone()
+    k[at] = 0.0
+    k[at, 0, 40:44] = 0.5                                    # a unit key in channels that nobody else uses
+    q[230, 0], q[at - 1, 0] = k[at, 0], k[at, 0]
+    v = torch.randn(T, H, dv, generator=g)
+    w = torch.full((T, H, dk), 0.995)
+    w[:, 0, 41] = 0.98
+    beta = torch.rand(T, H, generator=g)
+    beta[at] = 1.0
+    state = torch.zeros(1, H, dv, dk, device=DEV)
+    out = _chunked_run(K, [(q, k, v, w, beta)], [slice(0, T)], batch_of([T], [0]), state, H, dk, dv, G).cpu().double()
+    want = v[at, 0].double() * (3 * 0.25 * 0.995 ** back + 0.25 * 0.98 ** back)
+    assert float((out[230] - want).abs().max()) < 2e-4 and float(out[at - 1].abs().max()) < 1e-5
+    close(out, ref_scan(q, k, v, w, beta).flatten(1), 2e-4)
+
+
 # ---------------------------------------------------------------- experts
 
 @pytest.mark.parametrize("E,ident,top,groups,keep", [(7, 2, 3, 3, 2), (6, 2, 4, 2, 1), (3, 5, 4, 2, 2), (5, 0, 5, 1, 1), (1, 4, 2, 1, 1), (40, 8, 6, 8, 3)])
