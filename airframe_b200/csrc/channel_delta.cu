@@ -20,6 +20,7 @@
 // is the product g_(s+1) ... g_t itself, taken along a chain within 16 tokens, and across two groups of 16 tokens as the
 // product from s to its group's end times the product from the next group's start to t.
 #include "mma_pairs.cuh"
+#include "tma.cuh"
 
 namespace {
 
@@ -181,14 +182,14 @@ struct DeltaPromptArgs {
   const float *q, *k, *v, *beta, *z;   // rows of the step: unit queries and keys (G heads), values, step sizes, decays' logits
   long long qkv_ts, beta_ts, z_ts;
   const float *dt_bias, *rate;         // [H * dk]: decay = exp(-rate softplus(z + dt_bias))
-  __nv_bfloat16* ops;                  // [chunks * H][6][DP_C][dk]: W, Q . P, K . P_end / P, each hi then lo
-  __nv_bfloat16* b;                    // [chunks * H][2][DP_C][DP_C]: B, hi then lo
-  float* u0;                           // [chunks * H][DP_C][dv]
-  float* p_end;                        // [chunks * H][dk]
+  __nv_bfloat16* blob;                 // [chunks * H][dp_blob(dk).size]: what the second kernel needs of a chunk and head
+  float* u0;                           // [chunks * H][tiles of `tile` value columns][DP_C][tile + 4]
+  int tile;
   float* state;                        // [slots][H][dv][dk]
   float* out;                          // [tokens][H * dv]
   const int *chunk_starts, *seq_first_chunk, *slots;
   int G, H, dk, dv;
+  int* err;                            // set to 1 when a bounded wait ran out
 };
 
 __device__ __forceinline__ void dp_put(__nv_bfloat16* hi, __nv_bfloat16* lo, float y) {
@@ -197,24 +198,57 @@ __device__ __forceinline__ void dp_put(__nv_bfloat16* hi, __nv_bfloat16* lo, flo
   *lo = __float2bfloat16_rn(y - __bfloat162float(h));
 }
 
-size_t dp_prep_smem(int dk) { return ((size_t)(3 * DP_C + 3 * 16) * (dk + 4) + 2 * DP_C * 36 + DP_C) * sizeof(float); }
+// Where the pieces of a chunk lie, in global memory as in the walking kernel's shared memory (elements of bfloat16; rows of
+// dk + 8): W, Q . P, K . P_end / P (each hi then lo), B (hi, lo; rows of 40), P_end (floats).  A tile of U0 (floats, rows of
+// N + 4) follows in a stage.
+constexpr int DP_PB = DP_C + 8;
+struct DpBlob {
+  int pk, b, p_end, size;
+};
+__host__ __device__ inline DpBlob dp_blob(int dk) {
+  DpBlob s;
+  s.pk = dk + 8;
+  s.b = 6 * DP_C * s.pk;
+  s.p_end = s.b + 2 * DP_C * DP_PB;
+  s.size = s.p_end + 2 * dk;
+  return s;
+}
+
+size_t dp_prep_smem(int dk) { return ((size_t)3 * DP_C * (dk + 4) + 2 * DP_C * 36 + DP_C) * sizeof(float); }
+
+// 32 sums over the warp's lanes at once: lane l ends with the sum of everybody's v[l].
+__device__ __forceinline__ float dp_sum32(float* v) {
+  const int lane = threadIdx.x & 31;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const bool up = lane & o;
+#pragma unroll
+    for (int i = 0; i < o; ++i) {
+      const float keep = up ? v[i + o] : v[i], give = up ? v[i] : v[i + o];
+      v[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+    }
+  }
+  return v[0];
+}
 
 // Block (chunk, head), 256 threads; NE = channels a lane holds (dk / 32 rounded up).
 template <int NE>
-__global__ void __launch_bounds__(256, 2)
+__global__ void __launch_bounds__(256, NE <= 4 ? 3 : 1)
 delta_chunk_kernel(DeltaPromptArgs a) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) float sm[];
   const int dk = a.dk, dv = a.dv, DP = dk + 4, quads = dk / 4;
   float *k_s = sm, *q_s = k_s + DP_C * DP, *g_s = q_s + DP_C * DP;
-  float *kp_s = g_s + DP_C * DP, *qp_s = kp_s + 16 * DP, *kx_s = qp_s + 16 * DP;   // second group times P, first group times what follows
-  float *A_s = kx_s + 16 * DP, *B_s = A_s + DP_C * 36, *beta_s = B_s + DP_C * 36;
+  float *A_s = g_s + DP_C * DP, *B_s = A_s + DP_C * 36, *beta_s = B_s + DP_C * 36;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int ch = blockIdx.x, h = blockIdx.y, hk = h / (a.H / a.G);
   const int first = a.chunk_starts[ch], rows = a.chunk_starts[ch + 1] - first;
   const size_t unit = (size_t)ch * a.H + h;
+  const DpBlob L = dp_blob(dk);
+  __nv_bfloat16* blob = a.blob + unit * L.size;
   pdl_wait();
   a.q = pdl_fresh(a.q), a.k = pdl_fresh(a.k), a.v = pdl_fresh(a.v), a.beta = pdl_fresh(a.beta), a.z = pdl_fresh(a.z);
+#pragma unroll 2
   for (int i = tid; i < DP_C * quads; i += 256) {
     const int r = i / quads, c = (i - r * quads) * 4;
     float4 kq = make_float4(0.f, 0.f, 0.f, 0.f), qq = kq, gq = make_float4(1.f, 1.f, 1.f, 1.f);
@@ -240,91 +274,120 @@ delta_chunk_kernel(DeltaPromptArgs a) {
 #pragma unroll 1
   for (int job = 0; job < 4; ++job) {
     const int base = (job >> 1) * 16, s = base + ((job & 1) ? 15 - warp : warp);
-    float p[NE];
+    float p[NE], v[32];
 #pragma unroll
     for (int e = 0; e < NE; ++e) p[e] = lane + 32 * e < dk ? k_s[s * DP + lane + 32 * e] : 0.f;
-    for (int t = s; t < base + 16; ++t) {
-      float ak = 0.f, aq = 0.f;
 #pragma unroll
-      for (int e = 0; e < NE; ++e) {
-        const int c = lane + 32 * e;
-        if (c >= dk) continue;
-        if (t > s) p[e] *= g_s[t * DP + c];
-        ak = fmaf(k_s[t * DP + c], p[e], ak);
-        aq = fmaf(q_s[t * DP + c], p[e], aq);
+    for (int d = 0; d < 16; ++d) {
+      float ak = 0.f, aq = 0.f;
+      if (s + d < base + 16) {
+        const int at = (s + d) * DP + lane;
+#pragma unroll
+        for (int e = 0; e < NE; ++e) {
+          if (lane + 32 * e >= dk) continue;
+          if (d > 0) p[e] *= g_s[at + 32 * e];
+          ak = fmaf(k_s[at + 32 * e], p[e], ak);
+          aq = fmaf(q_s[at + 32 * e], p[e], aq);
+        }
       }
-      ak = warp_sum(ak), aq = warp_sum(aq);
-      if (lane == 0) {
-        if (t > s) A_s[t * 36 + s] = ak * beta_s[t];
-        B_s[t * 36 + s] = aq;
-      }
+      v[2 * d] = ak, v[2 * d + 1] = aq;
+    }
+    const float sum = dp_sum32(v);
+    const int t = s + (lane >> 1);
+    if (t < base + 16) {
+      if (lane & 1) B_s[t * 36 + s] = sum;
+      else if (t > s) A_s[t * 36 + s] = sum * beta_s[t];
     }
   }
-  // ---- a thread a channel: running products; the scaled queries and keys go out
-  __nv_bfloat16* ops = a.ops + unit * 6 * DP_C * dk;
-  for (int c = tid; c < dk; c += 256) {
-    float P = 1.f, half = 1.f;
-#pragma unroll 4
-    for (int t = 0; t < DP_C; ++t) {
-      const float g = g_s[t * DP + c];
-      if (t == 16) half = P, P = 1.f;
-      P *= g;
-      const float q = q_s[t * DP + c];
-      if (t >= 16) kp_s[(t - 16) * DP + c] = k_s[t * DP + c] * P, qp_s[(t - 16) * DP + c] = q * P;
-      dp_put(ops + (2 * DP_C + t) * dk + c, ops + (3 * DP_C + t) * dk + c, q * (t >= 16 ? half * P : P));
+  __syncthreads();
+  // ---- a thread a channel: running products from the front (half the threads) and from the back; the scaled queries and
+  // keys go out.  Left in place behind it: k times P from its group's start; q of the second group likewise; in the first
+  // group's place of q the keys times what follows them in their group; in g's first row the first group's whole product.
+  for (int c0 = 0; c0 < dk; c0 += 128) {
+    const int c = c0 + (tid & 127);
+    const bool on = c < dk, front = tid < 128;
+    float r[DP_C], half = 1.f;
+    if (on && front) {
+      __nv_bfloat16* o = blob + 2 * DP_C * L.pk + c;
+      float P = 1.f;
+#pragma unroll
+      for (int t = 0; t < DP_C; ++t) {
+        if (t == 16) half = P, P = 1.f;
+        P *= g_s[t * DP + c];
+        r[t] = k_s[t * DP + c] * P;
+        float q = q_s[t * DP + c] * P;
+        if (t >= 16) {
+          q_s[t * DP + c] = q;
+          q *= half;
+        }
+        dp_put(o, o + DP_C * L.pk, q);
+        o += L.pk;
+      }
+      reinterpret_cast<float*>(blob + L.p_end)[c] = half * P;
+    } else if (on) {
+      __nv_bfloat16* o = blob + (4 * DP_C + DP_C - 1) * L.pk + c;
+      float x = 1.f, second = 1.f;
+#pragma unroll
+      for (int s = DP_C - 1; s >= 0; --s) {
+        if (s == 15) second = x, x = 1.f;
+        r[s] = k_s[s * DP + c] * x;
+        dp_put(o, o + DP_C * L.pk, s < 16 ? r[s] * second : r[s]);
+        o -= L.pk;
+        x *= g_s[s * DP + c];
+      }
     }
-    a.p_end[unit * dk + c] = half * P;
-    const float second = P;                                           // (the second group's whole product)
-    float x = 1.f;                                                    // the product behind token s, to its group's end
-#pragma unroll 4
-    for (int s = DP_C - 1; s >= 0; --s) {
-      if (s == 15) x = 1.f;
-      const float k = k_s[s * DP + c];
-      if (s < 16) kx_s[s * DP + c] = k * x;
-      dp_put(ops + (4 * DP_C + s) * dk + c, ops + (5 * DP_C + s) * dk + c, k * (s < 16 ? x * second : x));
-      x *= g_s[s * DP + c];
+    __syncthreads();
+    if (on && front) {
+#pragma unroll
+      for (int t = 0; t < DP_C; ++t) k_s[t * DP + c] = r[t];
+      g_s[c] = half;
+    } else if (on) {
+#pragma unroll
+      for (int s = 0; s < 16; ++s) q_s[s * DP + c] = r[s];
     }
   }
   __syncthreads();
   // ---- the second group's tokens against the first group's: a thread a pair
   {
-    const float* kr = kp_s + (tid >> 4) * DP;
-    const float* qr = qp_s + (tid >> 4) * DP;
-    const float* xr = kx_s + (tid & 15) * DP;
-    float ak = 0.f, aq = 0.f;
+    const int t = 16 + (tid >> 4), s = tid & 15;
+    const float *kr = k_s + t * DP, *qr = q_s + t * DP, *xr = q_s + s * DP;
+    float ak = 0.f, aq = 0.f, ak2 = 0.f, aq2 = 0.f;
     for (int c = 0; c < dk; c += 4) {
       const float4 x = *reinterpret_cast<const float4*>(xr + c), kk = *reinterpret_cast<const float4*>(kr + c),
                    qq = *reinterpret_cast<const float4*>(qr + c);
-      ak = fmaf(kk.x, x.x, fmaf(kk.y, x.y, fmaf(kk.z, x.z, fmaf(kk.w, x.w, ak))));
-      aq = fmaf(qq.x, x.x, fmaf(qq.y, x.y, fmaf(qq.z, x.z, fmaf(qq.w, x.w, aq))));
+      ak = fmaf(kk.x, x.x, fmaf(kk.y, x.y, ak)), ak2 = fmaf(kk.z, x.z, fmaf(kk.w, x.w, ak2));
+      aq = fmaf(qq.x, x.x, fmaf(qq.y, x.y, aq)), aq2 = fmaf(qq.z, x.z, fmaf(qq.w, x.w, aq2));
     }
-    const int t = 16 + (tid >> 4), s = tid & 15;
-    A_s[t * 36 + s] = ak * beta_s[t];
-    B_s[t * 36 + s] = aq;
+    A_s[t * 36 + s] = (ak + ak2) * beta_s[t];
+    B_s[t * 36 + s] = aq + aq2;
   }
   __syncthreads();
-  __nv_bfloat16* b = a.b + unit * 2 * DP_C * DP_C;
-  for (int i = tid; i < DP_C * DP_C; i += 256) dp_put(b + i, b + DP_C * DP_C + i, B_s[(i >> 5) * 36 + (i & 31)]);
+  for (int i = tid; i < DP_C * DP_C; i += 256) {
+    __nv_bfloat16* o = blob + L.b + (i >> 5) * DP_PB + (i & 31);
+    dp_put(o, o + DP_C * DP_PB, B_s[(i >> 5) * 36 + (i & 31)]);
+  }
   // ---- (I + A) X = diag(beta) [K . P | V]: a thread a column, from the first row down
   for (int col = tid; col < dk + dv; col += 256) {
     const bool is_w = col < dk;
-    float x[DP_C], P = 1.f;
-    const float* src = a.v + (size_t)first * a.qkv_ts + (size_t)h * dv + (is_w ? 0 : col - dk);
-    __nv_bfloat16* w = ops + col;
-    float* u = a.u0 + unit * DP_C * dv + (is_w ? 0 : col - dk);
-    const float *gr = g_s + col, *kr = k_s + col;
+    float x[DP_C];
+    if (is_w) {
+      const float half = g_s[col];
 #pragma unroll
-    for (int t = 0; t < DP_C; ++t) {
-      float acc = 0.f, acc2 = 0.f;
-      if (is_w) {
-        P *= *gr;
-        acc = *kr * P;
-        gr += DP, kr += DP;
-      } else if (t < rows) {
-        acc = *src;
+      for (int t = 0; t < DP_C; ++t) x[t] = k_s[t * DP + col] * (t < 16 ? 1.f : half);
+    } else {
+      const float* src = a.v + (size_t)first * a.qkv_ts + (size_t)h * dv + col - dk;
+#pragma unroll
+      for (int t = 0; t < DP_C; ++t) {
+        x[t] = t < rows ? *src : 0.f;
         src += a.qkv_ts;
       }
-      acc *= beta_s[t];
+    }
+    __nv_bfloat16* w = blob + col;
+    const int j = is_w ? 0 : col - dk, n = a.tile;
+    float* u = a.u0 + ((unit * ((dv + n - 1) / n) + j / n) * DP_C) * (n + 4) + j % n;
+#pragma unroll
+    for (int t = 0; t < DP_C; ++t) {
+      float acc = x[t] * beta_s[t], acc2 = 0.f;
 #pragma unroll
       for (int s = 0; s < t; s += 4) {
         const float4 q = *reinterpret_cast<const float4*>(A_s + t * 36 + s);      // (zero from the diagonal on)
@@ -335,34 +398,28 @@ delta_chunk_kernel(DeltaPromptArgs a) {
       }
       x[t] = acc + acc2;
       if (is_w) {
-        dp_put(w, w + (size_t)DP_C * dk, x[t]);
-        w += dk;
+        dp_put(w, w + DP_C * L.pk, x[t]);
+        w += L.pk;
       } else {
         *u = x[t];
-        u += dv;
+        u += n + 4;
       }
-      asm volatile("" ::: "memory");               // (a row's factors are read when it is their turn: all at once they would fill the registers)
+      // (the factors are read when it is their rows' turn: all at once they would fill the registers)
+      if ((t & 3) == 3) asm volatile("" ::: "memory");
     }
   }
 }
 
-constexpr int DP_PB = DP_C + 8;
-
-// Where the pieces of a chunk lie in a stage (elements of bfloat16; rows of dk + 8).
-struct DpStage {
-  int pk, b, u0, p_end, size;
-};
-__host__ __device__ inline DpStage dp_stage(int dk, int n) {
-  DpStage s;
-  s.pk = dk + 8;
-  s.b = 6 * DP_C * s.pk;
-  s.u0 = s.b + 2 * DP_C * DP_PB;
-  s.p_end = s.u0 + 2 * DP_C * (n + 4);
-  s.size = (s.p_end + 2 * dk + 7) / 8 * 8;
-  return s;
-}
+size_t dp_stage_bytes(int dk, int n) { return (size_t)dp_blob(dk).size * 2 + (size_t)DP_C * (n + 4) * 4; }
 size_t dp_walk_smem(int dk, int n, int stages) {
-  return ((size_t)stages * dp_stage(dk, n).size + 2 * (size_t)dk * (n + 8) + 2 * (size_t)DP_C * (n + 8)) * sizeof(__nv_bfloat16);
+  return stages * dp_stage_bytes(dk, n) + (2 * (size_t)dk * (n + 8) + 2 * (size_t)DP_C * (n + 8)) * sizeof(__nv_bfloat16);
+}
+
+// A contiguous piece from global to shared memory, counted by an mbarrier (16-byte aligned, a multiple of 16 bytes).
+__device__ __forceinline__ void dp_bulk(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(dst)),
+               "l"(src), "r"(bytes), "r"(smem_u32(bar))
+               : "memory");
 }
 
 // Block (N value columns, head, sequence), eight warps, walks the sequence's chunks with its columns of the state in registers
@@ -373,18 +430,28 @@ template <int N, int MT>
 __global__ void __launch_bounds__(256)
 delta_walk_kernel(DeltaPromptArgs a, int stages) {
   pdl_launch_dependents();
-  extern __shared__ __align__(16) __nv_bfloat16 raw[];
+  extern __shared__ __align__(16) unsigned char raw[];
+  __shared__ uint64_t full[2];
+  __shared__ int give_up_s;
+  volatile int* give_up = &give_up_s;
   constexpr int PN = N + 8, NT = N / 16;           // NT: n8 tiles of a U or O warp
   const int dk = a.dk, dv = a.dv;
-  const DpStage L = dp_stage(dk, N);
-  __nv_bfloat16* s_hi = raw + (size_t)stages * L.size;
+  const DpBlob L = dp_blob(dk);
+  const uint32_t blob_bytes = (uint32_t)L.size * 2, u0_bytes = DP_C * (N + 4) * 4;
+  __nv_bfloat16* s_hi = reinterpret_cast<__nv_bfloat16*>(raw + (size_t)stages * (blob_bytes + u0_bytes));
   __nv_bfloat16* s_lo = s_hi + dk * PN;
   __nv_bfloat16* u_hi = s_lo + dk * PN;
   __nv_bfloat16* u_lo = u_hi + DP_C * PN;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
-  const int h = blockIdx.y, b = blockIdx.z, j0 = blockIdx.x * N;
+  const int h = blockIdx.y, b = blockIdx.z, j0 = blockIdx.x * N, tiles = gridDim.x;
   const int slot = a.slots[b], ch0 = a.seq_first_chunk[b], ch1 = a.seq_first_chunk[b + 1];
   if (slot < 0 || ch0 >= ch1) return;
+  if (tid == 0) {
+    mbar_init(&full[0], 1);
+    mbar_init(&full[1], 1);
+    give_up_s = 0;
+    mbar_fence_init();
+  }
   float* st = a.state + ((size_t)slot * a.H + h) * dv * dk;
   float S[MT][N / 8][4];
 #pragma unroll
@@ -413,62 +480,63 @@ delta_walk_kernel(DeltaPromptArgs a, int stages) {
     }
   };
   put_state();
+  __syncthreads();                                 // (the barriers are set up)
   pdl_wait();
-  auto load = [&](int ch, int which) {
-    __nv_bfloat16* sg = raw + (size_t)which * L.size;
+  auto load = [&](int ch, int which) {             // (one thread)
+    unsigned char* sg = raw + (size_t)which * (blob_bytes + u0_bytes);
     const size_t unit = (size_t)ch * a.H + h;
-    const __nv_bfloat16* ops = a.ops + unit * 6 * DP_C * dk;
-    const int pieces = dk / 8;
-    for (int i = tid; i < 6 * DP_C * pieces; i += 256) {
-      const int r = i / pieces, c = (i - r * pieces) * 8;
-      mp_cp16(sg + r * L.pk + c, ops + (size_t)r * dk + c, true);
-    }
-    const __nv_bfloat16* bb = a.b + unit * 2 * DP_C * DP_C;
-    for (int i = tid; i < 2 * DP_C * 4; i += 256) mp_cp16(sg + L.b + (i >> 2) * DP_PB + (i & 3) * 8, bb + i * 8, true);
-    const float* uu = a.u0 + unit * DP_C * dv + j0;
-    float* us = reinterpret_cast<float*>(sg + L.u0);
-    for (int i = tid; i < DP_C * (N / 4); i += 256) {
-      const int r = i / (N / 4), c = (i - r * (N / 4)) * 4;
-      const bool on = j0 + c < dv;
-      mp_cp16(us + r * (N + 4) + c, uu + (on ? (size_t)r * dv + c : 0), on);
-    }
-    const float* pe = a.p_end + unit * dk;
-    for (int i = tid; i < dk / 4; i += 256) mp_cp16(reinterpret_cast<float*>(sg + L.p_end) + i * 4, pe + i * 4, true);
-    mp_cp_commit();
+    mbar_expect_tx(&full[which], blob_bytes + u0_bytes);
+    dp_bulk(sg, a.blob + unit * L.size, blob_bytes, &full[which]);
+    dp_bulk(sg + blob_bytes, a.u0 + (unit * tiles + blockIdx.x) * (DP_C * (N + 4)), u0_bytes, &full[which]);
   };
-  load(ch0, 0);
-  const int kind = warp >> 2, mt = (warp >> 1) & 1, n0 = (warp & 1) * (N / 2);
+  if (tid == 0) load(ch0, 0);
+  const int kind = warp >> 2, mt = (warp >> 1) & 1, nh = warp & 1, n0 = nh * (N / 2);
+  const int nb = N == 32 ? n0 : 0;                 // (narrow tiles: a load brings both warps' columns)
+  bool ok = true;
   for (int ch = ch0; ch < ch1; ++ch) {
-    const int which = stages == 2 ? (ch - ch0) & 1 : 0;
-    mp_cp_wait();
+    const int i = ch - ch0, which = stages == 2 ? i & 1 : 0;
+    mbar_wait(&full[which], (stages == 2 ? i >> 1 : i) & 1, give_up);
     __syncthreads();                               // (the chunk's pieces and the state are there; the other stage is free)
-    if (stages == 2 && ch + 1 < ch1) load(ch + 1, which ^ 1);
-    const __nv_bfloat16* sg = raw + (size_t)which * L.size;
+    if (*give_up) {
+      ok = false;
+      break;
+    }
+    if (stages == 2 && ch + 1 < ch1 && tid == 0) load(ch + 1, which ^ 1);
+    const __nv_bfloat16* sg = reinterpret_cast<const __nv_bfloat16*>(raw + (size_t)which * (blob_bytes + u0_bytes));
     const int first = a.chunk_starts[ch], rows = a.chunk_starts[ch + 1] - first;
-    // ---- W S, or (Q . P) S
-    float acc[NT][4];
+    // ---- W S, or (Q . P) S: the three products of a pair in chains of their own
+    float part[3][NT][4];
 #pragma unroll
-    for (int n = 0; n < NT; ++n)
+    for (int p = 0; p < 3; ++p)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) acc[n][e] = 0.f;
+      for (int n = 0; n < NT; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) part[p][n][e] = 0.f;
     const __nv_bfloat16* left = sg + (size_t)kind * 2 * DP_C * L.pk + (mt * 16 + (lane & 15)) * L.pk + (lane >> 4) * 8;
-#pragma unroll 2
+#pragma unroll 4
     for (int kk = 0; kk < dk; kk += 16) {
       uint32_t ah[4], al[4], bh[4], bl[4];
       mp_ldm4(ah, left + kk);
       mp_ldm4(al, left + DP_C * L.pk + kk);
-      const int sa = (kk + (lane & 7) + ((lane >> 3) & 1) * 8) * PN + n0 + (lane >> 4) * 8;
+      const int sa = (kk + (lane & 7) + ((lane >> 3) & 1) * 8) * PN + nb + (lane >> 4) * 8;
       mp_ldm4t(bh, s_hi + sa);
       mp_ldm4t(bl, s_lo + sa);
 #pragma unroll
-      for (int n = 0; n < NT; ++n) mp_mma(acc[n], ah, bh[2 * n], bh[2 * n + 1]);
-#pragma unroll
-      for (int n = 0; n < NT; ++n) mp_mma(acc[n], ah, bl[2 * n], bl[2 * n + 1]);
-#pragma unroll
-      for (int n = 0; n < NT; ++n) mp_mma(acc[n], al, bh[2 * n], bh[2 * n + 1]);
+      for (int n = 0; n < NT; ++n) {
+        const uint32_t h0 = N == 32 ? bh[2 * n] : nh ? bh[2] : bh[0], h1 = N == 32 ? bh[2 * n + 1] : nh ? bh[3] : bh[1];
+        const uint32_t l0 = N == 32 ? bl[2 * n] : nh ? bl[2] : bl[0], l1 = N == 32 ? bl[2 * n + 1] : nh ? bl[3] : bl[1];
+        mp_mma(part[0][n], ah, h0, h1);
+        mp_mma(part[1][n], ah, l0, l1);
+        mp_mma(part[2][n], al, h0, h1);
+      }
     }
+    float acc[NT][4];
+#pragma unroll
+    for (int n = 0; n < NT; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[n][e] = part[0][n][e] + (part[1][n][e] + part[2][n][e]);
     if (kind == 0) {                               // U = U0 - W S, in two parts
-      const float* us = reinterpret_cast<const float*>(sg + L.u0);
+      const float* us = reinterpret_cast<const float*>(sg + L.size);
 #pragma unroll
       for (int n = 0; n < NT; ++n)
 #pragma unroll
@@ -482,33 +550,6 @@ delta_walk_kernel(DeltaPromptArgs a, int stages) {
         }
     }
     __syncthreads();                               // (U is there, and nobody reads the old state any more)
-    if (kind == 1) {                               // O += B U: the tokens up to this warp's
-      const __nv_bfloat16* bs = sg + L.b + (mt * 16 + (lane & 15)) * DP_PB + (lane >> 4) * 8;
-#pragma unroll
-      for (int ks = 0; ks < 2; ++ks) {
-        if (ks > mt) continue;
-        uint32_t ah[4], al[4], bh[4], bl[4];
-        mp_ldm4(ah, bs + ks * 16);
-        mp_ldm4(al, bs + DP_C * DP_PB + ks * 16);
-        const int ua = (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PN + n0 + (lane >> 4) * 8;
-        mp_ldm4t(bh, u_hi + ua);
-        mp_ldm4t(bl, u_lo + ua);
-#pragma unroll
-        for (int n = 0; n < NT; ++n) {
-          mp_mma(acc[n], ah, bh[2 * n], bh[2 * n + 1]);
-          mp_mma(acc[n], ah, bl[2 * n], bl[2 * n + 1]);
-          mp_mma(acc[n], al, bh[2 * n], bh[2 * n + 1]);
-        }
-      }
-#pragma unroll
-      for (int n = 0; n < NT; ++n)
-#pragma unroll
-        for (int r = 0; r < 2; ++r) {
-          const int row = mt * 16 + g + 8 * r, c = j0 + n0 + n * 8 + 2 * t4;
-          if (row < rows && c < dv)                // (dv is even: a pair lies inside or outside)
-            *reinterpret_cast<float2*>(a.out + ((size_t)(first + row) * a.H + h) * dv + c) = make_float2(acc[n][2 * r], acc[n][2 * r + 1]);
-        }
-    }
     // ---- S = P_end S + (K . P_end / P)^T U
     const __nv_bfloat16* d_hi = sg + (size_t)4 * DP_C * L.pk;
     const float* pe = reinterpret_cast<const float*>(sg + L.p_end);
@@ -541,10 +582,46 @@ delta_walk_kernel(DeltaPromptArgs a, int stages) {
       }
     }
     if (ch + 1 < ch1) put_state();
+    if (kind == 1) {                               // O += B U: the tokens up to this warp's
+      const __nv_bfloat16* bs = sg + L.b + (mt * 16 + (lane & 15)) * DP_PB + (lane >> 4) * 8;
+#pragma unroll
+      for (int ks = 0; ks < 2; ++ks) {
+        if (ks > mt) continue;
+        uint32_t ah[4], al[4], bh[4], bl[4];
+        mp_ldm4(ah, bs + ks * 16);
+        mp_ldm4(al, bs + DP_C * DP_PB + ks * 16);
+        const int ua = (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PN + nb + (lane >> 4) * 8;
+        mp_ldm4t(bh, u_hi + ua);
+        mp_ldm4t(bl, u_lo + ua);
+#pragma unroll
+        for (int n = 0; n < NT; ++n) {
+          const uint32_t h0 = N == 32 ? bh[2 * n] : nh ? bh[2] : bh[0], h1 = N == 32 ? bh[2 * n + 1] : nh ? bh[3] : bh[1];
+          const uint32_t l0 = N == 32 ? bl[2 * n] : nh ? bl[2] : bl[0], l1 = N == 32 ? bl[2 * n + 1] : nh ? bl[3] : bl[1];
+          mp_mma(acc[n], ah, h0, h1);
+          mp_mma(acc[n], ah, l0, l1);
+          mp_mma(acc[n], al, h0, h1);
+        }
+      }
+#pragma unroll
+      for (int n = 0; n < NT; ++n)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          const int row = mt * 16 + g + 8 * r, c = j0 + n0 + n * 8 + 2 * t4;
+          if (row < rows && c < dv)                // (dv is even: a pair lies inside or outside)
+            *reinterpret_cast<float2*>(a.out + ((size_t)(first + row) * a.H + h) * dv + c) = make_float2(acc[n][2 * r], acc[n][2 * r + 1]);
+        }
+    }
     if (stages == 1 && ch + 1 < ch1) {
       __syncthreads();                             // (the only stage is read)
-      load(ch + 1, 0);
+      if (tid == 0) load(ch + 1, 0);
     }
+  }
+  if (!ok) {
+    if (tid == 0) {
+      grace_period();
+      if (a.err) atomicExch(a.err, 1);
+    }
+    return;
   }
 #pragma unroll
   for (int m = 0; m < MT; ++m)
@@ -600,27 +677,32 @@ AF_EXPORT int af_delta_prompt_chunk() { return DP_C; }
 // A prefill step's recurrence.  q, k rows of G heads of dk, v rows of H heads of dv (qkv_ts elements between tokens), beta a
 // number per token and head, z the decays' logits [tokens][H * dk].  chunk_starts [n_chunks + 1], seq_first_chunk [n_seqs + 1]:
 // chunks of up to 32 tokens.  out float [tokens][H * dv]; state float [slots][H][dv][dk] is read and left updated.
-// Scratch: ops bfloat16 [n_chunks * H][6][32][dk], b bfloat16 [n_chunks * H][2][32][32], u0 float [n_chunks * H][32][dv],
-// p_end float [n_chunks * H][dk].
+// Scratch of af_delta_prompt_scratch(dk, dv, tile, 0 / 1) bytes a chunk and head, 16-byte aligned: blob and u0.  tile: value
+// columns of a block of the second kernel (16 or 32).
+AF_EXPORT long long af_delta_prompt_scratch(int dk, int dv, int tile, int which) {
+  return which == 0 ? (long long)dp_blob(dk).size * 2 : (long long)((dv + tile - 1) / tile) * DP_C * (tile + 4) * 4;
+}
 AF_EXPORT int af_delta_prompt(float* out, const float* q, const float* k, const float* v, long long qkv_ts, const float* beta,
                               long long beta_ts, const float* z, long long z_ts, const float* dt_bias, const float* rate,
-                              float* state, void* ops, void* b, float* u0, float* p_end, const int* chunk_starts,
+                              float* state, void* blob, float* u0, int tile, const int* chunk_starts,
                               const int* seq_first_chunk, const int* slots, int n_chunks, int n_seqs, int G, int H, int dk,
-                              int dv, cudaStream_t stream) {
+                              int dv, int* err, cudaStream_t stream) {
   if (n_chunks == 0) return 0;
   AF_REQUIRE(af_delta_prompt_supported(dk, dv), "af_delta_prompt: heads of %d keys and %d values", dk, dv);
   AF_REQUIRE(n_chunks > 0 && n_seqs > 0 && n_seqs < 65536 && G > 0 && H > 0 && H < 65536 && H % G == 0, "af_delta_prompt: bad sizes");
   AF_REQUIRE(qkv_ts % 4 == 0 && z_ts % 4 == 0 &&
-                 (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)z | (uintptr_t)dt_bias | (uintptr_t)rate | (uintptr_t)ops |
-                   (uintptr_t)b | (uintptr_t)u0 | (uintptr_t)p_end | (uintptr_t)out | (uintptr_t)state) & 15) == 0,
+                 (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)z | (uintptr_t)dt_bias | (uintptr_t)rate | (uintptr_t)blob |
+                   (uintptr_t)u0 | (uintptr_t)out | (uintptr_t)state) & 15) == 0,
              "af_delta_prompt: rows of whole 16-byte pieces");
-  DeltaPromptArgs a{q, k, v, beta, z, qkv_ts, beta_ts, z_ts, dt_bias, rate, (__nv_bfloat16*)ops, (__nv_bfloat16*)b, u0, p_end,
-                    state, out, chunk_starts, seq_first_chunk, slots, G, H, dk, dv};
+  AF_REQUIRE(tile == 16 || tile == 32, "af_delta_prompt: tiles of %d value columns", tile);
+  DeltaPromptArgs a{q, k, v, beta, z, qkv_ts, beta_ts, z_ts, dt_bias, rate, (__nv_bfloat16*)blob, u0, tile,
+                    state, out, chunk_starts, seq_first_chunk, slots, G, H, dk, dv, err};
   int e;
   if (dk <= 32) e = dp_launch_chunks<1>(a, n_chunks, stream);
   else if (dk <= 64) e = dp_launch_chunks<2>(a, n_chunks, stream);
   else if (dk <= 128) e = dp_launch_chunks<4>(a, n_chunks, stream);
   else e = dp_launch_chunks<8>(a, n_chunks, stream);
   if (e) return e;
+  if (tile == 16) return dk <= 128 ? dp_launch_walk<16, 1>(a, n_seqs, stream) : dp_launch_walk<16, 2>(a, n_seqs, stream);
   return dk <= 128 ? dp_launch_walk<32, 1>(a, n_seqs, stream) : dp_launch_walk<32, 2>(a, n_seqs, stream);
 }

@@ -1945,10 +1945,11 @@ def _delta_chunks(batch):
     return batch.aux["delta_chunks"]
 
 
-def delta_prompt(out, q, k, v, beta, z, dt_bias, rate, state, batch, heads: int, dk: int, dv: int) -> None:
+def delta_prompt(out, q, k, v, beta, z, dt_bias, rate, state, batch, heads: int, dk: int, dv: int, tile: int = 0) -> None:
     """:func:`state_scan`'s rule ``gated`` for a prefill step on the tensor cores, the sequences cut into chunks, with the
     decays exp(-rate softplus(z + dt_bias)) worked out from their logits ``z`` float32 [T, heads * dk]: q, k, v float32
-    sections of one row, out float32 [T, heads * dv].  32-bit sums; the operands are pairs of bfloat16."""
+    sections of one row, out float32 [T, heads * dv].  32-bit sums; the operands are pairs of bfloat16.  ``tile``: value
+    columns of a block of the kernel that walks the chunks (16 or 32; 0: chosen from the step's size)."""
     T = out.shape[0]
     key_heads = q.shape[1] // dk
     if tuple(q.shape) != (T, key_heads * dk) or q.shape != k.shape or tuple(v.shape) != (T, heads * dv) or heads % key_heads \
@@ -1961,17 +1962,18 @@ def delta_prompt(out, q, k, v, beta, z, dt_bias, rate, state, batch, heads: int,
         raise KernelError(f"delta_prompt: out contiguous float32 [{T}, {heads * dv}], state float32 [slots, {heads}, {dv}, {dk}]")
     starts, first, n = _delta_chunks(batch)
     dev, f32, i32 = out.device, torch.float32, torch.int32
-    chunk = int(_lib().af_delta_prompt_chunk())
-    ops = torch.empty(n * heads * 6 * chunk * dk, dtype=torch.bfloat16, device=dev)
-    b = torch.empty(n * heads * 2 * chunk * chunk, dtype=torch.bfloat16, device=dev)
-    u0 = torch.empty(n * heads * chunk * dv, dtype=f32, device=dev)
-    p_end = torch.empty(n * heads * dk, dtype=f32, device=dev)
+    # blocks of 32 value columns, or of 16 while the wider ones leave SMs without one
+    tile = tile or (16 if batch.n_seqs * heads * -(-dv // 32) < sm_count() else 32)
+    scratch = _lib().af_delta_prompt_scratch
+    scratch.restype = c_longlong
+    blob, u0 = (torch.empty(n * heads * scratch(c_int(dk), c_int(dv), c_int(tile), c_int(w)) // 4, dtype=f32, device=dev)
+                for w in (0, 1))
     (qp, ts), (kp, _), (vp, _) = _f32_rows(q, "q"), _f32_rows(k, "k"), _f32_rows(v, "v")
     _check(_lib().af_delta_prompt(
         _ptr(out), qp, kp, vp, ts, *_f32_rows(beta, "beta"), *_f32_rows(z, "z"), _ptr(dt_bias, "dt_bias", f32),
-        _ptr(rate, "rate", f32), _ptr(state), _ptr(ops), _ptr(b), _ptr(u0), _ptr(p_end), _ptr(starts, "chunk_starts", i32),
+        _ptr(rate, "rate", f32), _ptr(state), _ptr(blob), _ptr(u0), c_int(tile), _ptr(starts, "chunk_starts", i32),
         _ptr(first, "seq_first_chunk", i32), _ptr(batch.slots, "slots", i32), c_int(n), c_int(batch.n_seqs), c_int(key_heads),
-        c_int(heads), c_int(dk), c_int(dv), _stream()))
+        c_int(heads), c_int(dk), c_int(dv), _ptr(error_word(dev), "err", i32), _stream()))
 
 
 __all__ = [n for n in dir() if not n.startswith("_")]

@@ -253,7 +253,7 @@ def test_delta_rule_token_by_token(K, G, H, dk, dv):
     assert float(state[1].abs().max()) == 0.0
 
 
-def _chunked_run(K, parts, picks, batch, state, H, dk, dv, G):
+def _chunked_run(K, parts, picks, batch, state, H, dk, dv, G, tile=0):
     """:func:`kernels.delta_prompt` on rows whose logits give the parts' decays (rate 1, softplus inverted)."""
     rows = [torch.cat([p[i][s].flatten(1) for p, s in zip(parts, picks)]) for i in range(5)]
     q, k, v, w, beta = rows
@@ -264,7 +264,8 @@ def _chunked_run(K, parts, picks, batch, state, H, dk, dv, G):
     n = q.shape[1]
     out = torch.full((q.shape[0], H * dv), float("nan"), device=DEV)
     K.delta_prompt(out, mixed[:, :n], mixed[:, n: 2 * n], mixed[:, 2 * n: 2 * n + H * dv], mixed[:, 2 * n + H * dv: 2 * n + H * dv + H],
-                   (z - bias).to(DEV).contiguous(), bias.to(DEV), torch.ones(H * dk, device=DEV), state, batch, H, dk, dv)
+                   (z - bias).to(DEV).contiguous(), bias.to(DEV), torch.ones(H * dk, device=DEV), state, batch, H, dk, dv, tile=tile)
+    K.check_device_errors(DEV)
     return out
 
 
@@ -272,8 +273,8 @@ CHUNK_SHAPES = [(1, 3, 64, 64), (2, 2, 128, 128), (1, 2, 192, 96), (1, 2, 32, 20
 
 
 @pytest.mark.parametrize("G,H,dk,dv", CHUNK_SHAPES)
-@pytest.mark.parametrize("keep", [None, 1.0, 0.99])
-def test_delta_rule_in_chunks(K, G, H, dk, dv, keep):
+@pytest.mark.parametrize("keep,tile", [(None, 16), (None, 32), (1.0, 32), (0.99, 0)])
+def test_delta_rule_in_chunks(K, G, H, dk, dv, keep, tile):
     """Prompts of one token, of a group and a token, of a chunk and a token, of whole chunks and of many; decays from nothing to
     everything, none at all, and slow ones; then single tokens from the states the chunks left; slots in any order."""
     assert K.delta_prompt_supported(dk, dv) and not K.delta_prompt_supported(dk + 1, dv) and not K.delta_prompt_supported(dk, dv + 8)
@@ -283,7 +284,7 @@ def test_delta_rule_in_chunks(K, G, H, dk, dv, keep):
     refs = [ref_scan(*p) for p in parts]
     slots = [6, 2, 0, 5, 1, 7, 3]
     state = torch.zeros(8, H, dv, dk, device=DEV)
-    out = _chunked_run(K, parts, [slice(0, n) for n in lens], batch_of(lens, slots), state, H, dk, dv, G)
+    out = _chunked_run(K, parts, [slice(0, n) for n in lens], batch_of(lens, slots), state, H, dk, dv, G, tile)
     row = 0
     for n, r in zip(lens, refs):
         close(out[row: row + n], r[:n].flatten(1), 2e-4, n)
