@@ -631,6 +631,38 @@ head_gate_kernel(T* __restrict__ x, long long x_stride, const float* __restrict_
   *p = from_f32<T>(to_f32(*p) * gate_factor(gate, gate_stride, (int)t, per_value ? i : h));
 }
 
+// The same with four neighbours a thread (sizes, strides and bases in whole pieces).
+template <typename T>
+__global__ void __launch_bounds__(256)
+head_gate4_kernel(T* __restrict__ x, long long x_stride, const float* __restrict__ gate, long long gate_stride, int nq, int dv,
+                  int pitch, int per_value, size_t total) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t at = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  if (at >= total) return;
+  const int per_row = nq * dv;
+  const size_t t = at / per_row;
+  const int i = (int)(at - t * per_row), h = i / dv;
+  T* p = x + t * x_stride + (size_t)h * pitch + (i - h * dv);
+  float f[4], v[4];
+  if (per_value) {
+    const float4 z = *reinterpret_cast<const float4*>(gate + t * gate_stride + i);
+    f[0] = 1.f / (1.f + expf(-z.x)), f[1] = 1.f / (1.f + expf(-z.y)), f[2] = 1.f / (1.f + expf(-z.z)), f[3] = 1.f / (1.f + expf(-z.w));
+  } else {
+    f[0] = f[1] = f[2] = f[3] = gate_factor(gate, gate_stride, (int)t, h);
+  }
+  if constexpr (sizeof(T) == 2) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    v[0] = __uint_as_float(raw.x << 16), v[1] = __uint_as_float(raw.x & 0xffff0000u);
+    v[2] = __uint_as_float(raw.y << 16), v[3] = __uint_as_float(raw.y & 0xffff0000u);
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v[0] * f[0], v[1] * f[1]), b = __floats2bfloat162_rn(v[2] * f[2], v[3] * f[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+  } else {
+    const float4 q = *reinterpret_cast<const float4*>(p);
+    *reinterpret_cast<float4*>(p) = make_float4(q.x * f[0], q.y * f[1], q.z * f[2], q.w * f[3]);
+  }
+}
+
 AF_EXPORT int af_head_gate(void* x, long long x_stride, int dtype, const float* gate, long long gate_stride, int n_rows,
                            int nq, int dv, int pitch, int per_value, cudaStream_t stream) {
   if (n_rows == 0) return 0;
@@ -638,6 +670,12 @@ AF_EXPORT int af_head_gate(void* x, long long x_stride, int dtype, const float* 
   const size_t total = (size_t)n_rows * nq * dv;
   const size_t blocks = (total + 255) / 256;
   AF_REQUIRE(blocks < (1ull << 31), "af_head_gate: too many rows");
+  if (dv % 4 == 0 && pitch % 4 == 0 && x_stride % 4 == 0 && gate_stride % 4 == 0 && (((uintptr_t)x | (uintptr_t)gate) & 15) == 0) {
+    AF_DISPATCH_DTYPE(dtype, T,
+                      af_launch(head_gate4_kernel<T>, dim3((unsigned)((total / 4 + 255) / 256)), dim3(256), 0, stream, (T*)x,
+                                x_stride, gate, gate_stride, nq, dv, pitch, per_value, total));
+    AF_CHECK_LAUNCH("af_head_gate");
+  }
   AF_DISPATCH_DTYPE(dtype, T,
                     af_launch(head_gate_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, stream, (T*)x, x_stride, gate,
                               gate_stride, nq, dv, pitch, per_value, total));

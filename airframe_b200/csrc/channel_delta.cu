@@ -117,6 +117,107 @@ delta_conv_kernel(DeltaConvArgs a) {
   }
 }
 
+// The same where everything comes in 16-byte pieces, heads are 4 .. 128 channels (a power of two) and the convolution has up
+// to TAPS = 4 taps: a lane takes four channels of R tokens in a row, so that a row is read once for all taps, and a head's sum
+// of squares is joined over its dk / 4 lanes.  All loads of a warp are in flight at once; single tokens (R 1) ask for taps
+// and history before the wait.
+template <int R, bool SINGLE>
+__global__ void __launch_bounds__(128)
+delta_conv_row_kernel(DeltaConvArgs a, int n_tokens) {
+  pdl_launch_dependents();
+  constexpr int TAPS = 4;
+  const int lane = threadIdx.x & 31, t0 = blockIdx.x * R, slice = blockIdx.y * 4 + (threadIdx.x >> 5);
+  const int nq = a.G * a.dk, C = 2 * nq + a.H * a.dv, slices = (C + 127) / 128, keep = a.taps - 1;
+  if (slice > slices) return;
+  if (slice == slices) {                                     // step sizes, low-rank factors
+    pdl_wait();
+    a.proj = pdl_fresh(a.proj);
+    for (int r = 0; r < R && t0 + r < n_tokens; ++r) {
+      const size_t t = (size_t)t0 + r;
+      if (a.low != nullptr) {
+#pragma unroll
+        for (int f = 0; f < 2; ++f)
+          for (int i = lane; i < a.rank[f]; i += 32)
+            a.low[t * a.low_ld + (f ? a.low_at : 0) + i] = __float2bfloat16_rn(a.proj[t * a.ld + a.off_low[f] + i]);
+      }
+      for (int h = lane; h < a.H; h += 32) a.out[t * a.out_ld + C + h] = 1.f / (1.f + expf(-a.proj[t * a.ld + a.off_b + h]));
+    }
+    return;
+  }
+  const int c = slice * 128 + lane * 4;
+  const bool on = c < C;
+  const int cc = on ? c : 0, col = dc_col(a, cc), L = a.dk / 4;
+  // lane r knows token t0 + r: how many tokens of its sequence lie in the step before it, its slot, its position
+  int my_back = 0, my_slot = -1, my_pos = 0;
+  if (lane < R && t0 + lane < n_tokens) {
+    const int seq = a.seq_of_token[t0 + lane];
+    my_pos = a.positions[t0 + lane], my_slot = a.slots[seq], my_back = t0 + lane - a.seq_starts[seq];
+  }
+  float4 w[TAPS];                                            // w[d]: the tap that looks d tokens back
+#pragma unroll
+  for (int d = 0; d < TAPS; ++d)
+    w[d] = d <= keep ? *reinterpret_cast<const float4*>(a.taps_w + (size_t)(keep - d) * C + cc) : make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 old[TAPS - 1];                                      // single tokens: the history, newest last
+  float* hist = nullptr;
+  if (SINGLE) {
+    const int slot = __shfl_sync(0xffffffffu, my_slot, 0);
+    if (slot >= 0 && keep > 0) hist = a.history + (size_t)slot * keep * C + cc;
+#pragma unroll
+    for (int i = 0; i < TAPS - 1; ++i)
+      old[i] = hist != nullptr && i < keep ? *reinterpret_cast<const float4*>(hist + (size_t)i * C) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  pdl_wait();
+  a.proj = pdl_fresh(a.proj);
+  float4 u[R + TAPS - 1];
+#pragma unroll
+  for (int i = 0; i < R + TAPS - 1; ++i) {
+    const int t = t0 + i - (TAPS - 1);
+    u[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (t >= 0 && t < n_tokens && (!SINGLE || i == TAPS - 1)) u[i] = *reinterpret_cast<const float4*>(a.proj + (size_t)t * a.ld + col);
+  }
+  if (SINGLE) {
+#pragma unroll
+    for (int d = 1; d < TAPS; ++d) {                         // (history row keep - d holds the input d tokens back)
+      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int i = 0; i < TAPS - 1; ++i)
+        if (i == keep - d) x = old[i];
+      u[TAPS - 1 - d] = x;
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    const int t = t0 + r;
+    if (t >= n_tokens) break;
+    const int back = __shfl_sync(0xffffffffu, my_back, r), slot = __shfl_sync(0xffffffffu, my_slot, r),
+              pos = __shfl_sync(0xffffffffu, my_pos, r);
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int d = TAPS - 1; d >= 0; --d) {
+      float4 x = u[r + TAPS - 1 - d];
+      if (!SINGLE && d > back) {                             // (before the step: the history, or nothing before the sequence)
+        x = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (d <= pos && d <= keep && slot >= 0)
+          x = *reinterpret_cast<const float4*>(a.history + ((size_t)slot * keep + keep - (d - back)) * C + cc);
+      }
+      v.x = fmaf(w[d].x, x.x, v.x), v.y = fmaf(w[d].y, x.y, v.y), v.z = fmaf(w[d].z, x.z, v.z), v.w = fmaf(w[d].w, x.w, v.w);
+    }
+    v.x = v.x / (1.f + expf(-v.x)), v.y = v.y / (1.f + expf(-v.y)), v.z = v.z / (1.f + expf(-v.z)), v.w = v.w / (1.f + expf(-v.w));
+    float ss = v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    for (int o = 1; o < L; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (c < 2 * nq) {
+      const float f = (c < nq ? a.query_scale : 1.f) / sqrtf(ss + a.key_eps);
+      v.x *= f, v.y *= f, v.z *= f, v.w *= f;
+    }
+    if (on) *reinterpret_cast<float4*>(a.out + (size_t)t * a.out_ld + c) = v;
+  }
+  if (SINGLE && on && hist != nullptr) {
+#pragma unroll
+    for (int i = 0; i < TAPS - 1; ++i)
+      if (i < keep) *reinterpret_cast<float4*>(hist + (size_t)i * C) = i + 1 < keep ? old[i + 1 < TAPS - 1 ? i + 1 : i] : u[TAPS - 1];
+  }
+}
+
 // One thread a (sequence, channel): the history after a step of prompts = the last taps - 1 of (history, the step's inputs).
 __global__ void __launch_bounds__(256)
 delta_history_kernel(DeltaConvArgs a) {
@@ -160,7 +261,14 @@ AF_EXPORT int af_delta_conv(float* out, long long out_ld, const float* proj, lon
                   seq_starts, taps, G, H, dk, dv, key_eps, query_scale, (__nv_bfloat16*)low, {off_low0, off_low1},
                   {rank0, rank1}, low_at, low_ld};
   const bool single = n_tokens == n_seqs;
-  if (dk <= 32) dc_launch<1>(a, n_tokens, single, stream);
+  const bool rows = taps <= 4 && dk >= 4 && dk <= 128 && (dk & (dk - 1)) == 0 && (H * dv) % 4 == 0 &&
+                    ((ld | out_ld | off_q | off_k | off_v) & 3) == 0 &&
+                    (((uintptr_t)out | (uintptr_t)proj | (uintptr_t)taps_w | (uintptr_t)history) & 15) == 0;
+  if (rows) {
+    const int slices = (2 * G * dk + H * dv + 127) / 128 + 1;
+    if (single) af_launch(delta_conv_row_kernel<1, true>, dim3(n_tokens, (slices + 3) / 4), dim3(128), 0, stream, a, n_tokens);
+    else af_launch(delta_conv_row_kernel<8, false>, dim3((n_tokens + 7) / 8, (slices + 3) / 4), dim3(128), 0, stream, a, n_tokens);
+  } else if (dk <= 32) dc_launch<1>(a, n_tokens, single, stream);
   else if (dk <= 64) dc_launch<2>(a, n_tokens, single, stream);
   else if (dk <= 128) dc_launch<4>(a, n_tokens, single, stream);
   else if (dk <= 256) dc_launch<8>(a, n_tokens, single, stream);

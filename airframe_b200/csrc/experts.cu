@@ -35,8 +35,9 @@ __device__ __forceinline__ void load4_f32<__nv_bfloat16>(float* v, const __nv_bf
 // Scores first, the choice behind them.  A warp of the scores' kernel takes one row of the router (an expert, or
 // the shared expert's gate) and TM tokens, and adds a token's products in one fixed order whatever TM is, so that a
 // prompt and a decode step choose alike; the warps of a block share their tokens.  scores: [tokens, rows].
-// With `raw` the logits themselves are left there.
-template <typename TX, int TM>
+// With `raw` the logits themselves are left there.  RE > 1: a warp takes RE rows of the router (their number is a multiple of
+// RE), so that a token's values are read once for all of them; every (token, row) sum is the same whatever RE is.
+template <typename TX, int TM, int RE>
 __global__ void __launch_bounds__(256)
 expert_score_kernel(float* __restrict__ scores, const TX* __restrict__ h, const float* __restrict__ router, int n_tokens,
                     int hidden, int rows, int raw) {
@@ -44,49 +45,62 @@ expert_score_kernel(float* __restrict__ scores, const TX* __restrict__ h, const 
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const long long job = (long long)blockIdx.x * (blockDim.x >> 5) + warp;
   const long long groups = (n_tokens + TM - 1) / TM;
-  if (job >= groups * rows) return;
-  const int t0 = (int)(job / rows) * TM, e = (int)(job % rows);
+  const int sets = rows / RE;
+  if (job >= groups * sets) return;
+  const int t0 = (int)(job / sets) * TM, e = (int)(job % sets) * RE;
   const float* w = router + (size_t)e * hidden;
   const bool vec = hidden % 4 == 0 && (((uintptr_t)h | (uintptr_t)router) & 15) == 0;
   pdl_wait();
   h = pdl_fresh(h);
-  float z[TM];
+  float z[TM][RE];
   if (vec) {                                        // four values a lane and load, four loads in flight
-    float zz[TM][4];
+    float zz[TM][RE][4];
 #pragma unroll
-    for (int m = 0; m < TM; ++m) zz[m][0] = zz[m][1] = zz[m][2] = zz[m][3] = 0.f;
+    for (int m = 0; m < TM; ++m)
+#pragma unroll
+      for (int q = 0; q < RE; ++q) zz[m][q][0] = zz[m][q][1] = zz[m][q][2] = zz[m][q][3] = 0.f;
     for (int i0 = lane * 4; i0 < hidden; i0 += 512) {
 #pragma unroll
       for (int u = 0; u < 4; ++u) {
         const int i = i0 + u * 128;
         if (i < hidden) {
-          const float4 wv = *reinterpret_cast<const float4*>(w + i);
+          float4 wv[RE];
+#pragma unroll
+          for (int q = 0; q < RE; ++q) wv[q] = *reinterpret_cast<const float4*>(w + (size_t)q * hidden + i);
 #pragma unroll
           for (int m = 0; m < TM; ++m) {
             if (t0 + m >= n_tokens) continue;
             float xv[4];
             load4_f32<TX>(xv, h + (size_t)(t0 + m) * hidden + i);
-            zz[m][u] = fmaf(wv.x, xv[0], fmaf(wv.y, xv[1], fmaf(wv.z, xv[2], fmaf(wv.w, xv[3], zz[m][u]))));
+#pragma unroll
+            for (int q = 0; q < RE; ++q)
+              zz[m][q][u] = fmaf(wv[q].x, xv[0], fmaf(wv[q].y, xv[1], fmaf(wv[q].z, xv[2], fmaf(wv[q].w, xv[3], zz[m][q][u]))));
           }
         }
       }
     }
 #pragma unroll
-    for (int m = 0; m < TM; ++m) z[m] = (zz[m][0] + zz[m][1]) + (zz[m][2] + zz[m][3]);
+    for (int m = 0; m < TM; ++m)
+#pragma unroll
+      for (int q = 0; q < RE; ++q) z[m][q] = (zz[m][q][0] + zz[m][q][1]) + (zz[m][q][2] + zz[m][q][3]);
   } else {
 #pragma unroll
-    for (int m = 0; m < TM; ++m) {
-      z[m] = 0.f;
-      if (t0 + m >= n_tokens) continue;
-      const TX* x = h + (size_t)(t0 + m) * hidden;
-      for (int i = lane; i < hidden; i += 32) z[m] = fmaf(w[i], to_f32<TX>(x[i]), z[m]);
-    }
+    for (int m = 0; m < TM; ++m)
+#pragma unroll
+      for (int q = 0; q < RE; ++q) {
+        z[m][q] = 0.f;
+        if (t0 + m >= n_tokens) continue;
+        const TX* x = h + (size_t)(t0 + m) * hidden;
+        for (int i = lane; i < hidden; i += 32) z[m][q] = fmaf(w[(size_t)q * hidden + i], to_f32<TX>(x[i]), z[m][q]);
+      }
   }
 #pragma unroll
-  for (int m = 0; m < TM; ++m) {
-    const float zs = warp_sum(z[m]);
-    if (lane == 0 && t0 + m < n_tokens) scores[(size_t)(t0 + m) * rows + e] = raw ? zs : 1.f / (1.f + expf(-zs));
-  }
+  for (int m = 0; m < TM; ++m)
+#pragma unroll
+    for (int q = 0; q < RE; ++q) {
+      const float zs = warp_sum(z[m][q]);
+      if (lane == 0 && t0 + m < n_tokens) scores[(size_t)(t0 + m) * rows + e + q] = raw ? zs : 1.f / (1.f + expf(-zs));
+    }
 }
 
 // A warp a token: the `top` largest choice scores in turn (equal scores: the lower index), each struck out once
@@ -206,16 +220,21 @@ AF_EXPORT int af_expert_route(int* ids, float* wts, float* shared_gate, float* s
   const int rows = n_experts + (shared_gate != nullptr ? 1 : 0);
   // a prompt: four tokens a warp (a row of the router is read once for them); few tokens: a warp each
   const int tm = n_tokens >= 256 ? 4 : 1;
-  const long long jobs = (long long)((n_tokens + tm - 1) / tm) * rows;
+  const int re = tm == 4 && rows % 4 == 0 ? 4 : 1;
+  const long long jobs = (long long)((n_tokens + tm - 1) / tm) * (rows / re);
   const long long blocks = (jobs + 7) / 8;
   AF_REQUIRE(blocks < (1ll << 31), "af_expert_route: too many tokens");
-  if (tm == 4) {
+  if (re == 4) {
     AF_DISPATCH_DTYPE(h_dtype, TX,
-                      af_launch(expert_score_kernel<TX, 4>, dim3((unsigned)blocks), dim3(256), 0, stream, scores,
+                      af_launch(expert_score_kernel<TX, 4, 4>, dim3((unsigned)blocks), dim3(256), 0, stream, scores,
+                                (const TX*)h, router, n_tokens, hidden, rows, softmax));
+  } else if (tm == 4) {
+    AF_DISPATCH_DTYPE(h_dtype, TX,
+                      af_launch(expert_score_kernel<TX, 4, 1>, dim3((unsigned)blocks), dim3(256), 0, stream, scores,
                                 (const TX*)h, router, n_tokens, hidden, rows, softmax));
   } else {
     AF_DISPATCH_DTYPE(h_dtype, TX,
-                      af_launch(expert_score_kernel<TX, 1>, dim3((unsigned)blocks), dim3(256), 0, stream, scores,
+                      af_launch(expert_score_kernel<TX, 1, 1>, dim3((unsigned)blocks), dim3(256), 0, stream, scores,
                                 (const TX*)h, router, n_tokens, hidden, rows, softmax));
   }
   AF_COUNT_LAUNCH("af_expert_route");

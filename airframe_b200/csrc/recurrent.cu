@@ -696,11 +696,78 @@ gated_group_norm_kernel(TY* __restrict__ y, const float* __restrict__ o, const f
   }
 }
 
+// Groups of up to 1024 values in whole 16-byte pieces: a warp a group with its values in registers (NE groups of four a lane),
+// every load in flight before the first sum; the groups of all tokens over the grid.
+template <typename TY, int NE>
+__global__ void __launch_bounds__(128)
+gated_group_norm_warp_kernel(TY* __restrict__ y, const float* __restrict__ o, const float* __restrict__ w,
+                             const float* __restrict__ gate, long long gate_ts, int n, int group, float eps, int gate_act,
+                             float in_scale, long long jobs) {
+  pdl_launch_dependents();
+  const int lane = threadIdx.x & 31, per = n / group;
+  const long long job = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+  if (job >= jobs) return;
+  const size_t t = (size_t)(job / per);
+  const int c0 = (int)(job % per) * group;
+  float4 wv[NE], ov[NE], gv[NE];
+#pragma unroll
+  for (int e = 0; e < NE; ++e) {
+    const int c = (lane + 32 * e) * 4;
+    wv[e] = make_float4(1.f, 1.f, 1.f, 1.f), ov[e] = gv[e] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < group && w != nullptr) wv[e] = *reinterpret_cast<const float4*>(w + c0 + c);
+  }
+  pdl_wait();
+  o = pdl_fresh(o), gate = pdl_fresh(gate);
+  float ss = 0.f;
+#pragma unroll
+  for (int e = 0; e < NE; ++e) {
+    const int c = (lane + 32 * e) * 4;
+    if (c < group) {
+      ov[e] = *reinterpret_cast<const float4*>(o + t * n + c0 + c);
+      gv[e] = *reinterpret_cast<const float4*>(gate + t * gate_ts + c0 + c);
+    }
+  }
+#pragma unroll
+  for (int e = 0; e < NE; ++e) {
+    ov[e].x *= in_scale, ov[e].y *= in_scale, ov[e].z *= in_scale, ov[e].w *= in_scale;
+    ss += ov[e].x * ov[e].x + ov[e].y * ov[e].y + ov[e].z * ov[e].z + ov[e].w * ov[e].w;
+  }
+  const float inv = rsqrtf(warp_sum(ss) / (float)group + eps);
+  auto gated = [&](float g) { const float sg = 1.f / (1.f + expf(-g)); return gate_act ? g * sg : sg; };
+#pragma unroll
+  for (int e = 0; e < NE; ++e) {
+    const int c = (lane + 32 * e) * 4;
+    if (c >= group) continue;
+    const float v0 = ov[e].x * inv * wv[e].x * gated(gv[e].x), v1 = ov[e].y * inv * wv[e].y * gated(gv[e].y);
+    const float v2 = ov[e].z * inv * wv[e].z * gated(gv[e].z), v3 = ov[e].w * inv * wv[e].w * gated(gv[e].w);
+    TY* dst = y + t * n + c0 + c;
+    if constexpr (sizeof(TY) == 2) {
+      const __nv_bfloat162 a = __floats2bfloat162_rn(v0, v1), b = __floats2bfloat162_rn(v2, v3);
+      *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+    } else {
+      *reinterpret_cast<float4*>(dst) = make_float4(v0, v1, v2, v3);
+    }
+  }
+}
+
 AF_EXPORT int af_gated_group_norm(void* y, int y_dtype, const float* o, const float* w, const float* gate,
                                   long long gate_ts, int n_tokens, int n, int group, float eps, int gate_act,
                                   float in_scale, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   AF_REQUIRE(n_tokens > 0 && n > 0 && group > 0 && n % group == 0, "af_gated_group_norm: %d values in groups of %d", n, group);
+  if (group % 4 == 0 && group <= 1024 && gate_ts % 4 == 0 &&
+      (((uintptr_t)y | (uintptr_t)o | (uintptr_t)w | (uintptr_t)gate) & 15) == 0) {
+    const long long jobs = (long long)n_tokens * (n / group), blocks = (jobs + 3) / 4;
+    AF_REQUIRE(blocks < (1ll << 31), "af_gated_group_norm: too many groups for one grid");
+#define GN_LAUNCH(TY, NE)                                                                                                 \
+  af_launch(gated_group_norm_warp_kernel<TY, NE>, dim3((unsigned)blocks), dim3(128), 0, stream, (TY*)y, o, w, gate, gate_ts, n, \
+            group, eps, gate_act, in_scale, jobs)
+    if (group <= 128) AF_DISPATCH_DTYPE(y_dtype, TY, GN_LAUNCH(TY, 1));
+    else if (group <= 256) AF_DISPATCH_DTYPE(y_dtype, TY, GN_LAUNCH(TY, 2));
+    else AF_DISPATCH_DTYPE(y_dtype, TY, GN_LAUNCH(TY, 8));
+#undef GN_LAUNCH
+    AF_CHECK_LAUNCH("af_gated_group_norm");
+  }
   AF_DISPATCH_DTYPE(y_dtype, TY, af_launch(gated_group_norm_kernel<TY>, dim3(n_tokens), dim3(256), 0, stream, (TY*)y, o, w,
                                            gate, gate_ts, n, group, eps, gate_act, in_scale));
   AF_CHECK_LAUNCH("af_gated_group_norm");

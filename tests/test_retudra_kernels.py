@@ -132,15 +132,17 @@ def test_decoding_over_a_ring_behind_kept_pages(K, size, keep, hd, nq, nkv, dtyp
 
 # ---------------------------------------------------------------- the delta rule behind a decay per key channel
 
-def _delta_case(lens, G, H, dk, dv, taps, seed, pad=3):
+def _delta_case(lens, G, H, dk, dv, taps, seed, aligned):
     g = torch.Generator().manual_seed(seed)
     r = lambda *s: torch.randn(*s, generator=g)
     C = 2 * G * dk + H * dv
     T = sum(lens)
-    offs, at = [], 2
-    for n in (G * dk, G * dk, H * dv, H):                  # sections in an order of their own, with gaps
+    offs, at = [], 4 if aligned else 2
+    for n in (G * dk, G * dk, H * dv, H):                  # sections with gaps, on 16 bytes or not
         offs.append(at)
-        at += n + pad
+        at += n + 3
+        if aligned:
+            at = -(-at // 4) * 4
     return SimpleNamespace(proj=r(T, at), offs=offs, taps=r(C, taps), C=C, T=T, r=r)
 
 
@@ -156,13 +158,16 @@ def _ref_conv(c, rows, G, H, dk, dv, taps):
 
 
 @pytest.mark.parametrize("G,H,dk,dv,taps", [(2, 4, 12, 20, 3), (1, 3, 64, 64, 4), (1, 1, 5, 3, 9), (3, 3, 128, 128, 2), (2, 2, 192, 96, 4),
-                                            (1, 2, 300, 10, 1), (2, 2, 32, 48, 1), (1, 1, 520, 8, 5)])
-def test_convolution_unit_keys_and_step_sizes(K, G, H, dk, dv, taps):
+                                            (1, 2, 300, 10, 1), (2, 2, 32, 48, 1), (1, 1, 520, 8, 5), (3, 6, 16, 10, 3),
+                                            (5, 5, 4, 4, 4), (18, 18, 128, 128, 4), (1, 1, 8, 20, 2)])
+@pytest.mark.parametrize("aligned", [False, True])
+def test_convolution_unit_keys_and_step_sizes(K, G, H, dk, dv, taps, aligned):
     """Prompts of unequal lengths (one and two tokens among them: shorter than the convolution reaches), then single tokens one
     by one with the history carried on, a slot used again, a padding row."""
     lens, tail = [40, 1, 2, 17], 12
     full = [n + tail for n in lens]
-    c = _delta_case(full, G, H, dk, dv, taps, dk + taps)
+    c = _delta_case(full, G, H, dk, dv, taps, dk + taps, aligned)
+    wide = lambda T: torch.empty(T, -(-(c.C + H) // 4) * 4, device=DEV)[:, : c.C + H]
     seqs, at = [], 0
     for n in full:
         seqs.append(c.proj[at: at + n])
@@ -174,14 +179,17 @@ def test_convolution_unit_keys_and_step_sizes(K, G, H, dk, dv, taps):
         hist = torch.zeros(6, max(taps - 1, 1), c.C, device=DEV) if not again else hist
         if again:
             hist.zero_()                                    # (what taking a slot does)
-        out = torch.empty(sum(lens), c.C + H, device=DEV)
-        K.delta_conv(out, torch.cat([s[:n] for s, n in zip(seqs, lens)]).to(DEV), c.offs, tw, hist if taps > 1 else None,
-                     batch_of(lens, slots), G, H, dk, dv, 1e-6, 0.3)
+        out = wide(sum(lens))
+        low = torch.empty(sum(lens), 24, dtype=torch.bfloat16, device=DEV)
+        rows = torch.cat([s[:n] for s, n in zip(seqs, lens)])
+        K.delta_conv(out, rows.to(DEV), c.offs, tw, hist if taps > 1 else None, batch_of(lens, slots), G, H, dk, dv, 1e-6, 0.3,
+                     low=low, low_sections=((0, 5, 0), (2, 7, 8)))
+        assert torch.equal(low[:, :5].cpu(), rows[:, :5].bfloat16()) and torch.equal(low[:, 8:15].cpu(), rows[:, 2:9].bfloat16())
         close(out, torch.cat([r[:n] for r, n in zip(refs, lens)]), 2e-5)
         for j in range(tail):
             b = batch_of([1] * 5, [*slots, -1], [*(n + j for n in lens), 0])
             step = torch.cat([*(s[n + j: n + j + 1] for s, n in zip(seqs, lens)), torch.ones(1, c.proj.shape[1])]).to(DEV)
-            out = torch.empty(5, c.C + H, device=DEV)
+            out = wide(5)
             K.delta_conv(out, step, c.offs, tw, hist if taps > 1 else None, b, G, H, dk, dv, 1e-6, 0.3)
             close(out[:4], torch.cat([r[n + j: n + j + 1] for r, n in zip(refs, lens)]), 2e-5, j)
         if taps > 1:
@@ -437,21 +445,22 @@ def test_a_tokens_own_row(K, T, H, dim, layers, dtype):
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("T,heads,D,N,extra", [(3, 4, 20, 14, 0), (70, 2, 40, 300, 0), (8, 3, 96, 64, 16), (65, 5, 24, 33, 4)])
-def test_a_gate_per_value(K, T, heads, D, N, extra, dtype):
+@pytest.mark.parametrize("at,pad", [(3, 5), (4, 4)])
+def test_a_gate_per_value(K, T, heads, D, N, extra, dtype, at, pad):
     g = torch.Generator().manual_seed(T + N)
     r = lambda *s: torch.randn(*s, generator=g)
-    x, w, gate = r(T, heads, D + extra).to(dtype), r(heads, D, N).to(dtype), r(T, heads * N + 7)
+    x, w, gate = r(T, heads, D + extra).to(dtype), r(heads, D, N).to(dtype), r(T, -(-heads * N // 4) * 4 + 8)
     out = torch.empty(T, heads * (N + extra), dtype=dtype, device=DEV)
-    gd = gate.to(DEV)[:, 3: 3 + heads * N]
+    gd = gate.to(DEV)[:, at: at + heads * N]
     K.head_project(out, x.reshape(T, -1).to(DEV), w.to(DEV), heads, D, N, extra=extra, gate=gd)
-    s = plain.sigmoid(gate[:, 3: 3 + heads * N].double()).view(T, heads, N)
+    s = plain.sigmoid(gate[:, at: at + heads * N].double()).view(T, heads, N)
     ref = torch.einsum("thd,hdn->thn", x[..., :D].double(), w.double()) * s
     got = out.view(T, heads, N + extra).cpu()
     close(got[..., :N], ref, 1e-5 if dtype == torch.float32 else 1e-2)
     assert torch.equal(got[..., N:], x[..., D:])                              # (what is copied is not gated)
-    y = r(T, heads, N + 5).to(dtype)
+    y = r(T, heads, N + pad).to(dtype)
     yd = y.reshape(T, -1).to(DEV)
-    K.head_gate(yd, gd, heads, N, per_value=True, pitch=N + 5)
-    got = yd.view(T, heads, N + 5).cpu()
+    K.head_gate(yd, gd, heads, N, per_value=True, pitch=N + pad)
+    got = yd.view(T, heads, N + pad).cpu()
     close(got[..., :N], y[..., :N].double() * s, 1e-5 if dtype == torch.float32 else 1e-2)
     assert torch.equal(got[..., N:], y[..., N:])
