@@ -185,29 +185,39 @@ delta_conv_row_kernel(DeltaConvArgs a, int n_tokens) {
       u[TAPS - 1 - d] = x;
     }
   }
+  const bool heads = slice * 128 < 2 * nq;                   // (the whole warp: some of its channels are queries or keys)
+  const float scale = c < nq ? a.query_scale : 1.f;
 #pragma unroll
   for (int r = 0; r < R; ++r) {
     const int t = t0 + r;
     if (t >= n_tokens) break;
-    const int back = __shfl_sync(0xffffffffu, my_back, r), slot = __shfl_sync(0xffffffffu, my_slot, r),
-              pos = __shfl_sync(0xffffffffu, my_pos, r);
+    const int back = SINGLE ? TAPS : __shfl_sync(0xffffffffu, my_back, r);
+    float4 x[TAPS];
+#pragma unroll
+    for (int d = 0; d < TAPS; ++d) x[d] = u[r + TAPS - 1 - d];
+    if (!SINGLE && back < keep) {                            // taps that look before the step: the history, or nothing before the sequence
+      const int slot = __shfl_sync(0xffffffffu, my_slot, r), pos = __shfl_sync(0xffffffffu, my_pos, r);
+#pragma unroll
+      for (int d = 1; d < TAPS; ++d) {
+        if (d <= back) continue;
+        x[d] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (d <= pos && d <= keep && slot >= 0)
+          x[d] = *reinterpret_cast<const float4*>(a.history + ((size_t)slot * keep + keep - (d - back)) * C + cc);
+      }
+    }
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-    for (int d = TAPS - 1; d >= 0; --d) {
-      float4 x = u[r + TAPS - 1 - d];
-      if (!SINGLE && d > back) {                             // (before the step: the history, or nothing before the sequence)
-        x = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (d <= pos && d <= keep && slot >= 0)
-          x = *reinterpret_cast<const float4*>(a.history + ((size_t)slot * keep + keep - (d - back)) * C + cc);
+    for (int d = TAPS - 1; d >= 0; --d)
+      v.x = fmaf(w[d].x, x[d].x, v.x), v.y = fmaf(w[d].y, x[d].y, v.y), v.z = fmaf(w[d].z, x[d].z, v.z), v.w = fmaf(w[d].w, x[d].w, v.w);
+    v.x = __fdividef(v.x, 1.f + __expf(-v.x)), v.y = __fdividef(v.y, 1.f + __expf(-v.y));
+    v.z = __fdividef(v.z, 1.f + __expf(-v.z)), v.w = __fdividef(v.w, 1.f + __expf(-v.w));
+    if (heads) {
+      float ss = v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+      for (int o = 1; o < L; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      if (c < 2 * nq) {
+        const float f = scale * rsqrtf(ss + a.key_eps);
+        v.x *= f, v.y *= f, v.z *= f, v.w *= f;
       }
-      v.x = fmaf(w[d].x, x.x, v.x), v.y = fmaf(w[d].y, x.y, v.y), v.z = fmaf(w[d].z, x.z, v.z), v.w = fmaf(w[d].w, x.w, v.w);
-    }
-    v.x = v.x / (1.f + expf(-v.x)), v.y = v.y / (1.f + expf(-v.y)), v.z = v.z / (1.f + expf(-v.z)), v.w = v.w / (1.f + expf(-v.w));
-    float ss = v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
-    for (int o = 1; o < L; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-    if (c < 2 * nq) {
-      const float f = (c < nq ? a.query_scale : 1.f) / sqrtf(ss + a.key_eps);
-      v.x *= f, v.y *= f, v.z *= f, v.w *= f;
     }
     if (on) *reinterpret_cast<float4*>(a.out + (size_t)t * a.out_ld + c) = v;
   }

@@ -158,6 +158,9 @@ __device__ __forceinline__ T* pdl_fresh(T* p) {
   return p;
 }
 
+// Asks for the 128-byte line of `p` to come into L2 (before a wait, for weights that are read behind it).
+__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
+
 template <typename... KArgs, typename... Args>
 inline cudaError_t af_launch(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream,
                              Args&&... args) {

@@ -50,6 +50,8 @@ expert_score_kernel(float* __restrict__ scores, const TX* __restrict__ h, const 
   const int t0 = (int)(job / sets) * TM, e = (int)(job % sets) * RE;
   const float* w = router + (size_t)e * hidden;
   const bool vec = hidden % 4 == 0 && (((uintptr_t)h | (uintptr_t)router) & 15) == 0;
+  if (TM == 1)                                      // (a decode step: the router's row is cold)
+    for (int i = lane * 32; i < hidden; i += 1024) prefetch_l2(w + i);
   pdl_wait();
   h = pdl_fresh(h);
   float z[TM][RE];

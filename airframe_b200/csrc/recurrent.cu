@@ -942,16 +942,33 @@ channel_decay_kernel(float* __restrict__ alpha, const float* __restrict__ proj, 
   }
 }
 
-// Up to AF_CD_TOK tokens: block = 32 channels x AF_CD_SLICES runs (warp s takes run s).
+// One low-rank pair: what channel_decay is told of it.
+struct AfDecay {
+  float* alpha;
+  int off_low;
+  const float *w2t, *bias, *rate;
+  int rank, n;
+  float inv_tau;
+  int kind;
+};
+
+// Up to AF_CD_TOK tokens: block = 32 channels x AF_CD_SLICES runs (warp s takes run s).  The blocks behind the first
+// pair's work a second one.
 __global__ void __launch_bounds__(32 * AF_CD_SLICES)
-channel_decay_few_kernel(float* __restrict__ alpha, const float* __restrict__ proj, long long ld, int off_low,
-                         const float* __restrict__ w2t, const float* __restrict__ bias, const float* __restrict__ rate,
-                         int rank, int n, int n_tokens, float inv_tau, int kind) {
+channel_decay_few_kernel(AfDecay one, AfDecay two, const float* __restrict__ proj, long long ld, int n_tokens) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) float low[];                // [rank][AF_CD_TOK], then the runs' sums [runs][tokens][32]
+  const int first = (one.n + 31) / 32, bx = (int)blockIdx.x < first ? blockIdx.x : blockIdx.x - first;
+  const AfDecay d = (int)blockIdx.x < first ? one : two;
+  float* alpha = d.alpha;
+  const float* __restrict__ w2t = d.w2t;
+  const float *bias = d.bias, *rate = d.rate;
+  const int rank = d.rank, n = d.n, kind = d.kind, off_low = d.off_low;
+  const float inv_tau = d.inv_tau;
   float* sums = low + (size_t)rank * AF_CD_TOK;
   const int lane = threadIdx.x & 31, s = threadIdx.x >> 5;
-  const int c = blockIdx.x * 32 + lane;
+  const int c = bx * 32 + lane;
+  for (int r = threadIdx.x; r < rank; r += blockDim.x) prefetch_l2(w2t + (size_t)r * n + bx * 32);
   const float b = c < n && bias != nullptr ? bias[c] : 0.f;
   const float f = kind == AF_CD_SOFTPLUS ? (c < n ? rate[c] : 0.f) : inv_tau;
   pdl_wait();
@@ -976,6 +993,29 @@ channel_decay_few_kernel(float* __restrict__ alpha, const float* __restrict__ pr
   }
 }
 
+static int decay_few(const AfDecay& one, const AfDecay* two, const float* proj, long long ld, int n_tokens, cudaStream_t stream) {
+  const int rank = two != nullptr && two->rank > one.rank ? two->rank : one.rank;
+  const size_t smem = ((size_t)rank * AF_CD_TOK + AF_CD_SLICES * AF_CD_TOK * 32) * sizeof(float);
+  const int blocks = (one.n + 31) / 32 + (two != nullptr ? (two->n + 31) / 32 : 0);
+  af_launch(channel_decay_few_kernel, dim3(blocks), dim3(32 * AF_CD_SLICES), smem, stream, one, two != nullptr ? *two : one, proj, ld,
+            n_tokens);
+  AF_CHECK_LAUNCH("af_channel_decay");
+}
+
+// The decays exp(-rate softplus(bias + low w2t)) of one low-rank pair and the logits low2 g2t of another, for up to
+// AF_CD_TOK tokens in one launch.
+AF_EXPORT int af_decay_and_gate(float* decay, int off_a, const float* a2t, const float* bias, const float* rate, int rank_a,
+                                int n_a, float* gate, int off_g, const float* g2t, int rank_g, int n_g, const float* proj,
+                                long long ld, int n_tokens, cudaStream_t stream) {
+  if (n_tokens == 0) return 0;
+  AF_REQUIRE(n_tokens > 0 && n_tokens <= AF_CD_TOK && n_a > 0 && n_g > 0 && rank_a > 0 && rank_g > 0 && rank_a <= 512 &&
+                 rank_g <= 512 && bias != nullptr && rate != nullptr,
+             "af_decay_and_gate: bad sizes (up to %d tokens, ranks up to 512)", AF_CD_TOK);
+  const AfDecay one{decay, off_a, a2t, bias, rate, rank_a, n_a, 1.f, AF_CD_SOFTPLUS};
+  const AfDecay two{gate, off_g, g2t, nullptr, nullptr, rank_g, n_g, 1.f, AF_CD_LOGIT};
+  return decay_few(one, &two, proj, ld, n_tokens, stream);
+}
+
 AF_EXPORT int af_channel_decay(float* alpha, const float* proj, long long ld, int off_low, const float* w2t,
                                const float* bias, const float* rate, int rank, int n_tokens, int n, float tau, int kind,
                                cudaStream_t stream) {
@@ -984,10 +1024,8 @@ AF_EXPORT int af_channel_decay(float* alpha, const float* proj, long long ld, in
              "af_channel_decay: kind %d, a rate per channel with softplus", kind);
   AF_REQUIRE(n_tokens > 0 && n > 0 && rank > 0 && rank <= 512 && tau > 0.f, "af_channel_decay: bad sizes (rank up to 512)");
   if (n_tokens <= AF_CD_TOK) {
-    const size_t smem = ((size_t)rank * AF_CD_TOK + AF_CD_SLICES * AF_CD_TOK * 32) * sizeof(float);
-    af_launch(channel_decay_few_kernel, dim3((n + 31) / 32), dim3(32 * AF_CD_SLICES), smem, stream, alpha, proj, ld, off_low,
-              w2t, bias, rate, rank, n, n_tokens, 1.f / tau, kind);
-    AF_CHECK_LAUNCH("af_channel_decay");
+    const AfDecay one{alpha, off_low, w2t, bias, rate, rank, n, 1.f / tau, kind};
+    return decay_few(one, nullptr, proj, ld, n_tokens, stream);
   }
   const dim3 grid((n + 127) / 128, (n_tokens + AF_CD_TOK - 1) / AF_CD_TOK);
   AF_REQUIRE(grid.y < 65536, "af_channel_decay: too many tokens for one grid");

@@ -1673,6 +1673,25 @@ def channel_decay(alpha, proj, off_low: int, w2t, bias, tau: float = 1.0, kind: 
                                    c_float(tau), c_int(DECAY_KINDS[kind]), _stream()))
 
 
+DECAY_FEW = 16       # tokens that :func:`decay_and_gate` takes
+
+
+def decay_and_gate(decay, gate, proj, off_a: int, a2t, bias, rate, off_g: int, g2t) -> None:
+    """:func:`channel_decay` of the kinds "softplus" (into ``decay``) and "logit" (into ``gate``) from two low-rank sections of
+    the same projection rows, for up to ``DECAY_FEW`` tokens in one kernel."""
+    T, n_a = decay.shape
+    n_g = gate.shape[1]
+    if gate.shape[0] != T or proj.shape[0] != T or tuple(a2t.shape[1:]) != (n_a,) or tuple(g2t.shape[1:]) != (n_g,) \
+            or not all(t.is_contiguous() and t.dtype == torch.float32 for t in (decay, gate, a2t, g2t)) \
+            or bias.numel() != n_a or rate.numel() != n_a or max(off_a + a2t.shape[0], off_g + g2t.shape[0]) > proj.shape[1]:
+        raise KernelError("decay_and_gate: contiguous float32 rows and factors of one size, sections inside the projection row")
+    f32 = torch.float32
+    pp, ld = _f32_rows(proj, "proj")
+    _check(_lib().af_decay_and_gate(_ptr(decay), c_int(off_a), _ptr(a2t), _ptr(bias, "bias", f32), _ptr(rate, "rate", f32),
+                                    c_int(a2t.shape[0]), c_int(n_a), _ptr(gate), c_int(off_g), _ptr(g2t), c_int(g2t.shape[0]),
+                                    c_int(n_g), pp, ld, c_int(T), _stream()))
+
+
 SCAN_CHUNK = 128     # tokens of a chunk when a long prompt's scan is cut into chunks that run side by side
 
 
@@ -1962,8 +1981,8 @@ def delta_prompt(out, q, k, v, beta, z, dt_bias, rate, state, batch, heads: int,
         raise KernelError(f"delta_prompt: out contiguous float32 [{T}, {heads * dv}], state float32 [slots, {heads}, {dv}, {dk}]")
     starts, first, n = _delta_chunks(batch)
     dev, f32, i32 = out.device, torch.float32, torch.int32
-    # blocks of 32 value columns, or of 16 while the wider ones leave SMs without one
-    tile = tile or (16 if batch.n_seqs * heads * -(-dv // 32) < sm_count() else 32)
+    # blocks of 32 value columns, or of 16 while those all run at once (a block an SM)
+    tile = tile or (16 if batch.n_seqs * heads * -(-dv // 16) <= sm_count() else 32)
     scratch = _lib().af_delta_prompt_scratch
     scratch.restype = c_longlong
     blob, u0 = (torch.empty(n * heads * scratch(c_int(dk), c_int(dv), c_int(tile), c_int(w)) // 4, dtype=f32, device=dev)

@@ -619,11 +619,13 @@ class ChannelDelta(_StateMixer):
         kernels.delta_conv(mixed, proj, [off[n] for n in ("q", "k", "v", "b")], self.conv_w, history, batch, self.key_heads, H,
                            self.dk, self.dv, self.key_eps, self.query_scale, low=low,
                            low_sections=((off["a1"], ra, 0), (off["g1"], rg, (ra + 7) // 8 * 8)))
+        both = not chunked and T <= kernels.DECAY_FEW                 # decays and gates in one kernel
         if low is not None:
             gate = linear(low[:, (ra + 7) // 8 * 8:], self.g2_16, out_dtype=f32)
         else:
             gate = torch.empty(T, nv, dtype=f32, device=x.device)
-            kernels.channel_decay(gate, proj, off["g1"], self.g2t, None, kind="logit")
+            if not both:
+                kernels.channel_decay(gate, proj, off["g1"], self.g2t, None, kind="logit")
         o = torch.empty(T, nv, dtype=f32, device=x.device)
         if chunked:
             if low is not None:
@@ -634,7 +636,10 @@ class ChannelDelta(_StateMixer):
             kernels.delta_prompt(o, q, k, v, beta, z, self.dt_bias, self.rate, state, batch, H, self.dk, self.dv)
         else:
             decay = torch.empty(T, H * self.dk, dtype=f32, device=x.device)
-            kernels.channel_decay(decay, proj, off["a1"], self.a2t, self.dt_bias, kind="softplus", rate=self.rate)
+            if both:
+                kernels.decay_and_gate(decay, gate, proj, off["a1"], self.a2t, self.dt_bias, self.rate, off["g1"], self.g2t)
+            else:
+                kernels.channel_decay(decay, proj, off["a1"], self.a2t, self.dt_bias, kind="softplus", rate=self.rate)
             kernels.state_scan("gated", o, q, k, v, state, batch, H, self.dk, self.dv, w=decay, beta=beta)
         y = torch.empty(T, nv, dtype=x.dtype, device=x.device)
         kernels.gated_group_norm(y, o, self.norm_w, gate, self.dv, self.eps)

@@ -212,6 +212,11 @@ def test_decays_of_every_kind(K, T, rank, n):
     close(out, plain.sigmoid(z + bias.double()) ** (1.0 / 3.0), 2e-5)
     with pytest.raises(K.KernelError):
         K.channel_decay(out, d(proj), 4, d(w2.t()), d(bias), kind="softplus")
+    if T <= K.DECAY_FEW:                                      # both in one kernel, ranks and sizes apart
+        g2, gate = r(n + 45, rank + 3), torch.empty(T, n + 45, device=DEV)
+        K.decay_and_gate(out, gate, d(proj), 4, d(w2.t()), d(bias), d(rate), 5, d(g2.t()))
+        close(out, torch.exp(-rate.double() * plain.softplus(z + bias.double())), 2e-5)
+        close(gate, proj[:, 5: 8 + rank].double() @ g2.double().T, 1e-5)
 
 
 def delta_inputs(T, G, H, dk, dv, seed, keep=None):
