@@ -542,8 +542,9 @@ __device__ __forceinline__ void dp_bulk(void* dst, const void* src, uint32_t byt
 
 // Block (N value columns, head, sequence), eight warps, walks the sequence's chunks with its columns of the state in registers
 // (a warp holds MT tiles of 16 key channels) and, in two parts, in shared memory.  Warps 0 .. 3 make U = U0 - W S, warps 4 .. 7
-// O = (Q . P) S + B U (a warp: 16 tokens by N / 2 columns), all of them the new state; the next chunk's pieces are on their
-// way meanwhile if there is room for two.
+// O = (Q . P) S + B U (a warp: 16 tokens by 16 columns), all of them the new state; the next chunk's pieces are on their
+// way meanwhile if there is room for two.  In the narrow form the two warps of 16 tokens take all columns and halves of the
+// key channels, joined through shared memory: every piece of an operand is then loaded by one warp.
 template <int N, int MT>
 __global__ void __launch_bounds__(256)
 delta_walk_kernel(DeltaPromptArgs a, int stages) {
@@ -552,7 +553,9 @@ delta_walk_kernel(DeltaPromptArgs a, int stages) {
   __shared__ uint64_t full[2];
   __shared__ int give_up_s;
   volatile int* give_up = &give_up_s;
-  constexpr int PN = N + 8, NT = N / 16;           // NT: n8 tiles of a U or O warp
+  constexpr int PN = N + 8, NT = 2;                // NT: n8 tiles of a U or O warp
+  constexpr bool SPLIT = N == 16;
+  __shared__ float2 join_s[SPLIT ? 4 : 1][NT][2][32];
   const int dk = a.dk, dv = a.dv;
   const DpBlob L = dp_blob(dk);
   const uint32_t blob_bytes = (uint32_t)L.size * 2, u0_bytes = DP_C * (N + 4) * 4;
@@ -608,8 +611,7 @@ delta_walk_kernel(DeltaPromptArgs a, int stages) {
     dp_bulk(sg + blob_bytes, a.u0 + (unit * tiles + blockIdx.x) * (DP_C * (N + 4)), u0_bytes, &full[which]);
   };
   if (tid == 0) load(ch0, 0);
-  const int kind = warp >> 2, mt = (warp >> 1) & 1, nh = warp & 1, n0 = nh * (N / 2);
-  const int nb = N == 32 ? n0 : 0;                 // (narrow tiles: a load brings both warps' columns)
+  const int kind = warp >> 2, mt = (warp >> 1) & 1, half = warp & 1, n0 = SPLIT ? 0 : half * 16;
   bool ok = true;
   for (int ch = ch0; ch < ch1; ++ch) {
     const int i = ch - ch0, which = stages == 2 ? i & 1 : 0;
@@ -632,20 +634,18 @@ delta_walk_kernel(DeltaPromptArgs a, int stages) {
         for (int e = 0; e < 4; ++e) part[p][n][e] = 0.f;
     const __nv_bfloat16* left = sg + (size_t)kind * 2 * DP_C * L.pk + (mt * 16 + (lane & 15)) * L.pk + (lane >> 4) * 8;
 #pragma unroll 4
-    for (int kk = 0; kk < dk; kk += 16) {
+    for (int kk = SPLIT ? half * 16 : 0; kk < dk; kk += SPLIT ? 32 : 16) {
       uint32_t ah[4], al[4], bh[4], bl[4];
       mp_ldm4(ah, left + kk);
       mp_ldm4(al, left + DP_C * L.pk + kk);
-      const int sa = (kk + (lane & 7) + ((lane >> 3) & 1) * 8) * PN + nb + (lane >> 4) * 8;
+      const int sa = (kk + (lane & 7) + ((lane >> 3) & 1) * 8) * PN + n0 + (lane >> 4) * 8;
       mp_ldm4t(bh, s_hi + sa);
       mp_ldm4t(bl, s_lo + sa);
 #pragma unroll
       for (int n = 0; n < NT; ++n) {
-        const uint32_t h0 = N == 32 ? bh[2 * n] : nh ? bh[2] : bh[0], h1 = N == 32 ? bh[2 * n + 1] : nh ? bh[3] : bh[1];
-        const uint32_t l0 = N == 32 ? bl[2 * n] : nh ? bl[2] : bl[0], l1 = N == 32 ? bl[2 * n + 1] : nh ? bl[3] : bl[1];
-        mp_mma(part[0][n], ah, h0, h1);
-        mp_mma(part[1][n], ah, l0, l1);
-        mp_mma(part[2][n], al, h0, h1);
+        mp_mma(part[0][n], ah, bh[2 * n], bh[2 * n + 1]);
+        mp_mma(part[1][n], ah, bl[2 * n], bl[2 * n + 1]);
+        mp_mma(part[2][n], al, bh[2 * n], bh[2 * n + 1]);
       }
     }
     float acc[NT][4];
@@ -653,7 +653,27 @@ delta_walk_kernel(DeltaPromptArgs a, int stages) {
     for (int n = 0; n < NT; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[n][e] = part[0][n][e] + (part[1][n][e] + part[2][n][e]);
-    if (kind == 0) {                               // U = U0 - W S, in two parts
+    if constexpr (SPLIT) {                         // the second half of the key channels joins the first
+      float2(*mine)[2][32] = join_s[warp >> 1];
+      if (half == 1) {
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+          for (int r = 0; r < 2; ++r) mine[n][r][lane] = make_float2(acc[n][2 * r], acc[n][2 * r + 1]);
+      }
+      asm volatile("bar.sync %0, 64;" ::"r"(1 + (warp >> 1)) : "memory");
+      if (half == 0) {
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+          for (int r = 0; r < 2; ++r) {
+            const float2 v = mine[n][r][lane];
+            acc[n][2 * r] += v.x, acc[n][2 * r + 1] += v.y;
+          }
+      }
+    }
+    const bool owner = !SPLIT || half == 0;        // (of this warp pair's U or O)
+    if (kind == 0 && owner) {                               // U = U0 - W S, in two parts
       const float* us = reinterpret_cast<const float*>(sg + L.size);
 #pragma unroll
       for (int n = 0; n < NT; ++n)
@@ -700,7 +720,7 @@ delta_walk_kernel(DeltaPromptArgs a, int stages) {
       }
     }
     if (ch + 1 < ch1) put_state();
-    if (kind == 1) {                               // O += B U: the tokens up to this warp's
+    if (kind == 1 && owner) {                      // O += B U: the tokens up to this warp's
       const __nv_bfloat16* bs = sg + L.b + (mt * 16 + (lane & 15)) * DP_PB + (lane >> 4) * 8;
 #pragma unroll
       for (int ks = 0; ks < 2; ++ks) {
@@ -708,16 +728,14 @@ delta_walk_kernel(DeltaPromptArgs a, int stages) {
         uint32_t ah[4], al[4], bh[4], bl[4];
         mp_ldm4(ah, bs + ks * 16);
         mp_ldm4(al, bs + DP_C * DP_PB + ks * 16);
-        const int ua = (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PN + nb + (lane >> 4) * 8;
+        const int ua = (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PN + n0 + (lane >> 4) * 8;
         mp_ldm4t(bh, u_hi + ua);
         mp_ldm4t(bl, u_lo + ua);
 #pragma unroll
         for (int n = 0; n < NT; ++n) {
-          const uint32_t h0 = N == 32 ? bh[2 * n] : nh ? bh[2] : bh[0], h1 = N == 32 ? bh[2 * n + 1] : nh ? bh[3] : bh[1];
-          const uint32_t l0 = N == 32 ? bl[2 * n] : nh ? bl[2] : bl[0], l1 = N == 32 ? bl[2 * n + 1] : nh ? bl[3] : bl[1];
-          mp_mma(acc[n], ah, h0, h1);
-          mp_mma(acc[n], ah, l0, l1);
-          mp_mma(acc[n], al, h0, h1);
+          mp_mma(acc[n], ah, bh[2 * n], bh[2 * n + 1]);
+          mp_mma(acc[n], ah, bl[2 * n], bl[2 * n + 1]);
+          mp_mma(acc[n], al, bh[2 * n], bh[2 * n + 1]);
         }
       }
 #pragma unroll
@@ -763,7 +781,7 @@ int dp_raise(K kernel, bool* flags, size_t smem) {
   return 0;
 }
 
-constexpr size_t DP_SMEM = 226 * 1024;
+constexpr size_t DP_SMEM = 220 * 1024;      // (dynamic; a block has a few KB of its own besides)
 
 template <int NE>
 int dp_launch_chunks(const DeltaPromptArgs& a, int n_chunks, cudaStream_t stream) {

@@ -34,7 +34,7 @@ __device__ __forceinline__ void load4_f32<__nv_bfloat16>(float* v, const __nv_bf
 
 // Scores first, the choice behind them.  A warp of the scores' kernel takes one row of the router (an expert, or
 // the shared expert's gate) and TM tokens, and adds a token's products in one fixed order whatever TM is, so that a
-// prompt and a decode step choose alike; the warps of a block share their tokens.  scores: [tokens, rows].
+// prompt and a decode step choose alike.  scores: [tokens, rows].
 // With `raw` the logits themselves are left there.  RE > 1: a warp takes RE rows of the router (their number is a multiple of
 // RE), so that a token's values are read once for all of them; every (token, row) sum is the same whatever RE is.
 template <typename TX, int TM, int RE>
@@ -47,7 +47,8 @@ expert_score_kernel(float* __restrict__ scores, const TX* __restrict__ h, const 
   const long long groups = (n_tokens + TM - 1) / TM;
   const int sets = rows / RE;
   if (job >= groups * sets) return;
-  const int t0 = (int)(job / sets) * TM, e = (int)(job % sets) * RE;
+  // (the warps that run together share router rows, which stay in L1, and stream the tokens)
+  const int t0 = (int)(job % groups) * TM, e = (int)(job / groups) * RE;
   const float* w = router + (size_t)e * hidden;
   const bool vec = hidden % 4 == 0 && (((uintptr_t)h | (uintptr_t)router) & 15) == 0;
   if (TM == 1)                                      // (a decode step: the router's row is cold)
@@ -112,19 +113,24 @@ expert_score_kernel(float* __restrict__ scores, const TX* __restrict__ h, const 
 // the `keep` best groups (equal scores: the lower group) can be chosen.  With `softmax` the kernel finds logits and the
 // scores are their softmax over all experts.  With `normalise` the chosen weights are divided by their sum + 1e-20;
 // all weights are multiplied by `out_scale`.
-__global__ void __launch_bounds__(128)
-expert_choose_kernel(int* __restrict__ ids, float* __restrict__ wts, float* __restrict__ shared_gate,
-                     const float* __restrict__ scores, const float* __restrict__ correction, int n_tokens,
-                     int n_experts, int rows, int top, int groups, int keep, int normalise, float out_scale, int softmax,
-                     int group_max) {
-  pdl_launch_dependents();
-  extern __shared__ float score_all[];              // a warp: n_experts choice scores, n_experts scores, `groups` group scores
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int t = blockIdx.x * (blockDim.x >> 5) + warp;
-  pdl_wait();
-  if (t >= n_tokens) return;
-  scores = pdl_fresh(scores);
-  float* choice = score_all + (size_t)warp * (2 * n_experts + groups);
+struct ExpertChoice {
+  int* ids;
+  float *wts, *shared_gate;
+  const float *scores, *correction;
+  int n_tokens, n_experts, rows, top, groups, keep, normalise;
+  float out_scale;
+  int softmax, group_max;
+};
+
+// `choice`: the warp's piece of shared memory: n_experts choice scores, n_experts scores, `groups` group scores.
+__device__ __forceinline__ void choose_token(const ExpertChoice& a, int t, float* choice) {
+  int *ids = a.ids;
+  float *wts = a.wts, *shared_gate = a.shared_gate;
+  const float *scores = a.scores, *correction = a.correction;
+  const int n_experts = a.n_experts, rows = a.rows, top = a.top, groups = a.groups, keep = a.keep, normalise = a.normalise;
+  const int softmax = a.softmax, group_max = a.group_max;
+  const float out_scale = a.out_scale;
+  const int lane = threadIdx.x & 31;
   float* score = choice + n_experts;
   float* gscore = score + n_experts;
   const float OUT = -3.0e38f;                       // an expert of a group that is not kept (it still beats a struck one)
@@ -206,11 +212,30 @@ expert_choose_kernel(int* __restrict__ ids, float* __restrict__ wts, float* __re
   }
 }
 
+__global__ void __launch_bounds__(128)
+expert_choose_kernel(ExpertChoice a) {
+  pdl_launch_dependents();
+  extern __shared__ float score_all[];
+  const int warp = threadIdx.x >> 5, t = blockIdx.x * (blockDim.x >> 5) + warp;
+  pdl_wait();
+  if (t >= a.n_tokens) return;
+  a.scores = pdl_fresh(a.scores);
+  choose_token(a, t, score_all + (size_t)warp * (2 * a.n_experts + a.groups));
+}
+
+// What the plan of the same step needs besides the choices: the choice's kernel makes it too where the step's tokens are few
+// (perm null: no plan).
+struct ExpertPlanOut {
+  int *perm, *plan;
+  int n_experts, max_tiles, tile;
+};
+static int launch_choose_plan(const ExpertChoice& c, const ExpertPlanOut& p, cudaStream_t stream);
+
 // scores: room for n_tokens x (n_experts + 1) floats.
-AF_EXPORT int af_expert_route(int* ids, float* wts, float* shared_gate, float* scores, const void* h, int h_dtype,
+static int expert_route_impl(int* ids, float* wts, float* shared_gate, float* scores, const void* h, int h_dtype,
                               const float* router, int n_tokens, int hidden, int n_experts, int top,
                               const float* correction, int groups, int keep, int normalise, float out_scale, int softmax,
-                              int group_max, cudaStream_t stream) {
+                              int group_max, const ExpertPlanOut& out, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   AF_REQUIRE(n_tokens > 0 && hidden > 0 && n_experts > 0 && top >= 1 && top <= n_experts && scores != nullptr,
              "af_expert_route: %d of %d experts", top, n_experts);
@@ -240,11 +265,21 @@ AF_EXPORT int af_expert_route(int* ids, float* wts, float* shared_gate, float* s
                                 (const TX*)h, router, n_tokens, hidden, rows, softmax));
   }
   AF_COUNT_LAUNCH("af_expert_route");
+  const ExpertChoice c{ids, wts, shared_gate, scores, correction, n_tokens, n_experts, rows, top, groups, keep, normalise,
+                       out_scale, softmax, group_max};
+  if (out.perm != nullptr) return launch_choose_plan(c, out, stream);
   const int warps = n_experts <= 1024 ? 4 : 1;
   af_launch(expert_choose_kernel, dim3((n_tokens + warps - 1) / warps), dim3(32 * warps),
-            (size_t)warps * (2 * n_experts + groups) * sizeof(float), stream, ids, wts, shared_gate, (const float*)scores,
-            correction, n_tokens, n_experts, rows, top, groups, keep, normalise, out_scale, softmax, group_max);
+            (size_t)warps * (2 * n_experts + groups) * sizeof(float), stream, c);
   AF_CHECK_LAUNCH("af_expert_route");
+}
+
+AF_EXPORT int af_expert_route(int* ids, float* wts, float* shared_gate, float* scores, const void* h, int h_dtype,
+                              const float* router, int n_tokens, int hidden, int n_experts, int top,
+                              const float* correction, int groups, int keep, int normalise, float out_scale, int softmax,
+                              int group_max, cudaStream_t stream) {
+  return expert_route_impl(ids, wts, shared_gate, scores, h, h_dtype, router, n_tokens, hidden, n_experts, top, correction, groups,
+                           keep, normalise, out_scale, softmax, group_max, ExpertPlanOut{nullptr, nullptr, 0, 0, 0}, stream);
 }
 
 // ---------------------------------------------------------------- pairs by expert
@@ -254,21 +289,13 @@ AF_EXPORT int af_expert_route(int* ids, float* wts, float* shared_gate, float* s
 // token that the pair belongs to: expert = table[tokens[p / top]][p % top].  Block b takes the b-th table of
 // [blocks][vocab][top] and writes the b-th perm [n_pairs] and plan.  Numbers n_experts .. n_ids - 1 name identity
 // experts: their pairs end the permutation and belong to no tile.
-__global__ void __launch_bounds__(1024)
-expert_plan_kernel(int* __restrict__ perm, int* __restrict__ plan, const int* __restrict__ ids,
-                   const int* __restrict__ table, int vocab, int top, int n_pairs, int n_experts, int n_ids, int max_tiles,
-                   int tile) {
-  pdl_launch_dependents();
-  extern __shared__ int sh[];                       // count[E + 1], first[E + 1], cursor[E + 1] (the last: identity experts)
+// sh: count[E + 1], first[E + 1], cursor[E + 1] (the last: identity experts), count and cursor zero.
+__device__ __forceinline__ void plan_pairs(int* __restrict__ perm, int* __restrict__ plan, const int* ids,
+                                           const int* __restrict__ table, int vocab, int top, int n_pairs, int n_experts, int n_ids,
+                                           int max_tiles, int tile, int* sh) {
   int* count = sh;
   int* first = sh + n_experts + 1;
   int* cursor = sh + 2 * (n_experts + 1);
-  for (int e = threadIdx.x; e <= n_experts; e += blockDim.x) count[e] = 0, cursor[e] = 0;
-  __syncthreads();
-  pdl_wait();
-  ids = pdl_fresh(ids);
-  perm += (size_t)blockIdx.x * n_pairs;
-  plan += (size_t)blockIdx.x * (1 + 3 * max_tiles);
   if (table != nullptr) table += (size_t)blockIdx.x * vocab * top;
   auto expert_of = [&](int p) {
     if (table == nullptr) return ids[p];
@@ -284,29 +311,95 @@ expert_plan_kernel(int* __restrict__ perm, int* __restrict__ plan, const int* __
     if (ok) atomicAdd(&count[min(e, n_experts)], 1);
   }
   __syncthreads();
-  if (threadIdx.x == 0) {
+  if (threadIdx.x < 32) {                           // a lane an expert, 32 at a time: rows and tiles summed up over the lanes
+    const int lane = threadIdx.x;
     int rows = 0, tiles = 0;
-    for (int e = 0; e < n_experts; ++e) {
-      first[e] = rows;
+    for (int e0 = 0; e0 < n_experts; e0 += 32) {
+      const int e = e0 + lane, n = e < n_experts ? count[e] : 0;
       // an expert's rows in as few tiles as hold them, of equal size (a last tile of a few rows costs a wide
       // tile's set-up for nothing)
-      const int n_t = (count[e] + tile - 1) / tile;
-      const int per = n_t > 0 ? (count[e] + n_t - 1) / n_t : 0;
-      for (int r = 0; r < count[e] && tiles < max_tiles; r += per, ++tiles) {
-        plan[1 + 3 * tiles] = e;
-        plan[2 + 3 * tiles] = rows + r;
-        plan[3 + 3 * tiles] = min(per, count[e] - r);
+      const int n_t = (n + tile - 1) / tile, per = n_t > 0 ? (n + n_t - 1) / n_t : 0;
+      const int used = per > 0 ? (n + per - 1) / per : 0;
+      int r = n, u = used;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int ur = __shfl_up_sync(0xffffffffu, r, o), uu = __shfl_up_sync(0xffffffffu, u, o);
+        if (lane >= o) r += ur, u += uu;
       }
-      rows += count[e];
+      const int row0 = rows + r - n, tile0 = tiles + u - used;
+      if (e < n_experts) first[e] = row0;
+      for (int i = 0; i < used && tile0 + i < max_tiles; ++i) {
+        plan[1 + 3 * (tile0 + i)] = e;
+        plan[2 + 3 * (tile0 + i)] = row0 + i * per;
+        plan[3 + 3 * (tile0 + i)] = min(per, n - i * per);
+      }
+      rows += __shfl_sync(0xffffffffu, r, 31);
+      tiles += __shfl_sync(0xffffffffu, u, 31);
     }
-    first[n_experts] = rows;
-    plan[0] = tiles;
+    if (lane == 0) first[n_experts] = rows, plan[0] = min(tiles, max_tiles);
   }
   __syncthreads();
   for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
     const int id = expert_of(p), e = min(id, n_experts);
     if (id >= 0 && id < n_ids) perm[first[e] + atomicAdd(&cursor[e], 1)] = p;
   }
+}
+
+__global__ void __launch_bounds__(1024)
+expert_plan_kernel(int* __restrict__ perm, int* __restrict__ plan, const int* __restrict__ ids,
+                   const int* __restrict__ table, int vocab, int top, int n_pairs, int n_experts, int n_ids, int max_tiles,
+                   int tile) {
+  pdl_launch_dependents();
+  extern __shared__ int sh[];
+  for (int e = threadIdx.x; e < 3 * (n_experts + 1); e += blockDim.x) sh[e] = 0;
+  __syncthreads();
+  pdl_wait();
+  ids = pdl_fresh(ids);
+  plan_pairs(perm + (size_t)blockIdx.x * n_pairs, plan + (size_t)blockIdx.x * (1 + 3 * max_tiles), ids, table, vocab, top, n_pairs,
+             n_experts, n_ids, max_tiles, tile, sh);
+}
+
+// Few tokens: one block chooses (a warp a token in turn) and sorts the pairs.
+__global__ void __launch_bounds__(512)
+expert_choose_plan_kernel(ExpertChoice c, ExpertPlanOut p) {
+  pdl_launch_dependents();
+  extern __shared__ float score_all[];
+  const int warp = threadIdx.x >> 5, per = 2 * c.n_experts + c.groups;
+  int* sh = reinterpret_cast<int*>(score_all + 16 * per);
+  for (int e = threadIdx.x; e < 3 * (p.n_experts + 1); e += blockDim.x) sh[e] = 0;
+  pdl_wait();
+  c.scores = pdl_fresh(c.scores);
+  for (int t = warp; t < c.n_tokens; t += 16) {
+    choose_token(c, t, score_all + (size_t)warp * per);
+    __syncwarp();
+  }
+  __syncthreads();                                  // (the block's own ids, in global memory: visible behind the barrier)
+  plan_pairs(p.perm, p.plan, c.ids, nullptr, 0, 1, c.n_tokens * c.top, p.n_experts, c.n_experts, p.max_tiles, p.tile, sh);
+}
+
+static size_t choose_plan_smem(const ExpertChoice& c, const ExpertPlanOut& p) {
+  return ((size_t)16 * (2 * c.n_experts + c.groups) + 3 * (p.n_experts + 1)) * sizeof(float);
+}
+
+static int launch_choose_plan(const ExpertChoice& c, const ExpertPlanOut& p, cudaStream_t stream) {
+  const int n_pairs = c.n_tokens * c.top;
+  AF_REQUIRE(p.n_experts > 0 && p.n_experts <= c.n_experts && p.tile > 0 &&
+                 (p.max_tiles >= n_pairs / p.tile + p.n_experts || p.max_tiles >= n_pairs),
+             "af_expert_route_plan: room for %d tiles is too little", p.max_tiles);
+  AF_REQUIRE(choose_plan_smem(c, p) <= 48 * 1024, "af_expert_route_plan: %d experts are too many for one block", c.n_experts);
+  af_launch(expert_choose_plan_kernel, dim3(1), dim3(512), choose_plan_smem(c, p), stream, c, p);
+  AF_CHECK_LAUNCH("af_expert_route_plan");
+}
+
+// af_expert_route and af_expert_plan of the same step in one (n_experts of the router's n_choices have matrices).
+AF_EXPORT int af_expert_route_plan(int* ids, float* wts, float* shared_gate, float* scores, const void* h, int h_dtype,
+                                   const float* router, int n_tokens, int hidden, int n_choices, int top,
+                                   const float* correction, int groups, int keep, int normalise, float out_scale, int softmax,
+                                   int group_max, int* perm, int* plan, int n_experts, int max_tiles, int tile,
+                                   cudaStream_t stream) {
+  return expert_route_impl(ids, wts, shared_gate, scores, h, h_dtype, router, n_tokens, hidden, n_choices, top, correction, groups,
+                           keep, normalise, out_scale, softmax, group_max, ExpertPlanOut{perm, plan, n_experts, max_tiles, tile},
+                           stream);
 }
 
 AF_EXPORT int af_expert_plan(int* perm, int* plan, const int* ids, int n_pairs, int n_experts, int identity,

@@ -1409,14 +1409,17 @@ def expert_tc_tile(n_pairs: int, n_experts: int) -> int:
 
 
 def expert_route(ids, wts, shared_gate, h, router, n_experts: int, correction=None, groups: int = 1, keep: int = 1,
-                 normalise: bool = False, out_scale: float = 1.0, score: str = "sigmoid", group_score: str = "top2") -> None:
+                 normalise: bool = False, out_scale: float = 1.0, score: str = "sigmoid", group_score: str = "top2",
+                 plan_out=None) -> None:
     """Per row of h [T, H]: scores = sigmoid(router[:n_experts] h) in 32 bits; ids, wts [T, top] = the experts
     with the largest scores (equal scores: the lower index) and their scores; ``shared_gate`` float32 [T], when
     given, = sigmoid(router[n_experts] h).  ``correction`` (float32 [experts]) is added to the scores for the
     choice only.  ``groups`` > 1: the experts form so many equal groups of neighbours, a group's score is the sum
     of its two largest choice scores, and only experts of the ``keep`` best groups can be chosen.  ``normalise``:
     the chosen scores are divided by their sum + 1e-20; ``out_scale`` multiplies the weights.  ``score`` "softmax": the
-    scores are the softmax of the logits over all experts; ``group_score`` "max": a group's score is its largest alone."""
+    scores are the softmax of the logits over all experts; ``group_score`` "max": a group's score is its largest alone.
+    ``plan_out`` = (perm, plan, experts with matrices, tile): also :func:`expert_plan` of these choices, in the same kernel
+    (for the few tokens of a decode step: :func:`route_plans_fit`)."""
     if score not in ROUTER_SCORES or group_score not in GROUP_SCORES:
         raise KernelError(f"expert_route: score '{score}' or group score '{group_score}'")
     T, H = h.shape
@@ -1430,13 +1433,25 @@ def expert_route(ids, wts, shared_gate, h, router, n_experts: int, correction=No
     if correction is not None and (correction.numel() != n_experts or not correction.is_contiguous()):
         raise KernelError(f"expert_route: a correction of {n_experts} values")
     scores = torch.empty(T, rows, dtype=torch.float32, device=h.device)      # (between the two kernels)
-    _check(_lib().af_expert_route(_ptr(ids, "ids", torch.int32), _ptr(wts, "wts", torch.float32),
-                                  _ptr(shared_gate, "shared_gate", torch.float32, allow_none=True), _ptr(scores), _ptr(h),
-                                  c_int(dtype_code(h.dtype)), _ptr(router), c_int(T), c_int(H), c_int(n_experts),
-                                  c_int(top), _ptr(correction, "correction", torch.float32, allow_none=True),
-                                  c_int(groups), c_int(keep if groups > 1 else 1), c_int(1 if normalise else 0),
-                                  c_float(out_scale), c_int(ROUTER_SCORES[score]), c_int(GROUP_SCORES[group_score]),
-                                  _stream()))
+    args = (_ptr(ids, "ids", torch.int32), _ptr(wts, "wts", torch.float32),
+            _ptr(shared_gate, "shared_gate", torch.float32, allow_none=True), _ptr(scores), _ptr(h),
+            c_int(dtype_code(h.dtype)), _ptr(router), c_int(T), c_int(H), c_int(n_experts),
+            c_int(top), _ptr(correction, "correction", torch.float32, allow_none=True),
+            c_int(groups), c_int(keep if groups > 1 else 1), c_int(1 if normalise else 0),
+            c_float(out_scale), c_int(ROUTER_SCORES[score]), c_int(GROUP_SCORES[group_score]))
+    if plan_out is None:
+        _check(_lib().af_expert_route(*args, _stream()))
+        return
+    perm, plan, with_matrices, tile = plan_out
+    if perm.numel() != T * top or not (perm.is_contiguous() and plan.is_contiguous()):
+        raise KernelError("expert_route: one entry of perm per pair")
+    _check(_lib().af_expert_route_plan(*args, _ptr(perm, "perm", torch.int32), _ptr(plan, "plan", torch.int32),
+                                       c_int(with_matrices), c_int((plan.numel() - 1) // 3), c_int(tile), _stream()))
+
+
+def route_plans_fit(n_tokens: int, n_choices: int, groups: int) -> bool:
+    """Whether the choice's kernel makes the plan as well (one block: a decode step's few tokens)."""
+    return n_tokens <= 64 and 16 * (2 * n_choices + groups) + 3 * (n_choices + 1) <= 12 * 1024
 
 
 ROUTER_SCORES = {"sigmoid": 0, "softmax": 1}

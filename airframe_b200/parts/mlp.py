@@ -337,12 +337,15 @@ class RoutedExperts(FeedForward):
         ids = torch.empty(T, top, dtype=i32, device=dev)
         wts = torch.empty(T, top, dtype=torch.float32, device=dev)
         mix = torch.empty(T, dtype=torch.float32, device=dev) if self.mixed else None
-        kernels.expert_route(ids, wts, mix, x, self.router, self.n_choices, correction=self.correction,
-                             groups=self.groups, keep=self.keep, normalise=self.normalise, out_scale=self.route_scale,
-                             score=self.score, group_score=self.group_score)
         perm = torch.empty(T * top, dtype=i32, device=dev)
         plan = torch.empty(cells, dtype=i32, device=dev)
-        kernels.expert_plan(perm, plan, ids, self.n_experts, tile, identity=self.identity)
+        few = kernels.route_plans_fit(T, self.n_choices, self.groups)
+        kernels.expert_route(ids, wts, mix, x, self.router, self.n_choices, correction=self.correction,
+                             groups=self.groups, keep=self.keep, normalise=self.normalise, out_scale=self.route_scale,
+                             score=self.score, group_score=self.group_score,
+                             plan_out=(perm, plan, self.n_experts, tile) if few else None)
+        if not few:
+            kernels.expert_plan(perm, plan, ids, self.n_experts, tile, identity=self.identity)
         return perm, plan, wts, mix, ids if self.identity else None
 
     def forward(self, x, batch):

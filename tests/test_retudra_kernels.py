@@ -369,6 +369,26 @@ def test_router_with_softmax_scores(K, E, ident, top, groups, keep, T, H, dtype)
             want = plain.choose(s[t], corr.double(), top, groups, keep)
             assert ids[t].tolist() == want, t
             assert float((wts[t].cpu().double() - s[t, want]).abs().max()) < 1e-5
+        if not K.route_plans_fit(T, n, groups):
+            continue
+        # the same choices with the plan in the same kernel: every pair once, by expert, the identity experts' last
+        perm = torch.full((T * top,), -1, dtype=torch.int32, device=DEV)
+        plan = torch.empty(1 + 3 * K.expert_max_tiles(T * top, E, 16), dtype=torch.int32, device=DEV)
+        ids2, wts2 = torch.empty_like(ids), torch.empty_like(wts)
+        K.expert_route(ids2, wts2, None, h.to(DEV), router.to(DEV), n, correction=corr.to(DEV), groups=groups, keep=keep,
+                       score="softmax", group_score="max", plan_out=(perm, plan, E, 16))
+        assert torch.equal(ids2, ids) and torch.equal(wts2, wts)
+        order = perm.cpu().long()
+        assert sorted(order.tolist()) == list(range(T * top))
+        by = ids.cpu().flatten()[order].clamp(max=E)
+        assert torch.equal(by, by.sort().values)
+        cells = plan.cpu().tolist()
+        covered = []
+        for i in range(cells[0]):
+            e, r0, m = cells[1 + 3 * i: 4 + 3 * i]
+            assert 0 < m <= 16 and by[r0: r0 + m].tolist() == [e] * m
+            covered += range(r0, r0 + m)
+        assert covered == list(range(int((by < E).sum())))
     with pytest.raises(K.KernelError):
         K.expert_route(ids, wts, None, h.to(DEV), router.to(DEV), n, score="cosine")
 
